@@ -13,7 +13,7 @@ Here ONE manager serves all requests:
   need (kv heads, head size, window or chunk) form a **page group**: the group has one pool of page ids and
   one block table per request, and each entry of the group has key and value tensors of its own
   ``[pages, kv heads, page size, head dim]`` addressed by the group's page ids.  Groups with
-  different needs (all keys / a window of them) have pools and tables of their own.
+  different needs (all keys / a window of them / a row for every so many tokens) have pools and tables of their own.
 * A request's pages are allocated before a step for every token the step brings (``extend``),
   counted as held after it (``commit``), and given back when the request ends (``release``) or, in a
   window group (or one of chunks), as soon as the window has passed them or their chunk is over (in ``commit``); a page that is given back is
@@ -65,8 +65,8 @@ class PageGroup:
 
     @property
     def span(self) -> Optional[int]:
-        """The most keys a token reads (None: all of them)."""
-        return self.need.window if self.need.window is not None else self.need.chunk
+        """The most rows a request has to hold at once (None: all of them)."""
+        return self.need.span
 
 
 @dataclass
@@ -182,7 +182,8 @@ class CacheManager:
                  prefix_sharing: bool = False, min_prefix_share_tokens: int = 0, keep_finished: bool = False):
         """``needs[i]``: the cache need of run-order entry i (PagedKV, FixedState, a kind registered with
         ``register_cache_need``, or None).
-        ``num_pages``: pages per group (an int for all groups, or a dict gid -> int).
+        ``num_pages``: pages per group (an int for all groups, or a dict gid -> int).  An int counts pages of tokens: a
+        group with a row for every so many tokens gets what those tokens' rows need at most.
         ``device`` None: bookkeeping only (no tensors), as the CPU tests use it.
         ``keep_finished`` (with prefix sharing): shareable pages stay in the cache after their last
         holder has gone, until their room is needed."""
@@ -208,7 +209,7 @@ class CacheManager:
         self.requests: dict = {}
         # Pages of prompts are shared only where a page means the same for every layer: all page groups keep
         # every key (no window) and no mixer keeps a state of its own.
-        shareable = bool(self.groups) and all(g.keeps_all for g in self.groups) and not any(
+        shareable = bool(self.groups) and all(g.keeps_all and g.need.stride == 1 for g in self.groups) and not any(
             isinstance(leaf, FixedState) for n in needs for leaf in leaf_needs(n))
         self.prefix = PrefixIndex() if (prefix_sharing and shareable) else None
         self.min_prefix_share_tokens = int(min_prefix_share_tokens)
@@ -238,7 +239,11 @@ class CacheManager:
         gid = self._by_need.get(need)
         if gid is None:
             gid = len(self.groups)
-            n = self._num_pages[gid] if isinstance(self._num_pages, dict) else self._num_pages
+            if isinstance(self._num_pages, dict):
+                n = self._num_pages[gid]
+            else:  # every request may leave its last page of rows part-filled
+                n = self._num_pages if need.stride == 1 else min(
+                    self._num_pages, -(-self._num_pages // need.stride) + self.max_requests)
             self.groups.append(PageGroup(gid, need, [], self.page_size, PagePool(n)))
             self._by_need[need] = gid
         return self.groups[gid]
@@ -331,12 +336,16 @@ class CacheManager:
         """Lowest block that a query at position >= num_tokens can still read."""
         return g.need.first_needed(num_tokens) // self.page_size
 
+    def _blocks(self, g: PageGroup, num_tokens: int) -> int:
+        """How many blocks the rows of ``num_tokens`` tokens fill."""
+        return -(-g.need.rows(num_tokens) // self.page_size)
+
     def pages_needed(self, request_id, new_total: int) -> dict:
         """gid -> pages that ``extend(request_id, new_total)`` would take from the pool."""
         rc = self.get(request_id)
         out = {}
-        blocks = -(-new_total // self.page_size)
         for g in self.groups:
+            blocks = self._blocks(g, new_total)
             table = rc.tables[g.gid]
             first = self._first_needed_block(g, rc.num_tokens)
             # every block from `first` up to the table's end has a page (extend fills them, commit frees
@@ -396,8 +405,8 @@ class CacheManager:
         short = max(need[g.gid] - g.pool.num_free for g in self.groups) if self.groups else 0
         if short > 0:
             self._evict_idle(short)
-        blocks = -(-new_total // self.page_size)
         for g in self.groups:
+            blocks = self._blocks(g, new_total)
             table = rc.tables[g.gid]
             if blocks <= len(table):
                 continue
@@ -492,7 +501,8 @@ class CacheManager:
         return arr
 
     def slots_for(self, request_id, gid: int, start: int, count: int) -> list:
-        """Cache slot (page * page_size + offset) of positions start .. start + count - 1."""
+        """Cache slot (page * page_size + offset) of rows start .. start + count - 1 (a row is a position, or a run of
+        them in a group with a stride)."""
         table = self.get(request_id).tables[gid]
         ps = self.page_size
         out = []

@@ -41,6 +41,10 @@ def _of(d, key, kind, where, default=None, required=True):
         if isinstance(v, bool) or not isinstance(v, (int, float)) or not math.isfinite(float(v)):
             raise ConfigError(f"config.json: {where}.{key} must be a finite number, found {v!r}")
         return float(v)
+    if kind is bool:
+        if not isinstance(v, bool):
+            raise ConfigError(f"config.json: {where}.{key} must be true or false, found {v!r}")
+        return v
     if kind is dict:
         if not isinstance(v, dict):
             raise ConfigError(f"config.json: {where}.{key} must be an object")

@@ -8,6 +8,9 @@
 //   the start of P's chunk; softmax over them; out = sum w_j v_j.
 //   With `slopes` (one per query head; a position encoding that acts on the scores, not on q and k):
 //   s_j += slopes[hq] * (j - P), a penalty linear in the distance.
+//   With pooled keys (PooledKeys) beside a window: one key and value more for every run of `every` positions (counted off
+//   from 0) that lies wholly before the window, read from pages of their own (the means of the run's keys and values);
+//   tokens and runs share one softmax.  With lo the window's first position, the runs seen are 0 .. lo / every - 1.
 // (crates/ferrisinfer-kernel/src/cpu/attention.rs:729-781, 1125-1155: streaming softmax with a
 // running maximum, which this kernel keeps per warp).  The step's own keys are already in the
 // cache when this runs, so prompts, portions of prompts and single decoded tokens are one case.
@@ -33,6 +36,15 @@ struct ScoreTerms {
     const float* log_r2;
     const float* sink;
     int v_stride;
+};
+// Keys that stand for runs of positions before the window: k [pages, nkv, page_size, d] and v [.., dv], rows addressed by
+// tables [requests, max_blocks] as tokens are by the step's block tables.  Kernels with POOL walk the keys by one index
+// n: n < pooled is the run n, the others are the tokens from the window's first position on.
+struct PooledKeys {
+    const void* k;
+    const void* v;
+    const int* tables;
+    int max_blocks, every;
 };
 struct HeadTerms {
     int kind;  // 0: nothing, 1: slope, 2: logarithm
@@ -60,13 +72,13 @@ __device__ __forceinline__ int first_key(int P, int window) {
 // the sink's share of the denominator, relative to the maximum mm of the keys' scores
 __device__ __forceinline__ float sink_share(const ScoreTerms& st, int h, float mm) { return st.sink ? expf(st.sink[h] - mm) : 0.0f; }
 
-template <typename T>
+template <typename T, bool POOL>
 __global__ void __launch_bounds__(ATT_THREADS)
     paged_attention_simt_kernel(const T* q, int ldq, T* __restrict__ out, int ldo, const T* k_cache, const T* v_cache,
                                 const int* __restrict__ block_tables, int max_blocks,
                                 const int* __restrict__ token_seq, const int* __restrict__ positions, int nh,
                                 int nkv, int d, int dv, int page_size, int window, float scale,
-                                const ScoreTerms st) {
+                                const ScoreTerms st, const PooledKeys pk) {
     extern __shared__ float smem[];  // per warp: m, z, acc[dv]
     pdl_wait();
     pdl_launch_dependents();
@@ -89,18 +101,25 @@ __global__ void __launch_bounds__(ATT_THREADS)
         acc[r] = 0.0f;
     }
     float m = -INFINITY, z = 0.0f;
-    for (int j = lo + warp; j <= P; j += ATT_WARPS) {
-        const int page = table[j / page_size];
+    const int pooled = POOL ? lo / pk.every : 0;
+    const int shift = POOL ? lo - pooled : 0;  // key n >= pooled is the token at n + shift
+    const int* ptable = POOL ? pk.tables + (size_t)seq * pk.max_blocks : nullptr;
+    for (int n = (POOL ? 0 : lo) + warp; n <= P - shift; n += ATT_WARPS) {
+        const bool run = POOL && n < pooled;
+        const int j = run ? n : n + shift;
+        const int page = (run ? ptable : table)[j / page_size];
         if (page < 0) continue;  // a hole in the table: never reached for keys inside the window
         const size_t row = ((size_t)page * nkv + hk) * page_size + (j % page_size);
         const size_t base = row * d, vbase = row * vs;
+        const T* keys = run ? reinterpret_cast<const T*>(pk.k) : k_cache;
+        const T* vals = run ? reinterpret_cast<const T*>(pk.v) : v_cache;
         float dot = 0.0f;
 #pragma unroll
         for (int r = 0; r < MAX_PER_LANE; ++r) {
             const int i = lane + 32 * r;
-            if (i < d) dot = fmaf(qv[r], to_float(k_cache[base + i]), dot);
+            if (i < d) dot = fmaf(qv[r], to_float(keys[base + i]), dot);
         }
-        const float s = with_terms(warp_sum(dot) * scale, ht, j, P);
+        const float s = POOL ? warp_sum(dot) * scale : with_terms(warp_sum(dot) * scale, ht, j, P);
         float wgt;
         if (s > m) {
             const float rescale = expf(m - s);  // exp(-inf) = 0 on the first key
@@ -116,7 +135,7 @@ __global__ void __launch_bounds__(ATT_THREADS)
 #pragma unroll
         for (int r = 0; r < MAX_PER_LANE; ++r) {
             const int i = lane + 32 * r;
-            if (i < dv) acc[r] = fmaf(wgt, to_float(v_cache[vbase + i]), acc[r]);
+            if (i < dv) acc[r] = fmaf(wgt, to_float(vals[vbase + i]), acc[r]);
         }
     }
     float* mine = smem + warp * (dv + 2);
@@ -215,13 +234,13 @@ __device__ __forceinline__ void load_chunk(const bf16* p, int n, float (&o)[MAXC
 }
 
 // MAXC: most elements of a head that one lane holds (d, dv <= 8 * MAXC).  U: keys of a group in flight together.
-template <typename T, int MAXC, int U>
+template <typename T, int MAXC, int U, bool POOL>
 __global__ void __launch_bounds__(AL_THREADS)
     paged_attention_lanes_kernel(const T* q, int ldq, T* __restrict__ out, int ldo, const T* k_cache, const T* v_cache,
                                  const int* __restrict__ block_tables, int max_blocks,
                                  const int* __restrict__ token_seq, const int* __restrict__ positions, int nh, int nkv,
                                  int d, int dv, int page_size, int window, float scale,
-                                 const ScoreTerms st) {
+                                 const ScoreTerms st, const PooledKeys pk) {
     extern __shared__ float smem[];  // per group: m, z, acc[dv]
     pdl_wait();
     pdl_launch_dependents();
@@ -242,25 +261,31 @@ __global__ void __launch_bounds__(AL_THREADS)
     for (int i = 0; i < MAXC; ++i) qv[i] = 0.0f, acc[i] = 0.0f;
     load_chunk<MAXC>(q + (size_t)t * ldq + (size_t)hq * d + sub * ch, ch, qv);
     float m = -INFINITY, z = 0.0f;
-    const int rounds = (P - lo + AL_GROUPS * U) / (AL_GROUPS * U);  // every lane of a warp makes as many: the shuffles need all
+    const int pooled = POOL ? lo / pk.every : 0;
+    const int shift = POOL ? lo - pooled : 0;  // key n >= pooled is the token at n + shift
+    const int* ptable = POOL ? pk.tables + (size_t)seq * pk.max_blocks : nullptr;
+    const int n0 = POOL ? 0 : lo, n1 = P - shift;
+    const int rounds = (n1 - n0 + AL_GROUPS * U) / (AL_GROUPS * U);  // every lane of a warp makes as many: the shuffles need all
     for (int it = 0; it < rounds; ++it) {
         float kk[U][MAXC], vv[U][MAXC];
         bool ok[U];
         int jj[U];
 #pragma unroll
         for (int u = 0; u < U; ++u) {
-            const int j = lo + (it * U + u) * AL_GROUPS + grp;
+            const int n = n0 + (it * U + u) * AL_GROUPS + grp;
+            const bool run = POOL && n < pooled;
+            const int j = run ? n : n + shift;
             jj[u] = j;
             int page = -1;
-            if (j <= P) page = table[pshift >= 0 ? (j >> pshift) : (j / page_size)];
+            if (n <= n1) page = (run ? ptable : table)[pshift >= 0 ? (j >> pshift) : (j / page_size)];
             ok[u] = page >= 0;  // beyond the last key, or a hole in the table (never for keys inside the window)
             const int in_page = pshift >= 0 ? (j & (page_size - 1)) : (j % page_size);
             const size_t row = ((size_t)(ok[u] ? page : 0) * nkv + hk) * page_size + (ok[u] ? in_page : 0);
 #pragma unroll
             for (int i = 0; i < MAXC; ++i) kk[u][i] = 0.0f, vv[u][i] = 0.0f;
             if (ok[u]) {
-                load_chunk<MAXC>(k_cache + row * d + sub * ch, ch, kk[u]);
-                load_chunk<MAXC>(v_cache + row * vs + sub * cv, cv, vv[u]);
+                load_chunk<MAXC>((run ? reinterpret_cast<const T*>(pk.k) : k_cache) + row * d + sub * ch, ch, kk[u]);
+                load_chunk<MAXC>((run ? reinterpret_cast<const T*>(pk.v) : v_cache) + row * vs + sub * cv, cv, vv[u]);
             }
         }
         float dot[U];
@@ -278,7 +303,7 @@ __global__ void __launch_bounds__(AL_THREADS)
 #pragma unroll
         for (int u = 0; u < U; ++u) {
             if (!ok[u]) continue;
-            const float s = with_terms(dot[u] * scale, ht, jj[u], P);
+            const float s = POOL ? dot[u] * scale : with_terms(dot[u] * scale, ht, jj[u], P);
             float wgt;
             if (s > m) {
                 const float rescale = expf(m - s);  // exp(-inf) = 0 on the first key
@@ -331,13 +356,13 @@ __global__ void __launch_bounds__(AL_THREADS)
 constexpr int AG_THREADS = 128;
 constexpr int AG_GROUPS = AG_THREADS / 16;
 
-template <typename T, int MAXC, int G, int U>
+template <typename T, int MAXC, int G, int U, bool POOL>
 __global__ void __launch_bounds__(AG_THREADS)
     paged_attention_shared_kernel(const T* q, int ldq, T* __restrict__ out, int ldo, const T* k_cache, const T* v_cache,
                                   const int* __restrict__ block_tables, int max_blocks,
                                   const int* __restrict__ token_seq, const int* __restrict__ positions, int nh, int nkv,
                                   int d, int dv, int page_size, int window, float scale,
-                                  const ScoreTerms st, int splits, float* __restrict__ partial) {
+                                  const ScoreTerms st, const PooledKeys pk, int splits, float* __restrict__ partial) {
     extern __shared__ float smem[];  // per group and head: m, z, acc[dv]
     pdl_wait();
     pdl_launch_dependents();
@@ -363,10 +388,14 @@ __global__ void __launch_bounds__(AG_THREADS)
         m[a] = -INFINITY, z[a] = 0.0f;
         ht[a] = head_terms(st, h0 + a);
     }
-    // the block's share of the keys lo .. P: with several splits, a run of `span` keys each
-    const int span = (P - lo + splits) / splits;
-    const int first = lo + split * span;
-    const int lastk = min(P, first + span - 1);
+    const int pooled = POOL ? lo / pk.every : 0;
+    const int shift = POOL ? lo - pooled : 0;  // key n >= pooled is the token at n + shift
+    const int* ptable = POOL ? pk.tables + (size_t)seq * pk.max_blocks : nullptr;
+    const int n0 = POOL ? 0 : lo, n1 = P - shift;
+    // the block's share of the keys n0 .. n1: with several splits, a run of `span` keys each
+    const int span = (n1 - n0 + splits) / splits;
+    const int first = n0 + split * span;
+    const int lastk = min(n1, first + span - 1);
     const int rounds = lastk >= first ? (lastk - first + AG_GROUPS * U) / (AG_GROUPS * U) : 0;
     for (int it = 0; it < rounds; ++it) {
         float kk[U][MAXC], vv[U][MAXC];
@@ -374,18 +403,20 @@ __global__ void __launch_bounds__(AG_THREADS)
         int jj[U];
 #pragma unroll
         for (int u = 0; u < U; ++u) {
-            const int j = first + (it * U + u) * AG_GROUPS + grp;
+            const int n = first + (it * U + u) * AG_GROUPS + grp;
+            const bool run = POOL && n < pooled;
+            const int j = run ? n : n + shift;
             jj[u] = j;
             int page = -1;
-            if (j <= lastk) page = table[pshift >= 0 ? (j >> pshift) : (j / page_size)];
+            if (n <= lastk) page = (run ? ptable : table)[pshift >= 0 ? (j >> pshift) : (j / page_size)];
             ok[u] = page >= 0;
             const int in_page = pshift >= 0 ? (j & (page_size - 1)) : (j % page_size);
             const size_t row = ((size_t)(ok[u] ? page : 0) * nkv + hk) * page_size + (ok[u] ? in_page : 0);
 #pragma unroll
             for (int i = 0; i < MAXC; ++i) kk[u][i] = 0.0f, vv[u][i] = 0.0f;
             if (ok[u]) {
-                load_chunk<MAXC>(k_cache + row * d + sub * ch, ch, kk[u]);
-                load_chunk<MAXC>(v_cache + row * vs + sub * cv, cv, vv[u]);
+                load_chunk<MAXC>((run ? reinterpret_cast<const T*>(pk.k) : k_cache) + row * d + sub * ch, ch, kk[u]);
+                load_chunk<MAXC>((run ? reinterpret_cast<const T*>(pk.v) : v_cache) + row * vs + sub * cv, cv, vv[u]);
             }
         }
         float dot[U][G];
@@ -409,7 +440,7 @@ __global__ void __launch_bounds__(AG_THREADS)
             if (!ok[u]) continue;
 #pragma unroll
             for (int a = 0; a < G; ++a) {
-                const float s = with_terms(dot[u][a] * scale, ht[a], jj[u], P);
+                const float s = POOL ? dot[u][a] * scale : with_terms(dot[u][a] * scale, ht[a], jj[u], P);
                 float wgt;
                 if (s > m[a]) {
                     const float rescale = expf(m[a] - s);
@@ -491,18 +522,18 @@ __global__ void __launch_bounds__(128) attention_merge_shares_kernel(const float
     }
 }
 
-template <typename T, int G>
+template <typename T, int G, bool POOL>
 void launch_shared(const void* q, int ldq, void* out, int ldo, const void* k_cache, const void* v_cache,
                    const int* block_tables, int max_blocks, const int* token_seq, const int* positions, int tokens, int nh,
-                   int nkv, int d, int dv, int page_size, int window, float scale, const ScoreTerms st, int splits,
-                   float* partial, cudaStream_t s) {
+                   int nkv, int d, int dv, int page_size, int window, float scale, const ScoreTerms st, const PooledKeys pk,
+                   int splits, float* partial, cudaStream_t s) {
     const dim3 grid(tokens, nh / G, splits), block(AG_THREADS);
     const size_t smem = (size_t)AG_GROUPS * G * (dv + 2) * sizeof(float);
     const int most = d > dv ? d : dv;
 #define FERRIS_AG_LAUNCH(MAXC, U)                                                                                       \
-    ferris_launch(paged_attention_shared_kernel<T, MAXC, G, U>, grid, block, smem, s, (const T*)q, ldq, (T*)out, ldo,   \
+    ferris_launch(paged_attention_shared_kernel<T, MAXC, G, U, POOL>, grid, block, smem, s, (const T*)q, ldq, (T*)out, ldo,   \
                   (const T*)k_cache, (const T*)v_cache, block_tables, max_blocks, token_seq, positions, nh, nkv, d, dv,  \
-                  page_size, window, scale, st, splits, partial)
+                  page_size, window, scale, st, pk, splits, partial)
     if (most <= 128)
         FERRIS_AG_LAUNCH(8, 4);
     else
@@ -513,17 +544,18 @@ void launch_shared(const void* q, int ldq, void* out, int ldo, const void* k_cac
                       ldo, nh, dv, splits, st);
 }
 
-template <typename T>
+template <typename T, bool POOL>
 void launch_lanes(const void* q, int ldq, void* out, int ldo, const void* k_cache, const void* v_cache,
                   const int* block_tables, int max_blocks, const int* token_seq, const int* positions, int tokens, int nh,
-                  int nkv, int d, int dv, int page_size, int window, float scale, const ScoreTerms st, cudaStream_t s) {
+                  int nkv, int d, int dv, int page_size, int window, float scale, const ScoreTerms st, const PooledKeys pk,
+                  cudaStream_t s) {
     const dim3 grid(tokens, nh), block(AL_THREADS);
     const size_t smem = (size_t)AL_GROUPS * (dv + 2) * sizeof(float);
     const int most = d > dv ? d : dv;
 #define FERRIS_AL_LAUNCH(MAXC, U)                                                                                      \
-    ferris_launch(paged_attention_lanes_kernel<T, MAXC, U>, grid, block, smem, s, (const T*)q, ldq, (T*)out, ldo,      \
+    ferris_launch(paged_attention_lanes_kernel<T, MAXC, U, POOL>, grid, block, smem, s, (const T*)q, ldq, (T*)out, ldo,      \
                   (const T*)k_cache, (const T*)v_cache, block_tables, max_blocks, token_seq, positions, nh, nkv, d, dv, \
-                  page_size, window, scale, st)
+                  page_size, window, scale, st, pk)
     if (most <= 64)
         FERRIS_AL_LAUNCH(8, 2);
     else if (most <= 128)
@@ -564,13 +596,13 @@ __device__ __forceinline__ void zero_row(float* dst, int n, int part, int parts)
     for (int v = part; v * 4 < n; v += parts) *reinterpret_cast<float4*>(dst + v * 4) = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
 }
 
-template <typename T, int NC>  // NC: 4-column pieces of the value head that a lane adds up: dv <= 32 * NC
+template <typename T, int NC, bool POOL>  // NC: 4-column pieces of the value head that a lane adds up: dv <= 32 * NC
 __global__ void __launch_bounds__(TL_THREADS)
     paged_attention_tiled_kernel(const T* q, int ldq, T* __restrict__ out, int ldo, const T* k_cache, const T* v_cache,
                                  const int* __restrict__ block_tables, int max_blocks,
                                  const int* __restrict__ token_seq, const int* __restrict__ positions, int tokens, int nh,
                                  int nkv, int d, int dv, int page_size, int window, float scale,
-                                 const ScoreTerms st) {
+                                 const ScoreTerms st, const PooledKeys pk) {
     extern __shared__ __align__(16) float tl_smem[];
     const int dp = d + 4, dvp = dv + 4;
     float* Qs = tl_smem;                      // [64][d + 4], scaled
@@ -623,20 +655,27 @@ __global__ void __launch_bounds__(TL_THREADS)
         int tb = ta;  // its last token within the tile
         while (tb + 1 < t_end && token_seq[tb + 1] == sq) ++tb;
         const int pa = positions[ta], pb = positions[tb];
-        const int kmin = first_key(pa, window);  // of the first token: no later token of the request sees an earlier key
-        const int* table = block_tables + (size_t)sq * max_blocks;
-        for (int j0 = kmin & ~(TL_KEYS - 1); j0 <= pb; j0 += TL_KEYS) {
+        // with POOL the keys of runs before the window come first (seg 0, indexed by the run), then the tokens
+        for (int seg = POOL ? 0 : 1; seg < 2; ++seg) {
+        const bool runs = POOL && seg == 0;
+        // of the first token: no later token of the request sees an earlier key
+        const int kmin = runs ? 0 : first_key(pa, window);
+        const int kmax = runs ? first_key(pb, window) / pk.every - 1 : pb;
+        const int* table = runs ? pk.tables + (size_t)sq * pk.max_blocks : block_tables + (size_t)sq * max_blocks;
+        const T* keys = runs ? reinterpret_cast<const T*>(pk.k) : k_cache;
+        const T* vals = runs ? reinterpret_cast<const T*>(pk.v) : v_cache;
+        for (int j0 = kmin & ~(TL_KEYS - 1); j0 <= kmax; j0 += TL_KEYS) {
             __syncthreads();  // the tile before has been used (and, the first time, the queries are in place)
             {
                 const int key = tid >> 3, part = tid & 7;
                 const int j = j0 + key;
                 int page = -1;
-                if (j >= kmin && j <= pb) page = table[pshift >= 0 ? (j >> pshift) : (j / page_size)];
+                if (j >= kmin && j <= kmax) page = table[pshift >= 0 ? (j >> pshift) : (j / page_size)];
                 if (page >= 0) {
                     const int in_page = pshift >= 0 ? (j & (page_size - 1)) : (j % page_size);
                     const size_t row = ((size_t)page * nkv + hk) * page_size + in_page;
-                    stage_row(k_cache + row * d, Ks + key * dp, d, part, 8, 1.0f);
-                    stage_row(v_cache + row * (st.v_stride ? (size_t)st.v_stride : (size_t)dv), Vs + key * dvp, dv, part, 8, 1.0f);
+                    stage_row(keys + row * d, Ks + key * dp, d, part, 8, 1.0f);
+                    stage_row(vals + row * (st.v_stride ? (size_t)st.v_stride : (size_t)dv), Vs + key * dvp, dv, part, 8, 1.0f);
                 } else {
                     zero_row(Ks + key * dp, d, part, 8);
                     zero_row(Vs + key * dvp, dv, part, 8);
@@ -665,13 +704,17 @@ __global__ void __launch_bounds__(TL_THREADS)
             float alpha[2];
 #pragma unroll
             for (int a = 0; a < 2; ++a) {
-                const int lo = first_key(rpos[a], window);
+                int lo = first_key(rpos[a], window), hi = rpos[a];
+                if (runs) hi = lo / pk.every - 1, lo = 0;
                 float best = -INFINITY;
 #pragma unroll
                 for (int c = 0; c < 4; ++c) {
                     const int j = j0 + kx + 8 * c;
-                    const bool seen = rseq[a] == sq && j >= lo && j <= rpos[a];
-                    sc[a][c] = seen ? with_terms(sc[a][c], rterm[a], j, rpos[a]) : -INFINITY;
+                    const bool seen = rseq[a] == sq && j >= lo && j <= hi;
+                    if (POOL)
+                        sc[a][c] = seen ? sc[a][c] : -INFINITY;
+                    else
+                        sc[a][c] = seen ? with_terms(sc[a][c], rterm[a], j, rpos[a]) : -INFINITY;
                     best = fmaxf(best, sc[a][c]);
                 }
 #pragma unroll
@@ -713,6 +756,7 @@ __global__ void __launch_bounds__(TL_THREADS)
                 }
             }
         }
+        }
         ta = tb + 1;
     }
 #pragma unroll
@@ -742,20 +786,21 @@ bool tiled_takes(int dtype, int nh, int nkv, int d, int dv) {
            dv <= 256 && tiled_smem_bytes(d, dv) <= 200 * 1024;
 }
 
-template <typename T>
+template <typename T, bool POOL>
 int launch_tiled(const void* q, int ldq, void* out, int ldo, const void* k_cache, const void* v_cache,
                  const int* block_tables, int max_blocks, const int* token_seq, const int* positions, int tokens, int nh,
-                 int nkv, int d, int dv, int page_size, int window, float scale, const ScoreTerms st, cudaStream_t s) {
+                 int nkv, int d, int dv, int page_size, int window, float scale, const ScoreTerms st, const PooledKeys pk,
+                 cudaStream_t s) {
     const int qt = TL_ROWS / (nh / nkv);
     const dim3 grid((tokens + qt - 1) / qt, nkv), block(TL_THREADS);
     const size_t smem = tiled_smem_bytes(d, dv);
 #define FERRIS_TL_LAUNCH(NC)                                                                                        \
     do {                                                                                                            \
-        int e_ = ferris_allow_dynamic_smem((const void*)paged_attention_tiled_kernel<T, NC>, smem);                 \
+        int e_ = ferris_allow_dynamic_smem((const void*)paged_attention_tiled_kernel<T, NC, POOL>, smem);                 \
         if (e_ != FERRIS_OK) return e_;                                                                             \
-        ferris_launch(paged_attention_tiled_kernel<T, NC>, grid, block, smem, s, (const T*)q, ldq, (T*)out, ldo,   \
+        ferris_launch(paged_attention_tiled_kernel<T, NC, POOL>, grid, block, smem, s, (const T*)q, ldq, (T*)out, ldo,   \
                       (const T*)k_cache, (const T*)v_cache, block_tables, max_blocks, token_seq, positions, tokens, \
-                      nh, nkv, d, dv, page_size, window, scale, st);                                           \
+                      nh, nkv, d, dv, page_size, window, scale, st, pk);                                       \
     } while (0)
     if (dv <= 64)
         FERRIS_TL_LAUNCH(2);
@@ -767,6 +812,16 @@ int launch_tiled(const void* q, int ldq, void* out, int ldo, const void* k_cache
     FERRIS_LAUNCH_CHECK();
 }
 
+// Whether the arguments for pooled keys make sense (all null / 0: there are none).
+int check_pooled(const PooledKeys& pk, int window, const ScoreTerms& st) {
+    if (pk.every == 0 && !pk.k && !pk.v && !pk.tables) return FERRIS_OK;
+    if (pk.every <= 0 || !pk.k || !pk.v || !pk.tables || pk.max_blocks <= 0)
+        FERRIS_REFUSE("attention: pooled keys of %d positions want rows and block tables", pk.every);
+    if (window <= 0) FERRIS_REFUSE("attention: pooled keys stand before a window");
+    if (st.slopes || st.log_r1 || st.v_stride) FERRIS_REFUSE("attention: pooled keys go with no distance penalty and no values in keys");
+    return FERRIS_OK;
+}
+
 }  // namespace
 
 FERRIS_API int ferris_paged_attention_simt(const void* q, int ldq, void* out, int ldo, const void* k_cache,
@@ -774,12 +829,16 @@ FERRIS_API int ferris_paged_attention_simt(const void* q, int ldq, void* out, in
                                            const int* token_seq, const int* positions, int tokens, int nh, int nkv,
                                            int d, int dv, int page_size, int window, float scale, const float* slopes,
                                            const float* log_r1, const float* log_r2, const float* sink, int v_stride,
-                                           int kv_span, float* scratch, long long scratch_floats, void* stream) {
+                                           const void* pool_k, const void* pool_v, const int* pool_tables,
+                                           int pool_max_blocks, int pool_every, int kv_span, float* scratch, long long scratch_floats, void* stream) {
     if (tokens <= 0) return FERRIS_OK;
     if ((log_r1 == nullptr) != (log_r2 == nullptr)) FERRIS_REFUSE("attention: the logarithmic penalty needs both of its numbers per head");
     if (slopes && log_r1) FERRIS_REFUSE("attention: a slope and a logarithmic penalty at once");
     if (v_stride < 0 || (v_stride > 0 && v_stride < dv)) FERRIS_REFUSE("attention: value rows %d apart hold no %d values", v_stride, dv);
     const ScoreTerms st = {slopes, log_r1, log_r2, sink, v_stride};
+    const PooledKeys pk = {pool_k, pool_v, pool_tables, pool_max_blocks, pool_every};
+    if (int rc = check_pooled(pk, window, st)) return rc;
+    const bool pool = pk.every > 0;
     if (nh <= 0 || nkv <= 0 || nh % nkv != 0) FERRIS_REFUSE("attention: %d heads over %d kv heads", nh, nkv);
     if (d <= 0 || d > 32 * MAX_PER_LANE) FERRIS_REFUSE("attention: head size %d not in 1..%d", d, 32 * MAX_PER_LANE);
     if (dv <= 0 || dv > 32 * MAX_PER_LANE) FERRIS_REFUSE("attention: value head size %d not in 1..%d", dv, 32 * MAX_PER_LANE);
@@ -791,7 +850,8 @@ FERRIS_API int ferris_paged_attention_simt(const void* q, int ldq, void* out, in
     if (dtype != FERRIS_F32 && dtype != FERRIS_BF16) FERRIS_REFUSE("attention: unknown dtype %d", dtype);
     // head sizes that eight lanes can share evenly, rows that start on 16 bytes: the kernel with eight lanes to a key
     const size_t elt = dtype == FERRIS_F32 ? 4 : 2;
-    const bool aligned = (((uintptr_t)q | (uintptr_t)k_cache | (uintptr_t)v_cache) & 15) == 0 && ((size_t)ldq * elt) % 16 == 0;
+    const bool aligned = (((uintptr_t)q | (uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)pool_k | (uintptr_t)pool_v) & 15) == 0 &&
+                         ((size_t)ldq * elt) % 16 == 0;
     // Query heads that share keys, where the caller brings scratch for shares of the keys (a step of single tokens):
     // the keys of a token are cut into as many shares as fill the SMs about three times over, of 64 keys at least.
     const int g = nh / nkv;
@@ -815,31 +875,51 @@ FERRIS_API int ferris_paged_attention_simt(const void* q, int ldq, void* out, in
         if (splits > fit) splits = fit;
         if (splits >= 1) {
             const int sp = (int)splits;
+#define FERRIS_AG(T, G)                                                                                                   \
+    do {                                                                                                                  \
+        if (pool)                                                                                                         \
+            launch_shared<T, G, true>(q, ldq, out, ldo, k_cache, v_cache, block_tables, max_blocks, token_seq, positions,  \
+                                      tokens, nh, nkv, d, dv, page_size, window, scale, st, pk, sp, scratch, s);          \
+        else                                                                                                              \
+            launch_shared<T, G, false>(q, ldq, out, ldo, k_cache, v_cache, block_tables, max_blocks, token_seq, positions, \
+                                       tokens, nh, nkv, d, dv, page_size, window, scale, st, pk, sp, scratch, s);         \
+    } while (0)
             if (dtype == FERRIS_F32) {
-                if (four) launch_shared<float, 4>(q, ldq, out, ldo, k_cache, v_cache, block_tables, max_blocks, token_seq, positions, tokens, nh, nkv, d, dv, page_size, window, scale, st, sp, scratch, s);
-                else launch_shared<float, 2>(q, ldq, out, ldo, k_cache, v_cache, block_tables, max_blocks, token_seq, positions, tokens, nh, nkv, d, dv, page_size, window, scale, st, sp, scratch, s);
+                if (four) FERRIS_AG(float, 4); else FERRIS_AG(float, 2);
             } else {
-                if (four) launch_shared<bf16, 4>(q, ldq, out, ldo, k_cache, v_cache, block_tables, max_blocks, token_seq, positions, tokens, nh, nkv, d, dv, page_size, window, scale, st, sp, scratch, s);
-                else launch_shared<bf16, 2>(q, ldq, out, ldo, k_cache, v_cache, block_tables, max_blocks, token_seq, positions, tokens, nh, nkv, d, dv, page_size, window, scale, st, sp, scratch, s);
+                if (four) FERRIS_AG(bf16, 4); else FERRIS_AG(bf16, 2);
             }
+#undef FERRIS_AG
             FERRIS_LAUNCH_CHECK();
         }
     }
     if (d % 8 == 0 && dv % 8 == 0 && d <= 256 && dv <= 256 && aligned && (size_t)AL_GROUPS * (dv + 2) * sizeof(float) <= 48 * 1024) {
+#define FERRIS_AL(T)                                                                                                      \
+    do {                                                                                                                  \
+        if (pool)                                                                                                         \
+            launch_lanes<T, true>(q, ldq, out, ldo, k_cache, v_cache, block_tables, max_blocks, token_seq, positions,      \
+                                  tokens, nh, nkv, d, dv, page_size, window, scale, st, pk, s);                           \
+        else                                                                                                              \
+            launch_lanes<T, false>(q, ldq, out, ldo, k_cache, v_cache, block_tables, max_blocks, token_seq, positions,     \
+                                   tokens, nh, nkv, d, dv, page_size, window, scale, st, pk, s);                          \
+    } while (0)
         if (dtype == FERRIS_F32)
-            launch_lanes<float>(q, ldq, out, ldo, k_cache, v_cache, block_tables, max_blocks, token_seq, positions, tokens, nh, nkv, d, dv, page_size, window, scale, st, s);
+            FERRIS_AL(float);
         else
-            launch_lanes<bf16>(q, ldq, out, ldo, k_cache, v_cache, block_tables, max_blocks, token_seq, positions, tokens, nh, nkv, d, dv, page_size, window, scale, st, s);
+            FERRIS_AL(bf16);
+#undef FERRIS_AL
         FERRIS_LAUNCH_CHECK();
     }
-    if (dtype == FERRIS_F32)
-        ferris_launch(paged_attention_simt_kernel<float>, grid, dim3(ATT_THREADS), smem, s, (const float*)q, ldq, (float*)out, ldo, (const float*)k_cache, (const float*)v_cache, block_tables,
-            max_blocks, token_seq, positions, nh, nkv, d, dv, page_size, window, scale, st);
-    else if (dtype == FERRIS_BF16)
-        ferris_launch(paged_attention_simt_kernel<bf16>, grid, dim3(ATT_THREADS), smem, s, (const bf16*)q, ldq, (bf16*)out, ldo, (const bf16*)k_cache, (const bf16*)v_cache, block_tables, max_blocks,
-            token_seq, positions, nh, nkv, d, dv, page_size, window, scale, st);
-    else
-        FERRIS_REFUSE("attention: unknown dtype %d", dtype);
+#define FERRIS_ATT(T, POOL)                                                                                               \
+    ferris_launch(paged_attention_simt_kernel<T, POOL>, grid, dim3(ATT_THREADS), smem, s, (const T*)q, ldq, (T*)out, ldo,  \
+                  (const T*)k_cache, (const T*)v_cache, block_tables, max_blocks, token_seq, positions, nh, nkv, d, dv,    \
+                  page_size, window, scale, st, pk)
+    if (dtype == FERRIS_F32) {
+        if (pool) FERRIS_ATT(float, true); else FERRIS_ATT(float, false);
+    } else {
+        if (pool) FERRIS_ATT(bf16, true); else FERRIS_ATT(bf16, false);
+    }
+#undef FERRIS_ATT
     FERRIS_LAUNCH_CHECK();
 }
 
@@ -855,20 +935,28 @@ FERRIS_API int ferris_paged_attention_tiled(const void* q, int ldq, void* out, i
                                             const int* token_seq, const int* positions, int tokens, int nh, int nkv,
                                             int d, int dv, int page_size, int window, float scale, const float* slopes,
                                             const float* log_r1, const float* log_r2, const float* sink, int v_stride,
-                                            void* stream) {
+                                            const void* pool_k, const void* pool_v, const int* pool_tables,
+                                            int pool_max_blocks, int pool_every, void* stream) {
     if (tokens <= 0) return FERRIS_OK;
     if ((log_r1 == nullptr) != (log_r2 == nullptr) || (slopes && log_r1)) FERRIS_REFUSE("tiled attention: one kind of distance penalty, with all its numbers");
     if (v_stride < 0 || (v_stride > 0 && v_stride < dv)) FERRIS_REFUSE("tiled attention: value rows %d apart hold no %d values", v_stride, dv);
     const ScoreTerms st = {slopes, log_r1, log_r2, sink, v_stride};
+    const PooledKeys pk = {pool_k, pool_v, pool_tables, pool_max_blocks, pool_every};
+    if (int rc = check_pooled(pk, window, st)) return rc;
     if (dtype != FERRIS_F32 && dtype != FERRIS_BF16) FERRIS_REFUSE("attention: unknown dtype %d", dtype);
     if (page_size <= 0 || max_blocks <= 0) FERRIS_REFUSE("attention: page_size=%d max_blocks=%d", page_size, max_blocks);
     if (!tiled_takes(dtype, nh, nkv, d, dv)) FERRIS_REFUSE("tiled attention: %d heads over %d kv heads of %d / %d are not taken", nh, nkv, d, dv);
     const size_t elt = dtype == FERRIS_F32 ? 4 : 2;
-    if ((((uintptr_t)q | (uintptr_t)k_cache | (uintptr_t)v_cache) & 15) != 0 || ((size_t)ldq * elt) % 16 != 0)
+    if ((((uintptr_t)q | (uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)pool_k | (uintptr_t)pool_v) & 15) != 0 || ((size_t)ldq * elt) % 16 != 0)
         FERRIS_REFUSE("tiled attention: rows must start on 16 bytes");
     if (nkv > 65535) FERRIS_REFUSE("attention: %d kv heads are more than one launch takes", nkv);
     cudaStream_t s = (cudaStream_t)stream;
-    if (dtype == FERRIS_F32)
-        return launch_tiled<float>(q, ldq, out, ldo, k_cache, v_cache, block_tables, max_blocks, token_seq, positions, tokens, nh, nkv, d, dv, page_size, window, scale, st, s);
-    return launch_tiled<bf16>(q, ldq, out, ldo, k_cache, v_cache, block_tables, max_blocks, token_seq, positions, tokens, nh, nkv, d, dv, page_size, window, scale, st, s);
+#define FERRIS_TILED(T, POOL)                                                                                             \
+    return launch_tiled<T, POOL>(q, ldq, out, ldo, k_cache, v_cache, block_tables, max_blocks, token_seq, positions, tokens, \
+                                 nh, nkv, d, dv, page_size, window, scale, st, pk, s)
+    if (dtype == FERRIS_F32) {
+        if (pk.every > 0) FERRIS_TILED(float, true); else FERRIS_TILED(float, false);
+    }
+    if (pk.every > 0) FERRIS_TILED(bf16, true); else FERRIS_TILED(bf16, false);
+#undef FERRIS_TILED
 }

@@ -823,3 +823,141 @@ FERRIS_API int ferris_scale(float* x, long long n, float scale, void* stream) {
     ferris_launch(scale_kernel, dim3((unsigned)(want < 148 * 16 ? want : 148 * 16)), dim3(threads), 0, (cudaStream_t)stream, x, n, scale);
     FERRIS_LAUNCH_CHECK();
 }
+
+// ---------------------------------------------------------------------------------------------
+// Embedding with a learned vector per position, into the fp32 residual stream: out[t] = table[ids[t]] + pos_table[positions[t]].
+// `rows` (may be null): the same rows in the activations' type, for layers whose products read the residual itself.
+// An id outside [0, vocab) or a position outside [0, max_pos) writes zeros and is reported as by embed_gather.
+// ---------------------------------------------------------------------------------------------
+template <typename T>
+__global__ void embed_positions_kernel(const T* __restrict__ table, const T* __restrict__ pos_table, const int* ids,
+                                       const int* positions, float* out, T* rows, int hidden, int vocab, int max_pos,
+                                       int* status) {
+    pdl_wait();
+    pdl_launch_dependents();
+    const int t = blockIdx.x;
+    const int id = ids[t], pos = positions[t];
+    const bool ok = id >= 0 && id < vocab && pos >= 0 && pos < max_pos;
+    if (!ok && threadIdx.x == 0 && status) atomicCAS(status, 0, t + 1);
+    const T* a = table + (size_t)(ok ? id : 0) * hidden;
+    const T* b = pos_table + (size_t)(ok ? pos : 0) * hidden;
+    float* o = out + (size_t)t * hidden;
+    for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
+        const float v = ok ? to_float(a[i]) + to_float(b[i]) : 0.0f;
+        o[i] = v;
+        if (rows) rows[(size_t)t * hidden + i] = from_float<T>(v);
+    }
+}
+
+FERRIS_API int ferris_embed_positions(const void* table, const void* pos_table, int dtype, const int* ids, const int* positions,
+                                      float* out, void* rows, int tokens, int hidden, int vocab, int max_pos, int* status,
+                                      void* stream) {
+    if (tokens <= 0) return FERRIS_OK;
+    if (hidden <= 0 || vocab <= 0 || max_pos <= 0) FERRIS_REFUSE("embed_positions: hidden=%d vocab=%d positions=%d", hidden, vocab, max_pos);
+    const int threads = hidden >= 1024 ? 256 : 128;
+    cudaStream_t s = (cudaStream_t)stream;
+    if (dtype == FERRIS_F32)
+        ferris_launch(embed_positions_kernel<float>, dim3(tokens), dim3(threads), 0, s, (const float*)table, (const float*)pos_table,
+                      ids, positions, out, (float*)rows, hidden, vocab, max_pos, status);
+    else if (dtype == FERRIS_BF16)
+        ferris_launch(embed_positions_kernel<bf16>, dim3(tokens), dim3(threads), 0, s, (const bf16*)table, (const bf16*)pos_table,
+                      ids, positions, out, (bf16*)rows, hidden, vocab, max_pos, status);
+    else
+        FERRIS_REFUSE("embed_positions: unknown dtype %d", dtype);
+    FERRIS_LAUNCH_CHECK();
+}
+
+// ---------------------------------------------------------------------------------------------
+// The norm on a sublayer's output: h[r] += rmsnorm(y[r]) * w, both fp32 (statistics and sum in fp32), and, where `rows` is
+// given, rows[r] = h[r] in bf16, which is what the next sublayer's products read.  A warp per row with the row in
+// registers where the row is aligned and at most 4,096 wide, a block per row otherwise.  Without y (null): the rows alone.
+// ---------------------------------------------------------------------------------------------
+template <int VEC>
+__global__ void __launch_bounds__(256) rmsnorm_add_rows_kernel(const float* y, const float* __restrict__ w, float* h, bf16* rows,
+                                                               int n_rows, int hidden, float eps) {
+    pdl_wait();
+    pdl_launch_dependents();
+    const int lane = threadIdx.x & 31;
+    const int r = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (r >= n_rows) return;
+    const float4* yr = reinterpret_cast<const float4*>(y + (size_t)r * hidden);
+    float4* hr = reinterpret_cast<float4*>(h + (size_t)r * hidden);
+    const int n4 = hidden >> 2;
+    float4 v[VEC], a[VEC];
+    float ss = 0.0f;
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) {
+        const int i = lane + 32 * j;
+        v[j] = i < n4 ? yr[i] : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        a[j] = i < n4 ? hr[i] : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    }
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) {
+        ss = fmaf(v[j].x, v[j].x, ss);
+        ss = fmaf(v[j].y, v[j].y, ss);
+        ss = fmaf(v[j].z, v[j].z, ss);
+        ss = fmaf(v[j].w, v[j].w, ss);
+    }
+    ss = warp_sum(ss);
+    const float inv = 1.0f / sqrtf(ss / (float)hidden + eps);
+    const float4* w4 = reinterpret_cast<const float4*>(w);
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) {
+        const int i = lane + 32 * j;
+        if (i < n4) {
+            const float4 g = w4[i];
+            float4 x = a[j];
+            x.x = fmaf(v[j].x * inv, g.x, x.x), x.y = fmaf(v[j].y * inv, g.y, x.y);
+            x.z = fmaf(v[j].z * inv, g.z, x.z), x.w = fmaf(v[j].w * inv, g.w, x.w);
+            hr[i] = x;
+            if (rows) store4(rows + (size_t)r * hidden + 4 * i, x.x, x.y, x.z, x.w);
+        }
+    }
+}
+
+__global__ void __launch_bounds__(512) rmsnorm_add_kernel(const float* y, const float* __restrict__ w, float* h, bf16* rows,
+                                                          int hidden, float eps) {
+    __shared__ float scratch[33];
+    pdl_wait();
+    pdl_launch_dependents();
+    const size_t at = (size_t)blockIdx.x * hidden;
+    float inv = 0.0f;
+    if (y) {
+        float ss = 0.0f;
+        for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
+            const float v = y[at + i];
+            ss = fmaf(v, v, ss);
+        }
+        inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)hidden + eps);
+    }
+    for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
+        float x = h[at + i];
+        if (y) {
+            x = fmaf(y[at + i] * inv, w[i], x);
+            h[at + i] = x;
+        }
+        if (rows) rows[at + i] = from_float<bf16>(x);
+    }
+}
+
+FERRIS_API int ferris_rmsnorm_add(const float* y, const float* w, float* h, void* rows, int n_rows, int hidden, float eps,
+                                  void* stream) {
+    if (n_rows <= 0) return FERRIS_OK;
+    if (hidden <= 0 || (y && !w)) FERRIS_REFUSE("norm + add: hidden=%d", hidden);
+    cudaStream_t s = (cudaStream_t)stream;
+    const bool aligned = (((uintptr_t)y | (uintptr_t)w | (uintptr_t)h | (uintptr_t)rows) & 15) == 0;
+    if (y && hidden % 4 == 0 && hidden <= 4096 && aligned) {
+        const int warps = n_rows >= 148 * 8 ? 8 : (n_rows >= 148 * 2 ? 2 : 1);  // few rows: spread over the SMs
+        const dim3 grid((n_rows + warps - 1) / warps), block(32 * warps);
+#define FERRIS_NORM_ADD(VEC) ferris_launch(rmsnorm_add_rows_kernel<VEC>, grid, block, 0, s, y, w, h, (bf16*)rows, n_rows, hidden, eps)
+        if (hidden <= 512) FERRIS_NORM_ADD(4);
+        else if (hidden <= 1024) FERRIS_NORM_ADD(8);
+        else if (hidden <= 2048) FERRIS_NORM_ADD(16);
+        else FERRIS_NORM_ADD(32);
+#undef FERRIS_NORM_ADD
+        FERRIS_LAUNCH_CHECK();
+    }
+    const int threads = hidden >= 2048 ? 512 : (hidden >= 512 ? 256 : 128);
+    ferris_launch(rmsnorm_add_kernel, dim3(n_rows), dim3(threads), 0, s, y, w, h, (bf16*)rows, hidden, eps);
+    FERRIS_LAUNCH_CHECK();
+}

@@ -689,6 +689,9 @@ struct PTParams {
     // Written by the launch before this one, so never read through a read-only path.
     const int* tile_expert = nullptr;
     int expert_rows = 0;
+    // SwiGLU mode: a factor per row (written by an earlier launch) on both accumulators ahead of the activation: the
+    // product of a row that is multiplied by it.  Null: none.
+    const float* row_scale = nullptr;
 };
 
 // The first weight row of the expert that token tile `mt` meets (0 without experts), or -1 to skip the tile.
@@ -772,6 +775,8 @@ __device__ __forceinline__ void pt_epilogue_tile(const PTParams& p, const CUtens
                                                  int quarter, int half, int lane, int t, uint8_t* out_stage) {
     constexpr int ACCS = MODE == SWIGLU_BF16 ? 2 : 1;
     const int cols = p.bn;  // output columns of this tile
+    float row_scale = 1.0f;
+    if (MODE == SWIGLU_BF16 && p.row_scale && t < p.T) row_scale = *(reinterpret_cast<const volatile float*>(p.row_scale) + t);
     for (int c0 = half * 32; c0 < cols; c0 += 64) {
         uint32_t ra[32], rb[32];
         tmem_load_32x32(d0 + c0, ra);
@@ -814,7 +819,11 @@ __device__ __forceinline__ void pt_epilogue_tile(const PTParams& p, const CUtens
             for (int c = 0; c < 32; c += 2) {
                 float v0, v1;
                 if (MODE == SWIGLU_BF16) {
-                    if (p.act.kind) {  // another gated activation than SiLU
+                    if (p.row_scale) {
+                        const int kind = p.act.kind ? p.act.kind - FERRIS_EPILOGUE_GATED : FERRIS_GATED_SILU;
+                        v0 = ferris_gated_act(row_scale * __uint_as_float(ra[c]), row_scale * __uint_as_float(rb[c]), kind, p.act.a);
+                        v1 = ferris_gated_act(row_scale * __uint_as_float(ra[c + 1]), row_scale * __uint_as_float(rb[c + 1]), kind, p.act.a);
+                    } else if (p.act.kind) {  // another gated activation than SiLU
                         v0 = ferris_gated_act(__uint_as_float(ra[c]), __uint_as_float(rb[c]), p.act.kind - FERRIS_EPILOGUE_GATED, p.act.a);
                         v1 = ferris_gated_act(__uint_as_float(ra[c + 1]), __uint_as_float(rb[c + 1]), p.act.kind - FERRIS_EPILOGUE_GATED, p.act.a);
                     } else {
@@ -1554,7 +1563,8 @@ static FerrisEpilogueAct g_launch_act = {0, 0.0f, 0.0f};
 // The persistent token-major kernel for a long step (T >= 128 tokens; output rows aligned for 16-byte stores).
 static int run_tokens_m(const void* x, const void* w, const float* bias, void* out, int mode, int T, int N, int K,
                         int ldx, int ldw, int ldo, int rows_w, int up_row_offset, const RopeEpilogue* rope,
-                        cudaStream_t s, const int* tile_expert = nullptr, int expert_rows = 0) {
+                        cudaStream_t s, const int* tile_expert = nullptr, int expert_rows = 0,
+                        const float* row_scale = nullptr) {
     const int accs = mode == SWIGLU_BF16 ? 2 : 1;
     const int elt = (mode == STORE_F32 || mode == ACCUM_F32) ? 4 : 2;
     sm_count();
@@ -1593,6 +1603,7 @@ static int run_tokens_m(const void* x, const void* w, const float* bias, void* o
     q.rope = rope ? *rope : RopeEpilogue{};
     q.tile_expert = tile_expert;
     q.expert_rows = expert_rows;
+    q.row_scale = row_scale;
     CUtensorMap mx, mw;
     int rc = ferris_make_tensor_map_2d(&mx, x, (uint64_t)T, (uint64_t)K, (uint64_t)ldx, PT_BLOCK_M, BLOCK_K);
     if (rc != FERRIS_OK) return rc;
@@ -1619,10 +1630,11 @@ static int run_tokens_m(const void* x, const void* w, const float* bias, void* o
 // One product per group of token tiles (see PTParams::tile_expert): x holds `rows` rows (a multiple of 128), sorted by
 // expert with every expert's rows filled up to whole tiles of 128; w holds the experts' matrices stacked, expert_rows
 // rows each, of which the first N (and, in SwiGLU mode, the N from up_row_offset on) meet the rows of their tiles.
-// Modes: 0 bf16 store, 1 fp32 store, 3 SwiGLU from two accumulators.  A tile whose entry is negative is skipped.
+// Modes: 0 bf16 store, 1 fp32 store, 3 SwiGLU from two accumulators (with row_scale, fp32 [rows], both times the row's
+// factor first).  A tile whose entry is negative is skipped.
 FERRIS_API int ferris_gemm_grouped_tcgen05(const void* x, const void* w, void* out, int mode, int rows, int N, int K,
                                            int ldx, int ldw, int ldo, int experts, int expert_rows, int up_row_offset,
-                                           const int* tile_expert, void* stream) {
+                                           const int* tile_expert, const float* row_scale, void* stream) {
     if (rows <= 0 || N <= 0) return FERRIS_OK;
     if (rows % PT_BLOCK_M) FERRIS_REFUSE("grouped gemm: %d rows are no multiple of %d", rows, PT_BLOCK_M);
     if (K <= 0 || (K & 7) || (ldx & 7) || (ldw & 7) || ldx < K || ldw < K)
@@ -1630,6 +1642,7 @@ FERRIS_API int ferris_gemm_grouped_tcgen05(const void* x, const void* w, void* o
     if (((uintptr_t)x & 15) || ((uintptr_t)w & 15)) FERRIS_REFUSE("grouped gemm: operands must be 16-byte aligned");
     if (mode != STORE_BF16 && mode != STORE_F32 && mode != SWIGLU_BF16) FERRIS_REFUSE("grouped gemm: mode %d", mode);
     if (!tile_expert || experts <= 0 || expert_rows <= 0) FERRIS_REFUSE("grouped gemm: no experts");
+    if (row_scale && mode != SWIGLU_BF16) FERRIS_REFUSE("grouped gemm: a factor per row goes with mode %d", (int)SWIGLU_BF16);
     if ((mode == SWIGLU_BF16 ? up_row_offset + N : N) > expert_rows || up_row_offset < 0)
         FERRIS_REFUSE("grouped gemm: %d outputs (+%d) from %d rows an expert", N, up_row_offset, expert_rows);
     const int elt = mode == STORE_F32 ? 4 : 2;
@@ -1638,7 +1651,7 @@ FERRIS_API int ferris_gemm_grouped_tcgen05(const void* x, const void* w, void* o
     if (g_launch_act.kind && (g_launch_act.kind >= FERRIS_EPILOGUE_GATED) != (mode == SWIGLU_BF16))
         FERRIS_REFUSE("grouped gemm: activation %d does not go with mode %d", g_launch_act.kind, mode);
     return run_tokens_m(x, w, nullptr, out, mode, rows, N, K, ldx, ldw, ldo, experts * expert_rows, up_row_offset, nullptr,
-                        (cudaStream_t)stream, tile_expert, expert_rows);
+                        (cudaStream_t)stream, tile_expert, expert_rows, row_scale);
 }
 
 static int gemm_tcgen05_impl(const void* x, const void* w, const float* bias, void* out, int mode, int T, int N, int K,

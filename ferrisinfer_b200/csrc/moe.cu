@@ -14,6 +14,13 @@
 // the adding passes multiply the token's row by.  The experts' gated activation is one of the kinds of
 // ferris_gated_act.
 //
+// A third kind (`scored` = 2): s = sigmoid(z) of every output by itself, the `top` largest z are chosen (the sigmoid keeps
+// their order; the lowest index among equals) and the weights are their s as they are.
+//
+// Where a token's weight for an expert goes: onto the expert's result (o_e times weight_e, the default), or onto its INPUT
+// (`input_weights`): o_e = Wd_e (act(weight_e Wg_e y, weight_e Wu_e y)), which is the expert of weight_e y; both products are
+// linear in y, so the factor is applied to their fp32 sums, and the results are added unweighted.
+//
 // The experts' matrices lie stacked: gate and up as [experts, ff, width] each, down as [experts, width, ff].
 //
 // Three ways through the experts.  Token-major (a single choice; the 32-bit path of long steps): a block per (token, chosen expert) and
@@ -279,7 +286,7 @@ __global__ void __launch_bounds__(128) moe_router_kernel(const T* x, int ldx, co
     } else {
         __syncwarp();
     }
-    if (scored) {
+    if (scored == 1) {
         float* c = z + experts;
         float* gsc = c + experts;
         float mx = -INFINITY;
@@ -352,6 +359,7 @@ __global__ void __launch_bounds__(128) moe_router_kernel(const T* x, int ldx, co
         if (identity_w && lane == 0) identity_w[t] = idw;
         return;
     }
+    // (scored = 2 takes this path too: the choice by z, other weights)
     float chosen_z = 0.0f, first_z = 0.0f, sum = 0.0f;  // lane s keeps the s-th choice
     int chosen = 0;
     for (int s = 0; s < top; ++s) {
@@ -376,7 +384,7 @@ __global__ void __launch_bounds__(128) moe_router_kernel(const T* x, int ldx, co
     }
     if (lane < top) {
         ids[(size_t)t * top + lane] = chosen;
-        weights[(size_t)t * top + lane] = expf(chosen_z - first_z) / sum;
+        weights[(size_t)t * top + lane] = scored == 2 ? 1.0f / (1.0f + expf(-chosen_z)) : expf(chosen_z - first_z) / sum;
     }
 }
 
@@ -386,13 +394,14 @@ template <typename T>
 __global__ void __launch_bounds__(128) moe_gate_up_kernel(const T* x, int ldx, const T* __restrict__ gate,
                                                           const T* __restrict__ up, size_t expert_stride, const int* ids,
                                                           T* __restrict__ act, int width, int ff, int top, int slab,
-                                                          int experts, int act_kind, float act_limit) {
+                                                          int experts, int act_kind, float act_limit, const float* input_w) {
     extern __shared__ __align__(16) float xs[];  // the token's row
     pdl_wait();
     pdl_launch_dependents();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int pair = blockIdx.x, t = pair / top, e = ids[pair];
     if (e >= experts) return;  // an identity expert: nothing to form
+    const float w = input_w ? input_w[pair] : 1.0f;
     const T* xr = x + (size_t)t * ldx;
     stage_row(xs, xr, width, threadIdx.x, blockDim.x);
     __syncthreads();
@@ -408,14 +417,14 @@ __global__ void __launch_bounds__(128) moe_gate_up_kernel(const T* x, int ldx, c
             float d[4];
             dot_rows<4>(rows, xs, width, lane, vec, d);
             if (lane == 0) {
-                act[(size_t)pair * ff + j] = from_float<T>(ferris_gated_act(d[0], d[1], act_kind, act_limit));
-                act[(size_t)pair * ff + j + 4] = from_float<T>(ferris_gated_act(d[2], d[3], act_kind, act_limit));
+                act[(size_t)pair * ff + j] = from_float<T>(ferris_gated_act(w * d[0], w * d[1], act_kind, act_limit));
+                act[(size_t)pair * ff + j + 4] = from_float<T>(ferris_gated_act(w * d[2], w * d[3], act_kind, act_limit));
             }
         } else {
             const T* const rows[2] = {g + (size_t)j * width, u + (size_t)j * width};
             float d[2];
             dot_rows<2>(rows, xs, width, lane, vec, d);
-            if (lane == 0) act[(size_t)pair * ff + j] = from_float<T>(ferris_gated_act(d[0], d[1], act_kind, act_limit));
+            if (lane == 0) act[(size_t)pair * ff + j] = from_float<T>(ferris_gated_act(w * d[0], w * d[1], act_kind, act_limit));
         }
     }
 }
@@ -434,7 +443,7 @@ __global__ void __launch_bounds__(128) moe_down_kernel(const T* act, const T* __
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int t = blockIdx.x;
     const T* ar = act + (size_t)t * top * ff;
-    if (threadIdx.x < top) es[threadIdx.x] = ids[(size_t)t * top + threadIdx.x], ws[threadIdx.x] = weights[(size_t)t * top + threadIdx.x];
+    if (threadIdx.x < top) es[threadIdx.x] = ids[(size_t)t * top + threadIdx.x], ws[threadIdx.x] = weights ? weights[(size_t)t * top + threadIdx.x] : 1.0f;
     __syncthreads();
     for (int s = 0; s < top; ++s)  // the rows of identity experts were never written
         if (es[s] < experts) stage_row(as + (size_t)s * ff, ar + (size_t)s * ff, ff, threadIdx.x, blockDim.x);
@@ -500,7 +509,10 @@ __device__ __forceinline__ int pairs_of_expert(const int* ids, int pairs, int e,
 template <typename T, int M>
 __device__ __forceinline__ void gate_up_rows(const T* g, const T* u, const float* xs, int width, int ff, int j0, int j1,
                                              const int* pair, T* __restrict__ act, int lane, int warp, bool vec,
-                                             uint4* ring, int act_kind, float act_limit) {
+                                             uint4* ring, int act_kind, float act_limit, const float* input_w) {
+    float w[M];
+#pragma unroll
+    for (int m = 0; m < M; ++m) w[m] = input_w ? input_w[pair[m]] : 1.0f;
     for (int j = j0 + warp; j < j1; j += 2 * FEW_WARPS) {
         if (j + FEW_WARPS < j1) {
             const T* const rows[4] = {g + (size_t)j * width, u + (size_t)j * width, g + (size_t)(j + FEW_WARPS) * width,
@@ -510,8 +522,8 @@ __device__ __forceinline__ void gate_up_rows(const T* g, const T* u, const float
             if (lane == 0) {
 #pragma unroll
                 for (int m = 0; m < M; ++m) {
-                    act[(size_t)pair[m] * ff + j] = from_float<T>(ferris_gated_act(d[0][m], d[1][m], act_kind, act_limit));
-                    act[(size_t)pair[m] * ff + j + FEW_WARPS] = from_float<T>(ferris_gated_act(d[2][m], d[3][m], act_kind, act_limit));
+                    act[(size_t)pair[m] * ff + j] = from_float<T>(ferris_gated_act(w[m] * d[0][m], w[m] * d[1][m], act_kind, act_limit));
+                    act[(size_t)pair[m] * ff + j + FEW_WARPS] = from_float<T>(ferris_gated_act(w[m] * d[2][m], w[m] * d[3][m], act_kind, act_limit));
                 }
             }
         } else {
@@ -521,7 +533,7 @@ __device__ __forceinline__ void gate_up_rows(const T* g, const T* u, const float
             if (lane == 0) {
 #pragma unroll
                 for (int m = 0; m < M; ++m)
-                    act[(size_t)pair[m] * ff + j] = from_float<T>(ferris_gated_act(d[0][m], d[1][m], act_kind, act_limit));
+                    act[(size_t)pair[m] * ff + j] = from_float<T>(ferris_gated_act(w[m] * d[0][m], w[m] * d[1][m], act_kind, act_limit));
             }
         }
     }
@@ -531,7 +543,7 @@ template <typename T>
 __global__ void __launch_bounds__(32 * FEW_WARPS) moe_gate_up_few_kernel(const T* x, int ldx, const T* __restrict__ gate,
                                                               const T* __restrict__ up, size_t expert_stride, const int* ids,
                                                               T* __restrict__ act, int width, int ff, int pairs, int top,
-                                                              int slab, int act_kind, float act_limit) {
+                                                              int slab, int act_kind, float act_limit, const float* input_w) {
     extern __shared__ __align__(16) float dyn[];  // every warp's slots for weights in flight, then MOE_FEW_ROWS token rows
     __shared__ int list[MOE_FEW_MAX_PAIRS];
     __shared__ int count;
@@ -555,10 +567,10 @@ __global__ void __launch_bounds__(32 * FEW_WARPS) moe_gate_up_few_kernel(const T
         __syncthreads();
         const int* pair = list + first;
         switch (m) {
-            case 1: gate_up_rows<T, 1>(g, u, xs, width, ff, j0, j1, pair, act, lane, warp, vec, ring, act_kind, act_limit); break;
-            case 2: gate_up_rows<T, 2>(g, u, xs, width, ff, j0, j1, pair, act, lane, warp, vec, ring, act_kind, act_limit); break;
-            case 3: gate_up_rows<T, 3>(g, u, xs, width, ff, j0, j1, pair, act, lane, warp, vec, ring, act_kind, act_limit); break;
-            default: gate_up_rows<T, 4>(g, u, xs, width, ff, j0, j1, pair, act, lane, warp, vec, ring, act_kind, act_limit); break;
+            case 1: gate_up_rows<T, 1>(g, u, xs, width, ff, j0, j1, pair, act, lane, warp, vec, ring, act_kind, act_limit, input_w); break;
+            case 2: gate_up_rows<T, 2>(g, u, xs, width, ff, j0, j1, pair, act, lane, warp, vec, ring, act_kind, act_limit, input_w); break;
+            case 3: gate_up_rows<T, 3>(g, u, xs, width, ff, j0, j1, pair, act, lane, warp, vec, ring, act_kind, act_limit, input_w); break;
+            default: gate_up_rows<T, 4>(g, u, xs, width, ff, j0, j1, pair, act, lane, warp, vec, ring, act_kind, act_limit, input_w); break;
         }
     }
 }
@@ -627,14 +639,19 @@ __global__ void __launch_bounds__(32 * FEW_WARPS) moe_down_few_kernel(const T* a
 // One block.  pos[pair] = the row of pair (t, s) in the sorted order; row_token[row] = its token, or -1 for a row that
 // only fills a tile up; tile_expert[tile] = the expert of the tile's rows, or -1 beyond the last row.
 constexpr int MOE_TILE = 128;
+// row_scale (may be null): the pair's weight at its row, 0 at the rows that only fill up.
 __global__ void __launch_bounds__(1024) moe_sort_kernel(const int* ids, int* pos, int* row_token, int* tile_expert,
-                                                        int pairs, int top, int experts, int max_rows, int with_weights) {
+                                                        int pairs, int top, int experts, int max_rows, int with_weights,
+                                                        const float* weights, float* row_scale) {
     __shared__ int count[MOE_MAX_EXPERTS];
     __shared__ int first[MOE_MAX_EXPERTS + 1];
     pdl_wait();
     pdl_launch_dependents();
     for (int e = threadIdx.x; e < experts; e += blockDim.x) count[e] = 0;
-    for (int r = threadIdx.x; r < max_rows; r += blockDim.x) row_token[r] = -1;
+    for (int r = threadIdx.x; r < max_rows; r += blockDim.x) {
+        row_token[r] = -1;
+        if (row_scale) row_scale[r] = 0.0f;
+    }
     __syncthreads();
     for (int i = threadIdx.x; i < pairs; i += blockDim.x) pos[i] = atomicAdd(&count[ids[i]], 1);  // its rank, for now
     __syncthreads();
@@ -651,6 +668,7 @@ __global__ void __launch_bounds__(1024) moe_sort_kernel(const int* ids, int* pos
         const int row = first[ids[i]] + pos[i];
         pos[i] = row;
         row_token[row] = i / top;
+        if (row_scale) row_scale[row] = weights[i];
     }
     for (int tile = threadIdx.x; tile < max_rows / MOE_TILE; tile += blockDim.x) {
         const int row = tile * MOE_TILE;
@@ -697,7 +715,7 @@ __global__ void __launch_bounds__(256) moe_combine_kernel(const float* y, int ld
         float4 sum = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
         for (int s = 0; s < top; ++s) {
             if (ids && ids[(size_t)t * top + s] >= experts) continue;  // an identity expert: its row was never written
-            const float w = weights[(size_t)t * top + s];
+            const float w = weights ? weights[(size_t)t * top + s] : 1.0f;
             const size_t row = pos ? (size_t)pos[(size_t)t * top + s] : (size_t)t * top + s;
             const float4 v = reinterpret_cast<const float4*>(y + row * ldy)[i];
             sum.x = fmaf(w, v.x, sum.x), sum.y = fmaf(w, v.y, sum.y), sum.z = fmaf(w, v.z, sum.z), sum.w = fmaf(w, v.w, sum.w);
@@ -718,7 +736,7 @@ __global__ void __launch_bounds__(256) moe_combine_kernel(const float* y, int ld
 extern "C" void ferris_gemm_set_gated_activation(int kind, float limit);
 extern "C" int ferris_gemm_grouped_tcgen05(const void* x, const void* w, void* out, int mode, int rows, int N, int K,
                                            int ldx, int ldw, int ldo, int experts, int expert_rows, int up_row_offset,
-                                           const int* tile_expert, void* stream);
+                                           const int* tile_expert, const float* row_scale, void* stream);
 
 // Rows of the sorted order that `tokens` tokens choosing `top` of `experts` can need at most (whole tiles of 128).
 FERRIS_API int ferris_moe_sorted_rows(int tokens, int top, int experts) {
@@ -733,12 +751,12 @@ FERRIS_API int ferris_moe_sorted_rows(int tokens, int top, int experts) {
 // tile_expert int32 [rows / 128], xs bf16 [rows, width], act bf16 [rows, ff], y fp32 [rows, width].
 // identity_w (may be null): fp32 [tokens]; with it, ids may hold `experts` (an identity expert: the pair meets no weights)
 // and h also gets identity_w[t] x[t]; the scratch is then sized for experts + 1.  act_kind, act_limit: the gated
-// activation (ferris_gated_act).
+// activation (ferris_gated_act).  row_scale: scratch, fp32 [rows], where the weights go onto the experts' inputs; else null.
 FERRIS_API int ferris_moe_experts_grouped(const void* x, int ldx, const void* gate_up, const void* down, const int* ids,
                                           const float* weights, float* h, int ldh, int tokens, int width, int ff, int top,
                                           int experts, int rows, int* pos, int* row_token, int* tile_expert, void* xs,
                                           void* act, float* y, int accumulate, int act_kind, float act_limit,
-                                          const float* identity_w, void* stream) {
+                                          const float* identity_w, float* row_scale, void* stream) {
     if (tokens <= 0) return FERRIS_OK;
     const int sorted = experts + (identity_w ? 1 : 0);  // the identity experts' pairs sort behind the last expert's
     if (experts <= 0 || sorted > MOE_MAX_EXPERTS || top <= 0 || top > MOE_MAX_TOP)
@@ -748,27 +766,27 @@ FERRIS_API int ferris_moe_experts_grouped(const void* x, int ldx, const void* ga
         FERRIS_REFUSE("experts: width %d, ff %d and the rows must be multiples of 8 elements and start on 16 bytes", width, ff);
     cudaStream_t s = (cudaStream_t)stream;
     ferris_launch(moe_sort_kernel, dim3(1), dim3(1024), 0, s, ids, pos, row_token, tile_expert, tokens * top, top, sorted,
-                  rows, experts);
+                  rows, experts, weights, row_scale);
     const size_t n16 = (size_t)rows * (width / 8);
     const size_t want = (n16 + 255) / 256;
     ferris_launch(moe_gather_kernel, dim3((unsigned)(want < 148 * 16 ? want : 148 * 16)), dim3(256), 0, s, (const uint4*)x,
                   ldx / 8, (const int*)row_token, (uint4*)xs, rows, width / 8);
     ferris_gemm_set_gated_activation(act_kind, act_limit);  // taken by the product launched next
     int rc = ferris_gemm_grouped_tcgen05(xs, gate_up, act, 3, rows, ff, width, width, width, ff, experts, 2 * ff, ff,
-                                         tile_expert, stream);
+                                         tile_expert, row_scale, stream);
     ferris_gemm_set_gated_activation(0, 0.0f);
     if (rc != FERRIS_OK) return rc;
-    rc = ferris_gemm_grouped_tcgen05(act, down, y, 1, rows, width, ff, ff, ff, width, experts, width, 0, tile_expert, stream);
+    rc = ferris_gemm_grouped_tcgen05(act, down, y, 1, rows, width, ff, ff, ff, width, experts, width, 0, tile_expert, nullptr, stream);
     if (rc != FERRIS_OK) return rc;
     const size_t n4 = (size_t)tokens * (width / 4);
     const size_t want4 = (n4 + 255) / 256;
     ferris_launch(moe_combine_kernel<bf16>, dim3((unsigned)(want4 < 148 * 16 ? want4 : 148 * 16)), dim3(256), 0, s, (const float*)y,
-                  width, (const int*)pos, weights, h, ldh, tokens, width / 4, top, accumulate,
+                  width, (const int*)pos, row_scale ? (const float*)nullptr : weights, h, ldh, tokens, width / 4, top, accumulate,
                   identity_w ? ids : (const int*)nullptr, experts, (const bf16*)x, ldx, identity_w);
     FERRIS_LAUNCH_CHECK();
 }
 
-// scored = 0: the `top` largest logits (+ bias), softmax over those.  scored = 1: see the head of this file; `bias` is
+// scored = 2: the `top` largest logits (+ bias), weights = their sigmoids.  scored = 0: the `top` largest logits (+ bias), softmax over those.  scored = 1: see the head of this file; `bias` is
 // unused, `correction` fp32 [experts] (may be null), with_weights = the experts that have weights (the router outputs
 // from there on are identity experts, handed on as the index with_weights), identity_w fp32 [tokens] (the sum of a token's
 // identity weights; may be null when with_weights == experts).
@@ -780,7 +798,8 @@ FERRIS_API int ferris_moe_router(const void* x, int ldx, int dtype, const void* 
     if (experts <= 0 || experts > MOE_MAX_EXPERTS || top <= 0 || top > experts || top > MOE_MAX_TOP || width <= 0)
         FERRIS_REFUSE("router: %d experts (at most %d), %d chosen (at most %d), width %d", experts, MOE_MAX_EXPERTS, top,
                       MOE_MAX_TOP, width);
-    if (scored) {
+    if (scored < 0 || scored > 2) FERRIS_REFUSE("router: unknown kind %d", scored);
+    if (scored == 1) {
         if (groups <= 0 || experts % groups || keep < 1 || keep > groups || top > keep * (experts / groups))
             FERRIS_REFUSE("router: %d outputs in %d groups of which %d stay, %d chosen", experts, groups, keep, top);
         if (with_weights < 0 || with_weights > experts || (with_weights < experts && !identity_w))
@@ -814,13 +833,16 @@ FERRIS_API int ferris_moe_router(const void* x, int ldx, int dtype, const void* 
 // weights fp32 [tokens, top]; act [tokens x top, ff] (scratch, the activations' type); h fp32 rows ldh apart.
 // With y (scratch, fp32 [tokens x top, width]), `experts` and few enough tokens the weights are read once per expert
 // (the expert-major kernels for few tokens and the adding pass); the sums are the same bit for bit either way.
+// input_weights: a token's weight for an expert goes onto the expert's input instead of its result.
 FERRIS_API int ferris_moe_experts_token_major(const void* x, int ldx, int dtype, const void* gate, const void* up,
                                               long long gate_up_stride, const void* down, const int* ids,
                                               const float* weights, void* act, float* h,
                                               int ldh, int tokens, int width, int ff, int top, int accumulate,
                                               float* y, int experts, int act_kind, float act_limit,
-                                              const float* identity_w, void* stream) {
+                                              const float* identity_w, int input_weights, void* stream) {
     if (tokens <= 0) return FERRIS_OK;
+    const float* input_w = input_weights ? weights : nullptr;  // the weights go onto one side of the experts or the other
+    const float* output_w = input_weights ? nullptr : weights;
     if (experts <= 0) FERRIS_REFUSE("experts: %d experts", experts);
     if (act_kind < 0 || act_kind > 2) FERRIS_REFUSE("experts: unknown activation %d", act_kind);
     if (width <= 0 || ff <= 0 || top <= 0 || top > MOE_MAX_TOP) FERRIS_REFUSE("experts: width %d, ff %d, %d chosen", width, ff, top);
@@ -849,7 +871,7 @@ FERRIS_API int ferris_moe_experts_token_major(const void* x, int ldx, int dtype,
         if ((rc = ferris_allow_dynamic_smem((const void*)moe_down_few_kernel<T>, few_down)) != FERRIS_OK) return rc;      \
         ferris_launch(moe_gate_up_few_kernel<T>, grid_up, dim3(32 * FEW_WARPS), few_up, s, (const T*)x, ldx, (const T*)gate,         \
                       (const T*)up, (size_t)gate_up_stride, ids, (T*)act, width, ff, pairs, top, slab_up, act_kind,    \
-                      act_limit);                                                                                         \
+                      act_limit, input_w);                                                                                         \
         ferris_launch(moe_down_few_kernel<T>, grid_down, dim3(32 * FEW_WARPS), few_down, s, (const T*)act, (const T*)down, ids, y,   \
                       width, ff, pairs, slab_down);                                                                       \
     } while (0)
@@ -863,11 +885,11 @@ FERRIS_API int ferris_moe_experts_token_major(const void* x, int ldx, int dtype,
         const int* skip = identity_w ? ids : (const int*)nullptr;
         if (dtype == FERRIS_F32)
             ferris_launch(moe_combine_kernel<float>, dim3((unsigned)(want4 < 148 * 16 ? want4 : 148 * 16)), dim3(256), 0, s,
-                          (const float*)y, width, (const int*)nullptr, weights, h, ldh, tokens, width / 4, top, accumulate,
+                          (const float*)y, width, (const int*)nullptr, output_w, h, ldh, tokens, width / 4, top, accumulate,
                           skip, experts, (const float*)x, ldx, identity_w);
         else
             ferris_launch(moe_combine_kernel<bf16>, dim3((unsigned)(want4 < 148 * 16 ? want4 : 148 * 16)), dim3(256), 0, s,
-                          (const float*)y, width, (const int*)nullptr, weights, h, ldh, tokens, width / 4, top, accumulate,
+                          (const float*)y, width, (const int*)nullptr, output_w, h, ldh, tokens, width / 4, top, accumulate,
                           skip, experts, (const bf16*)x, ldx, identity_w);
         FERRIS_LAUNCH_CHECK();
     }
@@ -893,8 +915,8 @@ FERRIS_API int ferris_moe_experts_token_major(const void* x, int ldx, int dtype,
         if ((rc = ferris_allow_dynamic_smem((const void*)moe_down_kernel<T>, smem_down)) != FERRIS_OK) return rc;         \
         ferris_launch(moe_gate_up_kernel<T>, dim3(grid_up.x, grid_up.y, 1), dim3(128), smem_up, s, (const T*)x, ldx,      \
                       (const T*)gate, (const T*)up, (size_t)gate_up_stride, ids, (T*)act, width, ff, top, slab_up,      \
-                      experts, act_kind, act_limit);                                                                      \
-        ferris_launch(moe_down_kernel<T>, grid_down, dim3(128), smem_down, s, (const T*)act, (const T*)down, ids, weights, \
+                      experts, act_kind, act_limit, input_w);                                                                      \
+        ferris_launch(moe_down_kernel<T>, grid_down, dim3(128), smem_down, s, (const T*)act, (const T*)down, ids, output_w, \
                       h, ldh, width, ff, top, slab_down, accumulate, experts, (const T*)x, ldx, identity_w);              \
     } while (0)
     if (dtype == FERRIS_F32)

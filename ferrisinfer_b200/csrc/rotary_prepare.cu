@@ -17,6 +17,13 @@
 // reduction, and every thread loads, norms, rotates and stores two neighbouring elements at a time (in the
 // interleaved layout a pair that rotates together is one such load).  The general one takes every other geometry
 // element by element.
+//
+// Two things may ride along (PrepareExtras).  Value mixing: a layer stores (1 - lambda) v + lambda v1 as its values, v1
+// being what another layer projected for the same token in this pass; that layer leaves its rows in a buffer on its
+// way.  Pooled blocks: a cache of means, one row for every `pool` consecutive positions; in a step of single tokens the
+// block of the token that completes such a run reads the run's keys and values from the pages and writes their mean.
+// Steps that bring portions of prompts do the same in a launch of its own behind this one (a run's tokens then lie in
+// several blocks of the grid): pool_blocks_kernel.
 #include <math.h>
 #include <stdint.h>
 
@@ -24,12 +31,70 @@
 
 namespace {
 
+struct PrepareExtras {
+    void* first;            // the rows that values are mixed with, [tokens, nkv * dv] (null: nothing is mixed)
+    const float* lambda;    // one number on the device; null: this layer's values are copied INTO `first`
+    const int* pool_slots;  // [tokens]: the pooled row that the token completes, or < 0 (null: no pooling here)
+    void* pool_k;           // [pages, nkv, page_size, d] and [.., dv]: the pooled rows
+    void* pool_v;
+    int pool;               // positions to a pooled row
+    const int* tables;      // block tables of the unpooled pages, [requests, max_blocks]
+    const int* token_seq;
+    int max_blocks;
+};
+
+// The pooled row `slot` = the means of the keys and of the values of positions pos - pool + 1 .. pos, as the pages hold
+// them: fp32 sums in the order of the positions, one division, one rounding.  Elements `first`, `first + step`, ... of
+// the nkv heads' keys and then of their values.
+template <typename T>
+__device__ __forceinline__ void pool_run(const T* k_cache, const T* v_cache, const int* table, T* pool_k, T* pool_v, int slot,
+                                         int pos, int pool, int nkv, int d, int dv, int page_size, int first, int step) {
+    const int nk = nkv * d, total = nk + nkv * dv;
+    const int ppage = slot / page_size, pin = slot % page_size;
+    for (int e = first; e < total; e += step) {
+        const bool key = e < nk;
+        const int x = key ? e : e - nk, width = key ? d : dv;
+        const int head = x / width, i = x - head * width;
+        const T* base = key ? k_cache : v_cache;
+        float sum = 0.0f;
+        int j = pos - pool + 1;
+        while (j <= pos) {  // page by page
+            const int in_page = j % page_size;
+            const int n = min(page_size - in_page, pos - j + 1);
+            const int page = table[j / page_size];
+            if (page < 0) return;  // never: a run's pages stay until it is complete
+            const T* src = base + (((size_t)page * nkv + head) * page_size + in_page) * width + i;
+#pragma unroll 4
+            for (int r = 0; r < n; ++r) sum += to_float(src[(size_t)r * width]);
+            j += n;
+        }
+        T* dst = (key ? pool_k : pool_v) + (((size_t)ppage * nkv + head) * page_size + pin) * width + i;
+        *dst = from_float<T>(sum / (float)pool);
+    }
+}
+
+// The pooled rows that the tokens of a step complete, behind the launch that wrote the step's keys and values.
+template <typename T>
+__global__ void __launch_bounds__(128) pool_blocks_kernel(const T* k_cache, const T* v_cache, T* pool_k, T* pool_v,
+                                                          const int* __restrict__ tables, int max_blocks,
+                                                          const int* __restrict__ token_seq, const int* __restrict__ positions,
+                                                          const int* __restrict__ pool_slots, int tokens, int pool, int nkv,
+                                                          int d, int dv, int page_size) {
+    pdl_wait();
+    pdl_launch_dependents();
+    const int t = blockIdx.x;
+    const int slot = pool_slots[t];
+    if (slot < 0) return;
+    pool_run<T>(k_cache, v_cache, tables + (size_t)token_seq[t] * max_blocks, pool_k, pool_v, slot, positions[t], pool, nkv, d,
+                dv, page_size, blockIdx.y * blockDim.x + threadIdx.x, gridDim.y * blockDim.x);
+}
+
 template <typename T>
 __global__ void __launch_bounds__(128) qk_norm_rotary_cache_write_kernel(
     T* qkv, int ld, const int* __restrict__ positions, const int* __restrict__ slot_mapping, T* __restrict__ k_cache,
     T* __restrict__ v_cache, int nh, int nkv, int d, int dv, int page_size, const float* __restrict__ q_weight,
     const float* __restrict__ k_weight, float eps, const float* __restrict__ freq, int rotary, int interleaved, float mag,
-    int values_from_keys, int write_kv) {
+    int values_from_keys, int write_kv, const PrepareExtras ex) {
     __shared__ float scratch[33];
     pdl_wait();
     pdl_launch_dependents();
@@ -59,9 +124,18 @@ __global__ void __launch_bounds__(128) qk_norm_rotary_cache_write_kernel(
     const int in_page = slot >= 0 ? slot % page_size : 0;
     if (slot >= 0) {  // the values first: where they are the keys as projected, before anything touches those
         const T* vrow = values_from_keys ? row + nq : row + nq + nk;
+        T* mixed = reinterpret_cast<T*>(ex.first) + (size_t)t * nkv * dv;
+        const float lam = ex.first && ex.lambda ? *ex.lambda : 0.0f;
         for (int e = threadIdx.x; e < nkv * dv; e += blockDim.x) {
             const int h = e / dv, i = e % dv;
-            v_cache[(((size_t)page * nkv + h) * page_size + in_page) * dv + i] = vrow[e];
+            T v = vrow[e];
+            if (ex.first) {
+                if (ex.lambda)
+                    v = from_float<T>(fmaf(lam, to_float(mixed[e]), (1.0f - lam) * to_float(v)));
+                else
+                    mixed[e] = v;
+            }
+            v_cache[(((size_t)page * nkv + h) * page_size + in_page) * dv + i] = v;
         }
     }
     const int half = rotary >> 1;
@@ -95,6 +169,11 @@ __global__ void __launch_bounds__(128) qk_norm_rotary_cache_write_kernel(
         s *= mag, c *= mag;
         dst[i] = from_float<T>(u * c - v * s);
         dst[i + partner] = from_float<T>(v * c + u * s);
+    }
+    if (ex.pool_slots && slot >= 0 && ex.pool_slots[t] >= 0) {
+        __syncthreads();  // the token's own key and value are in their page
+        pool_run<T>(k_cache, v_cache, ex.tables + (size_t)ex.token_seq[t] * ex.max_blocks, reinterpret_cast<T*>(ex.pool_k),
+                    reinterpret_cast<T*>(ex.pool_v), ex.pool_slots[t], pos, ex.pool, nkv, d, dv, page_size, threadIdx.x, blockDim.x);
     }
 }
 
@@ -130,7 +209,7 @@ __global__ void __launch_bounds__(256) qk_norm_rotary_cache_write_paired_kernel(
     T* qkv, int ld, const int* __restrict__ positions, const int* __restrict__ slot_mapping, T* __restrict__ k_cache,
     T* __restrict__ v_cache, int nh, int nkv, int d, int dv, int page_size, const float* __restrict__ q_weight,
     const float* __restrict__ k_weight, float eps, const float* __restrict__ freq, int rotary, float mag,
-    int values_from_keys, int write_kv) {
+    int values_from_keys, int write_kv, const PrepareExtras ex) {
     extern __shared__ float cs[];
     __shared__ float scratch[66];
     pdl_wait();
@@ -164,9 +243,19 @@ __global__ void __launch_bounds__(256) qk_norm_rotary_cache_write_paired_kernel(
     const int in_page = slot >= 0 ? slot % page_size : 0;
     if (slot >= 0) {
         const T* vrow = values_from_keys ? row + nq : row + nq + nk;
+        T* mixed = reinterpret_cast<T*>(ex.first) + (size_t)t * nkv * dv;
+        const float lam = ex.first && ex.lambda ? *ex.lambda : 0.0f;
         for (int e = 2 * threadIdx.x; e < nkv * dv; e += 2 * blockDim.x) {
             const int h = e / dv, i = e - h * dv;
-            const float2 v = load2(vrow + e);
+            float2 v = load2(vrow + e);
+            if (ex.first) {
+                if (ex.lambda) {
+                    const float2 f = load2(mixed + e);
+                    v.x = fmaf(lam, f.x, (1.0f - lam) * v.x), v.y = fmaf(lam, f.y, (1.0f - lam) * v.y);
+                } else {
+                    store2(mixed + e, v.x, v.y);
+                }
+            }
             store2(v_cache + (((size_t)page * nkv + h) * page_size + in_page) * dv + i, v.x, v.y);
         }
     }
@@ -200,6 +289,11 @@ __global__ void __launch_bounds__(256) qk_norm_rotary_cache_write_paired_kernel(
             dst[j] = from_float<T>(u * c - v * s);
             dst[j + half] = from_float<T>(v * c + u * s);
         }
+    }
+    if (ex.pool_slots && slot >= 0 && ex.pool_slots[t] >= 0) {
+        __syncthreads();  // the token's own key and value are in their page
+        pool_run<T>(k_cache, v_cache, ex.tables + (size_t)ex.token_seq[t] * ex.max_blocks, reinterpret_cast<T*>(ex.pool_k),
+                    reinterpret_cast<T*>(ex.pool_v), ex.pool_slots[t], pos, ex.pool, nkv, d, dv, page_size, threadIdx.x, blockDim.x);
     }
 }
 
@@ -286,8 +380,15 @@ FERRIS_API int ferris_qk_norm_rotary_cache_write(void* qkv, int ld, int dtype, c
                                                  int nkv, int d, int dv, int page_size, const float* q_weight,
                                                  const float* k_weight, float eps, const float* freq, int rotary,
                                                  int interleaved, float mag, int values_from_keys, int write_kv,
-                                                 void* stream) {
+                                                 void* first_values, const float* mix_lambda, const int* pool_slots,
+                                                 void* pool_k, void* pool_v, int pool, const int* tables, int max_blocks,
+                                                 const int* token_seq, void* stream) {
     if (tokens <= 0) return FERRIS_OK;
+    if (mix_lambda && !first_values) FERRIS_REFUSE("qk norm + rotation: nothing to mix the values with");
+    if (first_values && !write_kv) FERRIS_REFUSE("qk norm + rotation: values are mixed where they are stored");
+    if (pool_slots && (!write_kv || !pool_k || !pool_v || pool <= 0 || !tables || max_blocks <= 0 || !token_seq))
+        FERRIS_REFUSE("qk norm + rotation: pooled rows of %d positions want a cache, pooled pages and block tables", pool);
+    const PrepareExtras ex = {first_values, mix_lambda, pool_slots, pool_k, pool_v, pool, tables, token_seq, max_blocks};
     if (nh <= 0 || nkv <= 0 || d <= 0 || dv <= 0 || page_size <= 0)
         FERRIS_REFUSE("qk norm + rotation: nh=%d nkv=%d d=%d dv=%d page_size=%d", nh, nkv, d, dv, page_size);
     if (rotary < 0 || rotary > d || (rotary & 1) || (rotary > 0 && !freq))
@@ -298,14 +399,14 @@ FERRIS_API int ferris_qk_norm_rotary_cache_write(void* qkv, int ld, int dtype, c
     cudaStream_t s = (cudaStream_t)stream;
     const size_t elem = dtype == FERRIS_F32 ? 4 : 2;
     const bool paired = !((d | dv | ld) & 1) && (uintptr_t)qkv % (2 * elem) == 0 && (uintptr_t)k_cache % (2 * elem) == 0 &&
-                        (uintptr_t)v_cache % (2 * elem) == 0 && ((uintptr_t)q_weight | (uintptr_t)k_weight) % 8 == 0 &&
+                        (uintptr_t)v_cache % (2 * elem) == 0 && (uintptr_t)first_values % (2 * elem) == 0 && ((uintptr_t)q_weight | (uintptr_t)k_weight) % 8 == 0 &&
                         (dtype == FERRIS_F32 || dtype == FERRIS_BF16);
     if (paired) {
         const size_t smem = (size_t)rotary * sizeof(float);
 #define FERRIS_PAIRED(T, I)                                                                                              \
     ferris_launch(qk_norm_rotary_cache_write_paired_kernel<T, I>, dim3(tokens), dim3(256), smem, s, (T*)qkv, ld, positions, \
                   slot_mapping, (T*)k_cache, (T*)v_cache, nh, nkv, d, dv, page_size, q_weight, k_weight, eps, freq, rotary,  \
-                  mag, values_from_keys, write_kv)
+                  mag, values_from_keys, write_kv, ex)
         if (dtype == FERRIS_F32) {
             if (interleaved) FERRIS_PAIRED(float, true); else FERRIS_PAIRED(float, false);
         } else {
@@ -317,11 +418,11 @@ FERRIS_API int ferris_qk_norm_rotary_cache_write(void* qkv, int ld, int dtype, c
     if (dtype == FERRIS_F32)
         ferris_launch(qk_norm_rotary_cache_write_kernel<float>, dim3(tokens), dim3(128), 0, s, (float*)qkv, ld, positions,
                       slot_mapping, (float*)k_cache, (float*)v_cache, nh, nkv, d, dv, page_size, q_weight, k_weight, eps,
-                      freq, rotary, interleaved, mag, values_from_keys, write_kv);
+                      freq, rotary, interleaved, mag, values_from_keys, write_kv, ex);
     else if (dtype == FERRIS_BF16)
         ferris_launch(qk_norm_rotary_cache_write_kernel<bf16>, dim3(tokens), dim3(128), 0, s, (bf16*)qkv, ld, positions,
                       slot_mapping, (bf16*)k_cache, (bf16*)v_cache, nh, nkv, d, dv, page_size, q_weight, k_weight, eps,
-                      freq, rotary, interleaved, mag, values_from_keys, write_kv);
+                      freq, rotary, interleaved, mag, values_from_keys, write_kv, ex);
     else
         FERRIS_REFUSE("qk norm + rotation: unknown dtype %d", dtype);
     FERRIS_LAUNCH_CHECK();
@@ -355,5 +456,28 @@ FERRIS_API int ferris_qk_head_norm_rotary_cache_write(void* qkv, int ld, int dty
                       freq, rotary, interleaved, mag, write_kv, freq_lo);
     else
         FERRIS_REFUSE("head norm + rotation: unknown dtype %d", dtype);
+    FERRIS_LAUNCH_CHECK();
+}
+
+// Pooled rows of the tokens of a step whose slot in `pool_slots` is not negative: the means of the `pool` keys and values up
+// to the token's position, read from the pages that `tables` [requests, max_blocks] name.
+FERRIS_API int ferris_pool_blocks(const void* k_cache, const void* v_cache, void* pool_k, void* pool_v, int dtype,
+                                  const int* tables, int max_blocks, const int* token_seq, const int* positions,
+                                  const int* pool_slots, int tokens, int pool, int nkv, int d, int dv, int page_size,
+                                  void* stream) {
+    if (tokens <= 0) return FERRIS_OK;
+    if (pool <= 0 || nkv <= 0 || d <= 0 || dv <= 0 || page_size <= 0 || max_blocks <= 0)
+        FERRIS_REFUSE("pooled rows: pool=%d nkv=%d d=%d dv=%d page_size=%d max_blocks=%d", pool, nkv, d, dv, page_size, max_blocks);
+    const int slabs = (nkv * (d + dv) + 255) / 256;
+    const dim3 grid(tokens, slabs < 64 ? slabs : 64), block(128);
+    cudaStream_t s = (cudaStream_t)stream;
+    if (dtype == FERRIS_F32)
+        ferris_launch(pool_blocks_kernel<float>, grid, block, 0, s, (const float*)k_cache, (const float*)v_cache, (float*)pool_k,
+                      (float*)pool_v, tables, max_blocks, token_seq, positions, pool_slots, tokens, pool, nkv, d, dv, page_size);
+    else if (dtype == FERRIS_BF16)
+        ferris_launch(pool_blocks_kernel<bf16>, grid, block, 0, s, (const bf16*)k_cache, (const bf16*)v_cache, (bf16*)pool_k,
+                      (bf16*)pool_v, tables, max_blocks, token_seq, positions, pool_slots, tokens, pool, nkv, d, dv, page_size);
+    else
+        FERRIS_REFUSE("pooled rows: unknown dtype %d", dtype);
     FERRIS_LAUNCH_CHECK();
 }

@@ -13,7 +13,7 @@ tokenizer's business and not part of the engine: requests are token ids.
 
 from __future__ import annotations
 
-from dataclasses import dataclass, field
+from dataclasses import dataclass, field, replace
 from typing import Any, Optional, Sequence as Seq
 
 import torch
@@ -97,6 +97,9 @@ class Engine:
         else:
             raise ValueError("give a model folder, or a configuration and a seed")
         self.scheduler_config = scheduler or SchedulerConfig()
+        plan = self.model.plan
+        if plan.positions_bounded and self.scheduler_config.max_sequence_length > plan.max_positions:
+            self.scheduler_config = replace(self.scheduler_config, max_sequence_length=plan.max_positions)
         sc = self.scheduler_config
         needs = self.model.cache_needs()
         if num_pages is None:
@@ -123,7 +126,9 @@ class Engine:
 
         needs = [leaf for n in needs for leaf in leaf_needs(n)]
         item = 2 if self.dtype == torch.bfloat16 else 4
-        per_page = sum(n.num_kv_heads * (n.head_dim + n.value_dim) * page_size * item for n in needs if isinstance(n, PagedKV))
+        # (a need with a row for every so many tokens gets as many pages fewer)
+        per_page = sum(-(-n.num_kv_heads * (n.head_dim + n.value_dim) * page_size * item // n.stride) for n in needs
+                       if isinstance(n, PagedKV))
         if per_page == 0:
             return 1
         states = [n for n in needs if isinstance(n, FixedState)] + [RNG_NEED]

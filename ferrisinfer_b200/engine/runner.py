@@ -51,6 +51,7 @@ class _HostStep:
     max_q: int
     max_kv: int
     max_blocks: int
+    widths: list  # of each page group's block tables
     seqs: list
     n_want: int
     real: int = 0
@@ -97,6 +98,8 @@ class ModelRunner:
         self.device = torch.device(device)
         self.vocab_size = model.vocab_size
         self.max_model_len = int(max_model_len or model.plan.max_positions)
+        if model.plan.positions_bounded:
+            self.max_model_len = min(self.max_model_len, model.plan.max_positions)
         self.cache = CacheManager(model.cache_needs(), page_size, num_pages, max_requests, dtype=dtype,
                                   device=self.device, extra_states=extra_states, prefix_sharing=prefix_sharing,
                                   min_prefix_share_tokens=min_prefix_share_tokens, keep_finished=keep_finished)
@@ -406,18 +409,29 @@ class ModelRunner:
         while max_blocks < need_blocks:
             max_blocks *= 2
         max_blocks = min(max_blocks, max(need_blocks, -(-self.max_model_len // ps)))
-        group_arrays = []
+        group_arrays, widths = [], []
         for g in cache.groups:
-            tables = np.full((S, max_blocks), NO_PAGE, dtype=np.int32)
+            stride = g.need.stride  # a row for so many tokens: tables of as many blocks fewer
+            widths.append(-(-max_blocks // stride))
+            tables = np.full((S, widths[-1]), NO_PAGE, dtype=np.int32)
             for i, e in enumerate(entries):
                 arr = cache.block_table_array(e.request_id, g.gid)
                 tables[i, :arr.size] = arr
             if pad:
                 tables[real:, 0] = cache.padding_page(g.gid)
-            pages = tables[token_seq, positions // ps]
-            if (pages < 0).any():
-                raise CacheError(f"a token of the step has no page in group {g.gid}")
-            slot_mapping = (pages * ps + positions % ps).astype(np.int32)
+            if stride == 1:
+                pages = tables[token_seq, positions // ps]
+                if (pages < 0).any():
+                    raise CacheError(f"a token of the step has no page in group {g.gid}")
+                slot_mapping = (pages * ps + positions % ps).astype(np.int32)
+            else:  # the slot of the row that a token completes
+                slot_mapping = np.full(T, -1, dtype=np.int32)
+                at = np.nonzero((positions + 1) % stride == 0)[0]
+                row = positions[at] // stride
+                pages = tables[token_seq[at], row // ps]
+                if (pages < 0).any():
+                    raise CacheError(f"a row of the step has no page in group {g.gid}")
+                slot_mapping[at] = pages * ps + row % ps
             group_arrays.append((slot_mapping, tables))
         want = np.asarray(want_rows, dtype=np.int32)
         pieces = [token_ids, positions, token_seq, q_start, start_pos, state_slot, want]
@@ -425,7 +439,7 @@ class ModelRunner:
             pieces += [slot_mapping, tables.reshape(-1)]
         singles = [s.q_start for s in seqs if s.q_len == 1] if max_q > 1 else []
         pieces.append(np.asarray(singles, dtype=np.int32))
-        return _HostStep(pieces, T, S, max_q, max_kv, max_blocks, seqs, int(want.size), real)
+        return _HostStep(pieces, T, S, max_q, max_kv, max_blocks, widths, seqs, int(want.size), real)
 
     def _context(self, host: _HostStep, dev: torch.Tensor):
         views = []
@@ -435,7 +449,7 @@ class ModelRunner:
             off += p.size
         paged = {}
         for k, g in enumerate(self.cache.groups):
-            paged[g.gid] = PagedMeta(block_tables=views[self.N_FIXED + 2 * k + 1].view(host.S, host.max_blocks),
+            paged[g.gid] = PagedMeta(block_tables=views[self.N_FIXED + 2 * k + 1].view(host.S, host.widths[k]),
                                      slot_mapping=views[self.N_FIXED + 2 * k], page_size=self.cache.page_size)
         ctx = StepContext(
             num_tokens=host.T, num_seqs=host.S, token_ids=views[0], positions=views[1], token_seq=views[2],

@@ -158,8 +158,9 @@ class Scheduler:
         most = min(len(prompt) + budget, cfg.max_sequence_length)
         ps = self.cache.page_size
         for g in self.cache.groups:
-            window = g.span  # the most keys a token reads: a window, a chunk, or None for all
-            span = most if window is None else min(most, window + 2 * ps)
+            window = g.span  # the most rows a request holds: a window's, a chunk's, or None for all
+            rows = g.need.rows(most)
+            span = rows if window is None else min(rows, window + 2 * ps)
             if -(-span // ps) > g.pool.num_pages:
                 raise SchedulerError(
                     f"request {request_id!r} can reach {most} tokens, which the cache ({g.pool.num_pages} pages "

@@ -781,6 +781,17 @@ class ScoreTerms:
         return any(t is not None for t in (self.slopes, self.log_r1, self.log_r2, self.sink))
 
 
+class PooledKeys:
+    """Keys and values that stand for whole runs of ``every`` positions ahead of an attention window: ``k`` [pages, kv
+    heads, page size, d] and ``v`` [.., dv] hold one row per run, addressed by ``block_tables`` (int32 [requests,
+    blocks]) as tokens are by the step's tables."""
+
+    __slots__ = ("k", "v", "block_tables", "every")
+
+    def __init__(self, k: torch.Tensor, v: torch.Tensor, block_tables: torch.Tensor, every: int):
+        self.k, self.v, self.block_tables, self.every = k, v, block_tables, int(every)
+
+
 def set_attention_tiled(on: bool = True) -> None:
     """Portions of prompts on the general attention's tiled kernel (True, the default) or on the kernel of single
     tokens (False), for comparisons."""
@@ -793,7 +804,7 @@ def paged_attention_simt(qkv: torch.Tensor, out: torch.Tensor, k_cache: torch.Te
                          num_heads: int, num_kv_heads: int, head_dim: int, window: int, scale: float,
                          score_slopes=None, v_head_dim: Optional[int] = None,
                          max_q_len: int = 1, max_kv_len: int = 0, workspace=None, values_in_keys: bool = False,
-                         chunk: int = 0):
+                         chunk: int = 0, pooled: Optional[PooledKeys] = None):
     """General attention over the paged cache; q is read from the first nh*d columns of ``qkv``.
     ``window``: the query at position P sees the keys P - window + 1 .. P (0: all).  ``chunk`` (instead of a window):
     positions are counted off in chunks of that many from 0, and a query sees the keys of its own chunk up to itself.
@@ -804,7 +815,8 @@ def paged_attention_simt(qkv: torch.Tensor, out: torch.Tensor, k_cache: torch.Te
     ``max_q_len``: the most tokens a request brings; above one (portions of prompts) the kernel that shares tiles of
     keys among 64 query rows runs where it takes the geometry.  ``max_kv_len`` and ``workspace`` (a step of single
     tokens): the most keys a request holds, and where scratch comes from; the keys of a token are then cut into
-    shares that run side by side, and query heads of one kv head share its keys."""
+    shares that run side by side, and query heads of one kv head share its keys.  ``pooled`` (with a window): beside the
+    window's tokens the query sees one row of ``pooled`` for every run of positions that lies wholly before the window."""
     dv = int(v_head_dim or head_dim)
     if chunk:
         if window or chunk < 0:
@@ -839,10 +851,23 @@ def paged_attention_simt(qkv: torch.Tensor, out: torch.Tensor, k_cache: torch.Te
         _need(score_slopes, "score slopes", torch.float32)
         if score_slopes.numel() != num_heads:
             raise KernelError("attention: one score slope per query head is needed")
+    pool_args = (_ptr(None), _ptr(None), _ptr(None), _c_int(0), _c_int(0))
+    if pooled is not None:
+        _need(pooled.k, "pooled keys", qkv.dtype)
+        _need(pooled.v, "pooled values", qkv.dtype)
+        _need(pooled.block_tables, "block tables of the pooled keys", torch.int32)
+        ps = k_cache.shape[2]
+        if (not window or chunk or pooled.every <= 0 or pooled.k.shape[1:] != (num_kv_heads, ps, head_dim)
+                or pooled.v.shape != (*pooled.k.shape[:3], dv) or pooled.block_tables.shape[0] != block_tables.shape[0]):
+            raise KernelError(f"attention: pooled keys {tuple(pooled.k.shape)} of {pooled.every} positions, window {window}")
+        pool_args = (_ptr(pooled.k), _ptr(pooled.v), _ptr(pooled.block_tables), _c_int(pooled.block_tables.shape[1]),
+                     _c_int(pooled.every))
     fn = _lib().ferris_paged_attention_simt
     extra = (_c_int(0), _ptr(None), ctypes.c_longlong(0))
     if max_q_len <= 1 and max_kv_len > 0 and workspace is not None:
         span = min(max_kv_len, window) if window else max_kv_len
+        if pooled is not None:
+            span += max_kv_len // pooled.every
         floats = T * num_heads * ATTENTION_MAX_SHARES * (dv + 2)
         scratch = workspace.get("attn_shares", (floats,), torch.float32)
         extra = (_c_int(span), _ptr(scratch), ctypes.c_longlong(floats))
@@ -858,9 +883,47 @@ def paged_attention_simt(qkv: torch.Tensor, out: torch.Tensor, k_cache: torch.Te
                                            _c_int(num_kv_heads), _c_int(head_dim), _c_int(dv), _c_int(k_cache.shape[2]),
                                            _c_int(-chunk if chunk else (window or 0)), _c_float(scale), _ptr(score_slopes),
                                            _ptr(terms.log_r1),
-                                           _ptr(terms.log_r2), _ptr(terms.sink), _c_int(v_stride), *extra, _stream()),
+                                           _ptr(terms.log_r2), _ptr(terms.sink), _c_int(v_stride), *pool_args, *extra,
+                                           _stream()),
         "paged attention", 2 if extra and extra[0].value > 0 else 1,
     )
+
+
+def embed_positions(table: torch.Tensor, pos_table: torch.Tensor, ids: torch.Tensor, positions: torch.Tensor, out: torch.Tensor,
+                    rows: Optional[torch.Tensor] = None, status: Optional[torch.Tensor] = None):
+    """out[t, :] = table[ids[t], :] + pos_table[positions[t], :] as fp32; ``rows`` (optional): the same in the tables' type."""
+    _need(table, "embedding table")
+    _need(pos_table, "position table", table.dtype)
+    _need(ids, "token ids", torch.int32)
+    _need(positions, "positions", torch.int32)
+    _need(out, "embedding output", torch.float32)
+    T, H = out.shape
+    if rows is not None:
+        _need(rows, "embedding rows", table.dtype)
+    if (table.dim() != 2 or table.shape[1] != H or pos_table.dim() != 2 or pos_table.shape[1] != H or ids.numel() != T
+            or positions.numel() != T or (rows is not None and rows.shape != (T, H))):
+        raise KernelError(f"embed_positions: tables {tuple(table.shape)} {tuple(pos_table.shape)}, ids {tuple(ids.shape)}, "
+                          f"out {tuple(out.shape)}")
+    _check(_lib().ferris_embed_positions(_ptr(table), _ptr(pos_table), _c_int(_dt(table, "embedding table")), _ptr(ids),
+                                         _ptr(positions), _ptr(out), _ptr(rows), _c_int(T), _c_int(H), _c_int(table.shape[0]),
+                                         _c_int(pos_table.shape[0]), _ptr(status), _stream()), "embed_positions")
+
+
+def rmsnorm_add(y: Optional[torch.Tensor], weight: Optional[torch.Tensor], eps: float, h: torch.Tensor,
+                rows: Optional[torch.Tensor] = None):
+    """h += rmsnorm(y) * weight, everything fp32; ``rows`` (optional, bf16): h rounded, what the next products read.
+    ``y`` None: h stays, the rows alone are written."""
+    _need(h, "residual rows", torch.float32)
+    T, H = h.shape
+    if y is not None:
+        _need(y, "norm input", torch.float32)
+        _need(weight, "norm weight", torch.float32)
+    if rows is not None:
+        _need(rows, "rounded residual rows", torch.bfloat16)
+    if (y is not None and (y.shape != (T, H) or weight.numel() != H)) or (rows is not None and rows.shape != (T, H)):
+        raise KernelError(f"norm + add: residual {tuple(h.shape)}, input {None if y is None else tuple(y.shape)}")
+    _check(_lib().ferris_rmsnorm_add(_ptr(y), _ptr(weight), _ptr(h), _ptr(rows), _c_int(T), _c_int(H), _c_float(eps),
+                                     _stream()), "norm + add")
 
 
 def embed_sinusoid(table: torch.Tensor, ids: torch.Tensor, positions: torch.Tensor, freq: torch.Tensor, scale: float,
@@ -1547,13 +1610,20 @@ def qk_norm_rotary_cache_write(qkv: torch.Tensor, ctx, slot_mapping: Optional[to
                                num_heads: int, num_kv_heads: int, head_dim: int, v_head_dim: int,
                                q_norm: Optional[torch.Tensor], k_norm: Optional[torch.Tensor], eps: float,
                                rotary: Optional[RotaryTable], values_from_keys: bool = False, write_kv: bool = True,
-                               per_head: bool = False):
+                               per_head: bool = False, mixed_values: Optional[torch.Tensor] = None,
+                               mix_lambda: Optional[torch.Tensor] = None, pooled: Optional[PooledKeys] = None,
+                               pool_slots: Optional[torch.Tensor] = None, block_tables: Optional[torch.Tensor] = None):
     """Between the q/k(/v) product and attention: q and k each divided by the root mean square of their WHOLE projection
     (all heads at once) and multiplied by ``q_norm`` / ``k_norm`` (fp32, one number per element; None: no norm), then
     rotated by the tokens' positions; q rewritten in place, k and the values into the paged cache.
     ``values_from_keys``: the values are the keys as projected (before norm and rotation); the rows then hold
     [nh d | nkv d] only.  ``per_head``: every head is divided by the root mean square of its own elements instead, and
-    the weights hold ``head_dim`` numbers that all heads share (not with ``values_from_keys``)."""
+    the weights hold ``head_dim`` numbers that all heads share (not with ``values_from_keys``).
+    ``mixed_values`` (rows [T, nkv dv] in the activations' type): with ``mix_lambda`` (one fp32 number on the device) the
+    values stored are (1 - lambda) v + lambda mixed_values, without it the layer's values are copied into the rows, for
+    later layers to mix with.  ``pooled`` with ``pool_slots`` (int32 [T], the pooled row that the token completes or a
+    negative number) and the step's ``block_tables``, in steps of SINGLE tokens only: the means of a completed run's keys
+    and values, as the pages hold them, go to its pooled row (other steps: ``pool_blocks`` behind this call)."""
     T, width, ld = _rows(qkv, "qkv")
     want = (num_heads + num_kv_heads) * head_dim + (0 if values_from_keys else num_kv_heads * v_head_dim)
     if width != want:
@@ -1577,6 +1647,24 @@ def qk_norm_rotary_cache_write(qkv: torch.Tensor, ctx, slot_mapping: Optional[to
             raise KernelError(f"qk norm + rotation: caches {tuple(k_cache.shape)} {tuple(v_cache.shape)} do not fit")
     positions, freq, rdim, inter, mag = _rotary_args(rotary, ctx, head_dim, qkv.device)
     _need(ctx.positions, "positions", torch.int32)
+    if (mixed_values is not None or pooled is not None) and (per_head or not write_kv):
+        raise KernelError("qk norm + rotation: mixed values and pooled rows go with a cache that is written and no norm per head")
+    if mixed_values is not None:
+        _need(mixed_values, "mixed values", qkv.dtype)
+        if mixed_values.shape != (T, num_kv_heads * v_head_dim):
+            raise KernelError(f"qk norm + rotation: mixed values {tuple(mixed_values.shape)}")
+        if mix_lambda is not None:
+            _need(mix_lambda, "mixing factor", torch.float32)
+    elif mix_lambda is not None:
+        raise KernelError("qk norm + rotation: a mixing factor and nothing to mix with")
+    pool_args = (_ptr(None), _ptr(None), _ptr(None), _c_int(0), _ptr(None), _c_int(0), _ptr(None))
+    if pooled is not None:
+        _check_pool(pooled, pool_slots, block_tables, k_cache, v_cache, T)
+        if ctx.max_q_len != 1:
+            raise KernelError("qk norm + rotation: runs are pooled on the way in steps of single tokens only")
+        _need(ctx.token_seq, "token-to-request map", torch.int32)
+        pool_args = (_ptr(pool_slots), _ptr(pooled.k), _ptr(pooled.v), _c_int(pooled.every), _ptr(block_tables),
+                     _c_int(block_tables.shape[1]), _ptr(ctx.token_seq))
     if per_head:
         _check(
             _lib().ferris_qk_head_norm_rotary_cache_write(
@@ -1594,20 +1682,47 @@ def qk_norm_rotary_cache_write(qkv: torch.Tensor, ctx, slot_mapping: Optional[to
             _ptr(k_cache if write_kv else None), _ptr(v_cache if write_kv else None), _c_int(T), _c_int(num_heads),
             _c_int(num_kv_heads), _c_int(head_dim), _c_int(v_head_dim), _c_int(page_size), _ptr(q_norm), _ptr(k_norm),
             _c_float(eps), freq, rdim, inter, mag, _c_int(1 if values_from_keys else 0), _c_int(1 if write_kv else 0),
-            _stream()),
+            _ptr(mixed_values), _ptr(mix_lambda), *pool_args, _stream()),
         "qk norm + rotation + cache write",
     )
 
 
+def _check_pool(pooled: "PooledKeys", pool_slots, block_tables, k_cache, v_cache, tokens: int) -> None:
+    _need(pooled.k, "pooled keys", k_cache.dtype)
+    _need(pooled.v, "pooled values", k_cache.dtype)
+    _need(pool_slots, "pooled slots", torch.int32)
+    _need(block_tables, "block tables", torch.int32)
+    if (pooled.every <= 0 or pool_slots.numel() != tokens or pooled.k.shape[1:] != k_cache.shape[1:]
+            or pooled.v.shape[1:] != v_cache.shape[1:] or pooled.k.shape[0] != pooled.v.shape[0] or block_tables.dim() != 2):
+        raise KernelError(f"pooled rows of {pooled.every} positions: {tuple(pooled.k.shape)} beside pages {tuple(k_cache.shape)}")
+
+
+def pool_blocks(k_cache: torch.Tensor, v_cache: torch.Tensor, pooled: PooledKeys, pool_slots: torch.Tensor,
+                block_tables: torch.Tensor, ctx):
+    """The pooled rows that the step's tokens complete (``pool_slots`` int32 [T]: the row, or a negative number): the means
+    of the keys and values of the ``pooled.every`` positions up to the token's, as the pages hold them (fp32 sums in the
+    order of the positions, rounded once)."""
+    T = ctx.num_tokens
+    _need(k_cache, "key cache")
+    _need(v_cache, "value cache", k_cache.dtype)
+    _check_pool(pooled, pool_slots, block_tables, k_cache, v_cache, T)
+    _check(_lib().ferris_pool_blocks(_ptr(k_cache), _ptr(v_cache), _ptr(pooled.k), _ptr(pooled.v),
+                                     _c_int(_dt(k_cache, "pooled rows")), _ptr(block_tables), _c_int(block_tables.shape[1]),
+                                     _ptr(ctx.token_seq), _ptr(ctx.positions), _ptr(pool_slots), _c_int(T),
+                                     _c_int(pooled.every), _c_int(k_cache.shape[1]), _c_int(k_cache.shape[3]),
+                                     _c_int(v_cache.shape[3]), _c_int(k_cache.shape[2]), _stream()), "pooled rows")
+
+
 def moe_router(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], ids: torch.Tensor,
-               weights: torch.Tensor, top: int, scored: Optional[dict] = None):
+               weights: torch.Tensor, top: int, scored: Optional[dict] = None, sigmoid: bool = False):
     """The ``top`` experts of every row of ``x`` and their weights: logits x weight^T + bias in fp32 sums, the largest
     ``top`` (lowest index among equals), softmax over those alone.  ids int32 [T, top], weights fp32 [T, top].
     ``scored`` = {"correction": fp32 [E] or None, "groups": n, "keep": n, "with_weights": n, "identity_w": fp32 [T] or
     None}: the scores are the softmax over ALL outputs, the choice is made by score + correction among the outputs of the
     ``keep`` groups (of ``groups`` equal groups of neighbours) whose best choice score is largest, and the weights are
     the chosen scores divided by their sum + 1e-20; outputs from ``with_weights`` on are identity experts, which come
-    out as the index ``with_weights`` and whose weights are summed per token into ``identity_w``."""
+    out as the index ``with_weights`` and whose weights are summed per token into ``identity_w``.
+    ``sigmoid``: the weights are the sigmoids of the chosen logits, as they are."""
     T, W, ldx = _rows(x, "router input")
     _need(weight, "router matrix", x.dtype)
     _need(ids, "expert ids", torch.int32)
@@ -1617,6 +1732,8 @@ def moe_router(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tenso
         raise KernelError(f"router: x {tuple(x.shape)}, matrix {tuple(weight.shape)}, ids {tuple(ids.shape)}")
     if bias is not None:
         _need(bias, "router bias", torch.float32)
+    if sigmoid and scored is not None:
+        raise KernelError("router: one kind of score at a time")
     corr = idw = None
     groups = keep = 1
     real = E
@@ -1631,7 +1748,7 @@ def moe_router(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tenso
             raise KernelError(f"router: correction / identity weights do not fit {E} outputs and {T} rows")
     _check(_lib().ferris_moe_router(_ptr(x), _c_int(ldx), _c_int(_dt(x, "router")), _ptr(weight), _ptr(bias), _ptr(ids),
                                     _ptr(weights), _c_int(T), _c_int(W), _c_int(E), _c_int(top),
-                                    _c_int(0 if scored is None else 1), _ptr(corr), _c_int(groups), _c_int(keep), _c_int(real),
+                                    _c_int(2 if sigmoid else (0 if scored is None else 1)), _ptr(corr), _c_int(groups), _c_int(keep), _c_int(real),
                                     _ptr(idw), _stream()), "router")
 
 
@@ -1641,7 +1758,8 @@ MOE_GROUPED_MIN_TOKENS = 17  # from here on (bf16) the experts' rows are sorted 
 
 def moe_experts(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor,
                 h: torch.Tensor, workspace=None, accumulate: bool = True, grouped: Optional[bool] = None,
-                activation: str = "silu", limit: float = 0.0, identity_w: Optional[torch.Tensor] = None):
+                activation: str = "silu", limit: float = 0.0, identity_w: Optional[torch.Tensor] = None,
+                input_weights: bool = False):
     """h (+)= sum over a row's chosen experts of weight x down_e (silu(gate_e x) * (up_e x)).  gate_up [E, 2 ff, W] (an
     expert's gate rows, then its up rows), down [E, W, ff] in x's type; ids int32 and weights fp32 [T, top]; h fp32
     [T, W].  Steps of few tokens (up to MOE_FEW_MAX_PAIRS choices): a block per (expert, slab of rows) reads the weights
@@ -1649,7 +1767,9 @@ def moe_experts(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, ids:
     whole dot products in the same order, so a token's result has the same bits.  Longer steps in bf16 (``grouped``; None = decide by size and alignment): the pairs sorted by expert, two
     tensor-core products over tiles that each meet their own expert's weights, and a pass that adds a token's results
     in the order of its choices.  ``activation``, ``limit``: the experts' gated activation (see ``gated_activation``).
-    ``identity_w`` fp32 [T]: ids may then hold E, an expert that meets no weights, and h also gets identity_w[t] x[t]."""
+    ``identity_w`` fp32 [T]: ids may then hold E, an expert that meets no weights, and h also gets identity_w[t] x[t].
+    ``input_weights``: a token's weight for an expert goes onto the expert's input (both first products times the weight
+    in fp32, ahead of the activation), and the results are added as they are."""
     T, W, ldx = _rows(x, "experts input")
     if activation not in GATED_ACTIVATIONS:
         raise KernelError(f"experts: activation '{activation}' is not known ({', '.join(GATED_ACTIVATIONS)})")
@@ -1687,11 +1807,12 @@ def moe_experts(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, ids:
         xs = get("moe_sorted_rows", (rows, W), x.dtype)
         act = get("moe_sorted_act", (rows, ff), x.dtype)
         y = get("moe_sorted_out", (rows, W), torch.float32)
+        row_scale = get("moe_row_scale", (rows,), torch.float32) if input_weights else None
         _check(_lib().ferris_moe_experts_grouped(_ptr(x), _c_int(ldx), _ptr(gate_up), _ptr(down), _ptr(ids), _ptr(weights),
                                                  _ptr(h), _c_int(ldh), _c_int(T), _c_int(W), _c_int(ff), _c_int(top),
                                                  _c_int(E), _c_int(rows), _ptr(pos), _ptr(row_token), _ptr(tile_expert),
                                                  _ptr(xs), _ptr(act), _ptr(y), _c_int(1 if accumulate else 0),
-                                                 _c_int(act_kind), _c_float(limit), _ptr(identity_w), _stream()),
+                                                 _c_int(act_kind), _c_float(limit), _ptr(identity_w), _ptr(row_scale), _stream()),
                "experts (sorted)", 5)
         return
     act = get("moe_act", (T * top, ff), x.dtype)
@@ -1704,7 +1825,8 @@ def moe_experts(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, ids:
                                                  _ptr(act), _ptr(h), _c_int(ldh), _c_int(T), _c_int(W), _c_int(ff),
                                                  _c_int(top), _c_int(1 if accumulate else 0),
                                                  _ptr(y) if few else ctypes.c_void_p(0), _c_int(E), _c_int(act_kind),
-                                                 _c_float(limit), _ptr(identity_w), _stream()),
+                                                 _c_float(limit), _ptr(identity_w), _c_int(1 if input_weights else 0),
+                                                 _stream()),
            "experts", 3 if few else 2)
 
 
@@ -1859,9 +1981,9 @@ def attention_step(qkv, out, k_cache, v_cache, meta, ctx, num_heads, num_kv_head
 
 def paged_attention(qkv, out, k_cache, v_cache, block_tables, ctx, num_heads, num_kv_heads, head_dim, window, scale,
                     score_slopes=None, v_head_dim: Optional[int] = None, values_in_keys: bool = False,
-                    chunk: int = 0, fp32_weights: bool = False):
+                    chunk: int = 0, fp32_weights: bool = False, pooled: Optional[PooledKeys] = None):
     """Attention of the step's tokens over the paged cache (their own keys are in it already).
-    ``chunk``: see ``paged_attention_simt``.  ``fp32_weights``: the softmax's weights and the weighted sum stay in 32-bit
+    ``chunk``, ``pooled``: see ``paged_attention_simt``.  ``fp32_weights``: the softmax's weights and the weighted sum stay in 32-bit
     (the tensor-core kernels round the weights to bf16 for their second product), so the general kernel runs.
     ``ctx`` is the step context.  bf16 with head size 64 / 128 runs on the tensor cores: the split-KV
     kernel when every request brings one token, the prefill kernel otherwise; every other geometry, the
@@ -1870,11 +1992,11 @@ def paged_attention(qkv, out, k_cache, v_cache, block_tables, ctx, num_heads, nu
     _need(k_cache, "key cache", qkv.dtype)
     if isinstance(score_slopes, ScoreTerms) and not score_slopes.any():
         score_slopes = None
-    if values_in_keys or chunk or fp32_weights or (v_head_dim is not None and v_head_dim != head_dim):
+    if values_in_keys or chunk or fp32_weights or pooled is not None or (v_head_dim is not None and v_head_dim != head_dim):
         paged_attention_simt(qkv, out, k_cache, v_cache, block_tables, ctx.token_seq, ctx.positions, num_heads,
                              num_kv_heads, head_dim, window, scale, score_slopes=score_slopes, v_head_dim=v_head_dim,
                              max_q_len=ctx.max_q_len, max_kv_len=ctx.max_kv_len, workspace=ctx.workspace,
-                             values_in_keys=values_in_keys, chunk=chunk)
+                             values_in_keys=values_in_keys, chunk=chunk, pooled=pooled)
         return
     _need(v_cache, "value cache", qkv.dtype)
     _need(block_tables, "block tables", torch.int32)

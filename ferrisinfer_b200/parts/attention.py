@@ -35,6 +35,13 @@ Options beyond the reference's layer, each a parameter of its own:
   ``output_scale``      a factor on the mixer's result (applied to the rows that enter the output product)
   ``chunk``             instead of a window: positions are counted off in chunks of that many from 0, and a token
                         sees the keys of its own chunk up to itself
+  ``pool``              (with a window) beside the window's tokens a token sees one key and value for every run of ``pool``
+                        positions (counted off from 0) that lies wholly before the window: the means of the run's keys
+                        and values as the cache holds them, kept in pages of their own (one row a run), in one softmax
+                        with the tokens
+  ``value_mix``         {"lambda": tensor name, "role": "source" or "mix"}: a layer with "mix" stores (1 - lambda) v +
+                        lambda v1 as its values, v1 being the values that the layer with "source" projected for the same
+                        token in this pass; the source's own number is read if the folder has it, and not used
   ``fp32_weights``      the softmax's weights and the weighted sum of values stay in 32-bit (the general kernel)
   a ``scaled_rotary`` position encoding (either pair layout, part of a head, scaled frequencies) rotates in the kernel
   that also norms and writes the cache; it goes with ``qk_norm``, ``values_from_keys``, ``chunk`` and value heads of
@@ -52,7 +59,7 @@ from typing import Optional
 import torch
 
 from ..kernels import ops
-from .base import LayerCache, Mixer, PagedKV, TensorSpec
+from .base import CombinedNeed, LayerCache, Mixer, PagedKV, PositionEncoding, TensorSpec
 from .plan import PartSpec, build_part, register_part
 
 
@@ -71,7 +78,8 @@ class GroupedQueryAttention(Mixer):
                  query_temperature: Optional[tuple] = None, tensor_names: Optional[dict] = None,
                  bias_names: Optional[dict] = None, sink_name: Optional[str] = None,
                  values_from_keys: bool = False, qk_norm: Optional[dict] = None, chunk: Optional[int] = None,
-                 fp32_weights: bool = False, output_gate: Optional[dict] = None, output_scale: float = 1.0):
+                 fp32_weights: bool = False, output_gate: Optional[dict] = None, output_scale: float = 1.0,
+                 pool: Optional[int] = None, value_mix: Optional[dict] = None):
         if num_heads % num_kv_heads:
             raise ValueError(f"{num_heads} heads cannot share {num_kv_heads} kv heads")
         self.hidden_size, self.num_heads = int(hidden_size), int(num_heads)
@@ -99,6 +107,21 @@ class GroupedQueryAttention(Mixer):
         self.qk_norm_per_head = bool(qk_norm and qk_norm.get("per_head", False))
         if self.qk_norm_per_head and self.values_from_keys:
             raise ValueError("a norm per head does not go with values taken from the keys")
+        self.pool = None if pool is None else int(pool)
+        if self.pool is not None and (self.pool <= 0 or not self.window or self.window < 0):
+            raise ValueError(f"pooled runs of {pool} positions stand before a window ({window})")
+        self.value_mix = None
+        if value_mix is not None:
+            self.value_mix = (value_mix["lambda"], value_mix["role"])
+            if self.value_mix[1] not in ("source", "mix"):
+                raise ValueError(f"value mixing: role '{self.value_mix[1]}' is not known (source, mix)")
+        self.mix_lambda = None
+        if (self.pool is not None or self.value_mix is not None) and (self.qk_norm_per_head or self.qk_norm is None
+                                                                      or self.values_from_keys):
+            raise ValueError("pooled runs and mixed values go with a norm over the whole projection and a value matrix")
+        if self.pool is not None and (type(self.position).score_slopes is not PositionEncoding.score_slopes
+                                      or type(self.position).score_log_penalty is not PositionEncoding.score_log_penalty):
+            raise ValueError("pooled runs go with no distance penalty: a run has no distance of its own")
         self.output_gate = None
         if output_gate is not None:
             self.output_gate = (output_gate["name"], output_gate.get("kind", "sigmoid"))
@@ -163,6 +186,8 @@ class GroupedQueryAttention(Mixer):
         specs += self.position.tensor_specs(prefix)  # learned numbers of the position encoding, if it has any
         if self.sink_name:
             specs.append(TensorSpec(f"{prefix}.{self.sink_name}", (self.num_heads,), "vector"))
+        if self.value_mix is not None:
+            specs.append(TensorSpec(f"{prefix}.{self.value_mix[0]}", (), "vector", required=self.value_mix[1] == "mix"))
         return specs + [TensorSpec(self._matrix_name(prefix, "o"), (H, self.o_size), "matrix")]
 
     @property
@@ -185,6 +210,8 @@ class GroupedQueryAttention(Mixer):
         self.position.bind(tensors, prefix)
         if self.sink_name:
             self.sink = tensors[f"{prefix}.{self.sink_name}"]
+        if self.value_mix is not None and self.value_mix[1] == "mix":
+            self.mix_lambda = tensors[f"{prefix}.{self.value_mix[0]}"].reshape(1)
         if any(b is not None for b in biases):
             sizes = (self.q_size, self.kv_size, self.v_size)[:len(biases)]
             if self.output_gate is not None:
@@ -200,13 +227,21 @@ class GroupedQueryAttention(Mixer):
 
     # -------------------------------------------------------------------- cache
     def cache_need(self):
-        return PagedKV(self.num_kv_heads, self.head_dim, self.window,
-                       None if self.v_head_dim == self.head_dim else self.v_head_dim, chunk=self.chunk)
+        dv = None if self.v_head_dim == self.head_dim else self.v_head_dim
+        need = PagedKV(self.num_kv_heads, self.head_dim, self.window, dv, chunk=self.chunk, run=self.pool)
+        if self.pool is None:
+            return need
+        return CombinedNeed((need, PagedKV(self.num_kv_heads, self.head_dim, None, dv, stride=self.pool)))
 
     # ------------------------------------------------------------------ forward
     def forward(self, x, h, ctx, cache: LayerCache, owns_cache: bool, accumulate: bool = True):
         T = x.shape[0]
         nh, nkv, d = self.num_heads, self.num_kv_heads, self.head_dim
+        pooled = pool_meta = None
+        if self.pool is not None:
+            cache, means = cache.parts
+            pool_meta = ctx.paged[means.group]
+            pooled = ops.PooledKeys(means.k, means.v, pool_meta.block_tables, self.pool)
         meta = ctx.paged[cache.group]
         n_qkv = self.q_size + self.kv_size + self.v_size
         qkv = ctx.workspace.get("attn_qkv", (T, self.qkv_weight.shape[0]), x.dtype)
@@ -218,11 +253,19 @@ class GroupedQueryAttention(Mixer):
                 qkv, gate = qkv[:, :n_qkv], qkv[:, n_qkv:]
             if self.rotary_prepare:
                 rotary = self.position.table(qkv.device) if hasattr(self.position, "table") else None
+                extra = {}
+                if self.value_mix is not None:
+                    extra.update(mixed_values=ctx.workspace.get("mixed_values", (T, self.v_size), x.dtype),
+                                 mix_lambda=self.mix_lambda)
+                if pooled is not None and owns_cache and ctx.max_q_len == 1:  # runs are pooled on the way
+                    extra.update(pooled=pooled, pool_slots=pool_meta.slot_mapping, block_tables=meta.block_tables)
                 ops.qk_norm_rotary_cache_write(qkv, ctx, meta.slot_mapping, cache.k, cache.v, nh, nkv, d, dv,
                                                self.q_norm_weight, self.k_norm_weight,
                                                self.qk_norm[0] if self.qk_norm else 0.0, rotary,
                                                values_from_keys=self.values_from_keys, write_kv=owns_cache,
-                                               per_head=self.qk_norm_per_head)
+                                               per_head=self.qk_norm_per_head, **extra)
+                if pooled is not None and owns_cache and ctx.max_q_len > 1:
+                    ops.pool_blocks(cache.k, cache.v, pooled, pool_meta.slot_mapping, meta.block_tables, ctx)
             else:
                 ops.qk_prepare_cache_write(qkv, ctx.positions, meta.slot_mapping, cache.k, cache.v, nh, nkv, d, dv,
                                            self.qk_unit_norm_eps, self.query_temperature, write_kv=owns_cache)
@@ -232,7 +275,7 @@ class GroupedQueryAttention(Mixer):
                                    log_r1=None if log is None else log[0], log_r2=None if log is None else log[1])
             ops.paged_attention(qkv, out, cache.k, cache.v, meta.block_tables, ctx, nh, nkv, d, self.window or 0,
                                 self.scale, score_slopes=terms, v_head_dim=dv, chunk=self.chunk or 0,
-                                fp32_weights=self.fp32_weights)
+                                fp32_weights=self.fp32_weights, pooled=pooled)
             if gate is not None:
                 ops.gate_mul(out, gate, out, self.output_gate[1], self.output_scale)
             ops.gemm(out, self.o_weight, None, h, accumulate=accumulate)

@@ -29,21 +29,41 @@ class PagedKV:
     ``chunk``: positions are counted off in chunks of that many from 0 and a token reads the keys of its own chunk only, so
     the pages of chunks that are over are given back while the request runs (not together with ``window``).
     ``v_head_dim``: size of a value head where it differs from a key head's (None = the same; 0 = no value rows are
-    kept, for a mixer whose keys carry their values)."""
+    kept, for a mixer whose keys carry their values).
+    ``run`` (with ``window``): positions are counted off in runs of that many from 0, and the pages of a run that is not
+    complete yet stay although the window may have passed its first positions (its rows are pooled when it is complete).
+    ``stride``: one row for every ``stride`` WHOLE tokens instead of one per token: row r stands for the tokens
+    r * stride .. r * stride + stride - 1 and exists once the last of them is in the cache."""
 
     num_kv_heads: int
     head_dim: int
     window: Optional[int] = None
     v_head_dim: Optional[int] = None
     chunk: Optional[int] = None
+    run: Optional[int] = None
+    stride: int = 1
 
     def first_needed(self, num_tokens: int) -> int:
-        """The lowest position that a query at position ``num_tokens`` or later can still read."""
+        """The lowest row that a query at position ``num_tokens`` or later can still read."""
         if self.chunk is not None:
             return num_tokens - num_tokens % self.chunk
         if self.window is not None:
-            return max(0, num_tokens - self.window + 1)
+            first = max(0, num_tokens - self.window + 1)
+            return first if self.run is None else min(first, num_tokens - num_tokens % self.run)
         return 0
+
+    def rows(self, num_tokens: int) -> int:
+        """How many rows ``num_tokens`` tokens have."""
+        return num_tokens // self.stride
+
+    @property
+    def span(self) -> Optional[int]:
+        """The most rows that have to stay in the cache at once, whatever the request's length (None: no such bound)."""
+        if self.chunk is not None:
+            return self.chunk
+        if self.window is not None:
+            return self.window if self.run is None else max(self.window, self.run)
+        return None
 
     @property
     def keeps_all(self) -> bool:
@@ -90,7 +110,9 @@ class PagedMeta:
     """Device metadata of one page group for one step."""
 
     block_tables: torch.Tensor  # int32 [S, max_blocks]; -1 = no page
-    slot_mapping: torch.Tensor  # int32 [T]; page * page_size + slot of each token of the step
+    # int32 [T]; page * page_size + slot of each token of the step; in a group with a stride the slot of the row that
+    # the token completes, or -1
+    slot_mapping: torch.Tensor
     page_size: int
 
 
@@ -188,6 +210,17 @@ class Norm(Part):
         self.forward(h, out)
         return out
 
+    def add_into(self, y: torch.Tensor, h: torch.Tensor, rows: Optional[torch.Tensor], workspace) -> None:
+        """h += norm(y), y and h fp32; ``rows`` (or None): h in the activations' type as well.  The default is a norm, a
+        sum and a cast; a norm with a kernel for all of it overrides this."""
+        from ..kernels import ops
+
+        normed = workspace.get("norm_add", tuple(h.shape), torch.float32)
+        self.forward(y, normed)
+        ops.add_(h, normed)
+        if rows is not None:
+            ops.rmsnorm_add(None, None, 0.0, h, rows)
+
 
 class PositionEncoding(Part):
     """How positions enter a mixer.  ``rotary_table`` lets the attention mixer fuse the
@@ -272,6 +305,9 @@ class FeedForward(Part):
 
 class Block(Part):
     graph_safe = False
+    # True for a block that keeps ctx.shared["residual_rows"] (the residual rows in the activations' type) in step with
+    # the residual stream; whatever else touches the stream makes the model forget those rows
+    keeps_rows = False
 
     def cache_need(self):
         return None

@@ -9,10 +9,18 @@ The parallel block, both branches from the same h:
 Both norms are taken before either branch adds, into buffers of their own.  A layer may have no feed-forward.
 
 The sums are made in the fp32 residual stream by the last matrix product of each branch.
+
+The output-norm block: the norms stand on the sublayers' results, and the sublayers read the residual stream itself:
+  h += norm_1(mixer(h));  h += norm_2(feed_forward(h))
+A sublayer's result is formed in fp32 rows of its own; one kernel norms it, adds it into the stream and leaves the
+stream's rows in the activations' type for the next sublayer's products.
 """
 
 from __future__ import annotations
 
+import torch
+
+from ..kernels import ops
 from .base import Block, TensorSpec
 from .plan import build_part, register_part
 
@@ -125,5 +133,45 @@ class ParallelResidualBlock(PreNormResidualBlock):
             self.feed_forward.forward(x2, h, ctx)
 
 
+class OutputNormBlock(ParallelResidualBlock):
+    """h += norm_1(mixer(h)); h += norm_2(feed_forward(h)); ``feed_forward`` None: the mixer's half alone (the second norm's
+    tensor is then read if the folder has it, and not used)."""
+
+    keeps_rows = True
+
+    @staticmethod
+    def rows_of(h, ctx):
+        """The residual rows as the sublayers read them: the stream itself in 32-bit, else its rounded rows, which the
+        embedding or the block before has left or which are written here."""
+        if ctx.act_dtype == torch.float32:
+            return h
+        rows = ctx.shared.get("residual_rows")
+        if rows is None:
+            rows = ctx.workspace.get("residual_rows", tuple(h.shape), ctx.act_dtype)
+            ops.rmsnorm_add(None, None, 0.0, h, rows)
+            ctx.shared["residual_rows"] = rows
+        return rows
+
+    def forward(self, h, ctx, cache, owns_cache):
+        y = ctx.workspace.get("sublayer_out", tuple(h.shape), torch.float32)
+        x = self.rows_of(h, ctx)
+        after = None if x is h else x  # the rows are rewritten in place: the sublayer has read them
+        if getattr(self.mixer, "can_overwrite", False):
+            self.mixer.forward(x, y, ctx, cache, owns_cache, accumulate=False)
+        else:
+            y.zero_()
+            self.mixer.forward(x, y, ctx, cache, owns_cache)
+        self.mixer_norm.add_into(y, h, after, ctx.workspace)
+        if self.feed_forward is None:
+            return
+        if getattr(self.feed_forward, "can_overwrite", False):
+            self.feed_forward.forward(x, y, ctx, accumulate=False)
+        else:
+            y.zero_()
+            self.feed_forward.forward(x, y, ctx)
+        self.feed_forward_norm.add_into(y, h, after, ctx.workspace)
+
+
+register_part("block", "output_norm", OutputNormBlock)
 register_part("block", "pre_norm_residual", PreNormResidualBlock)
 register_part("block", "parallel_residual", ParallelResidualBlock)

@@ -72,6 +72,34 @@ class ScaledSinusoidalEmbedding(Part):
         ops.embed_sinusoid(self.weight, token_ids, positions, self.frequencies(h.device), self.scale, h)
 
 
+class LearnedPositionEmbedding(Part):
+    """h[t, :] = E[id_t, :] + P[pos_t, :] with a second table P of ``max_positions`` rows (tensor ``position_name``, a name
+    of its own, not under the prefix).  ``emits_rows``: the model may hand ``forward`` a buffer in the activations' type
+    that gets the same rows, for blocks whose sublayers read the residual stream itself."""
+
+    needs_positions = True
+    emits_rows = True
+
+    def __init__(self, vocab_size: int, hidden_size: int, max_positions: int, weight_name: str = "weight",
+                 position_name: str = "position"):
+        self.vocab_size, self.hidden_size, self.max_positions = int(vocab_size), int(hidden_size), int(max_positions)
+        self.weight_name, self.position_name = weight_name, position_name
+        self.weight = self.positions = None
+
+    def _name(self, prefix):
+        return f"{prefix}.{self.weight_name}" if self.weight_name else prefix
+
+    def tensor_specs(self, prefix):
+        return [TensorSpec(self._name(prefix), (self.vocab_size, self.hidden_size), "embedding"),
+                TensorSpec(self.position_name, (self.max_positions, self.hidden_size), "embedding")]
+
+    def bind(self, tensors, prefix):
+        self.weight, self.positions = tensors[self._name(prefix)], tensors[self.position_name]
+
+    def forward(self, token_ids, h, positions=None, rows=None):
+        ops.embed_positions(self.weight, self.positions, token_ids, positions, h, rows)
+
+
 class OutputHead(Part):
     """``tied_to``: tensor name of the embedding table to use as the output matrix, or None
     when the folder has a matrix of its own under ``prefix``.  ``softcap``: the logits z become
@@ -122,6 +150,7 @@ class OutputHead(Part):
 
 register_part("embedding", "token_embedding", TokenEmbedding)
 register_part("embedding", "scaled_sinusoidal_embedding", ScaledSinusoidalEmbedding)
+register_part("embedding", "learned_position_embedding", LearnedPositionEmbedding)
 register_part("embedding", "scaled_embedding",
               lambda vocab_size, hidden_size, scale=1.0, weight_name="weight": ScaledSinusoidalEmbedding(
                   vocab_size, hidden_size, scale=scale, base=None, weight_name=weight_name))

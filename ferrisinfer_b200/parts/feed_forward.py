@@ -12,6 +12,8 @@ gate_proj: crates/ferrisinfer-io/src/hf.rs:437-457).  No bias.  Gate and up are 
 
 from __future__ import annotations
 
+from typing import Optional
+
 import torch
 
 from ..kernels import ops
@@ -143,16 +145,26 @@ class MixtureOfExperts(FeedForward):
     among the outputs of the ``keep`` best of ``groups`` equal groups of neighbours (a group's score is its largest
     choice score), the weights s_e / (sum of the chosen s + 1e-20).  ``identity``: that many router outputs after the
     experts stand for experts without tensors whose result is the token's row itself.  ``activation``, ``limit``: the
-    experts' gated activation (``ops.GATED_ACTIVATIONS``)."""
+    experts' gated activation (``ops.GATED_ACTIVATIONS``).
+
+    ``sigmoid_scores``: the weights are the sigmoids of the chosen outputs, as they are (not with ``scored``).
+    ``input_weights``: a weight multiplies its expert's input instead of its result: out = sum_e expert_e(weight_e y).
+    ``router_bias_name`` None: the router has no bias."""
 
     graph_safe = True
     can_overwrite = True
 
     def __init__(self, hidden_size: int, intermediate_size: int, experts: int, top: int, router_name: str = "router",
-                 router_bias_name: str = "router.b", expert_prefix: str = "e", gate_name: str = "gate",
+                 router_bias_name: Optional[str] = "router.b", expert_prefix: str = "e", gate_name: str = "gate",
                  up_name: str = "up", down_name: str = "down", scored: dict = None, identity: int = 0,
-                 activation: str = "silu", limit: float = 0.0):
+                 activation: str = "silu", limit: float = 0.0, sigmoid_scores: bool = False,
+                 input_weights: bool = False):
         self.hidden_size, self.intermediate_size = int(hidden_size), int(intermediate_size)
+        self.sigmoid_scores, self.input_weights = bool(sigmoid_scores), bool(input_weights)
+        if self.sigmoid_scores and scored is not None:
+            raise ValueError("a router scores by sigmoids or by the scored kind, not both")
+        if self.input_weights and identity:
+            raise ValueError("identity experts have no input for a weight to go onto")
         self.experts, self.top, self.identity = int(experts), int(top), int(identity)
         self.outputs = self.experts + self.identity  # of the router
         if not (1 <= self.top <= self.outputs) or self.identity < 0:
@@ -188,8 +200,8 @@ class MixtureOfExperts(FeedForward):
             if self.scored[0]:
                 specs.append(TensorSpec(f"{prefix}.{self.scored[0]}", (self.outputs,), "bias"))
             return specs
-        return specs + [TensorSpec(f"{prefix}.{r}", (self.experts, H), "matrix"),
-                        TensorSpec(f"{prefix}.{rb}", (self.experts,), "bias")]
+        specs.append(TensorSpec(f"{prefix}.{r}", (self.experts, H), "matrix"))
+        return specs + ([TensorSpec(f"{prefix}.{rb}", (self.experts,), "bias")] if rb else [])
 
     def bind(self, tensors, prefix):
         r, rb, _, g, u, d = self._names
@@ -202,7 +214,7 @@ class MixtureOfExperts(FeedForward):
             self.router_bias = None
             self.correction = tensors[f"{prefix}.{self.scored[0]}"] if self.scored[0] else None
         else:
-            self.router_bias = tensors[f"{prefix}.{rb}"]
+            self.router_bias = tensors[f"{prefix}.{rb}"] if rb else None
         if self.experts == 0:  # identity experts only: the kernels still want matrices to point at
             W, I = self.hidden_size, self.intermediate_size
             self.gate_up = self.router.new_zeros(1, 2 * I, W)
@@ -217,9 +229,9 @@ class MixtureOfExperts(FeedForward):
         if self.scored is not None:
             scored = {"correction": self.correction, "groups": self.scored[1], "keep": self.scored[2],
                       "with_weights": self.experts, "identity_w": identity_w}
-        ops.moe_router(x, self.router, self.router_bias, ids, weights, self.top, scored=scored)
+        ops.moe_router(x, self.router, self.router_bias, ids, weights, self.top, scored=scored, sigmoid=self.sigmoid_scores)
         ops.moe_experts(x, self.gate_up, self.down, ids, weights, h, ctx.workspace, accumulate=accumulate,
-                        activation=self.activation, limit=self.limit, identity_w=identity_w)
+                        activation=self.activation, limit=self.limit, identity_w=identity_w, input_weights=self.input_weights)
 
 
 register_part("feed_forward", "swiglu", SwiGLU)

@@ -96,7 +96,13 @@ class DecoderModel:
         ctx.shared.clear()  # what parts share belongs to one pass; a context may be run again (to record a graph)
         S = self.plan.residual_streams
         row = ctx.workspace.get("residual", (T, self.hidden_size), torch.float32)
-        if getattr(self.embedding, "needs_positions", False):
+        keeps_rows = [getattr(b, "keeps_rows", False) for b in self.blocks]
+        if (getattr(self.embedding, "emits_rows", False) and S == 1 and ctx.act_dtype != torch.float32 and self.plan.run_order
+                and keeps_rows[self.plan.run_order[0].layer]):
+            rows = ctx.workspace.get("residual_rows", (T, self.hidden_size), ctx.act_dtype)
+            self.embedding.forward(ctx.token_ids, row, ctx.positions, rows)
+            ctx.shared["residual_rows"] = rows
+        elif getattr(self.embedding, "needs_positions", False):
             self.embedding.forward(ctx.token_ids, row, ctx.positions)
         else:
             self.embedding.forward(ctx.token_ids, row)
@@ -112,6 +118,8 @@ class DecoderModel:
             owner = i if step.cache_of is None else step.cache_of
             if step.add_embedding:
                 ops.add_(h, embedded)
+            if step.add_embedding or not keeps_rows[step.layer]:
+                ctx.shared.pop("residual_rows", None)  # the stream moves on without its rounded rows
             self.blocks[step.layer].forward(h, ctx, caches[owner], owns_cache=step.cache_of is None)
             if self.after_run is not None:
                 flush_pending_write(ctx, h, S)

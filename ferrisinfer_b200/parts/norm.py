@@ -71,6 +71,12 @@ class GroupedRMSNorm(Norm):
         self.forward(h, out)
         return out
 
+    def add_into(self, y, h, rows, workspace):
+        if self.groups == 1:
+            ops.rmsnorm_add(y, self.weight, self.eps, h, rows)
+        else:
+            super().add_into(y, h, rows, workspace)
+
     def forward_pair(self, other, h, out, other_out) -> bool:
         """This norm and ``other`` of the same rows in one launch; False (nothing done) if ``other`` is not the same
         norm with another weight."""

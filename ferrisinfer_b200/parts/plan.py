@@ -93,6 +93,8 @@ class ModelPlan:
     # residual rows per token: above one, the blocks get [T, streams x hidden] rows that all start as the embedding
     # output, and the final norm reads their sum (block kinds made for it, such as ``residual_streams``)
     residual_streams: int = 1
+    # True where positions index a table of max_positions rows: no request may grow beyond it, whatever the engine allows
+    positions_bounded: bool = False
 
     def validate(self) -> None:
         if self.residual_streams < 1:
