@@ -1,9 +1,9 @@
 """Designs side by side at equal layer sizes: the Kugilix decoder beside the Qwen2 dense decoder, or (``design`` =
 "nusudra" / "netinex") the Nusudra or the Netinex decoder beside both, or (``design`` = "sumevik") the Sumevik decoder
 beside the Netinex decoder (the closest existing design: attention within chunks, a linear recurrence, experts) and
-Qwen2, random weights.
+Qwen2, or (``design`` = "retezen") the Retezen decoder beside the same two, random weights.
 
-Called by ``bench.py --designs [--design nusudra|netinex|sumevik]``.  For each of a few sizes that resemble a real model's layers it measures, through
+Called by ``bench.py --designs [--design nusudra|netinex|sumevik|retezen]``.  For each of a few sizes that resemble a real model's layers it measures, through
 the step function, the prefill of one prompt and decode steps at two batch sizes for both designs, and times the
 kernels that only the Kugilix design has (decayed linear attention, the windowed attention with slopes, the short
 convolution, the norms in groups, the gated norm, the activation) alone, with what they reach of the measured copy
@@ -137,6 +137,23 @@ def sumevik_config(s: dict) -> dict:
     order = [rec, rec, par]
     layers = [dict(order[i % 3], mlp=moe if i % 2 else dense) for i in range(kugilix_runs(s))]
     return {"architecture": "Sumevik", "vocab": VOCAB, "width": W, "norm": {"eps": 1e-6}, "logit_scale": 0.7, "layers": layers}
+
+
+RETEZEN_POOL = 16  # positions to a pooled block
+
+
+def retezen_config(s: dict) -> dict:
+    """As many layers as the Kugilix model has layer runs, all of them attention; the same width, heads, head size; a window
+    as long as the other designs' with blocks of ``RETEZEN_POOL`` before it; values mixed from the second layer on; a gated
+    feed-forward of as many weights as the plain one in the first layer, ``TOP`` of ``EXPERTS`` experts in the others."""
+    H, G, d = s["heads"], s["kv_heads"], s["dim"]
+    mixer = {"heads": H, "kv_heads": G, "dim": d, "vdim": d, "scale": 1.0 / math.sqrt(d), "v_mix": True,
+             "mask": {"size": WINDOW, "pool": RETEZEN_POOL}}
+    moe = {"kind": "moe", "expert": {"ff": netinex_expert_ff(s)}, "router": {"experts": EXPERTS, "top": TOP}}
+    dense = {"kind": "dense", "ff": sumevik_dense_ff(s), "limit": 7.0}
+    return {"architecture": "Retezen", "vocab": VOCAB, "width": s["width"], "max_positions": 8192, "norm": {"eps": 1e-6},
+            "logit_scale": 0.7, "layers": [{"type": "attention", "mixer": mixer, "mlp": moe if i else dense}
+                                           for i in range(kugilix_runs(s))]}
 
 
 def _timed(fn, flush, warmup=3, iters=5, reps=1):
@@ -666,11 +683,135 @@ def sumevik_kernel_numbers(s: dict, peaks: dict) -> dict:
     return out
 
 
+def retezen_kernel_numbers(s: dict, peaks: dict) -> dict:
+    """The Retezen design's own kernels alone at the layer sizes ``s``, measured as ``kernel_numbers`` measures; the attention
+    beside the same kernel without blocks, the clamped gate beside the SiLU one, experts whose weights go onto their inputs."""
+    import torch
+    from types import SimpleNamespace
+
+    from ferrisinfer_b200.engine.workspace import Workspace
+    from ferrisinfer_b200.kernels import ops
+
+    dev = torch.device("cuda")
+    bf = torch.bfloat16
+    flush = torch.zeros(96 << 20, dtype=torch.float32, device=dev)  # 384 MB
+    W, H, G, d = s["width"], s["heads"], s["kv_heads"], s["dim"]
+    hbm = peaks["hbm_gbs"] * 1e9
+    tensor = peaks["bf16_tflops"] * 1e12
+    ws = Workspace(dev)
+    out = {}
+
+    def ctx_of(q_lens, start):
+        S = len(q_lens)
+        q_start = [0]
+        for n in q_lens:
+            q_start.append(q_start[-1] + n)
+        i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+        return SimpleNamespace(num_tokens=q_start[-1], num_seqs=S, max_q_len=max(q_lens), workspace=ws,
+                               max_kv_len=start + max(q_lens),
+                               token_seq=i32([i for i in range(S) for _ in range(q_lens[i])]),
+                               positions=i32([start + j for i in range(S) for j in range(q_lens[i])]),
+                               seq_q_start=i32(q_start), seq_start_pos=i32([start] * S), seq_state_slot=i32(list(range(S))))
+
+    def record(name, seconds, bytes_=None, flops=None, tensor_flops=None):
+        e = {"us": round(seconds * 1e6, 1)}
+        if bytes_ is not None:
+            e["GBps"] = round(bytes_ / seconds / 1e9, 1)
+            e["frac_hbm"] = round(bytes_ / seconds / hbm, 3)
+        if flops is not None:
+            e["TFLOPs_fp32"] = round(flops / seconds / 1e12, 2)
+            e["frac_fp32_nominal"] = round(flops / seconds / (FP32_NOMINAL_TFLOPS * 1e12), 3)
+        if tensor_flops is not None:
+            e["TFLOPs_bf16"] = round(tensor_flops / seconds / 1e12, 1)
+            e["frac_bf16_measured"] = round(tensor_flops / seconds / tensor, 3)
+        out[name] = e
+
+    # ---- the attention over a window and blocks, beside the same kernel over the window alone, and what stands ahead of it
+    P = RETEZEN_POOL
+    for name, batch, q_len, ctx_len in (("decode_b64", 64, 1, 2047), ("decode_b8", 8, 1, 2047), ("prefill_2048", 1, 2048, 0)):
+        T = batch * q_len
+        reps = 10 if T <= 64 else 1
+        pages_each = (ctx_len + q_len + 15) // 16
+        runs_each = (pages_each + P - 1) // P
+        k = torch.randn(batch * pages_each + 1, G, 16, d, device=dev).to(bf)
+        v = torch.randn_like(k)
+        pk = torch.randn(batch * runs_each + 1, G, 16, d, device=dev).to(bf)
+        tables = torch.arange(batch * pages_each, dtype=torch.int32, device=dev).view(batch, pages_each)
+        ptables = torch.arange(batch * runs_each, dtype=torch.int32, device=dev).view(batch, runs_each)
+        pooled = ops.PooledKeys(pk, torch.randn_like(pk), ptables, P)
+        qkv = torch.randn(T, (H + 2 * G) * d, device=dev).to(bf)
+        o = torch.empty(T, H * d, dtype=bf, device=dev)
+        ctx = ctx_of([q_len] * batch, ctx_len)
+        window = [min(WINDOW, ctx_len + j + 1) for j in range(q_len)]
+        blocks = [max(0, ctx_len + j + 1 - WINDOW) // P for j in range(q_len)]
+        for what, pool_arg, keys in (("pooled_attention", pooled, sum(window) + sum(blocks)), ("window_attention", None, sum(window))):
+            t = _timed(lambda: ops.paged_attention_simt(qkv, o, k, v, tables, ctx.token_seq, ctx.positions, H, G, d, WINDOW,
+                                                        1.0 / math.sqrt(d), v_head_dim=d, max_q_len=q_len,
+                                                        max_kv_len=ctx_len + q_len, workspace=ws, pooled=pool_arg), flush)
+            record(f"{what}_{name}", t, flops=4.0 * keys * batch * H * d,
+                   bytes_=batch * G * keys * 2 * d * 2 + T * H * d * 4 if q_len == 1 else None)
+        slots = (tables[ctx.token_seq.long(), (ctx.positions // 16).long()] * 16 + ctx.positions % 16).int()
+        row = (ctx.positions // P).long()
+        pslots = (ptables[ctx.token_seq.long(), row // 16] * 16 + row % 16).int()
+        pslots = torch.where((ctx.positions + 1) % P == 0, pslots, torch.full_like(pslots, -1))
+        qn, kn, lam = torch.ones(H * d, device=dev), torch.ones(G * d, device=dev), torch.full((1,), 0.3, device=dev)
+        first = torch.randn(T, G * d, device=dev).to(bf)
+        extra = {}
+        if q_len == 1:  # (position 2,047 completes a block: the means are in this number)
+            extra = dict(pooled=pooled, pool_slots=pslots, block_tables=tables)
+        t = _timed(lambda: ops.qk_norm_rotary_cache_write(qkv, ctx, slots, k, v, H, G, d, d, qn, kn, 1e-6, None,
+                                                          mixed_values=first, mix_lambda=lam, **extra), flush, reps=10)
+        record(f"qk_norm_mix_{name}", t, bytes_=T * (2 * H * d + 4 * G * d + G * d) * 2 + (batch * (P + 1) * 2 * G * d * 2 if extra else 0))
+        if q_len > 1:
+            t = _timed(lambda: ops.pool_blocks(k, v, pooled, pslots, tables, ctx), flush, reps=10)
+            record(f"block_means_{name}", t, bytes_=(T // P) * (P + 1) * 2 * G * d * 2)
+    # ---- row-wise kernels of a long step and of a decode step
+    for tag, T in (("2048", 2048), ("b64", 64), ("b8", 8)):
+        reps = 10 if T <= 64 else 1
+        y, h, nw = torch.randn(T, W, device=dev), torch.zeros(T, W, device=dev), torch.ones(W, device=dev)
+        rows = torch.empty(T, W, dtype=bf, device=dev)
+        t = _timed(lambda: ops.rmsnorm_add(y, nw, 1e-6, h, rows), flush, reps=reps)
+        record(f"norm_add_{tag}", t, bytes_=T * W * (4 + 4 + 4 + 2))
+        table, pos = torch.randn(VOCAB, W, device=dev).to(bf), torch.randn(4096, W, device=dev).to(bf)
+        ids = torch.randint(0, VOCAB, (T,), dtype=torch.int32, device=dev)
+        ps = torch.arange(T, dtype=torch.int32, device=dev)
+        t = _timed(lambda: ops.embed_positions(table, pos, ids, ps, h, rows), flush, reps=reps)
+        record(f"embed_positions_{tag}", t, bytes_=T * W * (2 + 2 + 4 + 2))
+    # ---- the gated feed-forward: the clamped gate in the products' epilogues beside the SiLU one
+    inter = sumevik_dense_ff(s)
+    gate_up_w = (torch.randn(2 * inter, W, device=dev) / math.sqrt(W)).to(bf)
+    for tag, T in (("b8", 8), ("b64", 64), ("2048", 2048)):
+        x = torch.randn(T, W, device=dev).to(bf)
+        act = torch.empty(T, inter, dtype=bf, device=dev)
+        for kind in ("clamped_swish", "silu"):
+            t = _timed(lambda: ops.gemm_gated(x, gate_up_w, act, kind, 7.0, ws), flush)
+            record(f"gated_product_{kind}_{tag}", t, bytes_=2 * inter * W * 2 + T * (W + inter) * 2,
+                   tensor_flops=2.0 * T * 2 * inter * W)
+    # ---- the sigmoid router and the experts with weights on their inputs
+    eff = netinex_expert_ff(s)
+    gate_up = (torch.randn(EXPERTS, 2 * eff, W, device=dev) / math.sqrt(W)).to(bf)
+    down = (torch.randn(EXPERTS, W, eff, device=dev) / math.sqrt(eff)).to(bf)
+    router = torch.randn(EXPERTS, W, device=dev).to(bf)
+    for tag, T in (("b8", 8), ("b64", 64), ("2048", 2048)):
+        x = torch.randn(T, W, device=dev).to(bf)
+        hrow = torch.zeros(T, W, device=dev)
+        ids = torch.empty(T, TOP, dtype=torch.int32, device=dev)
+        wts = torch.empty(T, TOP, device=dev)
+        t = _timed(lambda: ops.moe_router(x, router, None, ids, wts, TOP, sigmoid=True), flush, reps=10)
+        record(f"sigmoid_router_{tag}", t, bytes_=T * W * 2 + EXPERTS * W * 2)
+        distinct = int(torch.unique(ids).numel())
+        t = _timed(lambda: ops.moe_experts(x, gate_up, down, ids, wts, hrow, ws, accumulate=False, input_weights=True), flush)
+        record(f"experts_input_weights_{tag}", t, bytes_=distinct * 3 * W * eff * 2 + T * W * (2 + 4),
+               tensor_flops=2.0 * T * TOP * 3 * W * eff)
+        out[f"experts_input_weights_{tag}"]["distinct_experts"] = distinct
+    return out
+
+
 def run(build_engine, time_decode, time_prefill, peaks, steps=32, warmup=4, sizes=("small", "1B-like"), context=2048,
         prompt=2048, batches=(8, 64), kernels_at="1B-like", design="kugilix") -> dict:
     """``build_engine(cfg, batch, context, extra_tokens)``, ``time_decode`` and ``time_prefill`` are bench.py's.
-    ``design`` "kugilix": that design beside Qwen2; "nusudra" or "netinex": that design beside both; "sumevik": that
-    design beside Netinex and Qwen2."""
+    ``design`` "kugilix": that design beside Qwen2; "nusudra" or "netinex": that design beside both; "sumevik" or "retezen":
+    that design beside Netinex and Qwen2."""
     import torch
 
     result = {"context": context, "prompt_tokens": prompt, "window": WINDOW, "sizes": {}}
@@ -682,8 +823,9 @@ def run(build_engine, time_decode, time_prefill, peaks, steps=32, warmup=4, size
             designs = (("nusudra", nusudra_config(s)),) + designs
         if design == "netinex":
             designs = (("netinex", netinex_config(s)),) + designs
-        if design == "sumevik":
-            designs = (("sumevik", sumevik_config(s)), ("netinex", netinex_config(s)), ("qwen2", qwen2_config(s)))
+        if design in ("sumevik", "retezen"):
+            own = sumevik_config(s) if design == "sumevik" else retezen_config(s)
+            designs = ((design, own), ("netinex", netinex_config(s)), ("qwen2", qwen2_config(s)))
         for design_name, cfg in designs:
             numbers = {}
             engine = build_engine(cfg, 1, context, extra_tokens=prompt)
@@ -703,7 +845,12 @@ def run(build_engine, time_decode, time_prefill, peaks, steps=32, warmup=4, size
                 torch.cuda.empty_cache()
             entry[design_name] = numbers
         result["sizes"][name] = entry
-    if kernels_at and design == "sumevik":
+    if kernels_at and design == "retezen":
+        result["kernels_retezen"] = {"at": kernels_at, "expert_ff": netinex_expert_ff(SIZES[kernels_at]), "experts": EXPERTS,
+                                     "top": TOP, "pool": RETEZEN_POOL, **retezen_kernel_numbers(SIZES[kernels_at], peaks)}
+        result["kernels_netinex"] = {"at": kernels_at, "expert_ff": netinex_expert_ff(SIZES[kernels_at]),
+                                     "experts": EXPERTS, "top": TOP, **netinex_kernel_numbers(SIZES[kernels_at], peaks)}
+    elif kernels_at and design == "sumevik":
         result["kernels_sumevik"] = {"at": kernels_at, "expert_ff": netinex_expert_ff(SIZES[kernels_at]), "experts": EXPERTS,
                                      "identity": SUMEVIK_IDENTITY, "top": TOP,
                                      **sumevik_kernel_numbers(SIZES[kernels_at], peaks)}
