@@ -1,0 +1,592 @@
+// The general attention over a bf16 cache on tensor cores, with the softmax's weights in 32-bit: head sizes of any multiple
+// of eight up to 256 (the values' may differ), any page size, any grouping of heads, a window, a chunk or every key, pooled
+// keys before the window, a sink.  The formulas and arguments are those of attention_simt.cu.
+//
+// q . k is a product of bf16 numbers with fp32 sums, as exact as FMAs on the widened numbers.  The second product, weights
+// times values, must not round the weights to bf16: a weight p is cut into three bf16 parts, p1 = bf16(p), p2 = bf16(p - p1),
+// p3 = bf16(p - p1 - p2), whose sum is p to the last of its 24 bits, and the three products with the values meet in one fp32
+// accumulator.  Scores, maximum, exponentials and sums are fp32 (powers of two: the scale carries log2 e).
+//
+// Two kernels.  Portions of prompts: a block takes 64 rows, the g query heads of one kv head for floor(64 / g) consecutive
+// tokens, and walks the keys in tiles that asynchronous copies bring into shared memory one tile ahead; each of its four
+// warps owns 16 rows.  Single tokens: a block takes one token, one kv head (its up to 16 query heads are the rows of the
+// fragments) and a share of the keys; each of its four warps walks chunks of 16 keys of its own through a ring of
+// asynchronous copies that only it reads (no block-wide barrier in the loop), and the four meet in shared memory at the
+// end; several shares of a token are merged by attention_merge_shares_kernel.
+#include <math.h>
+
+#include "attention_general.cuh"
+#include "common.cuh"
+#include "sm100.cuh"
+
+namespace {
+
+constexpr float LOG2E = 1.4426950408889634f;
+constexpr int AR_THREADS = 128, AR_WARPS = 4, AR_ROWS = 64;
+constexpr int AS_KEYS = 16, AS_STAGES = 3;  // single tokens: keys of a warp's chunk, chunks in its ring
+
+// 16 bytes into shared memory, or 16 zero bytes where the row is not there
+__device__ __forceinline__ void copy16_or_zero(uint32_t dst, const void* src, bool there) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(there ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ void ar_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void ar_wait() {
+    asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory");
+}
+
+// The pair (a, b) as three packed pairs of bf16 whose sums are a and b.
+__device__ __forceinline__ void split3(float a, float b, uint32_t& p1, uint32_t& p2, uint32_t& p3) {
+    p1 = pack_bf16(a, b);
+    a -= __uint_as_float(p1 << 16), b -= __uint_as_float(p1 & 0xffff0000u);
+    p2 = pack_bf16(a, b);
+    a -= __uint_as_float(p2 << 16), b -= __uint_as_float(p2 & 0xffff0000u);
+    p3 = pack_bf16(a, b);
+}
+
+// Fragments of 16 query rows straight from global memory (a null row reads as zero); nks steps of 16 columns, the columns
+// from d on are zero.
+template <int KS>
+__device__ __forceinline__ void load_q_rows(uint32_t (&qf)[KS][4], const bf16* row0, const bf16* row1, int d) {
+    const int t = threadIdx.x & 3;
+#pragma unroll
+    for (int ks = 0; ks < KS; ++ks) {
+        const int c = 16 * ks + 2 * t;
+        qf[ks][0] = row0 && c < d ? *reinterpret_cast<const uint32_t*>(row0 + c) : 0u;
+        qf[ks][1] = row1 && c < d ? *reinterpret_cast<const uint32_t*>(row1 + c) : 0u;
+        qf[ks][2] = row0 && c + 8 < d ? *reinterpret_cast<const uint32_t*>(row0 + c + 8) : 0u;
+        qf[ks][3] = row1 && c + 8 < d ? *reinterpret_cast<const uint32_t*>(row1 + c + 8) : 0u;
+    }
+}
+
+struct AttentionArgs {
+    const bf16* q;
+    bf16* out;
+    const bf16* k;
+    const bf16* v;
+    const int* tables;
+    const int* token_seq;
+    const int* positions;
+    const float* sink;
+    PooledKeys pk;  // every = 0: none
+    int ldq, ldo, max_blocks, tokens, nh, nkv, d, dv, page_size, window;
+    float scale2;  // scale x log2 e
+};
+
+__device__ __forceinline__ int page_of(const int* table, int j, int page_size, int pshift) {
+    return table[pshift >= 0 ? (j >> pshift) : (j / page_size)];
+}
+__device__ __forceinline__ size_t row_of(int page, int head, int nkv, int j, int page_size, int pshift) {
+    return ((size_t)page * nkv + head) * page_size + (pshift >= 0 ? (j & (page_size - 1)) : (j % page_size));
+}
+__device__ __forceinline__ int shift_of(int page_size) {
+    return (page_size & (page_size - 1)) == 0 ? __ffs(page_size) - 1 : -1;
+}
+
+// One row pair's step of the running softmax over a tile of scores s (NT blocks of 8 keys; scaled, unseen ones -inf):
+// scores become weights, the accumulators are brought to the new maximum.
+template <int NT, int DT>
+__device__ __forceinline__ void softmax_step(float (&s)[NT][4], float (&m)[2], float (&l)[2], float (&o)[DT][4]) {
+    float alpha[2];
+    bool moved = false;
+#pragma unroll
+    for (int a = 0; a < 2; ++a) {
+        float best = -INFINITY;
+#pragma unroll
+        for (int n = 0; n < NT; ++n) best = fmaxf(best, fmaxf(s[n][2 * a], s[n][2 * a + 1]));
+        best = fmaxf(best, __shfl_xor_sync(0xffffffffu, best, 1));
+        best = fmaxf(best, __shfl_xor_sync(0xffffffffu, best, 2));
+        const float m_new = fmaxf(m[a], best);
+        const float base = m_new == -INFINITY ? 0.0f : m_new;  // a row that has seen nothing yet: every weight is 0
+        alpha[a] = exp2f(m[a] - base);
+        moved |= m_new != m[a];
+        m[a] = m_new;
+        float sum = 0.0f;
+#pragma unroll
+        for (int n = 0; n < NT; ++n) {
+            s[n][2 * a] = exp2f(s[n][2 * a] - base);
+            s[n][2 * a + 1] = exp2f(s[n][2 * a + 1] - base);
+            sum += s[n][2 * a] + s[n][2 * a + 1];
+        }
+        l[a] = l[a] * alpha[a] + sum;
+    }
+    if (__any_sync(0xffffffffu, moved)) {
+#pragma unroll
+        for (int n = 0; n < DT; ++n) o[n][0] *= alpha[0], o[n][1] *= alpha[0], o[n][2] *= alpha[1], o[n][3] *= alpha[1];
+    }
+}
+
+// o += weights of 16 keys (blocks 2 kk and 2 kk + 1 of s) times their values (rows of pitch vp bytes from v_base).
+template <int NT, int DT>
+__device__ __forceinline__ void weights_times_values(float (&o)[DT][4], const float (&s)[NT][4], int kk, uint32_t v_base, int vp,
+                                                     int dv) {
+    const int lane = threadIdx.x & 31;
+    uint32_t p[3][4];
+    split3(s[2 * kk][0], s[2 * kk][1], p[0][0], p[1][0], p[2][0]);
+    split3(s[2 * kk][2], s[2 * kk][3], p[0][1], p[1][1], p[2][1]);
+    split3(s[2 * kk + 1][0], s[2 * kk + 1][1], p[0][2], p[1][2], p[2][2]);
+    split3(s[2 * kk + 1][2], s[2 * kk + 1][3], p[0][3], p[1][3], p[2][3]);
+    const uint32_t at = v_base + (uint32_t)(16 * kk + ((lane >> 3) & 1) * 8 + (lane & 7)) * vp + (lane >> 4) * 16;
+#pragma unroll
+    for (int n = 0; n < DT; n += 2) {
+        if (8 * n < dv) {
+            uint32_t b[4];
+            ldmatrix_x4_trans(b, at + n * 16);
+#pragma unroll
+            for (int x = 0; x < 3; ++x) {
+                mma_bf16_16816(o[n], p[x], b[0], b[1]);
+                mma_bf16_16816(o[n + 1], p[x], b[2], b[3]);
+            }
+        }
+    }
+}
+
+// ------------------------------------------------------------------------------------------ portions of prompts
+// D: columns held for a head (64, 128, 256; d, dv <= D).  KT: keys to a tile.  The query fragments stay in registers up to
+// D = 128 and come from shared memory beyond.
+template <int D, int KT, bool POOL>
+__global__ void __launch_bounds__(AR_THREADS) attention_rows_kernel(const AttentionArgs p) {
+    constexpr int KS = D / 16, DT = D / 8, NT = KT / 8;
+    constexpr bool QREG = D <= 128;
+    extern __shared__ __align__(16) uint8_t ar_smem[];
+    constexpr int PITCH = (D + 8) * 2;  // bytes of a row: 16 more than the columns, so that eight rows lie in different banks
+    const uint32_t base = smem_u32(ar_smem);
+    constexpr uint32_t V_OFF = KT * PITCH, STAGE = 2 * KT * PITCH, Q_OFF = 2 * STAGE;
+    pdl_wait();
+    pdl_launch_dependents();
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gq = lane >> 2, tq = lane & 3;
+    const int g = p.nh / p.nkv, qt = AR_ROWS / g;
+    const int hk = blockIdx.y;
+    const int t_first = (gridDim.x - 1 - blockIdx.x) * qt;  // the last tokens, which see most keys, first
+    const int t_end = min(t_first + qt, p.tokens);
+    const int pshift = shift_of(p.page_size);
+    const int d = p.d, dv = p.dv;
+    const int nks = (d + 15) >> 4;
+
+    // columns between d and the next multiple of 16 are zero on both sides
+    if (d & 15) {
+        for (int r = tid; r < 2 * KT; r += AR_THREADS)
+            *reinterpret_cast<uint4*>(ar_smem + (r / KT) * STAGE + (r % KT) * PITCH + d * 2) = make_uint4(0u, 0u, 0u, 0u);
+    }
+    int rt[2], rpos[2], rseq[2];
+    const bf16* qrow[2];
+#pragma unroll
+    for (int a = 0; a < 2; ++a) {
+        const int r = 16 * warp + gq + 8 * a;
+        rt[a] = r < qt * g ? t_first + r / g : p.tokens;
+        const bool ok = rt[a] < t_end;
+        rpos[a] = ok ? p.positions[rt[a]] : -1;
+        rseq[a] = ok ? p.token_seq[rt[a]] : -1;
+        qrow[a] = ok ? p.q + (size_t)rt[a] * p.ldq + (size_t)(hk * g + r % g) * d : nullptr;
+    }
+    uint32_t qf[QREG ? KS : 1][4];
+    if constexpr (QREG) {
+        load_q_rows<KS>(qf, qrow[0], qrow[1], d);
+    } else {
+        for (int x = tid; x < AR_ROWS * (D / 8); x += AR_THREADS) {
+            const int r = x / (D / 8), c = x % (D / 8);
+            const int t = r < qt * g ? t_first + r / g : p.tokens;
+            uint4 u = make_uint4(0u, 0u, 0u, 0u);
+            if (t < t_end && 8 * c < d)
+                u = *reinterpret_cast<const uint4*>(p.q + (size_t)t * p.ldq + (size_t)(hk * g + r % g) * d + 8 * c);
+            *reinterpret_cast<uint4*>(ar_smem + Q_OFF + r * PITCH + c * 16) = u;
+        }
+    }
+    float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.0f, 0.0f};
+    float o[DT][4];
+#pragma unroll
+    for (int n = 0; n < DT; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) o[n][e] = 0.0f;
+
+    const int seq_first = p.token_seq[t_first], seq_last = p.token_seq[t_end - 1];
+    int ta = t_first;  // first token of the current request within the tile
+    for (int sq = seq_first; sq <= seq_last; ++sq) {
+        int tb = ta;  // its last token within the tile
+        while (tb + 1 < t_end && p.token_seq[tb + 1] == sq) ++tb;
+        const int pa = p.positions[ta], pb = p.positions[tb];
+        const int kmin = first_key(pa, p.window);  // of the first token: no later token of the request sees an earlier key
+        const int runs = POOL ? first_key(pb, p.window) / p.pk.every : 0;
+        const int run_tiles = (runs + KT - 1) / KT;
+        const int tiles = run_tiles + (pb - kmin + KT) / KT;
+        const int* table = p.tables + (size_t)sq * p.max_blocks;
+        const int* ptable = POOL ? p.pk.tables + (size_t)sq * p.pk.max_blocks : nullptr;
+        constexpr int TPK = AR_THREADS / KT;  // threads that copy a key
+        const int key = tid / TPK, part = tid % TPK;
+        auto page_at = [&](int i) -> int {  // page of this thread's key in tile i, -1 if the tile does not hold it
+            if (i >= tiles) return -1;
+            if (POOL && i < run_tiles) {
+                const int j = i * KT + key;
+                return j < runs ? page_of(ptable, j, p.page_size, pshift) : -1;
+            }
+            const int j = kmin + (i - run_tiles) * KT + key;
+            return j <= pb ? page_of(table, j, p.page_size, pshift) : -1;
+        };
+        auto fetch = [&](int i, int page) {
+            if (i < tiles) {
+                const bool run = POOL && i < run_tiles;
+                const int j = run ? i * KT + key : kmin + (i - run_tiles) * KT + key;
+                const bool there = page >= 0;
+                const size_t row = there ? row_of(page, hk, p.nkv, j, p.page_size, pshift) : 0;
+                const bf16* ks = (run ? reinterpret_cast<const bf16*>(p.pk.k) : p.k) + row * d;
+                const bf16* vs = (run ? reinterpret_cast<const bf16*>(p.pk.v) : p.v) + row * dv;
+                const uint32_t dst = base + (i & 1) * STAGE + key * PITCH;
+                for (int c = part; c < (d >> 3); c += TPK) copy16_or_zero(dst + c * 16, ks + 8 * c, there);
+                for (int c = part; c < (dv >> 3); c += TPK) copy16_or_zero(dst + V_OFF + c * 16, vs + 8 * c, there);
+            }
+            ar_commit();
+        };
+        __syncthreads();  // the request before has been read (and, the first time, the zero columns and queries are in place)
+        fetch(0, page_at(0));
+        int next_page = page_at(1);
+        int hi[2], lo[2], seen_runs[2];
+#pragma unroll
+        for (int a = 0; a < 2; ++a) {
+            const bool mine = rseq[a] == sq;
+            lo[a] = mine ? first_key(rpos[a], p.window) : 0;
+            hi[a] = mine ? rpos[a] : -1;
+            seen_runs[a] = POOL && mine ? lo[a] / p.pk.every : 0;
+        }
+        for (int i = 0; i < tiles; ++i) {
+            fetch(i + 1, next_page);
+            next_page = page_at(i + 2);
+            ar_wait<1>();
+            __syncthreads();
+            const uint32_t kb = base + (i & 1) * STAGE;
+            float s[NT][4];
+#pragma unroll
+            for (int n = 0; n < NT; ++n)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) s[n][e] = 0.0f;
+            const uint32_t k_at = kb + (uint32_t)((lane >> 4) * 8 + (lane & 7)) * PITCH + ((lane >> 3) & 1) * 16;
+            const uint32_t q_at = base + Q_OFF + (uint32_t)(16 * warp + (lane & 7) + ((lane >> 3) & 1) * 8) * PITCH + (lane >> 4) * 16;
+#pragma unroll
+            for (int ks = 0; ks < KS; ++ks) {
+                if (ks < nks) {
+                    uint32_t af[4];
+                    if constexpr (QREG) {
+#pragma unroll
+                        for (int e = 0; e < 4; ++e) af[e] = qf[ks][e];
+                    } else {
+                        ldmatrix_x4(af, q_at + ks * 32);
+                    }
+#pragma unroll
+                    for (int n = 0; n < NT; n += 2) {
+                        uint32_t b[4];
+                        ldmatrix_x4(b, k_at + (uint32_t)(8 * n) * PITCH + ks * 32);
+                        mma_bf16_16816(s[n], af, b[0], b[1]);
+                        mma_bf16_16816(s[n + 1], af, b[2], b[3]);
+                    }
+                }
+            }
+            const bool run = POOL && i < run_tiles;
+            const int j0 = run ? i * KT : kmin + (i - run_tiles) * KT;
+            int from[2], to[2];  // of the tile's keys, those that the rows see
+#pragma unroll
+            for (int a = 0; a < 2; ++a) {
+                from[a] = run ? 0 : lo[a] - j0;
+                to[a] = (run ? seen_runs[a] - 1 : hi[a]) - j0;
+            }
+            const bool whole = from[0] <= 0 && from[1] <= 0 && to[0] >= KT - 1 && to[1] >= KT - 1;
+            if (__all_sync(0xffffffffu, whole)) {
+#pragma unroll
+                for (int n = 0; n < NT; ++n)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) s[n][e] *= p.scale2;
+            } else {
+#pragma unroll
+                for (int n = 0; n < NT; ++n)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        const int c = 8 * n + 2 * tq + (e & 1);
+                        s[n][e] = c >= from[e >> 1] && c <= to[e >> 1] ? s[n][e] * p.scale2 : -INFINITY;
+                    }
+            }
+            softmax_step<NT, DT>(s, m, l, o);
+#pragma unroll
+            for (int kk = 0; kk < KT / 16; ++kk) weights_times_values<NT, DT>(o, s, kk, kb + V_OFF, PITCH, dv);
+            __syncthreads();  // the stage is read: the copies after next may overwrite it
+        }
+        ta = tb + 1;
+    }
+    ar_wait<0>();
+#pragma unroll
+    for (int a = 0; a < 2; ++a) {
+        l[a] += __shfl_xor_sync(0xffffffffu, l[a], 1);
+        l[a] += __shfl_xor_sync(0xffffffffu, l[a], 2);
+        if (rt[a] >= t_end) continue;
+        const int head = hk * g + (16 * warp + gq + 8 * a) % g;
+        const float sink = p.sink ? exp2f(p.sink[head] * LOG2E - m[a]) : 0.0f;
+        const float inv = 1.0f / (l[a] + sink);
+        bf16* orow = p.out + (size_t)rt[a] * p.ldo + (size_t)head * dv;
+#pragma unroll
+        for (int n = 0; n < DT; ++n) {
+            const int c = 8 * n + 2 * tq;
+            if (c < dv) *reinterpret_cast<uint32_t*>(orow + c) = pack_bf16(o[n][2 * a] * inv, o[n][2 * a + 1] * inv);
+        }
+    }
+}
+
+template <int D>
+constexpr int rows_keys() { return D <= 128 ? 64 : 32; }
+template <int D>
+constexpr size_t rows_smem() {
+    return (size_t)4 * rows_keys<D>() * (D + 8) * 2 + (D <= 128 ? 0 : (size_t)AR_ROWS * (D + 8) * 2);
+}
+
+// ------------------------------------------------------------------------------------------ single tokens
+// partial (splits > 1): per (token, head, share): maximum (natural units), sum, weighted values, as the merge kernel reads.
+template <int D, bool POOL>
+__global__ void __launch_bounds__(AR_THREADS) attention_single_rows_kernel(const AttentionArgs p, int row_groups, int splits,
+                                                                           float* partial) {
+    constexpr int KS = D / 16, DT = D / 8, NT = AS_KEYS / 8;
+    constexpr int PITCH = (D + 8) * 2;
+    constexpr uint32_t V_OFF = AS_KEYS * PITCH, STAGE = 2 * AS_KEYS * PITCH;
+    extern __shared__ __align__(16) uint8_t ar_smem[];
+    pdl_wait();
+    pdl_launch_dependents();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gq = lane >> 2, tq = lane & 3;
+    const int t = blockIdx.x, hk = blockIdx.y / row_groups, r0 = (blockIdx.y % row_groups) * 16, split = blockIdx.z;
+    const int g = p.nh / p.nkv, rows = min(16, g - r0);
+    const int seq = p.token_seq[t], P = p.positions[t];
+    const int pshift = shift_of(p.page_size);
+    const int d = p.d, dv = p.dv;
+    const int nks = (d + 15) >> 4;
+    const int lo = first_key(P, p.window);
+    const int pooled = POOL ? lo / p.pk.every : 0;
+    const int shift = lo - pooled;  // key n >= pooled is the token at n + shift
+    const int total = pooled + P - lo + 1;
+    // this block's share of the keys, in whole chunks
+    const int chunks_all = (total + AS_KEYS - 1) / AS_KEYS;
+    const int per = (chunks_all + splits - 1) / splits;
+    const int c_first = split * per, c_end = min(chunks_all, c_first + per);
+    const int* table = p.tables + (size_t)seq * p.max_blocks;
+    const int* ptable = POOL ? p.pk.tables + (size_t)seq * p.pk.max_blocks : nullptr;
+
+    uint8_t* mine = ar_smem + warp * AS_STAGES * STAGE;
+    const uint32_t ring = smem_u32(mine);
+    if (d & 15) {
+        for (int r = lane; r < AS_STAGES * AS_KEYS; r += 32)
+            *reinterpret_cast<uint4*>(mine + (r / AS_KEYS) * STAGE + (r % AS_KEYS) * PITCH + d * 2) = make_uint4(0u, 0u, 0u, 0u);
+    }
+    const bf16* qbase = p.q + (size_t)t * p.ldq + (size_t)(hk * g + r0) * d;
+    uint32_t qf[KS][4];
+    load_q_rows<KS>(qf, gq < rows ? qbase + (size_t)gq * d : nullptr, gq + 8 < rows ? qbase + (size_t)(gq + 8) * d : nullptr, d);
+    float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.0f, 0.0f};
+    float o[DT][4];
+#pragma unroll
+    for (int n = 0; n < DT; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) o[n][e] = 0.0f;
+
+    const int key = lane >> 1, part = lane & 1;
+    // chunk number i of this warp is c_first + warp + 4 i
+    auto page_at = [&](int i) -> int {
+        const int n = (c_first + warp + AR_WARPS * i) * AS_KEYS + key;
+        if (c_first + warp + AR_WARPS * i >= c_end || n >= total) return -1;
+        return POOL && n < pooled ? page_of(ptable, n, p.page_size, pshift) : page_of(table, n + shift, p.page_size, pshift);
+    };
+    auto fetch = [&](int i, int stage, int page) {
+        if (c_first + warp + AR_WARPS * i < c_end) {
+            const int n = (c_first + warp + AR_WARPS * i) * AS_KEYS + key;
+            const bool run = POOL && n < pooled, there = page >= 0;
+            const size_t row = there ? row_of(page, hk, p.nkv, run ? n : n + shift, p.page_size, pshift) : 0;
+            const bf16* ks = (run ? reinterpret_cast<const bf16*>(p.pk.k) : p.k) + row * d;
+            const bf16* vs = (run ? reinterpret_cast<const bf16*>(p.pk.v) : p.v) + row * dv;
+            const uint32_t dst = ring + stage * STAGE + key * PITCH;
+            for (int c = part; c < (d >> 3); c += 2) copy16_or_zero(dst + c * 16, ks + 8 * c, there);
+            for (int c = part; c < (dv >> 3); c += 2) copy16_or_zero(dst + V_OFF + c * 16, vs + 8 * c, there);
+        }
+        ar_commit();
+    };
+    const int own = c_end - c_first - warp > 0 ? (c_end - c_first - warp + AR_WARPS - 1) / AR_WARPS : 0;
+    int pages[AS_STAGES];
+#pragma unroll
+    for (int i = 0; i < AS_STAGES; ++i) pages[i] = page_at(i);
+#pragma unroll
+    for (int i = 0; i < AS_STAGES - 1; ++i) fetch(i, i, pages[i]);
+    int next_page = pages[AS_STAGES - 1];
+    int stage = 0, fill = AS_STAGES - 1;
+    for (int i = 0; i < own; ++i) {
+        fetch(i + AS_STAGES - 1, fill, next_page);
+        next_page = page_at(i + AS_STAGES);
+        ar_wait<AS_STAGES - 1>();
+        __syncwarp();
+        const uint32_t kb = ring + stage * STAGE;
+        float s[NT][4];
+#pragma unroll
+        for (int n = 0; n < NT; ++n)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) s[n][e] = 0.0f;
+        const uint32_t k_at = kb + (uint32_t)((lane >> 4) * 8 + (lane & 7)) * PITCH + ((lane >> 3) & 1) * 16;
+#pragma unroll
+        for (int ks = 0; ks < KS; ++ks) {
+            if (ks < nks) {
+                uint32_t b[4];
+                ldmatrix_x4(b, k_at + ks * 32);
+                mma_bf16_16816(s[0], qf[ks], b[0], b[1]);
+                mma_bf16_16816(s[1], qf[ks], b[2], b[3]);
+            }
+        }
+        const int left = total - (c_first + warp + AR_WARPS * i) * AS_KEYS;  // keys of the chunk that exist
+#pragma unroll
+        for (int n = 0; n < NT; ++n)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) s[n][e] = 8 * n + 2 * tq + (e & 1) < left ? s[n][e] * p.scale2 : -INFINITY;
+        softmax_step<NT, DT>(s, m, l, o);
+        weights_times_values<NT, DT>(o, s, 0, kb + V_OFF, PITCH, dv);
+        __syncwarp();  // the stage is read: the copy after next may overwrite it
+        stage = stage + 1 == AS_STAGES ? 0 : stage + 1;
+        fill = fill + 1 == AS_STAGES ? 0 : fill + 1;
+    }
+    ar_wait<0>();
+    // the four warps meet: per warp and row its maximum, sum and weighted values
+    float* meet = reinterpret_cast<float*>(ar_smem);
+    const int stride = dv + 2;
+    __syncthreads();
+#pragma unroll
+    for (int a = 0; a < 2; ++a) {
+        l[a] += __shfl_xor_sync(0xffffffffu, l[a], 1);
+        l[a] += __shfl_xor_sync(0xffffffffu, l[a], 2);
+        const int r = gq + 8 * a;
+        if (r < rows) {
+            float* e = meet + (size_t)(warp * rows + r) * stride;
+            if (tq == 0) e[0] = m[a], e[1] = l[a];
+#pragma unroll
+            for (int n = 0; n < DT; ++n) {
+                const int c = 8 * n + 2 * tq;
+                if (c < dv) *reinterpret_cast<float2*>(e + 2 + c) = make_float2(o[n][2 * a], o[n][2 * a + 1]);
+            }
+        }
+    }
+    __syncthreads();
+    for (int x = threadIdx.x; x < rows * dv; x += AR_THREADS) {
+        const int r = x / dv, i = x - r * dv;
+        float mm = -INFINITY;
+#pragma unroll
+        for (int w = 0; w < AR_WARPS; ++w) mm = fmaxf(mm, meet[(size_t)(w * rows + r) * stride]);
+        float zz = 0.0f, acc = 0.0f;
+#pragma unroll
+        for (int w = 0; w < AR_WARPS; ++w) {
+            const float* e = meet + (size_t)(w * rows + r) * stride;
+            const float f = e[0] == -INFINITY ? 0.0f : exp2f(e[0] - mm);
+            zz = fmaf(e[1], f, zz), acc = fmaf(e[2 + i], f, acc);
+        }
+        const int head = hk * g + r0 + r;
+        if (splits == 1) {
+            if (p.sink) zz += exp2f(p.sink[head] * LOG2E - mm);
+            p.out[(size_t)t * p.ldo + (size_t)head * dv + i] = from_float<bf16>(acc / zz);
+        } else {
+            float* e = partial + (((size_t)t * p.nh + head) * splits + split) * stride;
+            if (i == 0) e[0] = mm / LOG2E, e[1] = zz;
+            e[2 + i] = acc;
+        }
+    }
+}
+
+template <int D>
+constexpr size_t single_smem() {
+    return (size_t)AR_WARPS * AS_STAGES * 2 * AS_KEYS * (D + 8) * 2;
+}
+
+int rows_bucket(int d, int dv) {
+    const int most = d > dv ? d : dv;
+    return most <= 64 ? 64 : (most <= 128 ? 128 : 256);
+}
+
+int device_sms() {
+    static int sms = 0;
+    if (sms <= 0) {
+        int dev = 0;
+        cudaGetDevice(&dev);
+        if (cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess || sms <= 0) sms = 148;
+    }
+    return sms;
+}
+
+template <int D, bool POOL>
+int launch_rows(const AttentionArgs& p, cudaStream_t s) {
+    const int qt = AR_ROWS / (p.nh / p.nkv);
+    constexpr int KT = rows_keys<D>();
+    constexpr size_t smem = rows_smem<D>();
+    int rc = ferris_allow_dynamic_smem((const void*)attention_rows_kernel<D, KT, POOL>, smem);
+    if (rc != FERRIS_OK) return rc;
+    ferris_launch(attention_rows_kernel<D, KT, POOL>, dim3((p.tokens + qt - 1) / qt, p.nkv), dim3(AR_THREADS), smem, s, p);
+    FERRIS_LAUNCH_CHECK();
+}
+
+template <int D, bool POOL>
+int launch_single(const AttentionArgs& p, int splits, float* partial, cudaStream_t s) {
+    const int groups = (p.nh / p.nkv + 15) / 16;
+    constexpr size_t smem = single_smem<D>();
+    static_assert((size_t)AR_WARPS * 16 * (D + 2) * sizeof(float) <= smem, "the warps meet in the ring's memory");
+    int rc = ferris_allow_dynamic_smem((const void*)attention_single_rows_kernel<D, POOL>, smem);
+    if (rc != FERRIS_OK) return rc;
+    ferris_launch(attention_single_rows_kernel<D, POOL>, dim3(p.tokens, p.nkv * groups, splits), dim3(AR_THREADS), smem, s, p,
+                  groups, splits, partial);
+    if (splits > 1) {
+        const ScoreTerms st = {nullptr, nullptr, nullptr, p.sink, 0};
+        ferris_launch(attention_merge_shares_kernel<bf16>, dim3(p.tokens, p.nh), dim3(128), 0, s, (const float*)partial, p.out,
+                      p.ldo, p.nh, p.dv, splits, st);
+    }
+    FERRIS_LAUNCH_CHECK();
+}
+
+}  // namespace
+
+// Whether ferris_attention_rows takes a geometry (bf16).  portions: 1 = the kernel for portions of prompts, 0 = single tokens.
+FERRIS_API int ferris_attention_rows_takes(int nh, int nkv, int d, int dv, int portions) {
+    if (nh <= 0 || nkv <= 0 || nh % nkv || d <= 0 || dv <= 0 || d % 8 || dv % 8 || d > 256 || dv > 256) return 0;
+    if (nkv > 65535 || (long long)nkv * ((nh / nkv + 15) / 16) > 65535) return 0;
+    return portions ? nh / nkv <= AR_ROWS : 1;
+}
+
+// Arguments as ferris_paged_attention_simt, bf16 throughout, no distance penalty, values in rows of their own.  portions:
+// requests bring several tokens each (the kernel of 64-row blocks); else kv_span (the most keys a token sees) and scratch
+// (fp32, for shares of the keys; may be null) as there.  Returns the number of launches through *launches.
+FERRIS_API int ferris_attention_rows(const void* q, int ldq, void* out, int ldo, const void* k_cache, const void* v_cache,
+                                     const int* block_tables, int max_blocks, const int* token_seq, const int* positions,
+                                     int tokens, int nh, int nkv, int d, int dv, int page_size, int window, float scale,
+                                     const float* sink, const void* pool_k, const void* pool_v, const int* pool_tables,
+                                     int pool_max_blocks, int pool_every, int portions, int kv_span, float* scratch,
+                                     long long scratch_floats, int* launches, void* stream) {
+    if (launches) *launches = 0;
+    if (tokens <= 0) return FERRIS_OK;
+    if (!ferris_attention_rows_takes(nh, nkv, d, dv, portions))
+        FERRIS_REFUSE("attention rows: %d heads over %d kv heads of %d / %d are not taken", nh, nkv, d, dv);
+    if (page_size <= 0 || max_blocks <= 0) FERRIS_REFUSE("attention: page_size=%d max_blocks=%d", page_size, max_blocks);
+    const ScoreTerms st = {nullptr, nullptr, nullptr, sink, 0};
+    const PooledKeys pk = {pool_k, pool_v, pool_tables, pool_max_blocks, pool_every};
+    if (int rc = check_pooled(pk, window, st)) return rc;
+    if ((((uintptr_t)q | (uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)pool_k | (uintptr_t)pool_v) & 15) != 0 || ldq % 8 ||
+        ((uintptr_t)out & 3) || (ldo & 1))
+        FERRIS_REFUSE("attention rows: rows must start on 16 bytes");
+    const AttentionArgs p = {(const bf16*)q, (bf16*)out, (const bf16*)k_cache, (const bf16*)v_cache, block_tables, token_seq,
+                             positions, sink, pk, ldq, ldo, max_blocks, tokens, nh, nkv, d, dv, page_size, window,
+                             scale * LOG2E};
+    cudaStream_t s = (cudaStream_t)stream;
+    const bool pool = pk.every > 0;
+    const int bucket = rows_bucket(d, dv);
+    if (portions) {
+        if (launches) *launches = 1;
+        if (bucket == 64) return pool ? launch_rows<64, true>(p, s) : launch_rows<64, false>(p, s);
+        if (bucket == 128) return pool ? launch_rows<128, true>(p, s) : launch_rows<128, false>(p, s);
+        return pool ? launch_rows<256, true>(p, s) : launch_rows<256, false>(p, s);
+    }
+    // shares of a token's keys: as many as fill the SMs about three times over, of 64 keys at least
+    int splits = 1;
+    if (scratch && kv_span > 0) {
+        const long long blocks = (long long)tokens * nkv * ((nh / nkv + 15) / 16);
+        long long want = 3LL * device_sms() / blocks;
+        const long long most = kv_span / 64;
+        if (want > most) want = most;
+        if (want > 16) want = 16;
+        const long long fit = scratch_floats / ((long long)tokens * nh * (dv + 2));
+        if (want > fit) want = fit;
+        if (want > 1) splits = (int)want;
+    }
+    if (launches) *launches = splits > 1 ? 2 : 1;
+    if (bucket == 64) return pool ? launch_single<64, true>(p, splits, scratch, s) : launch_single<64, false>(p, splits, scratch, s);
+    if (bucket == 128) return pool ? launch_single<128, true>(p, splits, scratch, s) : launch_single<128, false>(p, splits, scratch, s);
+    return pool ? launch_single<256, true>(p, splits, scratch, s) : launch_single<256, false>(p, splits, scratch, s);
+}

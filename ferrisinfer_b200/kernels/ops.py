@@ -792,6 +792,16 @@ class PooledKeys:
         self.k, self.v, self.block_tables, self.every = k, v, block_tables, int(every)
 
 
+_attention_rows = True
+
+
+def set_attention_rows(on: bool = True) -> None:
+    """The general attention in bf16 on tensor cores with weights in 32-bit where it takes the geometry (True, the default)
+    or on CUDA cores (False), for comparisons."""
+    global _attention_rows
+    _attention_rows = bool(on)
+
+
 def set_attention_tiled(on: bool = True) -> None:
     """Portions of prompts on the general attention's tiled kernel (True, the default) or on the kernel of single
     tokens (False), for comparisons."""
@@ -862,12 +872,30 @@ def paged_attention_simt(qkv: torch.Tensor, out: torch.Tensor, k_cache: torch.Te
             raise KernelError(f"attention: pooled keys {tuple(pooled.k.shape)} of {pooled.every} positions, window {window}")
         pool_args = (_ptr(pooled.k), _ptr(pooled.v), _ptr(pooled.block_tables), _c_int(pooled.block_tables.shape[1]),
                      _c_int(pooled.every))
+    span = min(max_kv_len, window) if window else max_kv_len
+    if pooled is not None:
+        span += max_kv_len // pooled.every
+    single = max_q_len <= 1 and max_kv_len > 0 and workspace is not None
+    # bf16 without a distance penalty: on tensor cores, with the weights' 24 bits kept (the tiled kernel switched off, the
+    # CUDA-core form of single tokens is asked for)
+    if (_attention_rows and qkv.dtype == torch.bfloat16 and not v_stride and terms.slopes is None and terms.log_r1 is None
+            and (max_q_len <= 1 or _attention_tiled) and ldq % 8 == 0 and ldo % 2 == 0 and qkv.data_ptr() % 16 == 0
+            and _lib().ferris_attention_rows_takes(num_heads, num_kv_heads, head_dim, dv, 1 if max_q_len > 1 else 0)):
+        floats = T * num_heads * ATTENTION_MAX_SHARES * (dv + 2) if single else 0
+        scratch = workspace.get("attn_shares", (floats,), torch.float32) if single else None
+        launches = _c_int(0)
+        rc = _lib().ferris_attention_rows(
+            _ptr(qkv), _c_int(ldq), _ptr(out), _c_int(ldo), _ptr(k_cache), _ptr(v_cache), _ptr(block_tables),
+            _c_int(block_tables.shape[1]), _ptr(token_seq), _ptr(positions), _c_int(T), _c_int(num_heads),
+            _c_int(num_kv_heads), _c_int(head_dim), _c_int(dv), _c_int(k_cache.shape[2]),
+            _c_int(-chunk if chunk else (window or 0)), _c_float(scale), _ptr(terms.sink), *pool_args,
+            _c_int(1 if max_q_len > 1 else 0), _c_int(span if single else 0), _ptr(scratch), ctypes.c_longlong(floats),
+            ctypes.byref(launches), _stream())
+        _check(rc, "attention rows", launches.value)
+        return
     fn = _lib().ferris_paged_attention_simt
     extra = (_c_int(0), _ptr(None), ctypes.c_longlong(0))
-    if max_q_len <= 1 and max_kv_len > 0 and workspace is not None:
-        span = min(max_kv_len, window) if window else max_kv_len
-        if pooled is not None:
-            span += max_kv_len // pooled.every
+    if single:
         floats = T * num_heads * ATTENTION_MAX_SHARES * (dv + 2)
         scratch = workspace.get("attn_shares", (floats,), torch.float32)
         extra = (_c_int(span), _ptr(scratch), ctypes.c_longlong(floats))
