@@ -9,8 +9,7 @@
 //
 // Two kernels.  Portions of prompts: a block takes 64 rows, the g query heads of one kv head for floor(64 / g) consecutive
 // tokens, and walks the keys in tiles that asynchronous copies bring into shared memory one tile ahead; each of its four
-// warps owns 16 rows.  Single tokens: a block takes one token, one kv head (its up to 16 query heads are the rows of the
-// fragments) and a share of the keys; each of its four warps walks chunks of 16 keys of its own through a ring of
+// warps owns 16 rows.  Single tokens: a block takes one token, up to eight query heads of one kv head and a share of the keys; each of its four warps walks chunks of 16 keys of its own through a ring of
 // asynchronous copies that only it reads (no block-wide barrier in the loop), and the four meet in shared memory at the
 // end; several shares of a token are merged by attention_merge_shares_kernel.
 #include <math.h>
@@ -23,7 +22,6 @@ namespace {
 
 constexpr float LOG2E = 1.4426950408889634f;
 constexpr int AR_THREADS = 128, AR_WARPS = 4, AR_ROWS = 64;
-constexpr int AS_KEYS = 16, AS_STAGES = 3;  // single tokens: keys of a warp's chunk, chunks in its ring
 
 // 16 bytes into shared memory, or 16 zero bytes where the row is not there
 __device__ __forceinline__ void copy16_or_zero(uint32_t dst, const void* src, bool there) {
@@ -335,127 +333,191 @@ constexpr size_t rows_smem() {
 }
 
 // ------------------------------------------------------------------------------------------ single tokens
+// A token's query heads of one kv head are few (a row group holds up to eight), so they stand on the narrow side of the
+// fragments: S^T = K Q^T (16 keys x 8 heads), O^T = V^T P^T (16 value columns x 8 heads).  A chunk is 16 positions that begin
+// at a multiple of 16, so that with FAST (heads of exactly D, pages of a multiple of 16) its keys lie in one piece of memory
+// and one table look-up finds them.  A warp's chunks: the pooled runs' first, then the tokens', every fourth of the share.
 // partial (splits > 1): per (token, head, share): maximum (natural units), sum, weighted values, as the merge kernel reads.
-template <int D, bool POOL>
+constexpr int AS_KEYS = 16, AS_ROWS = 8;
+template <int D>
+struct SingleStages {
+    static constexpr int value = D <= 64 ? 4 : (D <= 128 ? 3 : 2);
+};
+
+template <int D, bool POOL, bool FAST>
 __global__ void __launch_bounds__(AR_THREADS) attention_single_rows_kernel(const AttentionArgs p, int row_groups, int splits,
                                                                            float* partial) {
-    constexpr int KS = D / 16, DT = D / 8, NT = AS_KEYS / 8;
+    constexpr int KS = D / 16, MT = D / 16, STAGES = SingleStages<D>::value;
     constexpr int PITCH = (D + 8) * 2;
     constexpr uint32_t V_OFF = AS_KEYS * PITCH, STAGE = 2 * AS_KEYS * PITCH;
     extern __shared__ __align__(16) uint8_t ar_smem[];
     pdl_wait();
     pdl_launch_dependents();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gq = lane >> 2, tq = lane & 3;
-    const int t = blockIdx.x, hk = blockIdx.y / row_groups, r0 = (blockIdx.y % row_groups) * 16, split = blockIdx.z;
-    const int g = p.nh / p.nkv, rows = min(16, g - r0);
+    const int t = blockIdx.x, hk = blockIdx.y / row_groups, r0 = (blockIdx.y % row_groups) * AS_ROWS, split = blockIdx.z;
+    const int g = p.nh / p.nkv, rows = min(AS_ROWS, g - r0);
     const int seq = p.token_seq[t], P = p.positions[t];
     const int pshift = shift_of(p.page_size);
-    const int d = p.d, dv = p.dv;
-    const int nks = (d + 15) >> 4;
+    const int d = FAST ? D : p.d, dv = FAST ? D : p.dv;
+    const int nks = FAST ? KS : (d + 15) >> 4;
     const int lo = first_key(P, p.window);
     const int pooled = POOL ? lo / p.pk.every : 0;
-    const int shift = lo - pooled;  // key n >= pooled is the token at n + shift
-    const int total = pooled + P - lo + 1;
-    // this block's share of the keys, in whole chunks
-    const int chunks_all = (total + AS_KEYS - 1) / AS_KEYS;
+    const int run_chunks = (pooled + AS_KEYS - 1) / AS_KEYS;
+    const int token_chunk = lo / AS_KEYS - run_chunks;  // chunk c >= run_chunks holds the tokens from 16 (c + token_chunk) on
+    const int chunks_all = P / AS_KEYS - token_chunk + 1;
     const int per = (chunks_all + splits - 1) / splits;
-    const int c_first = split * per, c_end = min(chunks_all, c_first + per);
+    const int c_first = split * per + warp, c_end = min(chunks_all, split * per + per);
     const int* table = p.tables + (size_t)seq * p.max_blocks;
     const int* ptable = POOL ? p.pk.tables + (size_t)seq * p.pk.max_blocks : nullptr;
 
-    uint8_t* mine = ar_smem + warp * AS_STAGES * STAGE;
+    uint8_t* mine = ar_smem + warp * STAGES * STAGE;
     const uint32_t ring = smem_u32(mine);
-    if (d & 15) {
-        for (int r = lane; r < AS_STAGES * AS_KEYS; r += 32)
+    if (!FAST && (d & 15)) {  // columns between d and the next multiple of 16 are zero on both sides
+        for (int r = lane; r < STAGES * AS_KEYS; r += 32)
             *reinterpret_cast<uint4*>(mine + (r / AS_KEYS) * STAGE + (r % AS_KEYS) * PITCH + d * 2) = make_uint4(0u, 0u, 0u, 0u);
     }
-    const bf16* qbase = p.q + (size_t)t * p.ldq + (size_t)(hk * g + r0) * d;
-    uint32_t qf[KS][4];
-    load_q_rows<KS>(qf, gq < rows ? qbase + (size_t)gq * d : nullptr, gq + 8 < rows ? qbase + (size_t)(gq + 8) * d : nullptr, d);
-    float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.0f, 0.0f};
-    float o[DT][4];
+    uint32_t qf[KS][2];
+    {
+        const bf16* row = p.q + (size_t)t * p.ldq + (size_t)(hk * g + r0 + gq) * d;
 #pragma unroll
-    for (int n = 0; n < DT; ++n)
+        for (int ks = 0; ks < KS; ++ks) {
+            const int c = 16 * ks + 2 * tq;
+            qf[ks][0] = gq < rows && c < d ? *reinterpret_cast<const uint32_t*>(row + c) : 0u;
+            qf[ks][1] = gq < rows && c + 8 < d ? *reinterpret_cast<const uint32_t*>(row + c + 8) : 0u;
+        }
+    }
+    float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.0f, 0.0f};
+    float o[MT][4];
+#pragma unroll
+    for (int n = 0; n < MT; ++n)
 #pragma unroll
         for (int e = 0; e < 4; ++e) o[n][e] = 0.0f;
 
-    const int key = lane >> 1, part = lane & 1;
-    // chunk number i of this warp is c_first + warp + 4 i
-    auto page_at = [&](int i) -> int {
-        const int n = (c_first + warp + AR_WARPS * i) * AS_KEYS + key;
-        if (c_first + warp + AR_WARPS * i >= c_end || n >= total) return -1;
-        return POOL && n < pooled ? page_of(ptable, n, p.page_size, pshift) : page_of(table, n + shift, p.page_size, pshift);
+    // of chunk c (this warp's are c_first, c_first + 4, ...): its first position, and which of its 16 keys are seen
+    auto first_of = [&](int c) -> int { return POOL && c < run_chunks ? c * AS_KEYS : (c + token_chunk) * AS_KEYS; };
+    auto from_of = [&](int c) -> int { return POOL && c < run_chunks ? 0 : lo - first_of(c); };
+    auto to_of = [&](int c) -> int { return (POOL && c < run_chunks ? pooled - 1 : P) - first_of(c); };
+    const int key = FAST ? 0 : lane >> 1, part = lane & 1;
+    auto page_at = [&](int c) -> int {
+        if (c >= c_end || (!FAST && (key < from_of(c) || key > to_of(c)))) return -1;
+        return page_of(POOL && c < run_chunks ? ptable : table, first_of(c) + key, p.page_size, pshift);
     };
-    auto fetch = [&](int i, int stage, int page) {
-        if (c_first + warp + AR_WARPS * i < c_end) {
-            const int n = (c_first + warp + AR_WARPS * i) * AS_KEYS + key;
-            const bool run = POOL && n < pooled, there = page >= 0;
-            const size_t row = there ? row_of(page, hk, p.nkv, run ? n : n + shift, p.page_size, pshift) : 0;
+    auto fetch = [&](int c, int stage, int page) {
+        if (c < c_end) {
+            const bool run = POOL && c < run_chunks, there = page >= 0;
+            const size_t row = there ? row_of(page, hk, p.nkv, first_of(c) + key, p.page_size, pshift) : 0;
             const bf16* ks = (run ? reinterpret_cast<const bf16*>(p.pk.k) : p.k) + row * d;
             const bf16* vs = (run ? reinterpret_cast<const bf16*>(p.pk.v) : p.v) + row * dv;
-            const uint32_t dst = ring + stage * STAGE + key * PITCH;
-            for (int c = part; c < (d >> 3); c += 2) copy16_or_zero(dst + c * 16, ks + 8 * c, there);
-            for (int c = part; c < (dv >> 3); c += 2) copy16_or_zero(dst + V_OFF + c * 16, vs + 8 * c, there);
+            const uint32_t dst = ring + stage * STAGE;
+            if constexpr (FAST) {  // 16 keys in one piece: a warp copies 512 bytes of it at a time
+                const int from = from_of(c), to = to_of(c);
+                constexpr int PIECES = D / 8;  // of a row
+#pragma unroll
+                for (int it = 0; it < AS_KEYS * PIECES / 32; ++it) {
+                    const int x = it * 32 + lane, r = x / PIECES, col = x % PIECES;
+                    const bool seen = there && r >= from && r <= to;
+                    copy16_or_zero(dst + r * PITCH + col * 16, ks + 8 * x, seen);
+                    copy16_or_zero(dst + V_OFF + r * PITCH + col * 16, vs + 8 * x, seen);
+                }
+            } else {
+                for (int x = part; x < (d >> 3); x += 2) copy16_or_zero(dst + key * PITCH + x * 16, ks + 8 * x, there);
+                for (int x = part; x < (dv >> 3); x += 2) copy16_or_zero(dst + V_OFF + key * PITCH + x * 16, vs + 8 * x, there);
+            }
         }
         ar_commit();
     };
-    const int own = c_end - c_first - warp > 0 ? (c_end - c_first - warp + AR_WARPS - 1) / AR_WARPS : 0;
-    int pages[AS_STAGES];
+    {
+        int pages[STAGES - 1];
 #pragma unroll
-    for (int i = 0; i < AS_STAGES; ++i) pages[i] = page_at(i);
+        for (int i = 0; i < STAGES - 1; ++i) pages[i] = page_at(c_first + AR_WARPS * i);
 #pragma unroll
-    for (int i = 0; i < AS_STAGES - 1; ++i) fetch(i, i, pages[i]);
-    int next_page = pages[AS_STAGES - 1];
-    int stage = 0, fill = AS_STAGES - 1;
-    for (int i = 0; i < own; ++i) {
-        fetch(i + AS_STAGES - 1, fill, next_page);
-        next_page = page_at(i + AS_STAGES);
-        ar_wait<AS_STAGES - 1>();
+        for (int i = 0; i < STAGES - 1; ++i) fetch(c_first + AR_WARPS * i, i, pages[i]);
+    }
+    int next_page = page_at(c_first + AR_WARPS * (STAGES - 1));
+    int stage = 0, fill = STAGES - 1;
+    for (int c = c_first; c < c_end; c += AR_WARPS) {
+        fetch(c + AR_WARPS * (STAGES - 1), fill, next_page);
+        next_page = page_at(c + AR_WARPS * STAGES);
+        ar_wait<STAGES - 1>();
         __syncwarp();
         const uint32_t kb = ring + stage * STAGE;
-        float s[NT][4];
+        float s[2][4];  // two accumulators, so that the products do not wait for one another
 #pragma unroll
-        for (int n = 0; n < NT; ++n)
-#pragma unroll
-            for (int e = 0; e < 4; ++e) s[n][e] = 0.0f;
-        const uint32_t k_at = kb + (uint32_t)((lane >> 4) * 8 + (lane & 7)) * PITCH + ((lane >> 3) & 1) * 16;
+        for (int e = 0; e < 4; ++e) s[0][e] = 0.0f, s[1][e] = 0.0f;
+        const uint32_t k_at = kb + (uint32_t)((lane & 7) + ((lane >> 3) & 1) * 8) * PITCH + (lane >> 4) * 16;
 #pragma unroll
         for (int ks = 0; ks < KS; ++ks) {
             if (ks < nks) {
-                uint32_t b[4];
-                ldmatrix_x4(b, k_at + ks * 32);
-                mma_bf16_16816(s[0], qf[ks], b[0], b[1]);
-                mma_bf16_16816(s[1], qf[ks], b[2], b[3]);
+                uint32_t a[4];
+                ldmatrix_x4(a, k_at + ks * 32);
+                mma_bf16_16816(s[ks & 1], a, qf[ks][0], qf[ks][1]);
             }
         }
-        const int left = total - (c_first + warp + AR_WARPS * i) * AS_KEYS;  // keys of the chunk that exist
+        // keys gq and gq + 8 of the chunk against heads 2 tq and 2 tq + 1
+        const int from = from_of(c), to = to_of(c);
+        float w[4];
 #pragma unroll
-        for (int n = 0; n < NT; ++n)
+        for (int e = 0; e < 4; ++e) {
+            const int at = gq + (e >> 1) * 8;
+            w[e] = at >= from && at <= to ? (s[0][e] + s[1][e]) * p.scale2 : -INFINITY;
+        }
+        float alpha[2];
+        bool moved = false;
 #pragma unroll
-            for (int e = 0; e < 4; ++e) s[n][e] = 8 * n + 2 * tq + (e & 1) < left ? s[n][e] * p.scale2 : -INFINITY;
-        softmax_step<NT, DT>(s, m, l, o);
-        weights_times_values<NT, DT>(o, s, 0, kb + V_OFF, PITCH, dv);
+        for (int a = 0; a < 2; ++a) {
+            float best = fmaxf(w[a], w[2 + a]);
+            best = fmaxf(best, __shfl_xor_sync(0xffffffffu, best, 4));
+            best = fmaxf(best, __shfl_xor_sync(0xffffffffu, best, 8));
+            best = fmaxf(best, __shfl_xor_sync(0xffffffffu, best, 16));
+            const float m_new = fmaxf(m[a], best);
+            const float base = m_new == -INFINITY ? 0.0f : m_new;
+            alpha[a] = exp2f(m[a] - base);
+            moved |= m_new != m[a];
+            m[a] = m_new;
+            w[a] = exp2f(w[a] - base), w[2 + a] = exp2f(w[2 + a] - base);
+            l[a] = l[a] * alpha[a] + (w[a] + w[2 + a]);
+        }
+        if (__any_sync(0xffffffffu, moved)) {
+#pragma unroll
+            for (int n = 0; n < MT; ++n) o[n][0] *= alpha[0], o[n][1] *= alpha[1], o[n][2] *= alpha[0], o[n][3] *= alpha[1];
+        }
+        uint32_t pw[3][2];
+        split3(w[0], w[1], pw[0][0], pw[1][0], pw[2][0]);
+        split3(w[2], w[3], pw[0][1], pw[1][1], pw[2][1]);
+#pragma unroll
+        for (int x = 0; x < 3; ++x) pw[x][0] = movmatrix_trans(pw[x][0]), pw[x][1] = movmatrix_trans(pw[x][1]);
+        const uint32_t v_at = kb + V_OFF + (uint32_t)((lane & 7) + (lane >> 4) * 8) * PITCH + ((lane >> 3) & 1) * 16;
+#pragma unroll
+        for (int n = 0; n < MT; ++n) {
+            if (16 * n < dv) {
+                uint32_t a[4];
+                ldmatrix_x4_trans(a, v_at + n * 32);
+#pragma unroll
+                for (int x = 0; x < 3; ++x) mma_bf16_16816(o[n], a, pw[x][0], pw[x][1]);
+            }
+        }
         __syncwarp();  // the stage is read: the copy after next may overwrite it
-        stage = stage + 1 == AS_STAGES ? 0 : stage + 1;
-        fill = fill + 1 == AS_STAGES ? 0 : fill + 1;
+        stage = stage + 1 == STAGES ? 0 : stage + 1;
+        fill = fill + 1 == STAGES ? 0 : fill + 1;
     }
     ar_wait<0>();
-    // the four warps meet: per warp and row its maximum, sum and weighted values
+    // the four warps meet: per warp and head its maximum, sum and weighted values
     float* meet = reinterpret_cast<float*>(ar_smem);
     const int stride = dv + 2;
     __syncthreads();
 #pragma unroll
     for (int a = 0; a < 2; ++a) {
-        l[a] += __shfl_xor_sync(0xffffffffu, l[a], 1);
-        l[a] += __shfl_xor_sync(0xffffffffu, l[a], 2);
-        const int r = gq + 8 * a;
+#pragma unroll
+        for (int x = 4; x <= 16; x <<= 1) l[a] += __shfl_xor_sync(0xffffffffu, l[a], x);
+        const int r = 2 * tq + a;
         if (r < rows) {
             float* e = meet + (size_t)(warp * rows + r) * stride;
-            if (tq == 0) e[0] = m[a], e[1] = l[a];
+            if (gq == 0) e[0] = m[a], e[1] = l[a];
 #pragma unroll
-            for (int n = 0; n < DT; ++n) {
-                const int c = 8 * n + 2 * tq;
-                if (c < dv) *reinterpret_cast<float2*>(e + 2 + c) = make_float2(o[n][2 * a], o[n][2 * a + 1]);
+            for (int n = 0; n < MT; ++n) {
+                const int c = 16 * n + gq;
+                if (c < dv) e[2 + c] = o[n][a];
+                if (c + 8 < dv) e[2 + c + 8] = o[n][2 + a];
             }
         }
     }
@@ -486,7 +548,7 @@ __global__ void __launch_bounds__(AR_THREADS) attention_single_rows_kernel(const
 
 template <int D>
 constexpr size_t single_smem() {
-    return (size_t)AR_WARPS * AS_STAGES * 2 * AS_KEYS * (D + 8) * 2;
+    return (size_t)AR_WARPS * SingleStages<D>::value * 2 * AS_KEYS * (D + 8) * 2;
 }
 
 int rows_bucket(int d, int dv) {
@@ -515,15 +577,23 @@ int launch_rows(const AttentionArgs& p, cudaStream_t s) {
     FERRIS_LAUNCH_CHECK();
 }
 
+template <int D, bool POOL, bool FAST>
+int launch_single_form(const AttentionArgs& p, int splits, float* partial, cudaStream_t s) {
+    const int groups = (p.nh / p.nkv + AS_ROWS - 1) / AS_ROWS;
+    constexpr size_t smem = single_smem<D>();
+    static_assert((size_t)AR_WARPS * AS_ROWS * (D + 2) * sizeof(float) <= smem, "the warps meet in the ring's memory");
+    int rc = ferris_allow_dynamic_smem((const void*)attention_single_rows_kernel<D, POOL, FAST>, smem);
+    if (rc != FERRIS_OK) return rc;
+    ferris_launch(attention_single_rows_kernel<D, POOL, FAST>, dim3(p.tokens, p.nkv * groups, splits), dim3(AR_THREADS), smem, s,
+                  p, groups, splits, partial);
+    return FERRIS_OK;
+}
+
 template <int D, bool POOL>
 int launch_single(const AttentionArgs& p, int splits, float* partial, cudaStream_t s) {
-    const int groups = (p.nh / p.nkv + 15) / 16;
-    constexpr size_t smem = single_smem<D>();
-    static_assert((size_t)AR_WARPS * 16 * (D + 2) * sizeof(float) <= smem, "the warps meet in the ring's memory");
-    int rc = ferris_allow_dynamic_smem((const void*)attention_single_rows_kernel<D, POOL>, smem);
+    const bool fast = p.d == D && p.dv == D && p.page_size % AS_KEYS == 0;
+    const int rc = fast ? launch_single_form<D, POOL, true>(p, splits, partial, s) : launch_single_form<D, POOL, false>(p, splits, partial, s);
     if (rc != FERRIS_OK) return rc;
-    ferris_launch(attention_single_rows_kernel<D, POOL>, dim3(p.tokens, p.nkv * groups, splits), dim3(AR_THREADS), smem, s, p,
-                  groups, splits, partial);
     if (splits > 1) {
         const ScoreTerms st = {nullptr, nullptr, nullptr, p.sink, 0};
         ferris_launch(attention_merge_shares_kernel<bf16>, dim3(p.tokens, p.nh), dim3(128), 0, s, (const float*)partial, p.out,
@@ -537,7 +607,7 @@ int launch_single(const AttentionArgs& p, int splits, float* partial, cudaStream
 // Whether ferris_attention_rows takes a geometry (bf16).  portions: 1 = the kernel for portions of prompts, 0 = single tokens.
 FERRIS_API int ferris_attention_rows_takes(int nh, int nkv, int d, int dv, int portions) {
     if (nh <= 0 || nkv <= 0 || nh % nkv || d <= 0 || dv <= 0 || d % 8 || dv % 8 || d > 256 || dv > 256) return 0;
-    if (nkv > 65535 || (long long)nkv * ((nh / nkv + 15) / 16) > 65535) return 0;
+    if (nkv > 65535 || (long long)nkv * ((nh / nkv + 7) / 8) > 65535) return 0;
     return portions ? nh / nkv <= AR_ROWS : 1;
 }
 
@@ -573,11 +643,11 @@ FERRIS_API int ferris_attention_rows(const void* q, int ldq, void* out, int ldo,
         if (bucket == 128) return pool ? launch_rows<128, true>(p, s) : launch_rows<128, false>(p, s);
         return pool ? launch_rows<256, true>(p, s) : launch_rows<256, false>(p, s);
     }
-    // shares of a token's keys: as many as fill the SMs about three times over, of 64 keys at least
+    // shares of a token's keys: as many as fill the SMs about twice over (two blocks are resident on one), of 64 keys at least
     int splits = 1;
     if (scratch && kv_span > 0) {
-        const long long blocks = (long long)tokens * nkv * ((nh / nkv + 15) / 16);
-        long long want = 3LL * device_sms() / blocks;
+        const long long blocks = (long long)tokens * nkv * ((nh / nkv + AS_ROWS - 1) / AS_ROWS);
+        long long want = 2LL * device_sms() / blocks;
         const long long most = kv_span / 64;
         if (want > most) want = most;
         if (want > 16) want = 16;
