@@ -1,5 +1,5 @@
 // What the forms of the general attention share (attention_simt.cu on CUDA cores in either precision, attention_rows.cu on
-// tensor cores in bf16): what enters a score besides the product, which keys a token sees, the merge of shares.
+// tensor cores in bf16): what enters a score besides the product, which keys a token sees.
 #pragma once
 
 #include <math.h>
@@ -55,35 +55,6 @@ __device__ __forceinline__ int first_key(int P, int window) {
 }
 // the sink's share of the denominator, relative to the maximum mm of the keys' scores
 __device__ __forceinline__ float sink_share(const ScoreTerms& st, int h, float mm) { return st.sink ? expf(st.sink[h] - mm) : 0.0f; }
-
-// out = sum_s o_s e^(m_s - M) / sum_s z_s e^(m_s - M) over the shares of the keys that the kernel above left in `partial`
-// ([tokens, heads, splits, 2 + dv]: maximum, sum, weighted values).  A block per (token, head).
-template <typename T>
-__global__ void __launch_bounds__(128) attention_merge_shares_kernel(const float* partial, T* __restrict__ out, int ldo,
-                                                                     int nh, int dv, int splits, const ScoreTerms st) {
-    pdl_wait();
-    pdl_launch_dependents();
-    const int t = blockIdx.x, h = blockIdx.y;
-    const int stride = dv + 2;
-    const float* base = partial + ((size_t)t * nh + h) * splits * stride;
-    float mm = -INFINITY;
-    for (int s2 = 0; s2 < splits; ++s2) mm = fmaxf(mm, base[(size_t)s2 * stride]);
-    float zz = 0.0f;
-    for (int s2 = 0; s2 < splits; ++s2) {
-        const float ms = base[(size_t)s2 * stride];
-        zz += ms == -INFINITY ? 0.0f : base[(size_t)s2 * stride + 1] * expf(ms - mm);
-    }
-    zz += sink_share(st, h, mm);
-    const float inv = 1.0f / zz;
-    for (int i = threadIdx.x; i < dv; i += blockDim.x) {
-        float o = 0.0f;
-        for (int s2 = 0; s2 < splits; ++s2) {
-            const float ms = base[(size_t)s2 * stride];
-            if (ms != -INFINITY) o += base[(size_t)s2 * stride + 2 + i] * expf(ms - mm);
-        }
-        out[(size_t)t * ldo + (size_t)h * dv + i] = from_float<T>(o * inv);
-    }
-}
 
 // Whether the arguments for pooled keys make sense (all null / 0: there are none).
 int check_pooled(const PooledKeys& pk, int window, const ScoreTerms& st) {

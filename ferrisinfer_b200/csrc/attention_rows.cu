@@ -9,9 +9,9 @@
 //
 // Two kernels.  Portions of prompts: a block takes 64 rows, the g query heads of one kv head for floor(64 / g) consecutive
 // tokens, and walks the keys in tiles that asynchronous copies bring into shared memory one tile ahead; each of its four
-// warps owns 16 rows.  Single tokens: a block takes one token, up to eight query heads of one kv head and a share of the keys; each of its four warps walks chunks of 16 keys of its own through a ring of
-// asynchronous copies that only it reads (no block-wide barrier in the loop), and the four meet in shared memory at the
-// end; several shares of a token are merged by attention_merge_shares_kernel.
+// warps owns 16 rows.  Single tokens: a block takes one token, up to eight query heads of one kv head and a share of the
+// keys; each of its four warps walks chunks of 16 keys of its own through a ring of asynchronous copies that only it reads
+// (no block-wide barrier in the loop), and the four meet in shared memory at the end; the shares of a token are a cluster.
 #include <math.h>
 
 #include "attention_general.cuh"
@@ -337,16 +337,15 @@ constexpr size_t rows_smem() {
 // fragments: S^T = K Q^T (16 keys x 8 heads), O^T = V^T P^T (16 value columns x 8 heads).  A chunk is 16 positions that begin
 // at a multiple of 16, so that with FAST (heads of exactly D, pages of a multiple of 16) its keys lie in one piece of memory
 // and one table look-up finds them.  A warp's chunks: the pooled runs' first, then the tokens', every fourth of the share.
-// partial (splits > 1): per (token, head, share): maximum (natural units), sum, weighted values, as the merge kernel reads.
-constexpr int AS_KEYS = 16, AS_ROWS = 8;
+// The shares of a token's keys (splits > 1) are a thread-block cluster, which merges them through its shared memory.
+constexpr int AS_KEYS = 16, AS_ROWS = 8, AS_MAX_SPLITS = 8;
 template <int D>
 struct SingleStages {
     static constexpr int value = D <= 64 ? 4 : (D <= 128 ? 3 : 2);
 };
 
 template <int D, bool POOL, bool FAST>
-__global__ void __launch_bounds__(AR_THREADS) attention_single_rows_kernel(const AttentionArgs p, int row_groups, int splits,
-                                                                           float* partial) {
+__global__ void __launch_bounds__(AR_THREADS) attention_single_rows_kernel(const AttentionArgs p, int row_groups, int splits) {
     constexpr int KS = D / 16, MT = D / 16, STAGES = SingleStages<D>::value;
     constexpr int PITCH = (D + 8) * 2;
     constexpr uint32_t V_OFF = AS_KEYS * PITCH, STAGE = 2 * AS_KEYS * PITCH;
@@ -534,16 +533,42 @@ __global__ void __launch_bounds__(AR_THREADS) attention_single_rows_kernel(const
             const float f = e[0] == -INFINITY ? 0.0f : exp2f(e[0] - mm);
             zz = fmaf(e[1], f, zz), acc = fmaf(e[2 + i], f, acc);
         }
-        const int head = hk * g + r0 + r;
         if (splits == 1) {
+            const int head = hk * g + r0 + r;
             if (p.sink) zz += exp2f(p.sink[head] * LOG2E - mm);
             p.out[(size_t)t * p.ldo + (size_t)head * dv + i] = from_float<bf16>(acc / zz);
         } else {
-            float* e = partial + (((size_t)t * p.nh + head) * splits + split) * stride;
-            if (i == 0) e[0] = mm / LOG2E, e[1] = zz;
+            float* e = meet + (size_t)(AR_WARPS * rows + r) * stride;
+            if (i == 0) e[0] = mm, e[1] = zz;
             e[2 + i] = acc;
         }
     }
+    if (splits == 1) return;
+    // the shares of a token are the blocks of a cluster: each adds up its part of the outputs from all of them
+    cluster_sync();
+    const uint32_t shares = smem_u32(meet + (size_t)AR_WARPS * rows * stride);
+    for (int x = split * AR_THREADS + threadIdx.x; x < rows * dv; x += splits * AR_THREADS) {
+        const int r = x / dv, i = x - r * dv;
+        const uint32_t at = shares + (uint32_t)(r * stride) * 4;
+        float ms[AS_MAX_SPLITS], mm = -INFINITY;
+#pragma unroll
+        for (int w = 0; w < AS_MAX_SPLITS; ++w) {
+            ms[w] = w < splits ? ld_peer_shared_f32(at, w) : -INFINITY;
+            mm = fmaxf(mm, ms[w]);
+        }
+        float zz = 0.0f, acc = 0.0f;
+#pragma unroll
+        for (int w = 0; w < AS_MAX_SPLITS; ++w) {
+            if (w < splits && ms[w] != -INFINITY) {
+                const float f = exp2f(ms[w] - mm);
+                zz = fmaf(ld_peer_shared_f32(at + 4, w), f, zz), acc = fmaf(ld_peer_shared_f32(at + 8 + 4 * i, w), f, acc);
+            }
+        }
+        const int head = hk * g + r0 + r;
+        if (p.sink) zz += exp2f(p.sink[head] * LOG2E - mm);
+        p.out[(size_t)t * p.ldo + (size_t)head * dv + i] = from_float<bf16>(acc / zz);
+    }
+    cluster_sync();  // nobody leaves while a peer may still read its shared memory
 }
 
 template <int D>
@@ -578,28 +603,24 @@ int launch_rows(const AttentionArgs& p, cudaStream_t s) {
 }
 
 template <int D, bool POOL, bool FAST>
-int launch_single_form(const AttentionArgs& p, int splits, float* partial, cudaStream_t s) {
+int launch_single_form(const AttentionArgs& p, int splits, cudaStream_t s) {
     const int groups = (p.nh / p.nkv + AS_ROWS - 1) / AS_ROWS;
     constexpr size_t smem = single_smem<D>();
-    static_assert((size_t)AR_WARPS * AS_ROWS * (D + 2) * sizeof(float) <= smem, "the warps meet in the ring's memory");
+    static_assert((size_t)(AR_WARPS + 1) * AS_ROWS * (D + 2) * sizeof(float) <= smem, "the warps meet in the ring's memory");
     int rc = ferris_allow_dynamic_smem((const void*)attention_single_rows_kernel<D, POOL, FAST>, smem);
     if (rc != FERRIS_OK) return rc;
-    ferris_launch(attention_single_rows_kernel<D, POOL, FAST>, dim3(p.tokens, p.nkv * groups, splits), dim3(AR_THREADS), smem, s,
-                  p, groups, splits, partial);
-    return FERRIS_OK;
+    const dim3 grid(p.tokens, p.nkv * groups, splits);
+    if (splits > 1)
+        ferris_launch_cluster(attention_single_rows_kernel<D, POOL, FAST>, grid, dim3(AR_THREADS), smem, s, (unsigned)splits, p, groups, splits);
+    else
+        ferris_launch(attention_single_rows_kernel<D, POOL, FAST>, grid, dim3(AR_THREADS), smem, s, p, groups, splits);
+    FERRIS_LAUNCH_CHECK();
 }
 
 template <int D, bool POOL>
-int launch_single(const AttentionArgs& p, int splits, float* partial, cudaStream_t s) {
+int launch_single(const AttentionArgs& p, int splits, cudaStream_t s) {
     const bool fast = p.d == D && p.dv == D && p.page_size % AS_KEYS == 0;
-    const int rc = fast ? launch_single_form<D, POOL, true>(p, splits, partial, s) : launch_single_form<D, POOL, false>(p, splits, partial, s);
-    if (rc != FERRIS_OK) return rc;
-    if (splits > 1) {
-        const ScoreTerms st = {nullptr, nullptr, nullptr, p.sink, 0};
-        ferris_launch(attention_merge_shares_kernel<bf16>, dim3(p.tokens, p.nh), dim3(128), 0, s, (const float*)partial, p.out,
-                      p.ldo, p.nh, p.dv, splits, st);
-    }
-    FERRIS_LAUNCH_CHECK();
+    return fast ? launch_single_form<D, POOL, true>(p, splits, s) : launch_single_form<D, POOL, false>(p, splits, s);
 }
 
 }  // namespace
@@ -612,15 +633,13 @@ FERRIS_API int ferris_attention_rows_takes(int nh, int nkv, int d, int dv, int p
 }
 
 // Arguments as ferris_paged_attention_simt, bf16 throughout, no distance penalty, values in rows of their own.  portions:
-// requests bring several tokens each (the kernel of 64-row blocks); else kv_span (the most keys a token sees) and scratch
-// (fp32, for shares of the keys; may be null) as there.  Returns the number of launches through *launches.
+// requests bring several tokens each (the kernel of 64-row blocks); else kv_span is the most keys a token sees (0: unknown),
+// by which they are cut into shares.
 FERRIS_API int ferris_attention_rows(const void* q, int ldq, void* out, int ldo, const void* k_cache, const void* v_cache,
                                      const int* block_tables, int max_blocks, const int* token_seq, const int* positions,
                                      int tokens, int nh, int nkv, int d, int dv, int page_size, int window, float scale,
                                      const float* sink, const void* pool_k, const void* pool_v, const int* pool_tables,
-                                     int pool_max_blocks, int pool_every, int portions, int kv_span, float* scratch,
-                                     long long scratch_floats, int* launches, void* stream) {
-    if (launches) *launches = 0;
+                                     int pool_max_blocks, int pool_every, int portions, int kv_span, void* stream) {
     if (tokens <= 0) return FERRIS_OK;
     if (!ferris_attention_rows_takes(nh, nkv, d, dv, portions))
         FERRIS_REFUSE("attention rows: %d heads over %d kv heads of %d / %d are not taken", nh, nkv, d, dv);
@@ -638,25 +657,20 @@ FERRIS_API int ferris_attention_rows(const void* q, int ldq, void* out, int ldo,
     const bool pool = pk.every > 0;
     const int bucket = rows_bucket(d, dv);
     if (portions) {
-        if (launches) *launches = 1;
         if (bucket == 64) return pool ? launch_rows<64, true>(p, s) : launch_rows<64, false>(p, s);
         if (bucket == 128) return pool ? launch_rows<128, true>(p, s) : launch_rows<128, false>(p, s);
         return pool ? launch_rows<256, true>(p, s) : launch_rows<256, false>(p, s);
     }
     // shares of a token's keys: as many as fill the SMs about twice over (two blocks are resident on one), of 64 keys at least
     int splits = 1;
-    if (scratch && kv_span > 0) {
+    if (kv_span > 0) {
         const long long blocks = (long long)tokens * nkv * ((nh / nkv + AS_ROWS - 1) / AS_ROWS);
         long long want = 2LL * device_sms() / blocks;
-        const long long most = kv_span / 64;
-        if (want > most) want = most;
-        if (want > 16) want = 16;
-        const long long fit = scratch_floats / ((long long)tokens * nh * (dv + 2));
-        if (want > fit) want = fit;
+        if (want > kv_span / 64) want = kv_span / 64;
+        if (want > AS_MAX_SPLITS) want = AS_MAX_SPLITS;
         if (want > 1) splits = (int)want;
     }
-    if (launches) *launches = splits > 1 ? 2 : 1;
-    if (bucket == 64) return pool ? launch_single<64, true>(p, splits, scratch, s) : launch_single<64, false>(p, splits, scratch, s);
-    if (bucket == 128) return pool ? launch_single<128, true>(p, splits, scratch, s) : launch_single<128, false>(p, splits, scratch, s);
-    return pool ? launch_single<256, true>(p, splits, scratch, s) : launch_single<256, false>(p, splits, scratch, s);
+    if (bucket == 64) return pool ? launch_single<64, true>(p, splits, s) : launch_single<64, false>(p, splits, s);
+    if (bucket == 128) return pool ? launch_single<128, true>(p, splits, s) : launch_single<128, false>(p, splits, s);
+    return pool ? launch_single<256, true>(p, splits, s) : launch_single<256, false>(p, splits, s);
 }

@@ -869,41 +869,57 @@ FERRIS_API int ferris_embed_positions(const void* table, const void* pos_table, 
 
 // ---------------------------------------------------------------------------------------------
 // The norm on a sublayer's output: h[r] += rmsnorm(y[r]) * w, both fp32 (statistics and sum in fp32), and, where `rows` is
-// given, rows[r] = h[r] in bf16, which is what the next sublayer's products read.  A warp per row with the row in
-// registers where the row is aligned and at most 4,096 wide, a block per row otherwise.  Without y (null): the rows alone.
+// given, rows[r] = h[r] in bf16, which is what the next sublayer's products read.  Without y (null): the rows alone.
+// With top > 0, y[r] is itself a sum that is formed here first: sum over s < top of weights[r, s] * y[pos[r, s]] (without
+// weights: unweighted; without pos: y[r * top + s]), in that order: a mixture of experts whose results were left apart.
+// A block per row with the row in registers where it is aligned and at most 4,096 wide.
 // ---------------------------------------------------------------------------------------------
-template <int VEC>
-__global__ void __launch_bounds__(256) rmsnorm_add_rows_kernel(const float* y, const float* __restrict__ w, float* h, bf16* rows,
-                                                               int n_rows, int hidden, float eps) {
+struct RowSum {
+    const int* pos;
+    const float* weights;
+    int top;  // 0: y holds the rows themselves
+};
+template <int VPT>
+__global__ void __launch_bounds__(256) rmsnorm_add_block_kernel(const float* y, const RowSum sum, const float* __restrict__ w,
+                                                                float* h, bf16* rows, int hidden, float eps) {
+    __shared__ float scratch[33];
     pdl_wait();
     pdl_launch_dependents();
-    const int lane = threadIdx.x & 31;
-    const int r = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
-    if (r >= n_rows) return;
-    const float4* yr = reinterpret_cast<const float4*>(y + (size_t)r * hidden);
+    const int r = blockIdx.x, n4 = hidden >> 2;
     float4* hr = reinterpret_cast<float4*>(h + (size_t)r * hidden);
-    const int n4 = hidden >> 2;
-    float4 v[VEC], a[VEC];
+    const float4* w4 = reinterpret_cast<const float4*>(w);
+    float4 v[VPT], a[VPT];
+#pragma unroll
+    for (int j = 0; j < VPT; ++j) {
+        const int i = threadIdx.x + j * blockDim.x;
+        a[j] = i < n4 ? hr[i] : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        v[j] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (sum.top == 0 && i < n4) v[j] = reinterpret_cast<const float4*>(y + (size_t)r * hidden)[i];
+    }
+    for (int s = 0; s < sum.top; ++s) {
+        const size_t at = (size_t)r * sum.top + s;
+        const float4* yr = reinterpret_cast<const float4*>(y + (sum.pos ? (size_t)sum.pos[at] : at) * hidden);
+        const float f = sum.weights ? sum.weights[at] : 1.0f;
+#pragma unroll
+        for (int j = 0; j < VPT; ++j) {
+            const int i = threadIdx.x + j * blockDim.x;
+            if (i < n4) {
+                const float4 x = yr[i];
+                v[j].x = fmaf(f, x.x, v[j].x), v[j].y = fmaf(f, x.y, v[j].y);
+                v[j].z = fmaf(f, x.z, v[j].z), v[j].w = fmaf(f, x.w, v[j].w);
+            }
+        }
+    }
     float ss = 0.0f;
 #pragma unroll
-    for (int j = 0; j < VEC; ++j) {
-        const int i = lane + 32 * j;
-        v[j] = i < n4 ? yr[i] : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-        a[j] = i < n4 ? hr[i] : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    for (int j = 0; j < VPT; ++j) {
+        ss = fmaf(v[j].x, v[j].x, ss), ss = fmaf(v[j].y, v[j].y, ss);
+        ss = fmaf(v[j].z, v[j].z, ss), ss = fmaf(v[j].w, v[j].w, ss);
     }
+    const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)hidden + eps);
 #pragma unroll
-    for (int j = 0; j < VEC; ++j) {
-        ss = fmaf(v[j].x, v[j].x, ss);
-        ss = fmaf(v[j].y, v[j].y, ss);
-        ss = fmaf(v[j].z, v[j].z, ss);
-        ss = fmaf(v[j].w, v[j].w, ss);
-    }
-    ss = warp_sum(ss);
-    const float inv = 1.0f / sqrtf(ss / (float)hidden + eps);
-    const float4* w4 = reinterpret_cast<const float4*>(w);
-#pragma unroll
-    for (int j = 0; j < VEC; ++j) {
-        const int i = lane + 32 * j;
+    for (int j = 0; j < VPT; ++j) {
+        const int i = threadIdx.x + j * blockDim.x;
         if (i < n4) {
             const float4 g = w4[i];
             float4 x = a[j];
@@ -915,17 +931,27 @@ __global__ void __launch_bounds__(256) rmsnorm_add_rows_kernel(const float* y, c
     }
 }
 
-__global__ void __launch_bounds__(512) rmsnorm_add_kernel(const float* y, const float* __restrict__ w, float* h, bf16* rows,
-                                                          int hidden, float eps) {
+// any width: the row is summed a second time where it is needed a second time
+__global__ void __launch_bounds__(512) rmsnorm_add_kernel(const float* y, const RowSum sum, const float* __restrict__ w, float* h,
+                                                          bf16* rows, int hidden, float eps) {
     __shared__ float scratch[33];
     pdl_wait();
     pdl_launch_dependents();
     const size_t at = (size_t)blockIdx.x * hidden;
+    auto value = [&](int i) -> float {
+        if (sum.top == 0) return y[at + i];
+        float v = 0.0f;
+        for (int s = 0; s < sum.top; ++s) {
+            const size_t x = (size_t)blockIdx.x * sum.top + s;
+            v = fmaf(sum.weights ? sum.weights[x] : 1.0f, y[(sum.pos ? (size_t)sum.pos[x] : x) * hidden + i], v);
+        }
+        return v;
+    };
     float inv = 0.0f;
     if (y) {
         float ss = 0.0f;
         for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
-            const float v = y[at + i];
+            const float v = value(i);
             ss = fmaf(v, v, ss);
         }
         inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)hidden + eps);
@@ -933,31 +959,35 @@ __global__ void __launch_bounds__(512) rmsnorm_add_kernel(const float* y, const 
     for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
         float x = h[at + i];
         if (y) {
-            x = fmaf(y[at + i] * inv, w[i], x);
+            x = fmaf(value(i) * inv, w[i], x);
             h[at + i] = x;
         }
         if (rows) rows[at + i] = from_float<bf16>(x);
     }
 }
 
-FERRIS_API int ferris_rmsnorm_add(const float* y, const float* w, float* h, void* rows, int n_rows, int hidden, float eps,
-                                  void* stream) {
+FERRIS_API int ferris_rmsnorm_add(const float* y, const int* pos, const float* weights, int top, const float* w, float* h,
+                                  void* rows, int n_rows, int hidden, float eps, void* stream) {
     if (n_rows <= 0) return FERRIS_OK;
-    if (hidden <= 0 || (y && !w)) FERRIS_REFUSE("norm + add: hidden=%d", hidden);
+    if (hidden <= 0 || (y && !w) || top < 0 || (top == 0 && (pos || weights)))
+        FERRIS_REFUSE("norm + add: hidden=%d, sums of %d rows", hidden, top);
     cudaStream_t s = (cudaStream_t)stream;
+    const RowSum sum = {pos, weights, top};
     const bool aligned = (((uintptr_t)y | (uintptr_t)w | (uintptr_t)h | (uintptr_t)rows) & 15) == 0;
     if (y && hidden % 4 == 0 && hidden <= 4096 && aligned) {
-        const int warps = n_rows >= 148 * 8 ? 8 : (n_rows >= 148 * 2 ? 2 : 1);  // few rows: spread over the SMs
-        const dim3 grid((n_rows + warps - 1) / warps), block(32 * warps);
-#define FERRIS_NORM_ADD(VEC) ferris_launch(rmsnorm_add_rows_kernel<VEC>, grid, block, 0, s, y, w, h, (bf16*)rows, n_rows, hidden, eps)
-        if (hidden <= 512) FERRIS_NORM_ADD(4);
-        else if (hidden <= 1024) FERRIS_NORM_ADD(8);
-        else if (hidden <= 2048) FERRIS_NORM_ADD(16);
-        else FERRIS_NORM_ADD(32);
+        const int n4 = hidden / 4;
+        const dim3 grid(n_rows), block(n4 < 256 ? (n4 + 31) / 32 * 32 : 256);
+#define FERRIS_NORM_ADD(VPT) ferris_launch(rmsnorm_add_block_kernel<VPT>, grid, block, 0, s, y, sum, w, h, (bf16*)rows, hidden, eps)
+        switch ((n4 + 255) / 256) {
+            case 1: FERRIS_NORM_ADD(1); break;
+            case 2: FERRIS_NORM_ADD(2); break;
+            case 3: FERRIS_NORM_ADD(3); break;
+            default: FERRIS_NORM_ADD(4); break;
+        }
 #undef FERRIS_NORM_ADD
         FERRIS_LAUNCH_CHECK();
     }
     const int threads = hidden >= 2048 ? 512 : (hidden >= 512 ? 256 : 128);
-    ferris_launch(rmsnorm_add_kernel, dim3(n_rows), dim3(threads), 0, s, y, w, h, (bf16*)rows, hidden, eps);
+    ferris_launch(rmsnorm_add_kernel, dim3(n_rows), dim3(threads), 0, s, y, sum, w, h, (bf16*)rows, hidden, eps);
     FERRIS_LAUNCH_CHECK();
 }

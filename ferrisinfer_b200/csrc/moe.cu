@@ -752,6 +752,7 @@ FERRIS_API int ferris_moe_sorted_rows(int tokens, int top, int experts) {
 // identity_w (may be null): fp32 [tokens]; with it, ids may hold `experts` (an identity expert: the pair meets no weights)
 // and h also gets identity_w[t] x[t]; the scratch is then sized for experts + 1.  act_kind, act_limit: the gated
 // activation (ferris_gated_act).  row_scale: scratch, fp32 [rows], where the weights go onto the experts' inputs; else null.
+// h null: the pairs' results are left in y (row pos[pair]) and not added anywhere.
 FERRIS_API int ferris_moe_experts_grouped(const void* x, int ldx, const void* gate_up, const void* down, const int* ids,
                                           const float* weights, float* h, int ldh, int tokens, int width, int ff, int top,
                                           int experts, int rows, int* pos, int* row_token, int* tile_expert, void* xs,
@@ -777,7 +778,7 @@ FERRIS_API int ferris_moe_experts_grouped(const void* x, int ldx, const void* ga
     ferris_gemm_set_gated_activation(0, 0.0f);
     if (rc != FERRIS_OK) return rc;
     rc = ferris_gemm_grouped_tcgen05(act, down, y, 1, rows, width, ff, ff, ff, width, experts, width, 0, tile_expert, nullptr, stream);
-    if (rc != FERRIS_OK) return rc;
+    if (rc != FERRIS_OK || !h) return rc;  // without h the rows stay in y, for the caller to add
     const size_t n4 = (size_t)tokens * (width / 4);
     const size_t want4 = (n4 + 255) / 256;
     ferris_launch(moe_combine_kernel<bf16>, dim3((unsigned)(want4 < 148 * 16 ? want4 : 148 * 16)), dim3(256), 0, s, (const float*)y,
@@ -833,6 +834,7 @@ FERRIS_API int ferris_moe_router(const void* x, int ldx, int dtype, const void* 
 // weights fp32 [tokens, top]; act [tokens x top, ff] (scratch, the activations' type); h fp32 rows ldh apart.
 // With y (scratch, fp32 [tokens x top, width]), `experts` and few enough tokens the weights are read once per expert
 // (the expert-major kernels for few tokens and the adding pass); the sums are the same bit for bit either way.
+// h null (with y and few enough pairs): the pairs' results are left in y and not added anywhere.
 // input_weights: a token's weight for an expert goes onto the expert's input instead of its result.
 FERRIS_API int ferris_moe_experts_token_major(const void* x, int ldx, int dtype, const void* gate, const void* up,
                                               long long gate_up_stride, const void* down, const int* ids,
@@ -880,6 +882,7 @@ FERRIS_API int ferris_moe_experts_token_major(const void* x, int ldx, int dtype,
         else
             FERRIS_MOE_FEW(bf16);
 #undef FERRIS_MOE_FEW
+        if (!h) FERRIS_LAUNCH_CHECK();  // the pairs' results stay in y
         const size_t n4 = (size_t)tokens * (width / 4);
         const size_t want4 = (n4 + 255) / 256;
         const int* skip = identity_w ? ids : (const int*)nullptr;
@@ -893,6 +896,7 @@ FERRIS_API int ferris_moe_experts_token_major(const void* x, int ldx, int dtype,
                           skip, experts, (const bf16*)x, ldx, identity_w);
         FERRIS_LAUNCH_CHECK();
     }
+    if (!h) FERRIS_REFUSE("experts: the pairs' results stand apart only where few pairs share an expert's weights");
     const size_t smem_up = (size_t)width * sizeof(float), smem_down = (size_t)top * ff * sizeof(float);
     if (smem_up > 200 * 1024 || smem_down > 200 * 1024)
         FERRIS_REFUSE("experts: a row of %d or %d x %d activations do not fit shared memory", width, top, ff);

@@ -12,7 +12,8 @@
 // Rows: [nh d | nkv d | nkv dv unless values_from_keys].  Everything is computed in fp32 (position x frequency as one
 // fp32 product, sincosf in full precision); one block per token.
 //
-// Two kernels.  The paired one (even head sizes and row strides, rows that start on a pair): a token's cosines and
+// Three kernels.  The vector one (no rotation, values of their own): 16 bytes at a time, every element loaded once.  The
+// paired one (even head sizes and row strides, rows that start on a pair): a token's cosines and
 // sines are formed once in shared memory and serve all its heads, both sums of squares come out of one pass and one
 // reduction, and every thread loads, norms, rotates and stores two neighbouring elements at a time (in the
 // interleaved layout a pair that rotates together is one such load).  The general one takes every other geometry
@@ -73,8 +74,76 @@ __device__ __forceinline__ void pool_run(const T* k_cache, const T* v_cache, con
     }
 }
 
-// The pooled rows that the tokens of a step complete, behind the launch that wrote the step's keys and values.
+// 16 bytes as fp32 and back: eight bf16 or four floats
 template <typename T>
+struct Vec16 {
+    static constexpr int N = 16 / (int)sizeof(T);
+};
+__device__ __forceinline__ void widen(const uint4& u, float (&f)[4]) {
+    f[0] = __uint_as_float(u.x), f[1] = __uint_as_float(u.y), f[2] = __uint_as_float(u.z), f[3] = __uint_as_float(u.w);
+}
+__device__ __forceinline__ void widen(const uint4& u, float (&f)[8]) {
+    const uint32_t x[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) f[2 * i] = __uint_as_float(x[i] << 16), f[2 * i + 1] = __uint_as_float(x[i] & 0xffff0000u);
+}
+__device__ __forceinline__ uint4 narrow(const float (&f)[4]) {
+    return make_uint4(__float_as_uint(f[0]), __float_as_uint(f[1]), __float_as_uint(f[2]), __float_as_uint(f[3]));
+}
+__device__ __forceinline__ uint4 narrow(const float (&f)[8]) {
+    uint32_t x[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        __nv_bfloat162 v = __floats2bfloat162_rn(f[2 * i], f[2 * i + 1]);
+        x[i] = *reinterpret_cast<uint32_t*>(&v);
+    }
+    return make_uint4(x[0], x[1], x[2], x[3]);
+}
+
+// pool_run with 16 bytes of a row at a time (d and dv whole vectors, caches on 16 bytes); every element's sum is formed in
+// the same order.
+template <typename T>
+__device__ __forceinline__ void pool_run_vec(const T* k_cache, const T* v_cache, const int* table, T* pool_k, T* pool_v,
+                                             int slot, int pos, int pool, int nkv, int d, int dv, int page_size, int first,
+                                             int step) {
+    constexpr int E = Vec16<T>::N;
+    const int nk = nkv * d / E, total = nk + nkv * dv / E;
+    const int ppage = slot / page_size, pin = slot % page_size;
+    for (int x = first; x < total; x += step) {
+        const bool key = x < nk;
+        const int width = key ? d : dv, e = (key ? x : x - nk) * E;
+        const int head = e / width, i = e - head * width;
+        const T* base = key ? k_cache : v_cache;
+        float sum[E];
+#pragma unroll
+        for (int q = 0; q < E; ++q) sum[q] = 0.0f;
+        int j = pos - pool + 1;
+        while (j <= pos) {
+            const int in_page = j % page_size;
+            const int n = min(page_size - in_page, pos - j + 1);
+            const int page = table[j / page_size];
+            if (page < 0) return;  // never: a run's pages stay until it is complete
+            const T* src = base + (((size_t)page * nkv + head) * page_size + in_page) * width + i;
+#pragma unroll 8
+            for (int r = 0; r < n; ++r) {
+                float f[E];
+                widen(*reinterpret_cast<const uint4*>(src + (size_t)r * width), f);
+#pragma unroll
+                for (int q = 0; q < E; ++q) sum[q] += f[q];
+            }
+            j += n;
+        }
+#pragma unroll
+        for (int q = 0; q < E; ++q) sum[q] /= (float)pool;
+        T* dst = (key ? pool_k : pool_v) + (((size_t)ppage * nkv + head) * page_size + pin) * width + i;
+        *reinterpret_cast<uint4*>(dst) = narrow(sum);
+    }
+}
+
+// The pooled rows that the tokens of a step complete, behind the launch that wrote the step's keys and values.
+// A block looks at POOL_TOKENS tokens of the step.
+constexpr int POOL_TOKENS = 16;
+template <typename T, bool VEC>
 __global__ void __launch_bounds__(128) pool_blocks_kernel(const T* k_cache, const T* v_cache, T* pool_k, T* pool_v,
                                                           const int* __restrict__ tables, int max_blocks,
                                                           const int* __restrict__ token_seq, const int* __restrict__ positions,
@@ -82,11 +151,17 @@ __global__ void __launch_bounds__(128) pool_blocks_kernel(const T* k_cache, cons
                                                           int d, int dv, int page_size) {
     pdl_wait();
     pdl_launch_dependents();
-    const int t = blockIdx.x;
-    const int slot = pool_slots[t];
-    if (slot < 0) return;
-    pool_run<T>(k_cache, v_cache, tables + (size_t)token_seq[t] * max_blocks, pool_k, pool_v, slot, positions[t], pool, nkv, d,
-                dv, page_size, blockIdx.y * blockDim.x + threadIdx.x, gridDim.y * blockDim.x);
+    const int t0 = blockIdx.x * POOL_TOKENS, t1 = min(tokens, t0 + POOL_TOKENS);
+    for (int t = t0; t < t1; ++t) {
+        const int slot = pool_slots[t];
+        if (slot < 0) continue;
+        const int* table = tables + (size_t)token_seq[t] * max_blocks;
+        const int first = blockIdx.y * blockDim.x + threadIdx.x, step = gridDim.y * blockDim.x;
+        if (VEC)
+            pool_run_vec<T>(k_cache, v_cache, table, pool_k, pool_v, slot, positions[t], pool, nkv, d, dv, page_size, first, step);
+        else
+            pool_run<T>(k_cache, v_cache, table, pool_k, pool_v, slot, positions[t], pool, nkv, d, dv, page_size, first, step);
+    }
 }
 
 template <typename T>
@@ -297,6 +372,96 @@ __global__ void __launch_bounds__(256) qk_norm_rotary_cache_write_paired_kernel(
     }
 }
 
+// Without a rotation and with values of their own: rows of whole 16-byte vectors (d, dv, ld multiples of a vector), every
+// vector loaded once and kept in registers (VPT a thread) between the sums of squares and the scaling.
+template <typename T, int VPT>
+__global__ void __launch_bounds__(256) qk_norm_cache_write_vec_kernel(
+    T* qkv, int ld, const int* __restrict__ positions, const int* __restrict__ slot_mapping, T* __restrict__ k_cache,
+    T* __restrict__ v_cache, int nh, int nkv, int d, int dv, int page_size, const float* __restrict__ q_weight,
+    const float* __restrict__ k_weight, float eps, int write_kv, const PrepareExtras ex) {
+    constexpr int E = Vec16<T>::N;
+    __shared__ float scratch[66];
+    pdl_wait();
+    pdl_launch_dependents();
+    const int t = blockIdx.x;
+    const int slot = write_kv ? slot_mapping[t] : -1;
+    T* row = qkv + (size_t)t * ld;
+    const int nq = nh * d, nk = nkv * d, total = (nq + nk + (slot >= 0 ? nkv * dv : 0)) / E;
+    const int page = slot >= 0 ? slot / page_size : 0;
+    const int in_page = slot >= 0 ? slot % page_size : 0;
+    T* mixed = reinterpret_cast<T*>(ex.first) + (size_t)t * nkv * dv;
+    uint4 u[VPT], other[VPT];
+#pragma unroll
+    for (int j = 0; j < VPT; ++j) {
+        const int x = threadIdx.x + j * blockDim.x;
+        if (x < total) {
+            u[j] = *reinterpret_cast<const uint4*>(row + x * E);
+            if (ex.first && ex.lambda && x * E >= nq + nk) other[j] = *reinterpret_cast<const uint4*>(mixed + x * E - nq - nk);
+        }
+    }
+    const float lam = ex.first && ex.lambda ? *ex.lambda : 0.0f;
+    float sq = 0.0f, sk = 0.0f;
+#pragma unroll
+    for (int j = 0; j < VPT; ++j) {
+        const int e = (threadIdx.x + j * blockDim.x) * E;
+        if (e < nq + nk) {
+            float f[E];
+            widen(u[j], f);
+            float ss = 0.0f;
+#pragma unroll
+            for (int i = 0; i < E; ++i) ss = fmaf(f[i], f[i], ss);
+            if (e < nq) sq += ss; else sk += ss;
+        }
+    }
+    const float2 sums = block_sum2(sq, sk, scratch);
+    const float inv_q = q_weight ? 1.0f / sqrtf(sums.x / (float)nq + eps) : 1.0f;
+    const float inv_k = k_weight ? 1.0f / sqrtf(sums.y / (float)nk + eps) : 1.0f;
+#pragma unroll
+    for (int j = 0; j < VPT; ++j) {
+        const int x = threadIdx.x + j * blockDim.x, e = x * E;
+        if (x >= total) continue;
+        float f[E];
+        widen(u[j], f);
+        if (e < nq + nk) {  // without a cache to write, the keys are left alone
+            const bool is_q = e < nq;
+            if (!is_q && slot < 0) continue;
+            const int col = is_q ? e : e - nq;
+            const float* w = is_q ? q_weight : k_weight;
+            const float inv = is_q ? inv_q : inv_k;
+            if (w) {
+#pragma unroll
+                for (int i = 0; i < E; i += 4) {
+                    const float4 g = *reinterpret_cast<const float4*>(w + col + i);
+                    f[i] = (f[i] * inv) * g.x, f[i + 1] = (f[i + 1] * inv) * g.y;
+                    f[i + 2] = (f[i + 2] * inv) * g.z, f[i + 3] = (f[i + 3] * inv) * g.w;
+                }
+            }
+            const int head = col / d;
+            T* dst = is_q ? row + e : k_cache + (((size_t)page * nkv + head) * page_size + in_page) * d + col - head * d;
+            *reinterpret_cast<uint4*>(dst) = narrow(f);
+            continue;
+        }
+        const int col = e - nq - nk, head = col / dv;
+        if (ex.first) {
+            if (ex.lambda) {
+                float o[E];
+                widen(other[j], o);
+#pragma unroll
+                for (int i = 0; i < E; ++i) f[i] = fmaf(lam, o[i], (1.0f - lam) * f[i]);
+            } else {
+                *reinterpret_cast<uint4*>(mixed + col) = u[j];
+            }
+        }
+        *reinterpret_cast<uint4*>(v_cache + (((size_t)page * nkv + head) * page_size + in_page) * dv + col - head * dv) = narrow(f);
+    }
+    if (ex.pool_slots && slot >= 0 && ex.pool_slots[t] >= 0) {
+        __syncthreads();  // the token's own key and value are in their page
+        pool_run_vec<T>(k_cache, v_cache, ex.tables + (size_t)ex.token_seq[t] * ex.max_blocks, reinterpret_cast<T*>(ex.pool_k),
+                        reinterpret_cast<T*>(ex.pool_v), ex.pool_slots[t], positions[t], ex.pool, nkv, d, dv, page_size,
+                        threadIdx.x, blockDim.x);
+    }
+}
+
 // The norm per HEAD: every q and k head divided by the root mean square of its own d elements and multiplied by a
 // weight of d numbers that all heads share (wq for queries, wk for keys; null: that side is not normed), then rotated
 // and stored as above.  A warp per head: its lanes sum the head's squares, then norm, rotate and store it; the values
@@ -398,6 +563,24 @@ FERRIS_API int ferris_qk_norm_rotary_cache_write(void* qkv, int ld, int dtype, c
     if (write_kv && (!slot_mapping || !k_cache || !v_cache)) FERRIS_REFUSE("qk norm + rotation: no cache to write");
     cudaStream_t s = (cudaStream_t)stream;
     const size_t elem = dtype == FERRIS_F32 ? 4 : 2;
+    const int E = (int)(16 / elem);
+    const long long vectors = ((long long)(nh + nkv) * d + (long long)nkv * dv) / E;
+    if (rotary == 0 && !values_from_keys && (dtype == FERRIS_F32 || dtype == FERRIS_BF16) && d % E == 0 && dv % E == 0 && ld % E == 0 &&
+        vectors <= 4 * 256 && (((uintptr_t)qkv | (uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)first_values | (uintptr_t)pool_k |
+        (uintptr_t)pool_v | (uintptr_t)q_weight | (uintptr_t)k_weight) & 15) == 0) {
+        const dim3 block(vectors < 256 ? (unsigned)((vectors + 31) / 32 * 32) : 256);
+#define FERRIS_QK_VEC(T, VPT)                                                                                              \
+    ferris_launch(qk_norm_cache_write_vec_kernel<T, VPT>, dim3(tokens), block, 0, s, (T*)qkv, ld, positions, slot_mapping,  \
+                  (T*)k_cache, (T*)v_cache, nh, nkv, d, dv, page_size, q_weight, k_weight, eps, write_kv, ex)
+        const int vpt = (int)((vectors + 255) / 256);
+        if (dtype == FERRIS_F32) {
+            if (vpt <= 1) FERRIS_QK_VEC(float, 1); else if (vpt <= 2) FERRIS_QK_VEC(float, 2); else FERRIS_QK_VEC(float, 4);
+        } else {
+            if (vpt <= 1) FERRIS_QK_VEC(bf16, 1); else if (vpt <= 2) FERRIS_QK_VEC(bf16, 2); else FERRIS_QK_VEC(bf16, 4);
+        }
+#undef FERRIS_QK_VEC
+        FERRIS_LAUNCH_CHECK();
+    }
     const bool paired = !((d | dv | ld) & 1) && (uintptr_t)qkv % (2 * elem) == 0 && (uintptr_t)k_cache % (2 * elem) == 0 &&
                         (uintptr_t)v_cache % (2 * elem) == 0 && (uintptr_t)first_values % (2 * elem) == 0 && ((uintptr_t)q_weight | (uintptr_t)k_weight) % 8 == 0 &&
                         (dtype == FERRIS_F32 || dtype == FERRIS_BF16);
@@ -468,16 +651,21 @@ FERRIS_API int ferris_pool_blocks(const void* k_cache, const void* v_cache, void
     if (tokens <= 0) return FERRIS_OK;
     if (pool <= 0 || nkv <= 0 || d <= 0 || dv <= 0 || page_size <= 0 || max_blocks <= 0)
         FERRIS_REFUSE("pooled rows: pool=%d nkv=%d d=%d dv=%d page_size=%d max_blocks=%d", pool, nkv, d, dv, page_size, max_blocks);
-    const int slabs = (nkv * (d + dv) + 255) / 256;
-    const dim3 grid(tokens, slabs < 64 ? slabs : 64), block(128);
+    if (dtype != FERRIS_F32 && dtype != FERRIS_BF16) FERRIS_REFUSE("pooled rows: unknown dtype %d", dtype);
+    const int E = dtype == FERRIS_F32 ? 4 : 8;
+    const bool vec = d % E == 0 && dv % E == 0 &&
+                     (((uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)pool_k | (uintptr_t)pool_v) & 15) == 0;
+    const int items = vec ? nkv * (d + dv) / E : nkv * (d + dv), slabs = (items + 127) / 128;
+    const dim3 grid((tokens + POOL_TOKENS - 1) / POOL_TOKENS, slabs < 64 ? slabs : 64), block(128);
     cudaStream_t s = (cudaStream_t)stream;
-    if (dtype == FERRIS_F32)
-        ferris_launch(pool_blocks_kernel<float>, grid, block, 0, s, (const float*)k_cache, (const float*)v_cache, (float*)pool_k,
-                      (float*)pool_v, tables, max_blocks, token_seq, positions, pool_slots, tokens, pool, nkv, d, dv, page_size);
-    else if (dtype == FERRIS_BF16)
-        ferris_launch(pool_blocks_kernel<bf16>, grid, block, 0, s, (const bf16*)k_cache, (const bf16*)v_cache, (bf16*)pool_k,
-                      (bf16*)pool_v, tables, max_blocks, token_seq, positions, pool_slots, tokens, pool, nkv, d, dv, page_size);
-    else
-        FERRIS_REFUSE("pooled rows: unknown dtype %d", dtype);
+#define FERRIS_POOL(T, VEC)                                                                                                \
+    ferris_launch(pool_blocks_kernel<T, VEC>, grid, block, 0, s, (const T*)k_cache, (const T*)v_cache, (T*)pool_k, (T*)pool_v, \
+                  tables, max_blocks, token_seq, positions, pool_slots, tokens, pool, nkv, d, dv, page_size)
+    if (dtype == FERRIS_F32) {
+        if (vec) FERRIS_POOL(float, true); else FERRIS_POOL(float, false);
+    } else {
+        if (vec) FERRIS_POOL(bf16, true); else FERRIS_POOL(bf16, false);
+    }
+#undef FERRIS_POOL
     FERRIS_LAUNCH_CHECK();
 }

@@ -881,17 +881,12 @@ def paged_attention_simt(qkv: torch.Tensor, out: torch.Tensor, k_cache: torch.Te
     if (_attention_rows and qkv.dtype == torch.bfloat16 and not v_stride and terms.slopes is None and terms.log_r1 is None
             and (max_q_len <= 1 or _attention_tiled) and ldq % 8 == 0 and ldo % 2 == 0 and qkv.data_ptr() % 16 == 0
             and _lib().ferris_attention_rows_takes(num_heads, num_kv_heads, head_dim, dv, 1 if max_q_len > 1 else 0)):
-        floats = T * num_heads * ATTENTION_MAX_SHARES * (dv + 2) if single else 0
-        scratch = workspace.get("attn_shares", (floats,), torch.float32) if single else None
-        launches = _c_int(0)
-        rc = _lib().ferris_attention_rows(
+        _check(_lib().ferris_attention_rows(
             _ptr(qkv), _c_int(ldq), _ptr(out), _c_int(ldo), _ptr(k_cache), _ptr(v_cache), _ptr(block_tables),
             _c_int(block_tables.shape[1]), _ptr(token_seq), _ptr(positions), _c_int(T), _c_int(num_heads),
             _c_int(num_kv_heads), _c_int(head_dim), _c_int(dv), _c_int(k_cache.shape[2]),
             _c_int(-chunk if chunk else (window or 0)), _c_float(scale), _ptr(terms.sink), *pool_args,
-            _c_int(1 if max_q_len > 1 else 0), _c_int(span if single else 0), _ptr(scratch), ctypes.c_longlong(floats),
-            ctypes.byref(launches), _stream())
-        _check(rc, "attention rows", launches.value)
+            _c_int(1 if max_q_len > 1 else 0), _c_int(span if single else 0), _stream()), "attention rows")
         return
     fn = _lib().ferris_paged_attention_simt
     extra = (_c_int(0), _ptr(None), ctypes.c_longlong(0))
@@ -938,20 +933,28 @@ def embed_positions(table: torch.Tensor, pos_table: torch.Tensor, ids: torch.Ten
 
 
 def rmsnorm_add(y: Optional[torch.Tensor], weight: Optional[torch.Tensor], eps: float, h: torch.Tensor,
-                rows: Optional[torch.Tensor] = None):
+                rows: Optional[torch.Tensor] = None, parts: Optional["PairRows"] = None):
     """h += rmsnorm(y) * weight, everything fp32; ``rows`` (optional, bf16): h rounded, what the next products read.
-    ``y`` None: h stays, the rows alone are written."""
+    ``y`` None: h stays, the rows alone are written.  ``parts`` (instead of y): the rows to norm are the sums of a mixture's
+    results that ``moe_experts`` left apart."""
     _need(h, "residual rows", torch.float32)
     T, H = h.shape
+    pos = wts = None
+    top = 0
+    if parts is not None:
+        y, pos, wts, top = parts.y, parts.pos, parts.weights, parts.top
+        if y.shape[1] != H or (pos is not None and pos.numel() != T * top) or (wts is not None and wts.numel() != T * top) \
+                or (pos is None and y.shape[0] != T * top):
+            raise KernelError(f"norm + add: residual {tuple(h.shape)}, results {tuple(y.shape)} of {top} a row")
     if y is not None:
         _need(y, "norm input", torch.float32)
         _need(weight, "norm weight", torch.float32)
     if rows is not None:
         _need(rows, "rounded residual rows", torch.bfloat16)
-    if (y is not None and (y.shape != (T, H) or weight.numel() != H)) or (rows is not None and rows.shape != (T, H)):
+    if (y is not None and ((parts is None and y.shape != (T, H)) or weight.numel() != H)) or (rows is not None and rows.shape != (T, H)):
         raise KernelError(f"norm + add: residual {tuple(h.shape)}, input {None if y is None else tuple(y.shape)}")
-    _check(_lib().ferris_rmsnorm_add(_ptr(y), _ptr(weight), _ptr(h), _ptr(rows), _c_int(T), _c_int(H), _c_float(eps),
-                                     _stream()), "norm + add")
+    _check(_lib().ferris_rmsnorm_add(_ptr(y), _ptr(pos), _ptr(wts), _c_int(top), _ptr(weight), _ptr(h), _ptr(rows), _c_int(T),
+                                     _c_int(H), _c_float(eps), _stream()), "norm + add")
 
 
 def embed_sinusoid(table: torch.Tensor, ids: torch.Tensor, positions: torch.Tensor, freq: torch.Tensor, scale: float,
@@ -1780,12 +1783,31 @@ def moe_router(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tenso
                                     _ptr(idw), _stream()), "router")
 
 
+class PairRows:
+    """A mixture's results before they are added: row t of the sum is, over s < ``top`` in that order, weights[t, s] times
+    y[pos[t, s]] (``weights`` None: unweighted; ``pos`` None: y[t * top + s])."""
+
+    __slots__ = ("y", "pos", "weights", "top")
+
+    def __init__(self, y: torch.Tensor, pos: Optional[torch.Tensor], weights: Optional[torch.Tensor], top: int):
+        self.y, self.pos, self.weights, self.top = y, pos, weights, int(top)
+
+
 MOE_FEW_MAX_PAIRS = 1024  # up to here the token-major form reads an expert's weights once for all its tokens
+MOE_FEW_MAX_WIDTH = 8192  # four rows of that width and the weights' ring fit shared memory
 MOE_GROUPED_MIN_TOKENS = 17  # from here on (bf16) the experts' rows are sorted by expert and meet tensor-core tiles
 
 
+def moe_leaves_apart(tokens: int, top: int, width: int, ff: int, x: torch.Tensor) -> bool:
+    """Whether ``moe_experts`` can leave the results of such a step apart (``h`` None)."""
+    if (x.dtype == torch.bfloat16 and tokens >= MOE_GROUPED_MIN_TOKENS and width % 8 == 0 and ff % 8 == 0
+            and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0):
+        return True
+    return 1 < tokens * top <= MOE_FEW_MAX_PAIRS and width % 4 == 0 and max(width, ff) <= MOE_FEW_MAX_WIDTH
+
+
 def moe_experts(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor,
-                h: torch.Tensor, workspace=None, accumulate: bool = True, grouped: Optional[bool] = None,
+                h: Optional[torch.Tensor], workspace=None, accumulate: bool = True, grouped: Optional[bool] = None,
                 activation: str = "silu", limit: float = 0.0, identity_w: Optional[torch.Tensor] = None,
                 input_weights: bool = False):
     """h (+)= sum over a row's chosen experts of weight x down_e (silu(gate_e x) * (up_e x)).  gate_up [E, 2 ff, W] (an
@@ -1797,7 +1819,8 @@ def moe_experts(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, ids:
     in the order of its choices.  ``activation``, ``limit``: the experts' gated activation (see ``gated_activation``).
     ``identity_w`` fp32 [T]: ids may then hold E, an expert that meets no weights, and h also gets identity_w[t] x[t].
     ``input_weights``: a token's weight for an expert goes onto the expert's input (both first products times the weight
-    in fp32, ahead of the activation), and the results are added as they are."""
+    in fp32, ahead of the activation), and the results are added as they are.
+    ``h`` None (where ``moe_leaves_apart``): the results are left apart and returned as ``PairRows``."""
     T, W, ldx = _rows(x, "experts input")
     if activation not in GATED_ACTIVATIONS:
         raise KernelError(f"experts: activation '{activation}' is not known ({', '.join(GATED_ACTIVATIONS)})")
@@ -1806,21 +1829,21 @@ def moe_experts(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, ids:
         _need(identity_w, "identity weights", torch.float32)
         if identity_w.numel() != T:
             raise KernelError(f"experts: {identity_w.numel()} identity weights for {T} rows")
-    T2, W2, ldh = _rows(h, "experts output")
+    T2, W2, ldh = _rows(h, "experts output") if h is not None else (T, W, W)
     _need(gate_up, "gate and up matrices", x.dtype)
     _need(down, "down matrices", x.dtype)
     _need(ids, "expert ids", torch.int32)
     _need(weights, "expert weights", torch.float32)
     E, ff = gate_up.shape[0], gate_up.shape[1] // 2
     top = ids.shape[1]
-    if (gate_up.shape != (E, 2 * ff, W) or down.shape != (E, W, ff) or (T2, W2) != (T, W) or h.dtype != torch.float32
+    if (gate_up.shape != (E, 2 * ff, W) or down.shape != (E, W, ff) or (T2, W2) != (T, W) or (h is not None and h.dtype != torch.float32)
             or ids.shape != (T, top) or weights.shape != (T, top)):
         raise KernelError(f"experts: x {tuple(x.shape)}, gate/up {tuple(gate_up.shape)}, down {tuple(down.shape)}, "
                           f"ids {tuple(ids.shape)}")
     get = (lambda name, shape, dtype: workspace.get(name, shape, dtype)) if workspace is not None else \
         (lambda name, shape, dtype: torch.empty(shape, dtype=dtype, device=x.device))
     can_group = (x.dtype == torch.bfloat16 and W % 8 == 0 and ff % 8 == 0 and ldx % 8 == 0 and ldh % 4 == 0
-                 and x.data_ptr() % 16 == 0 and h.data_ptr() % 16 == 0)
+                 and x.data_ptr() % 16 == 0 and (h is None or h.data_ptr() % 16 == 0))
     if grouped is None:
         grouped = can_group and T >= MOE_GROUPED_MIN_TOKENS
     if grouped:
@@ -1841,12 +1864,14 @@ def moe_experts(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, ids:
                                                  _c_int(E), _c_int(rows), _ptr(pos), _ptr(row_token), _ptr(tile_expert),
                                                  _ptr(xs), _ptr(act), _ptr(y), _c_int(1 if accumulate else 0),
                                                  _c_int(act_kind), _c_float(limit), _ptr(identity_w), _ptr(row_scale), _stream()),
-               "experts (sorted)", 5)
-        return
+               "experts (sorted)", 5 if h is not None else 4)
+        return None if h is not None else PairRows(y, pos, None if input_weights else weights, top)
     act = get("moe_act", (T * top, ff), x.dtype)
     up = gate_up[:, ff:, :]
     # few pairs: the weights are read once per expert, the results of a pair stand in y until they are added
-    few = 1 < T * top <= MOE_FEW_MAX_PAIRS and W % 4 == 0 and ldh % 4 == 0 and h.data_ptr() % 16 == 0
+    few = 1 < T * top <= MOE_FEW_MAX_PAIRS and W % 4 == 0 and ldh % 4 == 0 and (h is None or h.data_ptr() % 16 == 0)
+    if h is None and (identity_w is not None or not moe_leaves_apart(T, top, W, ff, x)):
+        raise KernelError("experts: a step of this form adds its results itself")
     y = get("moe_pair_out", (T * top, W), torch.float32) if few else None
     _check(_lib().ferris_moe_experts_token_major(_ptr(x), _c_int(ldx), _c_int(_dt(x, "experts")), _ptr(gate_up), _ptr(up),
                                                  ctypes.c_longlong(2 * ff * W), _ptr(down), _ptr(ids), _ptr(weights),
@@ -1855,7 +1880,8 @@ def moe_experts(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, ids:
                                                  _ptr(y) if few else ctypes.c_void_p(0), _c_int(E), _c_int(act_kind),
                                                  _c_float(limit), _ptr(identity_w), _c_int(1 if input_weights else 0),
                                                  _stream()),
-           "experts", 3 if few else 2)
+           "experts", (3 if few else 2) if h is not None else 2)
+    return None if h is not None else PairRows(y, None, None if input_weights else weights, top)
 
 
 def kernel_status() -> int:

@@ -210,6 +210,9 @@ class Norm(Part):
         self.forward(h, out)
         return out
 
+    # True if add_into also takes ``ops.PairRows`` for y (a mixture's results that its own kernel adds first)
+    adds_parts = False
+
     def add_into(self, y: torch.Tensor, h: torch.Tensor, rows: Optional[torch.Tensor], workspace) -> None:
         """h += norm(y), y and h fp32; ``rows`` (or None): h in the activations' type as well.  The default is a norm, a
         sum and a cast; a norm with a kernel for all of it overrides this."""

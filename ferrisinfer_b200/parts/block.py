@@ -164,12 +164,16 @@ class OutputNormBlock(ParallelResidualBlock):
         self.mixer_norm.add_into(y, h, after, ctx.workspace)
         if self.feed_forward is None:
             return
-        if getattr(self.feed_forward, "can_overwrite", False):
-            self.feed_forward.forward(x, y, ctx, accumulate=False)
-        else:
-            y.zero_()
-            self.feed_forward.forward(x, y, ctx)
-        self.feed_forward_norm.add_into(y, h, after, ctx.workspace)
+        parts = None
+        if self.feed_forward_norm.adds_parts and hasattr(self.feed_forward, "forward_apart"):
+            parts = self.feed_forward.forward_apart(x, ctx)  # a mixture whose results the norm's kernel adds on its way
+        if parts is None:
+            if getattr(self.feed_forward, "can_overwrite", False):
+                self.feed_forward.forward(x, y, ctx, accumulate=False)
+            else:
+                y.zero_()
+                self.feed_forward.forward(x, y, ctx)
+        self.feed_forward_norm.add_into(y if parts is None else parts, h, after, ctx.workspace)
 
 
 register_part("block", "output_norm", OutputNormBlock)

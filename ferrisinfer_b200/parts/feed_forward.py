@@ -221,6 +221,14 @@ class MixtureOfExperts(FeedForward):
             self.down = self.router.new_zeros(1, W, I)
 
     def forward(self, x, h, ctx, accumulate: bool = True):
+        self._run(x, h, ctx, accumulate)
+
+    def forward_apart(self, x, ctx):
+        """The chosen experts' results before they are added, as ``ops.PairRows``, for a caller whose own kernel adds them on
+        its way; None (nothing computed that counts) where the step's form adds them itself."""
+        return None if self.identity else self._run(x, None, ctx, False)
+
+    def _run(self, x, h, ctx, accumulate):
         T = x.shape[0]
         ids = ctx.workspace.get("moe_ids", (T, self.top), torch.int32)
         weights = ctx.workspace.get("moe_weights", (T, self.top), torch.float32)
@@ -229,9 +237,11 @@ class MixtureOfExperts(FeedForward):
         if self.scored is not None:
             scored = {"correction": self.correction, "groups": self.scored[1], "keep": self.scored[2],
                       "with_weights": self.experts, "identity_w": identity_w}
+        if h is None and not ops.moe_leaves_apart(T, self.top, self.hidden_size, self.intermediate_size, x):
+            return None
         ops.moe_router(x, self.router, self.router_bias, ids, weights, self.top, scored=scored, sigmoid=self.sigmoid_scores)
-        ops.moe_experts(x, self.gate_up, self.down, ids, weights, h, ctx.workspace, accumulate=accumulate,
-                        activation=self.activation, limit=self.limit, identity_w=identity_w, input_weights=self.input_weights)
+        return ops.moe_experts(x, self.gate_up, self.down, ids, weights, h, ctx.workspace, accumulate=accumulate,
+                               activation=self.activation, limit=self.limit, identity_w=identity_w, input_weights=self.input_weights)
 
 
 register_part("feed_forward", "swiglu", SwiGLU)

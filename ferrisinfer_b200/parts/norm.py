@@ -71,8 +71,14 @@ class GroupedRMSNorm(Norm):
         self.forward(h, out)
         return out
 
+    @property
+    def adds_parts(self):
+        return self.groups == 1
+
     def add_into(self, y, h, rows, workspace):
-        if self.groups == 1:
+        if isinstance(y, ops.PairRows):
+            ops.rmsnorm_add(None, self.weight, self.eps, h, rows, parts=y)
+        elif self.groups == 1:
             ops.rmsnorm_add(y, self.weight, self.eps, h, rows)
         else:
             super().add_into(y, h, rows, workspace)

@@ -122,6 +122,23 @@ def test_norm_of_a_result_added_into_the_residual(device, width, T):
     assert torch.equal(rows, alone.to(BF16)) and torch.equal(alone, got)
 
 
+@pytest.mark.parametrize("width", [43, 64, 2048])
+@pytest.mark.parametrize("top,ordered,weighted", [(1, False, True), (3, True, False), (4, True, True), (2, False, False)])
+def test_results_of_a_mixture_added_on_the_norms_way(device, width, top, ordered, weighted):
+    """The rows to norm are sums of rows that stand apart, in an order of their own or not, weighted or not."""
+    ops = _ops()
+    torch.manual_seed(width + top)
+    T, R = 21, 21 * top + (9 if ordered else 0)
+    y, h, w = torch.randn(R, width), torch.randn(T, width), 1.0 + 0.2 * torch.randn(width)
+    pos = torch.randperm(R)[:T * top].view(T, top) if ordered else torch.arange(T * top).view(T, top)
+    f = torch.rand(T, top) if weighted else torch.ones(T, top)
+    want = h.double() + plain.rms((f.double().unsqueeze(-1) * y.double()[pos]).sum(1), 1e-4) * w.double()
+    got, rows = h.to(device), torch.empty(T, width, dtype=BF16, device=device)
+    parts = ops.PairRows(y.to(device), pos.int().to(device) if ordered else None, f.to(device) if weighted else None, top)
+    ops.rmsnorm_add(None, w.to(device), 1e-4, got, rows, parts=parts)
+    assert torch.allclose(got.cpu().double(), want, atol=3e-6, rtol=3e-6) and torch.equal(rows, got.to(BF16))
+
+
 def pooled_setup(device, dtype, T, nkv, d, dv, ps, pool, seed):
     """Random keys and values of ``T`` positions in pages out of order, and empty pages for their blocks' means:
     (keys, values, k cache, v cache, table, PooledKeys with everything zero, slot of every position's block or -1)."""
@@ -176,7 +193,8 @@ def test_means_of_blocks(device, nkv, d, dv, ps, pool, T, dtype):
 
 
 @pytest.mark.parametrize("dtype", [F32, BF16])
-@pytest.mark.parametrize("nh,nkv,d,dv", [(4, 2, 32, 24), (3, 3, 15, 9), (4, 1, 64, 64)])
+@pytest.mark.parametrize("nh,nkv,d,dv", [(4, 2, 32, 24), (3, 3, 15, 9), (4, 1, 64, 64), (2, 2, 20, 12), (16, 8, 128, 64),
+                                          (48, 4, 128, 128)])
 def test_norm_mixing_cache_write_and_means_of_single_tokens(device, nh, nkv, d, dv, dtype):
     """The kernel between the product and attention: values mixed with (or left for) another layer, and, in steps of single
     tokens, the means of the blocks that the tokens complete, bit for bit those of the launch behind a portion."""
