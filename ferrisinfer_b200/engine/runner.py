@@ -98,7 +98,7 @@ class ModelRunner:
         self.device = torch.device(device)
         self.vocab_size = model.vocab_size
         self.max_model_len = int(max_model_len or model.plan.max_positions)
-        if model.plan.positions_bounded:
+        if getattr(model.plan, "positions_bounded", False):
             self.max_model_len = min(self.max_model_len, model.plan.max_positions)
         self.cache = CacheManager(model.cache_needs(), page_size, num_pages, max_requests, dtype=dtype,
                                   device=self.device, extra_states=extra_states, prefix_sharing=prefix_sharing,
