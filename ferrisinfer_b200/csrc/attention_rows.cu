@@ -125,15 +125,19 @@ __device__ __forceinline__ void weights_times_values(float (&o)[DT][4], const fl
     split3(s[2 * kk + 1][0], s[2 * kk + 1][1], p[0][2], p[1][2], p[2][2]);
     split3(s[2 * kk + 1][2], s[2 * kk + 1][3], p[0][3], p[1][3], p[2][3]);
     const uint32_t at = v_base + (uint32_t)(16 * kk + ((lane >> 3) & 1) * 8 + (lane & 7)) * vp + (lane >> 4) * 16;
+    // four accumulators in turn, so that a part's product does not wait for the part's before it
 #pragma unroll
-    for (int n = 0; n < DT; n += 2) {
+    for (int n = 0; n < DT; n += 4) {
         if (8 * n < dv) {
-            uint32_t b[4];
-            ldmatrix_x4_trans(b, at + n * 16);
+            uint32_t b[2][4];
+            ldmatrix_x4_trans(b[0], at + n * 16);
+            ldmatrix_x4_trans(b[1], at + n * 16 + 32);
 #pragma unroll
             for (int x = 0; x < 3; ++x) {
-                mma_bf16_16816(o[n], p[x], b[0], b[1]);
-                mma_bf16_16816(o[n + 1], p[x], b[2], b[3]);
+                mma_bf16_16816(o[n], p[x], b[0][0], b[0][1]);
+                mma_bf16_16816(o[n + 1], p[x], b[0][2], b[0][3]);
+                mma_bf16_16816(o[n + 2], p[x], b[1][0], b[1][1]);
+                mma_bf16_16816(o[n + 3], p[x], b[1][2], b[1][3]);
             }
         }
     }
@@ -143,7 +147,7 @@ __device__ __forceinline__ void weights_times_values(float (&o)[DT][4], const fl
 // D: columns held for a head (64, 128, 256; d, dv <= D).  KT: keys to a tile.  The query fragments stay in registers up to
 // D = 128 and come from shared memory beyond.
 template <int D, int KT, bool POOL>
-__global__ void __launch_bounds__(AR_THREADS) attention_rows_kernel(const AttentionArgs p) {
+__global__ void __launch_bounds__(AR_THREADS, D <= 128 ? 3 : 2) attention_rows_kernel(const AttentionArgs p) {
     constexpr int KS = D / 16, DT = D / 8, NT = KT / 8;
     constexpr bool QREG = D <= 128;
     extern __shared__ __align__(16) uint8_t ar_smem[];
@@ -487,12 +491,15 @@ __global__ void __launch_bounds__(AR_THREADS) attention_single_rows_kernel(const
         for (int x = 0; x < 3; ++x) pw[x][0] = movmatrix_trans(pw[x][0]), pw[x][1] = movmatrix_trans(pw[x][1]);
         const uint32_t v_at = kb + V_OFF + (uint32_t)((lane & 7) + (lane >> 4) * 8) * PITCH + ((lane >> 3) & 1) * 16;
 #pragma unroll
-        for (int n = 0; n < MT; ++n) {
+        for (int n = 0; n < MT; n += 4) {  // four accumulators in turn
             if (16 * n < dv) {
-                uint32_t a[4];
-                ldmatrix_x4_trans(a, v_at + n * 32);
+                uint32_t a[4][4];
 #pragma unroll
-                for (int x = 0; x < 3; ++x) mma_bf16_16816(o[n], a, pw[x][0], pw[x][1]);
+                for (int i = 0; i < 4; ++i) ldmatrix_x4_trans(a[i], v_at + (n + i) * 32);
+#pragma unroll
+                for (int x = 0; x < 3; ++x)
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) mma_bf16_16816(o[n + i], a[i], pw[x][0], pw[x][1]);
             }
         }
         __syncwarp();  // the stage is read: the copy after next may overwrite it

@@ -108,12 +108,14 @@ def dense(x, w, prefix, limit):
 
 def router(x, w, prefix, mlp, margins=None):
     """(chosen experts, their scores) of every row.  ``margins`` (a list with one entry per token, or None): lowered to
-    the gap between the last chosen logit and the first that is not, over the logits' spread, where that is smaller."""
+    the gap between the last chosen logit and the first that is not, over the size a logit has (the row's root mean square
+    times that of the router rows' lengths; the logits' own spread says nothing where there are two), where that is smaller."""
     E, top = mlp["router"]["experts"], mlp["router"]["top"]
     z = x @ w[prefix + ".router"].T
     if margins is not None and top < E:
         ordered = torch.sort(z, dim=-1, descending=True).values
-        gap = (ordered[:, top - 1] - ordered[:, top]) / (ordered[:, 0] - ordered[:, -1])
+        size = (x * x).mean(dim=-1).sqrt() * (w[prefix + ".router"] ** 2).sum(dim=-1).mean().sqrt()
+        gap = (ordered[:, top - 1] - ordered[:, top]) / size
         for t in range(x.shape[0]):
             margins[t] = min(margins[t], float(gap[t]))
     s = torch.sigmoid(z)

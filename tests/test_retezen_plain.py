@@ -272,7 +272,8 @@ def test_mixture_by_hand():
     for t in range(3):
         z = [sum(float(w["m.router"][e, i]) * float(x[t, i]) for i in range(W)) for e in range(E)]
         order = sorted(range(E), key=lambda e: -z[e])
-        assert abs(margins[t] - (z[order[1]] - z[order[2]]) / (z[order[0]] - z[order[-1]])) < 1e-12
+        size = math.sqrt(sum(float(a) ** 2 for a in x[t]) / W) * math.sqrt(float((w["m.router"] ** 2).sum()) / E)
+        assert abs(margins[t] - (z[order[1]] - z[order[2]]) / size) < 1e-12
         want = [0.0] * W
         for e in order[:top]:
             s = 1.0 / (1.0 + math.exp(-z[e]))
