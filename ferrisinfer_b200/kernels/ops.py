@@ -826,7 +826,9 @@ def paged_attention_simt(qkv: torch.Tensor, out: torch.Tensor, k_cache: torch.Te
     keys among 64 query rows runs where it takes the geometry.  ``max_kv_len`` and ``workspace`` (a step of single
     tokens): the most keys a request holds, and where scratch comes from; the keys of a token are then cut into
     shares that run side by side, and query heads of one kv head share its keys.  ``pooled`` (with a window): beside the
-    window's tokens the query sees one row of ``pooled`` for every run of positions that lies wholly before the window."""
+    window's tokens the query sees one row of ``pooled`` for every run of positions that lies wholly before the window.
+    bf16 without a distance penalty and with values in rows of their own runs on tensor cores where the geometry allows it
+    (``set_attention_rows``); everything else on CUDA cores."""
     dv = int(v_head_dim or head_dim)
     if chunk:
         if window or chunk < 0:
