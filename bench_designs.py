@@ -363,8 +363,9 @@ def nusudra_kernel_numbers(s: dict, peaks: dict) -> dict:
         slots = (tables[ctx.token_seq.long(), (ctx.positions // 16).long()] * 16 + ctx.positions % 16).int()
         freq = torch.full((rot // 2,), 0.01, device=dev)
         nw = torch.ones(rank, device=dev)
-        t = _timed(lambda: ops.latent_prepare(proj, 0, H * (d + rot), nw, 1e-6, ctx.positions, freq, rot, slots, kl, ql, H, d, rot,
-                                              rank), flush, reps=10 if T <= 64 else 1)
+        qw, table = H * (d + rot), ops.RotaryTable(freq, rot)
+        t = _timed(lambda: ops.latent_prepare(ctx.positions, table, 1e-6, H, d, rot, rank, queries=(proj[:, :qw], ql),
+                                              keys=(proj[:, qw:], nw, slots, kl)), flush, reps=10 if T <= 64 else 1)
         record(f"latent_prepare_{name}", t, bytes_=T * (2 * H * rot + 2 * (rank + rot)) * 2)
     # ---- row-wise kernels of a long step and of a decode step
     S4 = 4

@@ -16,8 +16,8 @@ Here ONE manager serves all requests:
   different needs (all keys / a window of them / a row for every so many tokens) have pools and tables of their own.
 * A request's pages are allocated before a step for every token the step brings (``extend``),
   counted as held after it (``commit``), and given back when the request ends (``release``) or, in a
-  window group (or one of chunks), as soon as the window has passed them or their chunk is over (in ``commit``); a page that is given back is
-  the next one handed out.
+  window group (or one of chunks), as soon as the window has passed them or their chunk is over (in ``commit``; not the
+  pages of first tokens that a window keeps); a page that is given back is the next one handed out.
 * Mixers with a ``FixedState`` need, and the engine itself (sampler state), get a tensor
   ``[slots, *shape]``; a request holds one slot id from admission to release, and the slot's rows
   are zeroed at admission.
@@ -336,6 +336,10 @@ class CacheManager:
         """Lowest block that a query at position >= num_tokens can still read."""
         return g.need.first_needed(num_tokens) // self.page_size
 
+    def _blocks_kept(self, g: PageGroup) -> int:
+        """How many blocks from the first on stay until the request ends (those of tokens that no window passes)."""
+        return -(-g.need.keep_first // self.page_size)
+
     def _blocks(self, g: PageGroup, num_tokens: int) -> int:
         """How many blocks the rows of ``num_tokens`` tokens fill."""
         return -(-g.need.rows(num_tokens) // self.page_size)
@@ -447,7 +451,8 @@ class CacheManager:
             table = rc.tables[g.gid]
             upto = min(self._first_needed_block(g, new_total), len(table))
             b = upto - 1
-            while b >= 0 and table[b] != NO_PAGE:  # everything below an earlier hole went back before
+            kept = self._blocks_kept(g)
+            while b >= kept and table[b] != NO_PAGE:  # everything below an earlier hole went back before
                 g.pool.release(table[b])
                 table[b] = NO_PAGE
                 freed += 1

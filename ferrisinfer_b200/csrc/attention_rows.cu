@@ -66,10 +66,17 @@ struct AttentionArgs {
     const int* token_seq;
     const int* positions;
     const float* sink;
-    PooledKeys pk;  // every = 0: none
+    PooledKeys pk;  // every = keep = 0: none
     int ldq, ldo, max_blocks, tokens, nh, nkv, d, dv, page_size, window;
-    float scale2;  // scale x log2 e
+    float scale2;  // scale x log2 e; with a soft cap: cap x log2 e, and scale_cap = scale / cap
+    float scale_cap;  // 0: no cap
+    const bf16* gate;  // the heads' gates, rows ldgate apart (null: none)
+    int ldgate;
 };
+// sigmoid of the gate of head h at token t
+__device__ __forceinline__ float gate_of(const AttentionArgs& p, int t, int h) {
+    return p.gate ? 1.0f / (1.0f + expf(-to_float(p.gate[(size_t)t * p.ldgate + h]))) : 1.0f;
+}
 
 __device__ __forceinline__ int page_of(const int* table, int j, int page_size, int pshift) {
     return table[pshift >= 0 ? (j >> pshift) : (j / page_size)];
@@ -208,7 +215,7 @@ __global__ void __launch_bounds__(AR_THREADS, D <= 128 ? 3 : 2) attention_rows_k
         while (tb + 1 < t_end && p.token_seq[tb + 1] == sq) ++tb;
         const int pa = p.positions[ta], pb = p.positions[tb];
         const int kmin = first_key(pa, p.window);  // of the first token: no later token of the request sees an earlier key
-        const int runs = POOL ? first_key(pb, p.window) / p.pk.every : 0;
+        const int runs = POOL ? ahead_rows(p.pk, first_key(pb, p.window)) : 0;
         const int run_tiles = (runs + KT - 1) / KT;
         const int tiles = run_tiles + (pb - kmin + KT) / KT;
         const int* table = p.tables + (size_t)sq * p.max_blocks;
@@ -247,7 +254,7 @@ __global__ void __launch_bounds__(AR_THREADS, D <= 128 ? 3 : 2) attention_rows_k
             const bool mine = rseq[a] == sq;
             lo[a] = mine ? first_key(rpos[a], p.window) : 0;
             hi[a] = mine ? rpos[a] : -1;
-            seen_runs[a] = POOL && mine ? lo[a] / p.pk.every : 0;
+            seen_runs[a] = POOL && mine ? ahead_rows(p.pk, lo[a]) : 0;
         }
         for (int i = 0; i < tiles; ++i) {
             fetch(i + 1, next_page);
@@ -280,6 +287,12 @@ __global__ void __launch_bounds__(AR_THREADS, D <= 128 ? 3 : 2) attention_rows_k
                         mma_bf16_16816(s[n + 1], af, b[2], b[3]);
                     }
                 }
+            }
+            if (p.scale_cap > 0.0f) {
+#pragma unroll
+                for (int n = 0; n < NT; ++n)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) s[n][e] = tanhf(s[n][e] * p.scale_cap);
             }
             const bool run = POOL && i < run_tiles;
             const int j0 = run ? i * KT : kmin + (i - run_tiles) * KT;
@@ -319,7 +332,7 @@ __global__ void __launch_bounds__(AR_THREADS, D <= 128 ? 3 : 2) attention_rows_k
         if (rt[a] >= t_end) continue;
         const int head = hk * g + (16 * warp + gq + 8 * a) % g;
         const float sink = p.sink ? exp2f(p.sink[head] * LOG2E - m[a]) : 0.0f;
-        const float inv = 1.0f / (l[a] + sink);
+        const float inv = gate_of(p, rt[a], head) / (l[a] + sink);
         bf16* orow = p.out + (size_t)rt[a] * p.ldo + (size_t)head * dv;
 #pragma unroll
         for (int n = 0; n < DT; ++n) {
@@ -364,7 +377,7 @@ __global__ void __launch_bounds__(AR_THREADS) attention_single_rows_kernel(const
     const int d = FAST ? D : p.d, dv = FAST ? D : p.dv;
     const int nks = FAST ? KS : (d + 15) >> 4;
     const int lo = first_key(P, p.window);
-    const int pooled = POOL ? lo / p.pk.every : 0;
+    const int pooled = POOL ? ahead_rows(p.pk, lo) : 0;
     const int run_chunks = (pooled + AS_KEYS - 1) / AS_KEYS;
     const int token_chunk = lo / AS_KEYS - run_chunks;  // chunk c >= run_chunks holds the tokens from 16 (c + token_chunk) on
     const int chunks_all = P / AS_KEYS - token_chunk + 1;
@@ -462,7 +475,9 @@ __global__ void __launch_bounds__(AR_THREADS) attention_single_rows_kernel(const
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
             const int at = gq + (e >> 1) * 8;
-            w[e] = at >= from && at <= to ? (s[0][e] + s[1][e]) * p.scale2 : -INFINITY;
+            float x = s[0][e] + s[1][e];
+            if (p.scale_cap > 0.0f) x = tanhf(x * p.scale_cap);
+            w[e] = at >= from && at <= to ? x * p.scale2 : -INFINITY;
         }
         float alpha[2];
         bool moved = false;
@@ -543,7 +558,7 @@ __global__ void __launch_bounds__(AR_THREADS) attention_single_rows_kernel(const
         if (splits == 1) {
             const int head = hk * g + r0 + r;
             if (p.sink) zz += exp2f(p.sink[head] * LOG2E - mm);
-            p.out[(size_t)t * p.ldo + (size_t)head * dv + i] = from_float<bf16>(acc / zz);
+            p.out[(size_t)t * p.ldo + (size_t)head * dv + i] = from_float<bf16>(acc / zz * gate_of(p, t, head));
         } else {
             float* e = meet + (size_t)(AR_WARPS * rows + r) * stride;
             if (i == 0) e[0] = mm, e[1] = zz;
@@ -573,7 +588,7 @@ __global__ void __launch_bounds__(AR_THREADS) attention_single_rows_kernel(const
         }
         const int head = hk * g + r0 + r;
         if (p.sink) zz += exp2f(p.sink[head] * LOG2E - mm);
-        p.out[(size_t)t * p.ldo + (size_t)head * dv + i] = from_float<bf16>(acc / zz);
+        p.out[(size_t)t * p.ldo + (size_t)head * dv + i] = from_float<bf16>(acc / zz * gate_of(p, t, head));
     }
     cluster_sync();  // nobody leaves while a peer may still read its shared memory
 }
@@ -646,22 +661,24 @@ FERRIS_API int ferris_attention_rows(const void* q, int ldq, void* out, int ldo,
                                      const int* block_tables, int max_blocks, const int* token_seq, const int* positions,
                                      int tokens, int nh, int nkv, int d, int dv, int page_size, int window, float scale,
                                      const float* sink, const void* pool_k, const void* pool_v, const int* pool_tables,
-                                     int pool_max_blocks, int pool_every, int portions, int kv_span, void* stream) {
+                                     int pool_max_blocks, int pool_every, int keep, float softcap, const void* gate, int ldgate,
+                                     int portions, int kv_span, void* stream) {
     if (tokens <= 0) return FERRIS_OK;
     if (!ferris_attention_rows_takes(nh, nkv, d, dv, portions))
         FERRIS_REFUSE("attention rows: %d heads over %d kv heads of %d / %d are not taken", nh, nkv, d, dv);
     if (page_size <= 0 || max_blocks <= 0) FERRIS_REFUSE("attention: page_size=%d max_blocks=%d", page_size, max_blocks);
-    const ScoreTerms st = {nullptr, nullptr, nullptr, sink, 0};
-    const PooledKeys pk = {pool_k, pool_v, pool_tables, pool_max_blocks, pool_every};
+    const ScoreTerms st = {nullptr, nullptr, nullptr, sink, 0, softcap, gate, ldgate};
+    const PooledKeys pk = keys_beside(pool_k, pool_v, pool_tables, pool_max_blocks, pool_every, keep, k_cache, v_cache, block_tables, max_blocks);
     if (int rc = check_pooled(pk, window, st)) return rc;
     if ((((uintptr_t)q | (uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)pool_k | (uintptr_t)pool_v) & 15) != 0 || ldq % 8 ||
         ((uintptr_t)out & 3) || (ldo & 1))
         FERRIS_REFUSE("attention rows: rows must start on 16 bytes");
     const AttentionArgs p = {(const bf16*)q, (bf16*)out, (const bf16*)k_cache, (const bf16*)v_cache, block_tables, token_seq,
                              positions, sink, pk, ldq, ldo, max_blocks, tokens, nh, nkv, d, dv, page_size, window,
-                             scale * LOG2E};
+                             (softcap > 0.0f ? softcap : scale) * LOG2E, softcap > 0.0f ? scale / softcap : 0.0f,
+                             (const bf16*)gate, ldgate};
     cudaStream_t s = (cudaStream_t)stream;
-    const bool pool = pk.every > 0;
+    const bool pool = pk.every > 0 || pk.keep > 0;
     const int bucket = rows_bucket(d, dv);
     if (portions) {
         if (bucket == 64) return pool ? launch_rows<64, true>(p, s) : launch_rows<64, false>(p, s);

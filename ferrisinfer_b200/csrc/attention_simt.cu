@@ -11,6 +11,8 @@
 //   With pooled keys (PooledKeys) beside a window: one key and value more for every run of `every` positions (counted off
 //   from 0) that lies wholly before the window, read from pages of their own (the means of the run's keys and values);
 //   tokens and runs share one softmax.  With lo the window's first position, the runs seen are 0 .. lo / every - 1.
+//   With kept tokens beside a window: the sequence's first `keep` tokens stay visible when the window has passed them.
+//   With a soft cap c: s_j = c tanh((q . k_j) * scale / c).  With gates: a head's output times sigmoid of its gate.
 // (crates/ferrisinfer-kernel/src/cpu/attention.rs:729-781, 1125-1155: streaming softmax with a
 // running maximum, which this kernel keeps per warp).  The step's own keys are already in the
 // cache when this runs, so prompts, portions of prompts and single decoded tokens are one case.
@@ -54,7 +56,7 @@ __global__ void __launch_bounds__(ATT_THREADS)
         acc[r] = 0.0f;
     }
     float m = -INFINITY, z = 0.0f;
-    const int pooled = POOL ? lo / pk.every : 0;
+    const int pooled = POOL ? ahead_rows(pk, lo) : 0;
     const int shift = POOL ? lo - pooled : 0;  // key n >= pooled is the token at n + shift
     const int* ptable = POOL ? pk.tables + (size_t)seq * pk.max_blocks : nullptr;
     for (int n = (POOL ? 0 : lo) + warp; n <= P - shift; n += ATT_WARPS) {
@@ -72,7 +74,7 @@ __global__ void __launch_bounds__(ATT_THREADS)
             const int i = lane + 32 * r;
             if (i < d) dot = fmaf(qv[r], to_float(keys[base + i]), dot);
         }
-        const float s = POOL ? warp_sum(dot) * scale : with_terms(warp_sum(dot) * scale, ht, j, P);
+        const float s = with_terms(warp_sum(dot) * scale, ht, j, P);
         float wgt;
         if (s > m) {
             const float rescale = expf(m - s);  // exp(-inf) = 0 on the first key
@@ -114,7 +116,7 @@ __global__ void __launch_bounds__(ATT_THREADS)
         zz += smem[w * (dv + 2) + 1] * f[w];
     }
     zz += sink_share(st, hq, mm);
-    const float inv = 1.0f / zz;
+    const float inv = head_gate<T>(st, t, hq) / zz;
     T* orow = out + (size_t)t * ldo + (size_t)hq * dv;
     for (int i = threadIdx.x; i < dv; i += ATT_THREADS) {
         float o = 0.0f;
@@ -214,7 +216,7 @@ __global__ void __launch_bounds__(AL_THREADS)
     for (int i = 0; i < MAXC; ++i) qv[i] = 0.0f, acc[i] = 0.0f;
     load_chunk<MAXC>(q + (size_t)t * ldq + (size_t)hq * d + sub * ch, ch, qv);
     float m = -INFINITY, z = 0.0f;
-    const int pooled = POOL ? lo / pk.every : 0;
+    const int pooled = POOL ? ahead_rows(pk, lo) : 0;
     const int shift = POOL ? lo - pooled : 0;  // key n >= pooled is the token at n + shift
     const int* ptable = POOL ? pk.tables + (size_t)seq * pk.max_blocks : nullptr;
     const int n0 = POOL ? 0 : lo, n1 = P - shift;
@@ -256,7 +258,7 @@ __global__ void __launch_bounds__(AL_THREADS)
 #pragma unroll
         for (int u = 0; u < U; ++u) {
             if (!ok[u]) continue;
-            const float s = POOL ? dot[u] * scale : with_terms(dot[u] * scale, ht, jj[u], P);
+            const float s = with_terms(dot[u] * scale, ht, jj[u], P);
             float wgt;
             if (s > m) {
                 const float rescale = expf(m - s);  // exp(-inf) = 0 on the first key
@@ -293,7 +295,7 @@ __global__ void __launch_bounds__(AL_THREADS)
         zz += smem[g * (dv + 2) + 1] * f[g];
     }
     zz += sink_share(st, hq, mm);
-    const float inv = 1.0f / zz;
+    const float inv = head_gate<T>(st, t, hq) / zz;
     T* orow = out + (size_t)t * ldo + (size_t)hq * dv;
     for (int i = threadIdx.x; i < dv; i += AL_THREADS) {
         float o = 0.0f;
@@ -341,7 +343,7 @@ __global__ void __launch_bounds__(AG_THREADS)
         m[a] = -INFINITY, z[a] = 0.0f;
         ht[a] = head_terms(st, h0 + a);
     }
-    const int pooled = POOL ? lo / pk.every : 0;
+    const int pooled = POOL ? ahead_rows(pk, lo) : 0;
     const int shift = POOL ? lo - pooled : 0;  // key n >= pooled is the token at n + shift
     const int* ptable = POOL ? pk.tables + (size_t)seq * pk.max_blocks : nullptr;
     const int n0 = POOL ? 0 : lo, n1 = P - shift;
@@ -393,7 +395,7 @@ __global__ void __launch_bounds__(AG_THREADS)
             if (!ok[u]) continue;
 #pragma unroll
             for (int a = 0; a < G; ++a) {
-                const float s = POOL ? dot[u][a] * scale : with_terms(dot[u][a] * scale, ht[a], jj[u], P);
+                const float s = with_terms(dot[u][a] * scale, ht[a], jj[u], P);
                 float wgt;
                 if (s > m[a]) {
                     const float rescale = expf(m[a] - s);
@@ -437,7 +439,7 @@ __global__ void __launch_bounds__(AG_THREADS)
         }
         if (splits == 1) {
             zz += sink_share(st, h0 + a, mm);
-            out[(size_t)t * ldo + (size_t)(h0 + a) * dv + i] = from_float<T>(o / zz);
+            out[(size_t)t * ldo + (size_t)(h0 + a) * dv + i] = from_float<T>(o / zz * head_gate<T>(st, t, h0 + a));
         } else {  // the share's maximum, sum and weighted values, for the merge kernel
             float* e = partial + (((size_t)t * nh + h0 + a) * splits + split) * stride;
             if (i == 0) e[0] = mm, e[1] = zz;
@@ -464,7 +466,7 @@ __global__ void __launch_bounds__(128) attention_merge_shares_kernel(const float
         zz += ms == -INFINITY ? 0.0f : base[(size_t)s2 * stride + 1] * expf(ms - mm);
     }
     zz += sink_share(st, h, mm);
-    const float inv = 1.0f / zz;
+    const float inv = head_gate<T>(st, t, h) / zz;
     for (int i = threadIdx.x; i < dv; i += blockDim.x) {
         float o = 0.0f;
         for (int s2 = 0; s2 < splits; ++s2) {
@@ -613,7 +615,7 @@ __global__ void __launch_bounds__(TL_THREADS)
         const bool runs = POOL && seg == 0;
         // of the first token: no later token of the request sees an earlier key
         const int kmin = runs ? 0 : first_key(pa, window);
-        const int kmax = runs ? first_key(pb, window) / pk.every - 1 : pb;
+        const int kmax = runs ? ahead_rows(pk, first_key(pb, window)) - 1 : pb;
         const int* table = runs ? pk.tables + (size_t)sq * pk.max_blocks : block_tables + (size_t)sq * max_blocks;
         const T* keys = runs ? reinterpret_cast<const T*>(pk.k) : k_cache;
         const T* vals = runs ? reinterpret_cast<const T*>(pk.v) : v_cache;
@@ -658,16 +660,13 @@ __global__ void __launch_bounds__(TL_THREADS)
 #pragma unroll
             for (int a = 0; a < 2; ++a) {
                 int lo = first_key(rpos[a], window), hi = rpos[a];
-                if (runs) hi = lo / pk.every - 1, lo = 0;
+                if (runs) hi = ahead_rows(pk, lo) - 1, lo = 0;
                 float best = -INFINITY;
 #pragma unroll
                 for (int c = 0; c < 4; ++c) {
                     const int j = j0 + kx + 8 * c;
                     const bool seen = rseq[a] == sq && j >= lo && j <= hi;
-                    if (POOL)
-                        sc[a][c] = seen ? sc[a][c] : -INFINITY;
-                    else
-                        sc[a][c] = seen ? with_terms(sc[a][c], rterm[a], j, rpos[a]) : -INFINITY;
+                    sc[a][c] = seen ? with_terms(sc[a][c], rterm[a], j, rpos[a]) : -INFINITY;
                     best = fmaxf(best, sc[a][c]);
                 }
 #pragma unroll
@@ -715,7 +714,7 @@ __global__ void __launch_bounds__(TL_THREADS)
 #pragma unroll
     for (int a = 0; a < 2; ++a) {
         if (rt[a] >= t_end) continue;
-        const float inv = 1.0f / (l[a] + sink_share(st, hk * g + (r0 + a) % g, m[a]));
+        const float inv = head_gate<T>(st, rt[a], hk * g + (r0 + a) % g) / (l[a] + sink_share(st, hk * g + (r0 + a) % g, m[a]));
         T* orow = out + (size_t)rt[a] * ldo + (size_t)(hk * g + (r0 + a) % g) * dv;
 #pragma unroll
         for (int c = 0; c < NC; ++c) {
@@ -773,15 +772,16 @@ FERRIS_API int ferris_paged_attention_simt(const void* q, int ldq, void* out, in
                                            int d, int dv, int page_size, int window, float scale, const float* slopes,
                                            const float* log_r1, const float* log_r2, const float* sink, int v_stride,
                                            const void* pool_k, const void* pool_v, const int* pool_tables,
-                                           int pool_max_blocks, int pool_every, int kv_span, float* scratch, long long scratch_floats, void* stream) {
+                                           int pool_max_blocks, int pool_every, int keep, float softcap, const void* gate, int ldgate,
+                                           int kv_span, float* scratch, long long scratch_floats, void* stream) {
     if (tokens <= 0) return FERRIS_OK;
     if ((log_r1 == nullptr) != (log_r2 == nullptr)) FERRIS_REFUSE("attention: the logarithmic penalty needs both of its numbers per head");
     if (slopes && log_r1) FERRIS_REFUSE("attention: a slope and a logarithmic penalty at once");
     if (v_stride < 0 || (v_stride > 0 && v_stride < dv)) FERRIS_REFUSE("attention: value rows %d apart hold no %d values", v_stride, dv);
-    const ScoreTerms st = {slopes, log_r1, log_r2, sink, v_stride};
-    const PooledKeys pk = {pool_k, pool_v, pool_tables, pool_max_blocks, pool_every};
+    const ScoreTerms st = {slopes, log_r1, log_r2, sink, v_stride, softcap, gate, ldgate};
+    const PooledKeys pk = keys_beside(pool_k, pool_v, pool_tables, pool_max_blocks, pool_every, keep, k_cache, v_cache, block_tables, max_blocks);
     if (int rc = check_pooled(pk, window, st)) return rc;
-    const bool pool = pk.every > 0;
+    const bool pool = pk.every > 0 || pk.keep > 0;
     if (nh <= 0 || nkv <= 0 || nh % nkv != 0) FERRIS_REFUSE("attention: %d heads over %d kv heads", nh, nkv);
     if (d <= 0 || d > 32 * MAX_PER_LANE) FERRIS_REFUSE("attention: head size %d not in 1..%d", d, 32 * MAX_PER_LANE);
     if (dv <= 0 || dv > 32 * MAX_PER_LANE) FERRIS_REFUSE("attention: value head size %d not in 1..%d", dv, 32 * MAX_PER_LANE);
@@ -879,12 +879,13 @@ FERRIS_API int ferris_paged_attention_tiled(const void* q, int ldq, void* out, i
                                             int d, int dv, int page_size, int window, float scale, const float* slopes,
                                             const float* log_r1, const float* log_r2, const float* sink, int v_stride,
                                             const void* pool_k, const void* pool_v, const int* pool_tables,
-                                            int pool_max_blocks, int pool_every, void* stream) {
+                                            int pool_max_blocks, int pool_every, int keep, float softcap,
+                                            const void* gate, int ldgate, void* stream) {
     if (tokens <= 0) return FERRIS_OK;
     if ((log_r1 == nullptr) != (log_r2 == nullptr) || (slopes && log_r1)) FERRIS_REFUSE("tiled attention: one kind of distance penalty, with all its numbers");
     if (v_stride < 0 || (v_stride > 0 && v_stride < dv)) FERRIS_REFUSE("tiled attention: value rows %d apart hold no %d values", v_stride, dv);
-    const ScoreTerms st = {slopes, log_r1, log_r2, sink, v_stride};
-    const PooledKeys pk = {pool_k, pool_v, pool_tables, pool_max_blocks, pool_every};
+    const ScoreTerms st = {slopes, log_r1, log_r2, sink, v_stride, softcap, gate, ldgate};
+    const PooledKeys pk = keys_beside(pool_k, pool_v, pool_tables, pool_max_blocks, pool_every, keep, k_cache, v_cache, block_tables, max_blocks);
     if (int rc = check_pooled(pk, window, st)) return rc;
     if (dtype != FERRIS_F32 && dtype != FERRIS_BF16) FERRIS_REFUSE("attention: unknown dtype %d", dtype);
     if (page_size <= 0 || max_blocks <= 0) FERRIS_REFUSE("attention: page_size=%d max_blocks=%d", page_size, max_blocks);
@@ -898,8 +899,8 @@ FERRIS_API int ferris_paged_attention_tiled(const void* q, int ldq, void* out, i
     return launch_tiled<T, POOL>(q, ldq, out, ldo, k_cache, v_cache, block_tables, max_blocks, token_seq, positions, tokens, \
                                  nh, nkv, d, dv, page_size, window, scale, st, pk, s)
     if (dtype == FERRIS_F32) {
-        if (pk.every > 0) FERRIS_TILED(float, true); else FERRIS_TILED(float, false);
+        if (pk.every > 0 || pk.keep > 0) FERRIS_TILED(float, true); else FERRIS_TILED(float, false);
     }
-    if (pk.every > 0) FERRIS_TILED(bf16, true); else FERRIS_TILED(bf16, false);
+    if (pk.every > 0 || pk.keep > 0) FERRIS_TILED(bf16, true); else FERRIS_TILED(bf16, false);
 #undef FERRIS_TILED
 }

@@ -9,9 +9,10 @@
 // or a gate) are one fp32 number per token and head, made by `recurrence_gates`; q and k come in `qk_heads` heads
 // shared by heads / qk_heads value heads each, and may carry one fp32 factor per (token, qk head) each (unit norms:
 // the factor is 1 / |x|, formed in fp32 by the gates kernel, so that the vectors themselves are read once as stored).
-// The plain form also takes a decay per ROW of the state (per key channel) that changes with every token, given as
-// fp32 numbers z per (token, head, row): the row's decay is sigmoid(z)^power = exp(-softplus(-z) * power), formed
-// in fp32 where the rows are staged; the decay per head is then left out (gated linear attention).  What is staged is
+// Either form also takes a decay per ROW of the state (per key channel) that changes with every token, given as
+// fp32 numbers z per (token, head, row): the row's decay is sigmoid(z)^power = exp(-softplus(-z) * power), or, with a rate
+// per head, exp(-softplus(z) * rate[head]), formed in fp32 where the rows are staged; the decay per head is then left out
+// (gated linear attention; a delta rule whose channels forget at their own pace).  What is staged is
 // the decay MINUS ONE, expm1(-softplus(-z) power), and a row moves on as s + ((decay - 1) s + k u): a decay close to one
 // rounded to 24 bits is off by a fixed share of what it takes away, with the same sign at every step where the row's
 // decay hardly changes, which over a thousand tokens shows in 32-bit logits; this way only the sum rounds, at the state's
@@ -44,6 +45,8 @@ constexpr int GR_STAGE = 16;  // tokens in shared memory at a time
 constexpr int GR_MAX_DIM = 256;
 
 __device__ __forceinline__ float softplus_g(float v) { return fmaxf(v, 0.0f) + log1pf(expf(-fabsf(v))); }
+// the logarithm of a row's decay: sign = -1 and rate = power, or sign = 1 and rate = the head's
+__device__ __forceinline__ float row_log_decay(float z, float sign, float rate) { return -softplus_g(sign * z) * rate; }
 
 // decay[t, h] = exp(-exp(A_log[h]) * dt), dt = softplus(a[t, h] + dt_bias[h]);  beta[t, h] = sigmoid(b[t, h]) (kind 0)
 // or dt itself (kind 1).  With unit norms: qscale[t, g] = q_mul / sqrt(sum q^2 + eps), kscale[t, g] = 1 / sqrt(sum k^2 + eps).
@@ -60,8 +63,11 @@ __global__ void __launch_bounds__(128) recurrence_gates_kernel(const T* proj, in
     const int t = blockIdx.x;
     const T* row = proj + (size_t)t * ld;
     for (int h = threadIdx.x; h < heads; h += blockDim.x) {
-        const float dt = softplus_g(to_float(row[a_off + h]) + dt_bias[h]);
-        decay[(size_t)t * heads + h] = expf(-expf(A_log[h]) * dt);
+        float dt = 0.0f;
+        if (A_log) {  // without: the step size alone (the decays are formed elsewhere)
+            dt = softplus_g(to_float(row[a_off + h]) + dt_bias[h]);
+            decay[(size_t)t * heads + h] = expf(-expf(A_log[h]) * dt);
+        }
         beta[(size_t)t * heads + h] = beta_kind == 0 ? 1.0f / (1.0f + expf(-to_float(row[b_off + h]))) : dt;
     }
     if (!qscale) return;
@@ -94,8 +100,8 @@ __global__ void __launch_bounds__(GR_THREADS) gated_recurrence_kernel(
     const T* q, int ldq, const T* k, int ldk, const T* v, int ldv, const float* decay, const float* beta,
     const float* qscale, const float* kscale, const float* __restrict__ skip, float* __restrict__ out, int ldo,
     float* state, const int* __restrict__ seq_q_start, const int* __restrict__ seq_state_slot, int heads, int qk_heads,
-    int dim, int vdim, int write_state, const float* row_z, int ldz, float row_power, float q_mul, int seg_len = 0,
-    int segs_max = 1, float* scratch_s = nullptr, float* scratch_p = nullptr) {
+    int dim, int vdim, int write_state, const float* row_z, int ldz, float row_power, const float* __restrict__ row_rate,
+    float q_mul, int seg_len = 0, int segs_max = 1, float* scratch_s = nullptr, float* scratch_p = nullptr) {
     constexpr int COLS = GR_THREADS / LANES;  // columns of a block
     constexpr int STAGE = (ROWDECAY && LANES == 32) ? GR_STAGE / 2 : GR_STAGE;  // three staged vectors of 256 rows: fewer tokens
     constexpr int ROWS = GR_KPL * LANES;      // rows of the state that the lanes of a column hold
@@ -140,6 +146,7 @@ __global__ void __launch_bounds__(GR_THREADS) gated_recurrence_kernel(
         if (ROWDECAY) (&as[0][0])[i] = 0.0f;
     }
     const float d_skip = skip ? skip[head] : 0.0f;
+    const float z_sign = row_rate ? 1.0f : -1.0f, z_rate = row_rate ? row_rate[head] : row_power;
     // A stage's q, k, v and per-token numbers are requested into registers while the stage before it is worked on
     // (the requests of a stage are all in flight together), and go to shared memory when that one is done.
     // (they stay as they were loaded until then: an instruction that touched one would wait for its load)
@@ -186,7 +193,7 @@ __global__ void __launch_bounds__(GR_THREADS) gated_recurrence_kernel(
                 const size_t row = (size_t)(t0 + r);
                 qs[r][c] = to_float(q[row * ldq + (size_t)qh * dim + c]);
                 ks[r][c] = to_float(k[row * ldk + (size_t)qh * dim + c]);
-                if (ROWDECAY) as[r][c] = expm1f(-softplus_g(-row_z[row * ldz + (size_t)head * dim + c]) * row_power);
+                if (ROWDECAY) as[r][c] = expm1f(row_log_decay(row_z[row * ldz + (size_t)head * dim + c], z_sign, z_rate));
             }
             for (int i = tid; i < n * COLS; i += GR_THREADS) {
                 const int r = i / COLS, c = i - r * COLS;
@@ -209,7 +216,7 @@ __global__ void __launch_bounds__(GR_THREADS) gated_recurrence_kernel(
                 const int c = tid + j * GR_THREADS;
                 if (c < dim) {
                     qs[r][c] = to_float(pq[r][j]), ks[r][c] = to_float(pk[r][j]);
-                    if (ROWDECAY) as[r][c] = expm1f(-softplus_g(-pz[r][j]) * row_power);
+                    if (ROWDECAY) as[r][c] = expm1f(row_log_decay(pz[r][j], z_sign, z_rate));
                 }
             }
         }
@@ -233,7 +240,12 @@ __global__ void __launch_bounds__(GR_THREADS) gated_recurrence_kernel(
                 float d0 = 0.0f, d1 = 0.0f;  // two chains, so that the sum waits for half as many dependent FMAs
 #pragma unroll
                 for (int i = 0; i < GR_KPL; i += 2) {
-                    s[i] *= g, s[i + 1] *= g;
+                    if (ROWDECAY) {  // s + (decay - 1) s
+                        s[i] = fmaf(as[r][sub + LANES * i], s[i], s[i]);
+                        s[i + 1] = fmaf(as[r][sub + LANES * (i + 1)], s[i + 1], s[i + 1]);
+                    } else {
+                        s[i] *= g, s[i + 1] *= g;
+                    }
                     d0 = fmaf(s[i], kr[i], d0), d1 = fmaf(s[i + 1], kr[i + 1], d1);
                 }
                 float dot = d0 + d1;
@@ -297,7 +309,7 @@ __global__ void __launch_bounds__(256) row_decay_products_kernel(const float* ro
     const size_t place = (size_t)(first / seg_len + seq);
     for (int r = threadIdx.x; r < dim; r += blockDim.x) {
         float sum = 0.0f;
-        for (int t = first; t < first + seg_len; ++t) sum -= softplus_g(-row_z[(size_t)t * ldz + (size_t)head * dim + r]) * row_power;
+        for (int t = first; t < first + seg_len; ++t) sum += row_log_decay(row_z[(size_t)t * ldz + (size_t)head * dim + r], -1.0f, row_power);
         scratch_p[(place * heads + head) * (size_t)dim + r] = expm1f(sum);
     }
 }
@@ -412,15 +424,15 @@ int launch_recurrence(const void* q, int ldq, const void* k, int ldk, const void
                       const float* beta, const float* qscale, const float* kscale, const float* skip, float* out, int ldo,
                       float* state, const int* seq_q_start, const int* seq_state_slot, int seqs, int heads, int qk_heads,
                       int dim, int vdim, int write_state, cudaStream_t s, const float* row_z = nullptr, int ldz = 0,
-                      float row_power = 1.0f, float q_mul = 1.0f, int seg_len = 0, int segs_max = 1,
-                      float* scratch_s = nullptr, float* scratch_p = nullptr) {
+                      float row_power = 1.0f, const float* row_rate = nullptr, float q_mul = 1.0f, int seg_len = 0,
+                      int segs_max = 1, float* scratch_s = nullptr, float* scratch_p = nullptr) {
     const dim3 block(GR_THREADS);
 #define FERRIS_GR_LAUNCH(LANES)                                                                                         \
     ferris_launch(gated_recurrence_kernel<T, LANES, DELTA, AHEAD, ROWDECAY, MODE>,                                    \
                   dim3(seqs * segs_max, heads, (vdim + GR_THREADS / LANES - 1) / (GR_THREADS / LANES)), block, 0, s,   \
                   (const T*)q, ldq, (const T*)k, ldk, (const T*)v, ldv, decay, beta, qscale, kscale, skip, out, ldo,    \
                   state, seq_q_start, seq_state_slot, heads, qk_heads, dim, vdim, write_state, row_z, ldz, row_power,   \
-                  q_mul, seg_len, segs_max, scratch_s, scratch_p)
+                  row_rate, q_mul, seg_len, segs_max, scratch_s, scratch_p)
     if (dim <= 32)
         FERRIS_GR_LAUNCH(4);
     else if (dim <= 64)
@@ -437,13 +449,14 @@ int launch_recurrence(const void* q, int ldq, const void* k, int ldk, const void
 
 // proj: [tokens, ld] rows holding a (heads columns from a_off) and, for beta_kind 0, b (heads columns from b_off).
 // qk: rows holding q and k heads (qk_heads x dim each) from q_off / k_off; qscale / kscale (null: no unit norms):
-// fp32 [tokens, qk_heads].  decay, beta: fp32 [tokens, heads].
+// fp32 [tokens, qk_heads].  decay, beta: fp32 [tokens, heads].  A_log, dt_bias and decay all null: beta (kind 0) alone.
 FERRIS_API int ferris_recurrence_gates(const void* proj, int ld, int dtype, int a_off, int b_off, const float* A_log,
                                        const float* dt_bias, float* decay, float* beta, int beta_kind, const void* qk,
                                        int ldqk, int q_off, int k_off, int qk_heads, int dim, float unit_eps, float q_mul,
                                        float* qscale, float* kscale, int tokens, int heads, void* stream) {
     if (tokens <= 0) return FERRIS_OK;
-    if (heads <= 0 || !A_log || !dt_bias || !decay || !beta) FERRIS_REFUSE("recurrence gates: %d heads, or a table is missing", heads);
+    if (heads <= 0 || (A_log == nullptr) != (dt_bias == nullptr) || (A_log == nullptr) != (decay == nullptr) || !beta) FERRIS_REFUSE("recurrence gates: %d heads, or a table is missing", heads);
+    if (!A_log && beta_kind != 0) FERRIS_REFUSE("recurrence gates: a step size without its tables");
     if (beta_kind != 0 && beta_kind != 1) FERRIS_REFUSE("recurrence gates: unknown kind %d of the second number", beta_kind);
     if ((qscale == nullptr) != (kscale == nullptr)) FERRIS_REFUSE("recurrence gates: unit norms of q and k go together");
     if (qscale && (!qk || qk_heads <= 0 || dim <= 0)) FERRIS_REFUSE("recurrence gates: unit norms of %d heads of %d", qk_heads, dim);
@@ -463,21 +476,35 @@ FERRIS_API int ferris_recurrence_gates(const void* proj, int ld, int dtype, int 
 
 // q, k: [tokens, qk_heads x dim] from their first column, rows ldq / ldk apart; v: [tokens, heads x vdim], rows ldv apart;
 // out: fp32 [tokens, heads x vdim]; state: fp32 [slots, heads, vdim, dim] (transposed); skip: fp32 [heads] or null.
+// row_z (with the delta rule only; decay is then null): fp32 [tokens, heads x dim], rows ldz apart, and row_rate fp32 [heads]:
+// the decay of row r of head h at token t is exp(-softplus(row_z[t, h, r]) row_rate[h]).
 FERRIS_API int ferris_gated_recurrence(const void* q, int ldq, const void* k, int ldk, const void* v, int ldv, int dtype,
                                        const float* decay, const float* beta, const float* qscale, const float* kscale,
                                        const float* skip, float* out, int ldo, float* state, const int* seq_q_start,
                                        const int* seq_state_slot, int seqs, int heads, int qk_heads, int dim, int vdim,
-                                       int delta_rule, int write_state, int longest, void* stream) {
+                                       int delta_rule, int write_state, int longest, const float* row_z, int ldz,
+                                       const float* row_rate, void* stream) {
     if (seqs <= 0) return FERRIS_OK;
     if (heads <= 0 || qk_heads <= 0 || heads % qk_heads) FERRIS_REFUSE("recurrence: %d heads over %d q/k heads", heads, qk_heads);
     if (dim <= 0 || dim > GR_MAX_DIM || vdim <= 0) FERRIS_REFUSE("recurrence: heads of %d x %d (at most %d rows)", dim, vdim, GR_MAX_DIM);
     if (heads > 65535 || (vdim + 3) / 4 > 65535) FERRIS_REFUSE("recurrence: too many heads or columns for one launch");
     cudaStream_t s = (cudaStream_t)stream;
     if (dtype != FERRIS_F32 && dtype != FERRIS_BF16) FERRIS_REFUSE("recurrence: unknown dtype %d", dtype);
+    if (row_z && (!delta_rule || !row_rate || decay)) FERRIS_REFUSE("recurrence: decays per row come with a rate per head, the delta rule and no decay per head");
+    if (!row_z && !decay) FERRIS_REFUSE("recurrence: no decays");
     const bool ahead = longest > GR_STAGE;  // `longest`: the most tokens a request brings (0: not known)
 #define FERRIS_GR_GO(T, D, A)                                                                                                \
     return launch_recurrence<T, D, A>(q, ldq, k, ldk, v, ldv, decay, beta, qscale, kscale, skip, out, ldo, state, seq_q_start, \
                                       seq_state_slot, seqs, heads, qk_heads, dim, vdim, write_state, s)
+    if (row_z) {
+#define FERRIS_CD_GO(T, A)                                                                                                    \
+    return launch_recurrence<T, true, A, true>(q, ldq, k, ldk, v, ldv, nullptr, beta, qscale, kscale, skip, out, ldo, state,    \
+                                               seq_q_start, seq_state_slot, seqs, heads, qk_heads, dim, vdim, write_state, s,   \
+                                               row_z, ldz, 1.0f, row_rate)
+        if (dtype == FERRIS_F32) { if (ahead) FERRIS_CD_GO(float, true); else FERRIS_CD_GO(float, false); }
+        if (ahead) FERRIS_CD_GO(bf16, true); else FERRIS_CD_GO(bf16, false);
+#undef FERRIS_CD_GO
+    }
     if (dtype == FERRIS_F32) {
         if (delta_rule) { if (ahead) FERRIS_GR_GO(float, true, true); else FERRIS_GR_GO(float, true, false); }
         if (ahead) FERRIS_GR_GO(float, false, true); else FERRIS_GR_GO(float, false, false);
@@ -507,7 +534,7 @@ FERRIS_API int ferris_row_decay_recurrence(const void* q, int ldq, const void* k
 #define FERRIS_RD_GO(T, A, M)                                                                                                \
     launch_recurrence<T, false, A, true, M>(q, ldq, k, ldk, v, ldv, nullptr, nullptr, nullptr, nullptr, nullptr, out, ldo,    \
                                             state, seq_q_start, seq_state_slot, seqs, heads, heads, dim, vdim, write_state,  \
-                                            s, row_z, ldz, row_power, q_mul, seg_len, M ? segs_max : 1, scratch_s, scratch_p)
+                                            s, row_z, ldz, row_power, (const float*)nullptr, q_mul, seg_len, M ? segs_max : 1, scratch_s, scratch_p)
     if (segs_max > 1) {  // segments side by side: sums, carry, outputs.  Many blocks hide one another's loads, so a stage
         // goes straight to shared memory: the form that requests the next tokens into registers holds four blocks an SM
         int rc = dtype == FERRIS_F32 ? FERRIS_RD_GO(float, false, 1) : FERRIS_RD_GO(bf16, false, 1);

@@ -689,8 +689,8 @@ struct PTParams {
     // Written by the launch before this one, so never read through a read-only path.
     const int* tile_expert = nullptr;
     int expert_rows = 0;
-    // SwiGLU mode: a factor per row (written by an earlier launch) on both accumulators ahead of the activation: the
-    // product of a row that is multiplied by it.  Null: none.
+    // SwiGLU mode, or the bf16 store with an activation: a factor per row (written by an earlier launch) on the accumulators
+    // ahead of the activation: the product of a row that is multiplied by it.  Null: none.
     const float* row_scale = nullptr;
 };
 
@@ -776,7 +776,7 @@ __device__ __forceinline__ void pt_epilogue_tile(const PTParams& p, const CUtens
     constexpr int ACCS = MODE == SWIGLU_BF16 ? 2 : 1;
     const int cols = p.bn;  // output columns of this tile
     float row_scale = 1.0f;
-    if (MODE == SWIGLU_BF16 && p.row_scale && t < p.T) row_scale = *(reinterpret_cast<const volatile float*>(p.row_scale) + t);
+    if ((MODE == SWIGLU_BF16 || MODE == STORE_BF16) && p.row_scale && t < p.T) row_scale = *(reinterpret_cast<const volatile float*>(p.row_scale) + t);
     for (int c0 = half * 32; c0 < cols; c0 += 64) {
         uint32_t ra[32], rb[32];
         tmem_load_32x32(d0 + c0, ra);
@@ -833,7 +833,7 @@ __device__ __forceinline__ void pt_epilogue_tile(const PTParams& p, const CUtens
                 } else {
                     v0 = __uint_as_float(ra[c]) + ((p.bias && n + c < p.N) ? __ldg(p.bias + n + c) : 0.0f);
                     v1 = __uint_as_float(ra[c + 1]) + ((p.bias && n + c + 1 < p.N) ? __ldg(p.bias + n + c + 1) : 0.0f);
-                    if (p.act.kind) v0 = ferris_epilogue_act(v0, p.act), v1 = ferris_epilogue_act(v1, p.act);
+                    if (p.act.kind) v0 = ferris_epilogue_act(row_scale * v0, p.act), v1 = ferris_epilogue_act(row_scale * v1, p.act);
                 }
                 packed[c >> 1] = pack_bf16(v0, v1);
             }
@@ -1630,8 +1630,8 @@ static int run_tokens_m(const void* x, const void* w, const float* bias, void* o
 // One product per group of token tiles (see PTParams::tile_expert): x holds `rows` rows (a multiple of 128), sorted by
 // expert with every expert's rows filled up to whole tiles of 128; w holds the experts' matrices stacked, expert_rows
 // rows each, of which the first N (and, in SwiGLU mode, the N from up_row_offset on) meet the rows of their tiles.
-// Modes: 0 bf16 store, 1 fp32 store, 3 SwiGLU from two accumulators (with row_scale, fp32 [rows], both times the row's
-// factor first).  A tile whose entry is negative is skipped.
+// Modes: 0 bf16 store (with the activation of ferris_gemm_set_activation), 1 fp32 store, 3 SwiGLU from two accumulators; with
+// row_scale (fp32 [rows]; mode 3, or mode 0 with an activation) the accumulators times the row's factor first.  A tile whose entry is negative is skipped.
 FERRIS_API int ferris_gemm_grouped_tcgen05(const void* x, const void* w, void* out, int mode, int rows, int N, int K,
                                            int ldx, int ldw, int ldo, int experts, int expert_rows, int up_row_offset,
                                            const int* tile_expert, const float* row_scale, void* stream) {
@@ -1642,7 +1642,6 @@ FERRIS_API int ferris_gemm_grouped_tcgen05(const void* x, const void* w, void* o
     if (((uintptr_t)x & 15) || ((uintptr_t)w & 15)) FERRIS_REFUSE("grouped gemm: operands must be 16-byte aligned");
     if (mode != STORE_BF16 && mode != STORE_F32 && mode != SWIGLU_BF16) FERRIS_REFUSE("grouped gemm: mode %d", mode);
     if (!tile_expert || experts <= 0 || expert_rows <= 0) FERRIS_REFUSE("grouped gemm: no experts");
-    if (row_scale && mode != SWIGLU_BF16) FERRIS_REFUSE("grouped gemm: a factor per row goes with mode %d", (int)SWIGLU_BF16);
     if ((mode == SWIGLU_BF16 ? up_row_offset + N : N) > expert_rows || up_row_offset < 0)
         FERRIS_REFUSE("grouped gemm: %d outputs (+%d) from %d rows an expert", N, up_row_offset, expert_rows);
     const int elt = mode == STORE_F32 ? 4 : 2;
@@ -1650,6 +1649,8 @@ FERRIS_API int ferris_gemm_grouped_tcgen05(const void* x, const void* w, void* o
     g_launch_act = ferris_take_epilogue_act();
     if (g_launch_act.kind && (g_launch_act.kind >= FERRIS_EPILOGUE_GATED) != (mode == SWIGLU_BF16))
         FERRIS_REFUSE("grouped gemm: activation %d does not go with mode %d", g_launch_act.kind, mode);
+    if (row_scale && mode != SWIGLU_BF16 && !(mode == STORE_BF16 && g_launch_act.kind))
+        FERRIS_REFUSE("grouped gemm: a factor per row goes with an activation (mode %d)", mode);
     return run_tokens_m(x, w, nullptr, out, mode, rows, N, K, ldx, ldw, ldo, experts * expert_rows, up_row_offset, nullptr,
                         (cudaStream_t)stream, tile_expert, expert_rows, row_scale);
 }

@@ -1,4 +1,4 @@
-// A mixture of gated feed-forward experts of which every token uses a few.
+// A mixture of feed-forward experts (gated ones, or plain ones) of which every token uses a few.
 //
 //   router    z = Wr y + br (fp32 sums whatever the storage type); the `top` largest z (the lowest index among
 //             equals); weights = softmax over those alone
@@ -20,6 +20,8 @@
 // Where a token's weight for an expert goes: onto the expert's result (o_e times weight_e, the default), or onto its INPUT
 // (`input_weights`): o_e = Wd_e (act(weight_e Wg_e y, weight_e Wu_e y)), which is the expert of weight_e y; both products are
 // linear in y, so the factor is applied to their fp32 sums, and the results are added unweighted.
+//
+// Experts without a gate (`plain`): a_e = act(Wu_e y), act one of the kinds of ferris_epilogue_act.
 //
 // The experts' matrices lie stacked: gate and up as [experts, ff, width] each, down as [experts, width, ff].
 //
@@ -390,7 +392,8 @@ __global__ void __launch_bounds__(128) moe_router_kernel(const T* x, int ldx, co
 
 // ------------------------------------------------------------------------------------------ token-major experts
 // act[(t, s), j] = silu(Wg_e[j] . y_t) * (Wu_e[j] . y_t) for e = ids[t, s]; a block per (t, s) and slab of `slab` rows j.
-template <typename T>
+// PLAIN: act[(t, s), j] = a(Wu_e[j] . y_t), `gate` is not read.
+template <typename T, bool PLAIN>
 __global__ void __launch_bounds__(128) moe_gate_up_kernel(const T* x, int ldx, const T* __restrict__ gate,
                                                           const T* __restrict__ up, size_t expert_stride, const int* ids,
                                                           T* __restrict__ act, int width, int ff, int top, int slab,
@@ -405,10 +408,28 @@ __global__ void __launch_bounds__(128) moe_gate_up_kernel(const T* x, int ldx, c
     const T* xr = x + (size_t)t * ldx;
     stage_row(xs, xr, width, threadIdx.x, blockDim.x);
     __syncthreads();
-    const T* g = gate + (size_t)e * expert_stride;
     const T* u = up + (size_t)e * expert_stride;
-    const bool vec = rows_vectorise(g, width) && rows_vectorise(u, width);
     const int j0 = blockIdx.y * slab, j1 = min(ff, j0 + slab);
+    if (PLAIN) {  // a warp takes rows j, j + 4, j + 8 and j + 12 at a time
+        const FerrisEpilogueAct a = {act_kind, act_limit, 0.0f};
+        const bool uvec = rows_vectorise(u, width);
+        for (int j = j0 + warp; j < j1; j += 16) {
+            const int n = min(4, (j1 - j + 3) / 4);
+            const T* first = u + (size_t)j * width;
+            float d[4];
+            if (n == 4) {
+                const T* const rows[4] = {first, first + (size_t)4 * width, first + (size_t)8 * width, first + (size_t)12 * width};
+                dot_rows<4>(rows, xs, width, lane, uvec, d);
+            } else {
+                for (int r = 0; r < n; ++r) d[r] = dot_row(first + (size_t)4 * r * width, xs, width, lane, uvec);
+            }
+            if (lane == 0)
+                for (int r = 0; r < n; ++r) act[(size_t)pair * ff + j + 4 * r] = from_float<T>(ferris_epilogue_act(w * d[r], a));
+        }
+        return;
+    }
+    const T* g = gate + (size_t)e * expert_stride;
+    const bool vec = rows_vectorise(g, width) && rows_vectorise(u, width);
     // a warp takes rows j and j + 4 of both matrices at a time: four weight rows in flight for one read of the token's row
     for (int j = j0 + warp; j < j1; j += 8) {
         if (j + 4 < j1) {
@@ -539,7 +560,41 @@ __device__ __forceinline__ void gate_up_rows(const T* g, const T* u, const float
     }
 }
 
-template <typename T>
+// the same for experts without a gate: rows j, j + FEW_WARPS, .. of the up matrix alone
+template <typename T, int M>
+__device__ __forceinline__ void up_rows(const T* u, const float* xs, int width, int ff, int j0, int j1, const int* pair,
+                                        T* __restrict__ act, int lane, int warp, bool vec, uint4* ring, int act_kind,
+                                        float act_limit, const float* input_w) {
+    const FerrisEpilogueAct a = {act_kind, act_limit, 0.0f};
+    float w[M];
+#pragma unroll
+    for (int m = 0; m < M; ++m) w[m] = input_w ? input_w[pair[m]] : 1.0f;
+    for (int j = j0 + warp; j < j1; j += 4 * FEW_WARPS) {
+        const int n = min(4, (j1 - j + FEW_WARPS - 1) / FEW_WARPS);
+        float d[4][M];
+        if (n == 4) {
+            const T* const rows[4] = {u + (size_t)j * width, u + (size_t)(j + FEW_WARPS) * width,
+                                      u + (size_t)(j + 2 * FEW_WARPS) * width, u + (size_t)(j + 3 * FEW_WARPS) * width};
+            dot_tile_few<4, M>(rows, xs, width, width, lane, vec, ring, d);
+        } else {
+            for (int r = 0; r < n; ++r) {
+                const T* const row[1] = {u + (size_t)(j + FEW_WARPS * r) * width};
+                float one[1][M];
+                dot_tile_few<1, M>(row, xs, width, width, lane, vec, ring, one);
+#pragma unroll
+                for (int m = 0; m < M; ++m) d[r][m] = one[0][m];
+            }
+        }
+        if (lane == 0) {
+            for (int r = 0; r < n; ++r)
+#pragma unroll
+                for (int m = 0; m < M; ++m)
+                    act[(size_t)pair[m] * ff + j + FEW_WARPS * r] = from_float<T>(ferris_epilogue_act(w[m] * d[r][m], a));
+        }
+    }
+}
+
+template <typename T, bool PLAIN>
 __global__ void __launch_bounds__(32 * FEW_WARPS) moe_gate_up_few_kernel(const T* x, int ldx, const T* __restrict__ gate,
                                                               const T* __restrict__ up, size_t expert_stride, const int* ids,
                                                               T* __restrict__ act, int width, int ff, int pairs, int top,
@@ -555,9 +610,9 @@ __global__ void __launch_bounds__(32 * FEW_WARPS) moe_gate_up_few_kernel(const T
     const int e = blockIdx.x;
     const int n = pairs_of_expert(ids, pairs, e, list, &count);
     if (n == 0) return;
-    const T* g = gate + (size_t)e * expert_stride;
+    const T* g = PLAIN ? nullptr : gate + (size_t)e * expert_stride;
     const T* u = up + (size_t)e * expert_stride;
-    const bool vec = rows_vectorise(g, width) && rows_vectorise(u, width);
+    const bool vec = (PLAIN || rows_vectorise(g, width)) && rows_vectorise(u, width);
     const int j0 = blockIdx.y * slab, j1 = min(ff, j0 + slab);
     for (int first = 0; first < n; first += MOE_FEW_ROWS) {
         const int m = min(MOE_FEW_ROWS, n - first);
@@ -566,6 +621,15 @@ __global__ void __launch_bounds__(32 * FEW_WARPS) moe_gate_up_few_kernel(const T
         if (warp < m) stage_row(xs + (size_t)warp * width, x + (size_t)(list[first + warp] / top) * ldx, width, lane, 32);
         __syncthreads();
         const int* pair = list + first;
+        if (PLAIN) {
+            switch (m) {
+                case 1: up_rows<T, 1>(u, xs, width, ff, j0, j1, pair, act, lane, warp, vec, ring, act_kind, act_limit, input_w); break;
+                case 2: up_rows<T, 2>(u, xs, width, ff, j0, j1, pair, act, lane, warp, vec, ring, act_kind, act_limit, input_w); break;
+                case 3: up_rows<T, 3>(u, xs, width, ff, j0, j1, pair, act, lane, warp, vec, ring, act_kind, act_limit, input_w); break;
+                default: up_rows<T, 4>(u, xs, width, ff, j0, j1, pair, act, lane, warp, vec, ring, act_kind, act_limit, input_w); break;
+            }
+            continue;
+        }
         switch (m) {
             case 1: gate_up_rows<T, 1>(g, u, xs, width, ff, j0, j1, pair, act, lane, warp, vec, ring, act_kind, act_limit, input_w); break;
             case 2: gate_up_rows<T, 2>(g, u, xs, width, ff, j0, j1, pair, act, lane, warp, vec, ring, act_kind, act_limit, input_w); break;
@@ -734,6 +798,7 @@ __global__ void __launch_bounds__(256) moe_combine_kernel(const float* y, int ld
 }  // namespace
 
 extern "C" void ferris_gemm_set_gated_activation(int kind, float limit);
+extern "C" void ferris_gemm_set_activation(int kind, float a, float b);
 extern "C" int ferris_gemm_grouped_tcgen05(const void* x, const void* w, void* out, int mode, int rows, int N, int K,
                                            int ldx, int ldw, int ldo, int experts, int expert_rows, int up_row_offset,
                                            const int* tile_expert, const float* row_scale, void* stream);
@@ -753,15 +818,17 @@ FERRIS_API int ferris_moe_sorted_rows(int tokens, int top, int experts) {
 // and h also gets identity_w[t] x[t]; the scratch is then sized for experts + 1.  act_kind, act_limit: the gated
 // activation (ferris_gated_act).  row_scale: scratch, fp32 [rows], where the weights go onto the experts' inputs; else null.
 // h null: the pairs' results are left in y (row pos[pair]) and not added anywhere.
+// plain: the experts have no gate; gate_up is then [experts, ff, width], act_kind a kind of ferris_epilogue_act (2 or 3).
 FERRIS_API int ferris_moe_experts_grouped(const void* x, int ldx, const void* gate_up, const void* down, const int* ids,
                                           const float* weights, float* h, int ldh, int tokens, int width, int ff, int top,
                                           int experts, int rows, int* pos, int* row_token, int* tile_expert, void* xs,
                                           void* act, float* y, int accumulate, int act_kind, float act_limit,
-                                          const float* identity_w, float* row_scale, void* stream) {
+                                          const float* identity_w, float* row_scale, int plain, void* stream) {
     if (tokens <= 0) return FERRIS_OK;
     const int sorted = experts + (identity_w ? 1 : 0);  // the identity experts' pairs sort behind the last expert's
     if (experts <= 0 || sorted > MOE_MAX_EXPERTS || top <= 0 || top > MOE_MAX_TOP)
         FERRIS_REFUSE("experts: %d of %d experts", top, experts);
+    if (plain && act_kind != 2 && act_kind != 3) FERRIS_REFUSE("experts: unknown activation %d without a gate", act_kind);
     if (rows != ferris_moe_sorted_rows(tokens, top, sorted)) FERRIS_REFUSE("experts: scratch for %d rows", rows);
     if (width % 8 || ff % 8 || ldx % 8 || ldh % 4 || (((uintptr_t)x | (uintptr_t)xs | (uintptr_t)y | (uintptr_t)h) & 15))
         FERRIS_REFUSE("experts: width %d, ff %d and the rows must be multiples of 8 elements and start on 16 bytes", width, ff);
@@ -772,10 +839,17 @@ FERRIS_API int ferris_moe_experts_grouped(const void* x, int ldx, const void* ga
     const size_t want = (n16 + 255) / 256;
     ferris_launch(moe_gather_kernel, dim3((unsigned)(want < 148 * 16 ? want : 148 * 16)), dim3(256), 0, s, (const uint4*)x,
                   ldx / 8, (const int*)row_token, (uint4*)xs, rows, width / 8);
-    ferris_gemm_set_gated_activation(act_kind, act_limit);  // taken by the product launched next
-    int rc = ferris_gemm_grouped_tcgen05(xs, gate_up, act, 3, rows, ff, width, width, width, ff, experts, 2 * ff, ff,
+    int rc;
+    if (plain) {
+        ferris_gemm_set_activation(act_kind, act_limit, 0.0f);  // taken by the product launched next
+        rc = ferris_gemm_grouped_tcgen05(xs, gate_up, act, 0, rows, ff, width, width, width, ff, experts, ff, 0, tile_expert, row_scale, stream);
+        ferris_gemm_set_activation(0, 0.0f, 0.0f);
+    } else {
+        ferris_gemm_set_gated_activation(act_kind, act_limit);
+        rc = ferris_gemm_grouped_tcgen05(xs, gate_up, act, 3, rows, ff, width, width, width, ff, experts, 2 * ff, ff,
                                          tile_expert, row_scale, stream);
-    ferris_gemm_set_gated_activation(0, 0.0f);
+        ferris_gemm_set_gated_activation(0, 0.0f);
+    }
     if (rc != FERRIS_OK) return rc;
     rc = ferris_gemm_grouped_tcgen05(act, down, y, 1, rows, width, ff, ff, ff, width, experts, width, 0, tile_expert, nullptr, stream);
     if (rc != FERRIS_OK || !h) return rc;  // without h the rows stay in y, for the caller to add
@@ -836,6 +910,7 @@ FERRIS_API int ferris_moe_router(const void* x, int ldx, int dtype, const void* 
 // (the expert-major kernels for few tokens and the adding pass); the sums are the same bit for bit either way.
 // h null (with y and few enough pairs): the pairs' results are left in y and not added anywhere.
 // input_weights: a token's weight for an expert goes onto the expert's input instead of its result.
+// gate null: the experts have no gate, up is [experts, ff, width] and act_kind a kind of ferris_epilogue_act (2 or 3).
 FERRIS_API int ferris_moe_experts_token_major(const void* x, int ldx, int dtype, const void* gate, const void* up,
                                               long long gate_up_stride, const void* down, const int* ids,
                                               const float* weights, void* act, float* h,
@@ -846,7 +921,8 @@ FERRIS_API int ferris_moe_experts_token_major(const void* x, int ldx, int dtype,
     const float* input_w = input_weights ? weights : nullptr;  // the weights go onto one side of the experts or the other
     const float* output_w = input_weights ? nullptr : weights;
     if (experts <= 0) FERRIS_REFUSE("experts: %d experts", experts);
-    if (act_kind < 0 || act_kind > 2) FERRIS_REFUSE("experts: unknown activation %d", act_kind);
+    const bool plain = gate == nullptr;
+    if (plain ? (act_kind != 2 && act_kind != 3) : (act_kind < 0 || act_kind > 2)) FERRIS_REFUSE("experts: unknown activation %d", act_kind);
     if (width <= 0 || ff <= 0 || top <= 0 || top > MOE_MAX_TOP) FERRIS_REFUSE("experts: width %d, ff %d, %d chosen", width, ff, top);
     if (dtype != FERRIS_F32 && dtype != FERRIS_BF16) FERRIS_REFUSE("experts: unknown dtype %d", dtype);
     const size_t few_up = FEW_WARPS * FEW_RING_BYTES + (size_t)MOE_FEW_ROWS * width * sizeof(float);
@@ -867,20 +943,21 @@ FERRIS_API int ferris_moe_experts_token_major(const void* x, int ldx, int dtype,
         const dim3 grid_up(experts, (ff + slab_up - 1) / slab_up), grid_down(experts, (width + slab_down - 1) / slab_down);
         if (grid_up.y > 65535 || grid_down.y > 65535) FERRIS_REFUSE("experts: too many slabs");
         int rc;
-#define FERRIS_MOE_FEW(T)                                                                                                 \
+#define FERRIS_MOE_FEW(T, P)                                                                                               \
     do {                                                                                                                  \
-        if ((rc = ferris_allow_dynamic_smem((const void*)moe_gate_up_few_kernel<T>, few_up)) != FERRIS_OK) return rc;     \
+        if ((rc = ferris_allow_dynamic_smem((const void*)moe_gate_up_few_kernel<T, P>, few_up)) != FERRIS_OK) return rc;     \
         if ((rc = ferris_allow_dynamic_smem((const void*)moe_down_few_kernel<T>, few_down)) != FERRIS_OK) return rc;      \
-        ferris_launch(moe_gate_up_few_kernel<T>, grid_up, dim3(32 * FEW_WARPS), few_up, s, (const T*)x, ldx, (const T*)gate,         \
+        ferris_launch(moe_gate_up_few_kernel<T, P>, grid_up, dim3(32 * FEW_WARPS), few_up, s, (const T*)x, ldx, (const T*)gate,         \
                       (const T*)up, (size_t)gate_up_stride, ids, (T*)act, width, ff, pairs, top, slab_up, act_kind,    \
                       act_limit, input_w);                                                                                         \
         ferris_launch(moe_down_few_kernel<T>, grid_down, dim3(32 * FEW_WARPS), few_down, s, (const T*)act, (const T*)down, ids, y,   \
                       width, ff, pairs, slab_down);                                                                       \
     } while (0)
-        if (dtype == FERRIS_F32)
-            FERRIS_MOE_FEW(float);
-        else
-            FERRIS_MOE_FEW(bf16);
+        if (dtype == FERRIS_F32) {
+            if (plain) FERRIS_MOE_FEW(float, true); else FERRIS_MOE_FEW(float, false);
+        } else {
+            if (plain) FERRIS_MOE_FEW(bf16, true); else FERRIS_MOE_FEW(bf16, false);
+        }
 #undef FERRIS_MOE_FEW
         if (!h) FERRIS_LAUNCH_CHECK();  // the pairs' results stay in y
         const size_t n4 = (size_t)tokens * (width / 4);
@@ -913,21 +990,21 @@ FERRIS_API int ferris_moe_experts_token_major(const void* x, int ldx, int dtype,
     const dim3 grid_up(pairs, (ff + slab_up - 1) / slab_up), grid_down(tokens, (width + slab_down - 1) / slab_down);
     if (grid_up.y > 65535 || grid_down.y > 65535) FERRIS_REFUSE("experts: too many slabs");
     int rc;
-#define FERRIS_MOE_RUN(T)                                                                                                 \
+#define FERRIS_MOE_RUN(T, P)                                                                                               \
     do {                                                                                                                  \
-        if ((rc = ferris_allow_dynamic_smem((const void*)moe_gate_up_kernel<T>, smem_up)) != FERRIS_OK) return rc;        \
+        if ((rc = ferris_allow_dynamic_smem((const void*)moe_gate_up_kernel<T, P>, smem_up)) != FERRIS_OK) return rc;        \
         if ((rc = ferris_allow_dynamic_smem((const void*)moe_down_kernel<T>, smem_down)) != FERRIS_OK) return rc;         \
-        ferris_launch(moe_gate_up_kernel<T>, dim3(grid_up.x, grid_up.y, 1), dim3(128), smem_up, s, (const T*)x, ldx,      \
+        ferris_launch(moe_gate_up_kernel<T, P>, dim3(grid_up.x, grid_up.y, 1), dim3(128), smem_up, s, (const T*)x, ldx,      \
                       (const T*)gate, (const T*)up, (size_t)gate_up_stride, ids, (T*)act, width, ff, top, slab_up,      \
                       experts, act_kind, act_limit, input_w);                                                                      \
         ferris_launch(moe_down_kernel<T>, grid_down, dim3(128), smem_down, s, (const T*)act, (const T*)down, ids, output_w, \
                       h, ldh, width, ff, top, slab_down, accumulate, experts, (const T*)x, ldx, identity_w);              \
     } while (0)
-    if (dtype == FERRIS_F32)
-        FERRIS_MOE_RUN(float);
-    else if (dtype == FERRIS_BF16)
-        FERRIS_MOE_RUN(bf16);
-    else
+    if (dtype == FERRIS_F32) {
+        if (plain) FERRIS_MOE_RUN(float, true); else FERRIS_MOE_RUN(float, false);
+    } else if (dtype == FERRIS_BF16) {
+        if (plain) FERRIS_MOE_RUN(bf16, true); else FERRIS_MOE_RUN(bf16, false);
+    } else
         FERRIS_REFUSE("experts: unknown dtype %d", dtype);
 #undef FERRIS_MOE_RUN
     FERRIS_LAUNCH_CHECK();

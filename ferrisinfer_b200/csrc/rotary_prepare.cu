@@ -9,8 +9,8 @@
 //   c = mag cos(pos * freq[i]), s = mag sin(pos * freq[i]); the other elements pass
 //   q rewritten in place, k and the values stored into the paged cache.
 //
-// Rows: [nh d | nkv d | nkv dv unless values_from_keys].  Everything is computed in fp32 (position x frequency as one
-// fp32 product, sincosf in full precision); one block per token.
+// Rows: [nh d | nkv d | nkv dv unless values_from_keys].  Everything is computed in fp32 (angles as position_angle
+// forms them, sincosf in full precision); one block per token.
 //
 // Three kernels.  The vector one (no rotation, values of their own): 16 bytes at a time, every element loaded once.  The
 // paired one (even head sizes and row strides, rows that start on a pair): a token's cosines and
@@ -42,7 +42,23 @@ struct PrepareExtras {
     const int* tables;      // block tables of the unpooled pages, [requests, max_blocks]
     const int* token_seq;
     int max_blocks;
+    const float* freq_lo;   // what the 32-bit frequencies lack of their 64-bit values (null: nothing)
 };
+
+// Cosine and sine of position x frequency.  With freq_lo the angle keeps the digits that one 32-bit product rounds away: the
+// product's own rounding error comes from an FMA, the frequency's from freq_lo, and the small sum e of the two enters as
+// sin(a + e) = sin a + e cos a, cos(a + e) = cos a - e sin a.  At position 1,000 a 32-bit angle is off by up to 6e-5 rad, which
+// shows in 32-bit logits.
+__device__ __forceinline__ void position_angle(float p, const float* __restrict__ freq, const float* __restrict__ freq_lo, int f,
+                                               float& s, float& c) {
+    const float hi = freq[f], angle = p * hi;
+    sincosf(angle, &s, &c);
+    if (freq_lo) {
+        const float e = fmaf(p, hi, -angle) + p * freq_lo[f];
+        const float s0 = s;
+        s = fmaf(e, c, s), c = fmaf(-e, s0, c);
+    }
+}
 
 // The pooled row `slot` = the means of the keys and of the values of positions pos - pool + 1 .. pos, as the pages hold
 // them: fp32 sums in the order of the positions, one division, one rounding.  Elements `first`, `first + step`, ... of
@@ -240,7 +256,7 @@ __global__ void __launch_bounds__(128) qk_norm_rotary_cache_write_kernel(
         float u = to_float(row[e]), v = to_float(row[e + partner]);
         if (w) u = (u * inv) * w[col], v = (v * inv) * w[col + partner];
         float s, c;
-        sincosf((float)pos * freq[f], &s, &c);
+        position_angle((float)pos, freq, ex.freq_lo, f, s, c);
         s *= mag, c *= mag;
         dst[i] = from_float<T>(u * c - v * s);
         dst[i + partner] = from_float<T>(v * c + u * s);
@@ -294,7 +310,7 @@ __global__ void __launch_bounds__(256) qk_norm_rotary_cache_write_paired_kernel(
     const int pos = positions[t];
     for (int f = threadIdx.x; f < half; f += blockDim.x) {
         float s, c;
-        sincosf((float)pos * freq[f], &s, &c);
+        position_angle((float)pos, freq, ex.freq_lo, f, s, c);
         cs[f] = c * mag, cs[half + f] = s * mag;
     }
     const int slot = write_kv ? slot_mapping[t] : -1;
@@ -465,10 +481,7 @@ __global__ void __launch_bounds__(256) qk_norm_cache_write_vec_kernel(
 // The norm per HEAD: every q and k head divided by the root mean square of its own d elements and multiplied by a
 // weight of d numbers that all heads share (wq for queries, wk for keys; null: that side is not normed), then rotated
 // and stored as above.  A warp per head: its lanes sum the head's squares, then norm, rotate and store it; the values
-// are copied by the whole block.  With freq_lo (what the 32-bit frequencies lack of their 64-bit values) the angle
-// position x frequency keeps the digits that one 32-bit product rounds away: the product's own rounding error comes
-// from an FMA, the frequency's from freq_lo, and the small sum e of the two enters as sin(a + e) = sin a + e cos a,
-// cos(a + e) = cos a - e sin a.  At position 1,000 a 32-bit angle is off by up to 6e-5 rad, which shows in 32-bit logits.
+// are copied by the whole block.
 template <typename T>
 __global__ void __launch_bounds__(256) qk_head_norm_rotary_cache_write_kernel(
     T* qkv, int ld, const int* __restrict__ positions, const int* __restrict__ slot_mapping, T* __restrict__ k_cache,
@@ -482,15 +495,8 @@ __global__ void __launch_bounds__(256) qk_head_norm_rotary_cache_write_kernel(
     const int pos = positions[t];
     const int half = rotary >> 1;
     for (int f = threadIdx.x; f < half; f += blockDim.x) {
-        const float p = (float)pos, hi = freq[f];
-        const float angle = p * hi;
         float s, c;
-        sincosf(angle, &s, &c);
-        if (freq_lo) {
-            const float e = fmaf(p, hi, -angle) + p * freq_lo[f];
-            const float s0 = s;
-            s = fmaf(e, c, s), c = fmaf(-e, s0, c);
-        }
+        position_angle((float)pos, freq, freq_lo, f, s, c);
         cs[f] = c * mag, cs[half + f] = s * mag;
     }
     __syncthreads();
@@ -547,13 +553,13 @@ FERRIS_API int ferris_qk_norm_rotary_cache_write(void* qkv, int ld, int dtype, c
                                                  int interleaved, float mag, int values_from_keys, int write_kv,
                                                  void* first_values, const float* mix_lambda, const int* pool_slots,
                                                  void* pool_k, void* pool_v, int pool, const int* tables, int max_blocks,
-                                                 const int* token_seq, void* stream) {
+                                                 const int* token_seq, const float* freq_lo, void* stream) {
     if (tokens <= 0) return FERRIS_OK;
     if (mix_lambda && !first_values) FERRIS_REFUSE("qk norm + rotation: nothing to mix the values with");
     if (first_values && !write_kv) FERRIS_REFUSE("qk norm + rotation: values are mixed where they are stored");
     if (pool_slots && (!write_kv || !pool_k || !pool_v || pool <= 0 || !tables || max_blocks <= 0 || !token_seq))
         FERRIS_REFUSE("qk norm + rotation: pooled rows of %d positions want a cache, pooled pages and block tables", pool);
-    const PrepareExtras ex = {first_values, mix_lambda, pool_slots, pool_k, pool_v, pool, tables, token_seq, max_blocks};
+    const PrepareExtras ex = {first_values, mix_lambda, pool_slots, pool_k, pool_v, pool, tables, token_seq, max_blocks, freq_lo};
     if (nh <= 0 || nkv <= 0 || d <= 0 || dv <= 0 || page_size <= 0)
         FERRIS_REFUSE("qk norm + rotation: nh=%d nkv=%d d=%d dv=%d page_size=%d", nh, nkv, d, dv, page_size);
     if (rotary < 0 || rotary > d || (rotary & 1) || (rotary > 0 && !freq))

@@ -200,65 +200,101 @@ __global__ void __launch_bounds__(256) branch_norm_sum_kernel(Branches br, float
 }
 
 // ---------------------------------------------------------------------------------------------
-// Attention over a shared latent.  A token's projection row holds, per query head, [dim plain | rot rotated] query
-// dimensions, and once [rank latent | rot rotated key] dimensions.  This kernel norms the latent (RMS norm with a
-// weight), rotates the key part and the heads' rotated query parts (rotate-half over the first `rot_dims` of the
-// part; angle = position * inv_freq[i], fp32), writes [latent | rotated key] as the token's one cache row and the
-// rotated query parts into the attention's query rows behind the place of the absorbed plain part:
-//   q_att[t, h] = [rank: left for the product of the plain query with the key up-projection | rot: rotated part].
+// Attention over a shared latent.  A token's projection row holds [rank latent | rot rotated key] dimensions; its query rows
+// hold, per head, [dim plain | rot rotated] dimensions (in the same projection row, or, where queries go through a latent of
+// their own, in the rows of a later product).  Three pieces of work, any of which may be left out of a launch:
+//   keys       the latent is normed (RMS norm with a weight), the key part rotated, [latent | rotated key] written as the
+//              token's one cache row;
+//   queries    the heads' rotated query parts go into the attention's query rows behind the place of the absorbed plain part:
+//              q_att[t, h] = [rank: left for the product of the plain query with the key up-projection | rot: rotated part];
+//   q latent   the query latent is normed (RMS norm with a weight of its own) into rows for the next product.
+// Rotation: the first `rot_dims` of the part, elements (i, i + rot_dims / 2) or (2i, 2i + 1) together (interleaved), angle =
+// position * freq[i] in fp32; with freq_lo (what the 32-bit frequencies lack of their 64-bit values) the angle keeps the digits
+// that one 32-bit product rounds away.
 // ---------------------------------------------------------------------------------------------
+struct LatentArgs {
+    const void* q;  // null: no queries
+    const void* dkv;  // null: no keys
+    const void* cq;  // null: no query latent
+    void* cq_out;
+    const float* cq_norm;
+    const float* norm;
+    const float* freq;
+    const float* freq_lo;
+    const int* positions;
+    const int* slots;
+    void* cache;
+    void* q_att;
+    int ldq, lddkv, ldcq, ldcq_out, ldqa, q_rank, rot_dims, interleaved, heads, dim, rot, rank;
+    float eps;
+};
+
 template <typename T>
-__global__ void __launch_bounds__(128) latent_prepare_kernel(const T* proj, int ld, int q_off, int dkv_off,
-                                                             const float* __restrict__ norm_w, float eps,
-                                                             const int* __restrict__ positions,
-                                                             const float* __restrict__ inv_freq, int rot_dims,
-                                                             const int* __restrict__ slot_mapping, T* __restrict__ cache,
-                                                             T* __restrict__ q_att, int ldqa, int heads, int dim, int rot,
-                                                             int rank, int write_kv) {
-    __shared__ float scratch[33];
-    __shared__ float cs_tab[256], sn_tab[256];  // the token's angles, once for the key part and every head
-    pdl_wait();
-    pdl_launch_dependents();
-    const int t = blockIdx.x;
-    const float pos = (float)positions[t];
-    const T* row = proj + (size_t)t * ld;
+__device__ __forceinline__ float rotated(const T* src, int e, int rot_dims, int interleaved, const float* cs, const float* sn) {
+    const float v = to_float(src[e]);
+    if (e >= rot_dims) return v;
     const int half = rot_dims >> 1;
-    for (int f = threadIdx.x; f < half; f += blockDim.x) sincosf(pos * inv_freq[f], &sn_tab[f], &cs_tab[f]);
-    __syncthreads();
-    // the heads' rotated query parts
-    for (int i = threadIdx.x; i < heads * rot; i += blockDim.x) {
-        const int h = i / rot, e = i - h * rot;
-        const T* src = row + q_off + (size_t)h * (dim + rot) + dim;
-        float v = to_float(src[e]);
-        if (e < rot_dims) {
-            const int f = e < half ? e : e - half;
-            const float sn = sn_tab[f], cs = cs_tab[f];
-            const float other = to_float(src[e < half ? e + half : e - half]);
-            v = e < half ? v * cs - other * sn : v * cs + other * sn;
-        }
-        q_att[(size_t)t * ldqa + (size_t)h * (rank + rot) + rank + e] = from_float<T>(v);
-    }
-    if (!write_kv) return;
-    const T* dkv = row + dkv_off;
+    const bool first = interleaved ? !(e & 1) : e < half;
+    const int f = interleaved ? e >> 1 : (first ? e : e - half);
+    const float other = to_float(src[interleaved ? (e ^ 1) : (first ? e + half : e - half)]);
+    return first ? v * cs[f] - other * sn[f] : v * cs[f] + other * sn[f];
+}
+
+template <typename T>
+__device__ __forceinline__ void normed_row(const T* src, T* dst, int n, const float* __restrict__ w, float eps, float* scratch) {
     float ss = 0.0f;
-    for (int i = threadIdx.x; i < rank; i += blockDim.x) {
-        const float v = to_float(dkv[i]);
+    for (int i = threadIdx.x; i < n; i += blockDim.x) {
+        const float v = to_float(src[i]);
         ss = fmaf(v, v, ss);
     }
     ss = block_sum(ss, scratch);
-    const float inv = 1.0f / sqrtf(ss / (float)rank + eps);
-    T* dst = cache + (size_t)slot_mapping[t] * (rank + rot);
-    for (int i = threadIdx.x; i < rank; i += blockDim.x) dst[i] = from_float<T>((to_float(dkv[i]) * inv) * norm_w[i]);
-    for (int e = threadIdx.x; e < rot; e += blockDim.x) {
-        float v = to_float(dkv[rank + e]);
-        if (e < rot_dims) {
-            const int f = e < half ? e : e - half;
-            const float sn = sn_tab[f], cs = cs_tab[f];
-            const float other = to_float(dkv[rank + (e < half ? e + half : e - half)]);
-            v = e < half ? v * cs - other * sn : v * cs + other * sn;
-        }
-        dst[rank + e] = from_float<T>(v);
+    const float inv = 1.0f / sqrtf(ss / (float)n + eps);
+    for (int i = threadIdx.x; i < n; i += blockDim.x) dst[i] = from_float<T>((to_float(src[i]) * inv) * w[i]);
+}
+
+template <typename T>
+__global__ void __launch_bounds__(128) latent_prepare_kernel(const LatentArgs p) {
+    __shared__ float scratch[33];
+    __shared__ float cs[256], sn[256];  // the token's angles, once for the key part and every head
+    pdl_wait();
+    pdl_launch_dependents();
+    // the pieces of a token side by side: blockIdx.y 0 takes keys and queries, 1 the query latent
+    const int t = blockIdx.x;
+    if (p.cq && (blockIdx.y == 1 || gridDim.y == 1)) {
+        normed_row(reinterpret_cast<const T*>(p.cq) + (size_t)t * p.ldcq, reinterpret_cast<T*>(p.cq_out) + (size_t)t * p.ldcq_out,
+                   p.q_rank, p.cq_norm, p.eps, scratch);
+        if (gridDim.y > 1) return;
+        __syncthreads();
     }
+    if (!p.q && !p.dkv) return;
+    const float pos = (float)p.positions[t];
+    for (int f = threadIdx.x; f < (p.rot_dims >> 1); f += blockDim.x) {
+        const float hi = p.freq[f], angle = pos * hi;
+        float s, c;
+        sincosf(angle, &s, &c);
+        if (p.freq_lo) {  // sin(a + e) = sin a + e cos a, cos(a + e) = cos a - e sin a
+            const float e = fmaf(pos, hi, -angle) + pos * p.freq_lo[f];
+            const float s0 = s;
+            s = fmaf(e, c, s), c = fmaf(-e, s0, c);
+        }
+        cs[f] = c, sn[f] = s;
+    }
+    __syncthreads();
+    if (p.q) {
+        const T* row = reinterpret_cast<const T*>(p.q) + (size_t)t * p.ldq;
+        T* dst = reinterpret_cast<T*>(p.q_att) + (size_t)t * p.ldqa;
+        for (int i = threadIdx.x; i < p.heads * p.rot; i += blockDim.x) {
+            const int h = i / p.rot, e = i - h * p.rot;
+            const float v = rotated(row + (size_t)h * (p.dim + p.rot) + p.dim, e, p.rot_dims, p.interleaved, cs, sn);
+            dst[(size_t)h * (p.rank + p.rot) + p.rank + e] = from_float<T>(v);
+        }
+    }
+    if (!p.dkv) return;
+    const T* dkv = reinterpret_cast<const T*>(p.dkv) + (size_t)t * p.lddkv;
+    T* dst = reinterpret_cast<T*>(p.cache) + (size_t)p.slots[t] * (p.rank + p.rot);
+    for (int e = threadIdx.x; e < p.rot; e += blockDim.x)
+        dst[p.rank + e] = from_float<T>(rotated(dkv + p.rank, e, p.rot_dims, p.interleaved, cs, sn));
+    normed_row(dkv, dst, p.rank, p.norm, p.eps, scratch);
 }
 
 // ---------------------------------------------------------------------------------------------
@@ -410,23 +446,30 @@ FERRIS_API int ferris_branch_norm_sum(const float* const* ys, const float* const
     FERRIS_LAUNCH_CHECK();
 }
 
-// proj: [tokens, ld]; cache: [rows, rank + rot] (one kv head: a cache row per slot); q_att: [tokens, ldqa].
-FERRIS_API int ferris_latent_prepare(const void* proj, int ld, int dtype, int q_off, int dkv_off, const float* norm_w,
-                                     float eps, const int* positions, const float* inv_freq, int rot_dims,
-                                     const int* slot_mapping, void* cache, void* q_att, int ldqa, int tokens, int heads,
-                                     int dim, int rot, int rank, int write_kv, void* stream) {
+// q (null: no queries): rows ldq apart of heads x (dim + rot); dkv (null: no keys): rows lddkv apart of rank + rot; cq (null: no
+// query latent): rows ldcq apart of q_rank, normed into cq_out.  cache: [rows, rank + rot] (one kv head: a cache row per
+// slot); q_att: rows ldqa apart.  The norms share eps.
+FERRIS_API int ferris_latent_prepare(const void* q, int ldq, const void* dkv, int lddkv, int dtype, const float* norm_w, float eps,
+                                     const int* positions, const float* freq, const float* freq_lo, int rot_dims, int interleaved,
+                                     const int* slot_mapping, void* cache, void* q_att, int ldqa, const void* cq, int ldcq,
+                                     const float* cq_norm, void* cq_out, int ldcq_out, int q_rank, int tokens, int heads,
+                                     int dim, int rot, int rank, void* stream) {
     if (tokens <= 0) return FERRIS_OK;
     if (heads <= 0 || dim < 0 || rot < 0 || rank <= 0) FERRIS_REFUSE("latent prepare: %d heads of %d + %d over a latent of %d", heads, dim, rot, rank);
     if (rot_dims < 0 || rot_dims > rot || (rot_dims & 1) || rot_dims > 512) FERRIS_REFUSE("latent prepare: %d of %d dimensions rotate (at most 512)", rot_dims, rot);
-    if (rot_dims > 0 && !inv_freq) FERRIS_REFUSE("latent prepare: no frequencies");
-    if (write_kv && (!slot_mapping || !cache || !norm_w)) FERRIS_REFUSE("latent prepare: no cache to write");
+    if (rot_dims > 0 && !freq) FERRIS_REFUSE("latent prepare: no frequencies");
+    if (!positions || (q && !q_att)) FERRIS_REFUSE("latent prepare: no positions, or no rows for the queries");
+    if (dkv && (!slot_mapping || !cache || !norm_w)) FERRIS_REFUSE("latent prepare: no cache to write");
+    if (cq && (!cq_norm || !cq_out || q_rank <= 0)) FERRIS_REFUSE("latent prepare: a query latent of %d", q_rank);
+    if (!q && !dkv && !cq) return FERRIS_OK;
+    const LatentArgs p = {q, dkv, cq, cq_out, cq_norm, norm_w, freq, freq_lo, positions, slot_mapping, cache, q_att,
+                          ldq, lddkv, ldcq, ldcq_out, ldqa, q_rank, rot_dims, interleaved, heads, dim, rot, rank, eps};
+    const dim3 grid(tokens, cq && (q || dkv) ? 2 : 1);
     cudaStream_t s = (cudaStream_t)stream;
     if (dtype == FERRIS_F32)
-        ferris_launch(latent_prepare_kernel<float>, dim3(tokens), dim3(128), 0, s, (const float*)proj, ld, q_off, dkv_off, norm_w, eps,
-                      positions, inv_freq, rot_dims, slot_mapping, (float*)cache, (float*)q_att, ldqa, heads, dim, rot, rank, write_kv);
+        ferris_launch(latent_prepare_kernel<float>, grid, dim3(128), 0, s, p);
     else if (dtype == FERRIS_BF16)
-        ferris_launch(latent_prepare_kernel<bf16>, dim3(tokens), dim3(128), 0, s, (const bf16*)proj, ld, q_off, dkv_off, norm_w, eps,
-                      positions, inv_freq, rot_dims, slot_mapping, (bf16*)cache, (bf16*)q_att, ldqa, heads, dim, rot, rank, write_kv);
+        ferris_launch(latent_prepare_kernel<bf16>, grid, dim3(128), 0, s, p);
     else
         FERRIS_REFUSE("latent prepare: unknown dtype %d", dtype);
     FERRIS_LAUNCH_CHECK();

@@ -770,15 +770,18 @@ class ScoreTerms:
     """What else enters an attention score and its softmax, per query head (fp32 [num_heads] tensors on the device, or
     None): ``slopes`` (the score of the key at j for the query at P gets slopes[h] * (j - P) added), ``log_r1`` and
     ``log_r2`` (it loses log_r1[h] * ln(1 + log_r2[h] * (P - j))), ``sink`` (the softmax's denominator also holds
-    exp(sink[h]): a weight with no key and no value)."""
+    exp(sink[h]): a weight with no key and no value), ``softcap`` (a number c > 0: the scaled product x becomes c tanh(x / c)
+    ahead of any penalty; 0: it stays).  ``gate``: [T, num_heads] in the queries' type (a view with contiguous rows): head h's
+    output is multiplied by sigmoid(gate[t, h])."""
 
-    __slots__ = ("slopes", "log_r1", "log_r2", "sink")
+    __slots__ = ("slopes", "log_r1", "log_r2", "sink", "softcap", "gate")
 
-    def __init__(self, slopes=None, log_r1=None, log_r2=None, sink=None):
+    def __init__(self, slopes=None, log_r1=None, log_r2=None, sink=None, softcap: float = 0.0, gate=None):
         self.slopes, self.log_r1, self.log_r2, self.sink = slopes, log_r1, log_r2, sink
+        self.softcap, self.gate = float(softcap or 0.0), gate
 
     def any(self) -> bool:
-        return any(t is not None for t in (self.slopes, self.log_r1, self.log_r2, self.sink))
+        return self.softcap > 0.0 or any(t is not None for t in (self.slopes, self.log_r1, self.log_r2, self.sink, self.gate))
 
 
 class PooledKeys:
@@ -814,7 +817,7 @@ def paged_attention_simt(qkv: torch.Tensor, out: torch.Tensor, k_cache: torch.Te
                          num_heads: int, num_kv_heads: int, head_dim: int, window: int, scale: float,
                          score_slopes=None, v_head_dim: Optional[int] = None,
                          max_q_len: int = 1, max_kv_len: int = 0, workspace=None, values_in_keys: bool = False,
-                         chunk: int = 0, pooled: Optional[PooledKeys] = None):
+                         chunk: int = 0, pooled: Optional[PooledKeys] = None, keep_first: int = 0):
     """General attention over the paged cache; q is read from the first nh*d columns of ``qkv``.
     ``window``: the query at position P sees the keys P - window + 1 .. P (0: all).  ``chunk`` (instead of a window):
     positions are counted off in chunks of that many from 0, and a query sees the keys of its own chunk up to itself.
@@ -827,6 +830,8 @@ def paged_attention_simt(qkv: torch.Tensor, out: torch.Tensor, k_cache: torch.Te
     tokens): the most keys a request holds, and where scratch comes from; the keys of a token are then cut into
     shares that run side by side, and query heads of one kv head share its keys.  ``pooled`` (with a window): beside the
     window's tokens the query sees one row of ``pooled`` for every run of positions that lies wholly before the window.
+    ``keep_first`` (with a window, without ``pooled``): beside the window's tokens the query sees the request's first
+    ``keep_first`` tokens.
     bf16 without a distance penalty and with values in rows of their own runs on tensor cores where the geometry allows it
     (``set_attention_rows``); everything else on CUDA cores."""
     dv = int(v_head_dim or head_dim)
@@ -874,7 +879,15 @@ def paged_attention_simt(qkv: torch.Tensor, out: torch.Tensor, k_cache: torch.Te
             raise KernelError(f"attention: pooled keys {tuple(pooled.k.shape)} of {pooled.every} positions, window {window}")
         pool_args = (_ptr(pooled.k), _ptr(pooled.v), _ptr(pooled.block_tables), _c_int(pooled.block_tables.shape[1]),
                      _c_int(pooled.every))
-    span = min(max_kv_len, window) if window else max_kv_len
+    if keep_first and (keep_first < 0 or not window or chunk or pooled is not None):
+        raise KernelError(f"attention: {keep_first} kept tokens go with a window and no pooled keys")
+    ldgate = 0
+    if terms.gate is not None:
+        Tg, ng, ldgate = _rows(terms.gate, "head gates")
+        if (Tg, ng) != (T, num_heads) or terms.gate.dtype != qkv.dtype:
+            raise KernelError(f"attention: gates {tuple(terms.gate.shape)} of {T} rows and {num_heads} heads")
+    pool_args += (_c_int(keep_first), _c_float(terms.softcap), _ptr(terms.gate), _c_int(ldgate))
+    span = min(max_kv_len, window + keep_first) if window else max_kv_len
     if pooled is not None:
         span += max_kv_len // pooled.every
     single = max_q_len <= 1 and max_kv_len > 0 and workspace is not None
@@ -1179,20 +1192,25 @@ def gated_rmsnorm(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps
     )
 
 
-def recurrence_gates(proj: torch.Tensor, a_off: int, b_off: Optional[int], A_log: torch.Tensor, dt_bias: torch.Tensor,
-                     decay: torch.Tensor, beta: torch.Tensor, heads: int, unit_norm: Optional[tuple] = None):
+def recurrence_gates(proj: torch.Tensor, a_off: Optional[int], b_off: Optional[int], A_log: Optional[torch.Tensor],
+                     dt_bias: Optional[torch.Tensor], decay: Optional[torch.Tensor], beta: torch.Tensor, heads: int, unit_norm: Optional[tuple] = None):
     """Per token and head: decay = exp(-exp(A_log) * dt) with dt = softplus(proj[:, a_off + h] + dt_bias); beta =
     sigmoid(proj[:, b_off + h]), or dt itself where ``b_off`` is None.  ``unit_norm`` = (rows, q_off, k_off, qk_heads,
     dim, eps, q_mul, qscale, kscale): the factors that make the q and k heads of ``rows`` unit vectors
-    (1 / sqrt(sum x^2 + eps); q's also times q_mul), fp32 [T, qk_heads] each.  All in fp32."""
+    (1 / sqrt(sum x^2 + eps); q's also times q_mul), fp32 [T, qk_heads] each.  All in fp32.  ``a_off``, ``A_log``, ``dt_bias``
+    and ``decay`` all None: no decays (a recurrence whose rows decay one by one forms its own)."""
     T, width, ld = _rows(proj, "recurrence gates input")
-    _need(A_log, "A_log", torch.float32)
-    _need(dt_bias, "dt_bias", torch.float32)
-    _need(decay, "decays", torch.float32)
+    if a_off is None and (A_log is not None or dt_bias is not None or decay is not None or b_off is None):
+        raise KernelError("recurrence gates: decays without the columns they come from")
+    if a_off is not None:
+        _need(A_log, "A_log", torch.float32)
+        _need(dt_bias, "dt_bias", torch.float32)
+        _need(decay, "decays", torch.float32)
+        if A_log.numel() != heads or dt_bias.numel() != heads or decay.shape != (T, heads) or a_off + heads > width:
+            raise KernelError(f"recurrence gates: proj {tuple(proj.shape)}, {heads} heads, decay {tuple(decay.shape)}")
     _need(beta, "step sizes", torch.float32)
-    if (A_log.numel() != heads or dt_bias.numel() != heads or decay.shape != (T, heads) or beta.shape != (T, heads)
-            or a_off + heads > width or (b_off is not None and b_off + heads > width)):
-        raise KernelError(f"recurrence gates: proj {tuple(proj.shape)}, {heads} heads, decay {tuple(decay.shape)}")
+    if beta.shape != (T, heads) or (b_off is not None and b_off + heads > width):
+        raise KernelError(f"recurrence gates: proj {tuple(proj.shape)}, {heads} heads, step sizes {tuple(beta.shape)}")
     qk, ldqk, q_off, k_off, qk_heads, dim, eps, q_mul, qscale, kscale = None, 0, 0, 0, 0, 0, 0.0, 1.0, None, None
     if unit_norm is not None:
         qk, q_off, k_off, qk_heads, dim, eps, q_mul, qscale, kscale = unit_norm
@@ -1203,7 +1221,7 @@ def recurrence_gates(proj: torch.Tensor, a_off: int, b_off: Optional[int], A_log
                 or kscale.shape != (T, qk_heads)):
             raise KernelError(f"recurrence gates: q/k rows {tuple(qk.shape)} for {qk_heads} heads of {dim}")
     _check(
-        _lib().ferris_recurrence_gates(_ptr(proj), _c_int(ld), _c_int(_dt(proj, "recurrence gates")), _c_int(a_off),
+        _lib().ferris_recurrence_gates(_ptr(proj), _c_int(ld), _c_int(_dt(proj, "recurrence gates")), _c_int(a_off or 0),
                                        _c_int(-1 if b_off is None else b_off), _ptr(A_log), _ptr(dt_bias), _ptr(decay),
                                        _ptr(beta), _c_int(1 if b_off is None else 0), _ptr(qk), _c_int(ldqk), _c_int(q_off),
                                        _c_int(k_off), _c_int(qk_heads), _c_int(dim), _c_float(eps), _c_float(q_mul),
@@ -1212,25 +1230,39 @@ def recurrence_gates(proj: torch.Tensor, a_off: int, b_off: Optional[int], A_log
     )
 
 
-def gated_recurrence(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, beta: torch.Tensor,
+def gated_recurrence(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: Optional[torch.Tensor], beta: torch.Tensor,
                      out: torch.Tensor, state: torch.Tensor, ctx, heads: int, qk_heads: int, dim: int, vdim: int,
                      delta_rule: bool, qscale: Optional[torch.Tensor] = None, kscale: Optional[torch.Tensor] = None,
-                     skip: Optional[torch.Tensor] = None, write_state: bool = True):
+                     skip: Optional[torch.Tensor] = None, write_state: bool = True,
+                     row_decay: Optional[tuple] = None):
     """The recurrence of the step's tokens, request by request from each request's state (fp32 [slots, heads, vdim, dim]: S transposed):
     plain: S <- decay S + k (beta v)^T, o = S^T q + skip v;  delta rule: S <- decay S, u = beta (v - S^T k), S <- S + k u^T,
     o = S^T q.  ``q``, ``k``: [T, qk_heads x dim] (views with contiguous rows; value head h uses q/k head
     h / (heads / qk_heads)), optionally times one fp32 factor per (token, q/k head) each; ``v``: [T, heads x vdim];
-    ``decay``, ``beta``: fp32 [T, heads]; ``out``: fp32 [T, heads x vdim]."""
+    ``decay``, ``beta``: fp32 [T, heads]; ``out``: fp32 [T, heads x vdim].  ``row_decay`` = (z fp32 [T, heads x dim], rates fp32
+    [heads]), with the delta rule and ``decay`` None: every row (key channel) of the state decays by a number of its own,
+    exp(-softplus(z) rate), formed in the kernel."""
     T, wq, ldq = _rows(q, "recurrence queries")
     T1, wk, ldk = _rows(k, "recurrence keys")
     T2, wv, ldv = _rows(v, "recurrence values")
     T3, wo, ldo = _rows(out, "recurrence output")
     _need(state, "recurrence state", torch.float32)
-    _need(decay, "decays", torch.float32)
+    z = rates = None
+    ldz = 0
+    if row_decay is not None:
+        z, rates = row_decay
+        T4, wz, ldz = _rows(z, "row decays")
+        _need(rates, "decay rates", torch.float32)
+        if not delta_rule or decay is not None or T4 != T or wz != heads * dim or z.dtype != torch.float32 or rates.numel() != heads:
+            raise KernelError(f"recurrence: row decays {tuple(z.shape)} for {heads} heads of {dim} rows")
+    else:
+        _need(decay, "decays", torch.float32)
+        if decay.shape != (T, heads):
+            raise KernelError(f"recurrence: decays {tuple(decay.shape)}")
     _need(beta, "step sizes", torch.float32)
     if (not (T == T1 == T2 == T3) or wq != qk_heads * dim or wk != qk_heads * dim or wv != heads * vdim or wo != heads * vdim
             or out.dtype != torch.float32 or k.dtype != q.dtype or v.dtype != q.dtype or state.shape[1:] != (heads, vdim, dim)
-            or decay.shape != (T, heads) or beta.shape != (T, heads)):
+            or beta.shape != (T, heads)):
         raise KernelError(f"recurrence: q {tuple(q.shape)}, k {tuple(k.shape)}, v {tuple(v.shape)}, out {tuple(out.shape)}, "
                           f"state {tuple(state.shape)}")
     for name, t_ in (("q factors", qscale), ("k factors", kscale)):
@@ -1249,7 +1281,7 @@ def gated_recurrence(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: t
                                        _ptr(ctx.seq_state_slot), _c_int(ctx.num_seqs), _c_int(heads), _c_int(qk_heads),
                                        _c_int(dim), _c_int(vdim), _c_int(1 if delta_rule else 0),
                                        _c_int(1 if write_state else 0), _c_int(int(getattr(ctx, "max_q_len", 0) or T)),
-                                       _stream()),
+                                       _ptr(z), _c_int(ldz), _ptr(rates), _stream()),
         "gated recurrence",
     )
 
@@ -1521,38 +1553,56 @@ def branch_norm_sum(h: torch.Tensor, branches: list, coef: float, eps: float, ac
                                          _c_int(h.shape[1]), _c_int(1 if accumulate else 0), _stream()), "branch norm sum")
 
 
-def latent_prepare(proj: torch.Tensor, q_off: int, dkv_off: int, norm_weight: torch.Tensor, eps: float,
-                   positions: torch.Tensor, inv_freq: Optional[torch.Tensor], rot_dims: int,
-                   slot_mapping: Optional[torch.Tensor], cache: Optional[torch.Tensor], q_att: torch.Tensor, heads: int,
-                   dim: int, rot: int, rank: int, write_kv: bool = True):
-    """Between the input product and attention over a shared latent.  ``proj`` rows hold ``heads`` x [dim plain | rot
-    rotated] query dimensions from ``q_off`` and [rank latent | rot key] from ``dkv_off``.  The latent is RMS-normed
-    with ``norm_weight``, the key part and the heads' rotated query parts are rotated (rotate-half over the first
-    ``rot_dims``, angle = position * inv_freq[i]), [latent | key part] becomes the token's cache row (``cache``
-    [pages, 1, page size, rank + rot]) and the rotated query parts go to ``q_att`` [T, heads x (rank + rot)], behind
-    the first ``rank`` columns of each head (which the absorbed plain queries fill)."""
-    T, width, ld = _rows(proj, "latent input")
-    T2, wq, ldqa = _rows(q_att, "latent queries")
+def latent_prepare(positions: torch.Tensor, rotary: Optional["RotaryTable"], eps: float, heads: int, dim: int, rot: int,
+                   rank: int, queries: Optional[tuple] = None, keys: Optional[tuple] = None, q_latent: Optional[tuple] = None):
+    """What stands around the products of attention over a shared latent; each piece is done where its tuple is given.
+    ``queries`` = (q, q_att): q's rows hold ``heads`` x [dim plain | rot rotated]; the rotated parts go, rotated by position, to
+    ``q_att`` [T, heads x (rank + rot)], behind the first ``rank`` columns of each head (which the absorbed plain queries
+    fill).  ``keys`` = (dkv, norm weight, slot mapping, cache): dkv's rows hold [rank latent | rot key]; the latent is
+    RMS-normed, the key part rotated, and [latent | key part] becomes the token's cache row (``cache`` [pages, 1, page size,
+    rank + rot]).  ``q_latent`` = (rows, norm weight, out): rows RMS-normed into ``out``, for the product that forms the
+    queries."""
     _need(positions, "positions", torch.int32)
-    if (T2 != T or q_att.dtype != proj.dtype or wq != heads * (rank + rot) or q_off + heads * (dim + rot) > width
-            or dkv_off + rank + rot > width or positions.numel() != T):
-        raise KernelError(f"latent prepare: proj {tuple(proj.shape)}, q_att {tuple(q_att.shape)}")
-    if rot_dims:
-        _need(inv_freq, "rotary frequencies", torch.float32)
-        if inv_freq.numel() != rot_dims // 2:
-            raise KernelError("latent prepare: one frequency per rotated pair is needed")
-    if write_kv:
-        _need(slot_mapping, "slot mapping", torch.int32)
-        _need(cache, "latent cache", proj.dtype)
-        _need(norm_weight, "latent norm weight", torch.float32)
-        if cache.dim() != 4 or cache.shape[1] != 1 or cache.shape[3] != rank + rot or norm_weight.numel() != rank:
-            raise KernelError(f"latent prepare: cache {tuple(cache.shape)} for rows of {rank} + {rot}")
+    T = positions.numel()
+    some = next((x[0] for x in (queries, keys, q_latent) if x is not None), None)
+    if some is None:
+        return
+    q = dkv = cq = q_att = cq_out = norm_w = cq_norm = slots = cache = None
+    ldq = lddkv = ldcq = ldqa = ldco = q_rank = 0
+    if queries is not None:
+        q, q_att = queries
+        T1, w1, ldq = _rows(q, "latent queries")
+        T2, w2, ldqa = _rows(q_att, "attention queries")
+        if T1 != T or T2 != T or w1 != heads * (dim + rot) or w2 != heads * (rank + rot) or q_att.dtype != q.dtype:
+            raise KernelError(f"latent prepare: q {tuple(q.shape)}, q_att {tuple(q_att.shape)}")
+    if keys is not None:
+        dkv, norm_w, slots, cache = keys
+        T1, w1, lddkv = _rows(dkv, "latent rows")
+        _need(slots, "slot mapping", torch.int32)
+        _need(cache, "latent cache", dkv.dtype)
+        _need(norm_w, "latent norm weight", torch.float32)
+        if (T1 != T or w1 != rank + rot or dkv.dtype != some.dtype or cache.dim() != 4 or cache.shape[1] != 1
+                or cache.shape[3] != rank + rot or norm_w.numel() != rank or slots.numel() != T):
+            raise KernelError(f"latent prepare: rows {tuple(dkv.shape)}, cache {tuple(cache.shape)} for {rank} + {rot}")
+    if q_latent is not None:
+        cq, cq_norm, cq_out = q_latent
+        T1, q_rank, ldcq = _rows(cq, "query latent")
+        T2, w2, ldco = _rows(cq_out, "normed query latent")
+        _need(cq_norm, "query latent norm weight", torch.float32)
+        if (T1, T2, w2, cq_norm.numel()) != (T, T, q_rank, q_rank) or cq.dtype != some.dtype or cq_out.dtype != cq.dtype:
+            raise KernelError(f"latent prepare: query latent {tuple(cq.shape)}, output {tuple(cq_out.shape)}")
+    rot_dims, inter, freq, freq_lo = 0, False, None, None
+    if rotary is not None and rotary.rotary_dim:
+        rot_dims, inter, freq, freq_lo = rotary.rotary_dim, rotary.interleaved, rotary.freq, rotary.freq_lo
+        _need(freq, "rotary frequencies", torch.float32)
+        if freq.numel() != rot_dims // 2 or rotary.magnitude != 1.0:
+            raise KernelError("latent prepare: one frequency per rotated pair is needed, and no factor on cosines and sines")
     _check(
-        _lib().ferris_latent_prepare(_ptr(proj), _c_int(ld), _c_int(_dt(proj, "latent prepare")), _c_int(q_off),
-                                     _c_int(dkv_off), _ptr(norm_weight), _c_float(eps), _ptr(positions), _ptr(inv_freq),
-                                     _c_int(rot_dims), _ptr(slot_mapping if write_kv else None),
-                                     _ptr(cache if write_kv else None), _ptr(q_att), _c_int(ldqa), _c_int(T), _c_int(heads),
-                                     _c_int(dim), _c_int(rot), _c_int(rank), _c_int(1 if write_kv else 0), _stream()),
+        _lib().ferris_latent_prepare(_ptr(q), _c_int(ldq), _ptr(dkv), _c_int(lddkv), _c_int(_dt(some, "latent prepare")),
+                                     _ptr(norm_w), _c_float(eps), _ptr(positions), _ptr(freq), _ptr(freq_lo), _c_int(rot_dims),
+                                     _c_int(1 if inter else 0), _ptr(slots), _ptr(cache), _ptr(q_att), _c_int(ldqa), _ptr(cq),
+                                     _c_int(ldcq), _ptr(cq_norm), _ptr(cq_out), _c_int(ldco), _c_int(q_rank), _c_int(T),
+                                     _c_int(heads), _c_int(dim), _c_int(rot), _c_int(rank), _stream()),
         "latent prepare",
     )
 
@@ -1715,7 +1765,8 @@ def qk_norm_rotary_cache_write(qkv: torch.Tensor, ctx, slot_mapping: Optional[to
             _ptr(k_cache if write_kv else None), _ptr(v_cache if write_kv else None), _c_int(T), _c_int(num_heads),
             _c_int(num_kv_heads), _c_int(head_dim), _c_int(v_head_dim), _c_int(page_size), _ptr(q_norm), _ptr(k_norm),
             _c_float(eps), freq, rdim, inter, mag, _c_int(1 if values_from_keys else 0), _c_int(1 if write_kv else 0),
-            _ptr(mixed_values), _ptr(mix_lambda), *pool_args, _stream()),
+            _ptr(mixed_values), _ptr(mix_lambda), *pool_args,
+            _ptr(rotary.freq_lo if rotary is not None and rotary.rotary_dim else None), _stream()),
         "qk norm + rotation + cache write",
     )
 
@@ -1808,10 +1859,13 @@ def moe_leaves_apart(tokens: int, top: int, width: int, ff: int, x: torch.Tensor
     return 1 < tokens * top <= MOE_FEW_MAX_PAIRS and width % 4 == 0 and max(width, ff) <= MOE_FEW_MAX_WIDTH
 
 
+PLAIN_ACTIVATIONS = {"silu": 2, "relu2": 3}  # of experts without a gate
+
+
 def moe_experts(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor,
                 h: Optional[torch.Tensor], workspace=None, accumulate: bool = True, grouped: Optional[bool] = None,
                 activation: str = "silu", limit: float = 0.0, identity_w: Optional[torch.Tensor] = None,
-                input_weights: bool = False):
+                input_weights: bool = False, plain: bool = False):
     """h (+)= sum over a row's chosen experts of weight x down_e (silu(gate_e x) * (up_e x)).  gate_up [E, 2 ff, W] (an
     expert's gate rows, then its up rows), down [E, W, ff] in x's type; ids int32 and weights fp32 [T, top]; h fp32
     [T, W].  Steps of few tokens (up to MOE_FEW_MAX_PAIRS choices): a block per (expert, slab of rows) reads the weights
@@ -1822,11 +1876,13 @@ def moe_experts(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, ids:
     ``identity_w`` fp32 [T]: ids may then hold E, an expert that meets no weights, and h also gets identity_w[t] x[t].
     ``input_weights``: a token's weight for an expert goes onto the expert's input (both first products times the weight
     in fp32, ahead of the activation), and the results are added as they are.
+    ``plain``: the experts have no gate, down_e act(up_e x): gate_up is [E, ff, W], ``activation`` one of PLAIN_ACTIVATIONS.
     ``h`` None (where ``moe_leaves_apart``): the results are left apart and returned as ``PairRows``."""
     T, W, ldx = _rows(x, "experts input")
-    if activation not in GATED_ACTIVATIONS:
-        raise KernelError(f"experts: activation '{activation}' is not known ({', '.join(GATED_ACTIVATIONS)})")
-    act_kind = GATED_ACTIVATIONS[activation]
+    kinds = PLAIN_ACTIVATIONS if plain else GATED_ACTIVATIONS
+    if activation not in kinds:
+        raise KernelError(f"experts: activation '{activation}' is not known ({', '.join(kinds)})")
+    act_kind = kinds[activation]
     if identity_w is not None:
         _need(identity_w, "identity weights", torch.float32)
         if identity_w.numel() != T:
@@ -1836,9 +1892,9 @@ def moe_experts(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, ids:
     _need(down, "down matrices", x.dtype)
     _need(ids, "expert ids", torch.int32)
     _need(weights, "expert weights", torch.float32)
-    E, ff = gate_up.shape[0], gate_up.shape[1] // 2
+    E, ff = gate_up.shape[0], gate_up.shape[1] if plain else gate_up.shape[1] // 2
     top = ids.shape[1]
-    if (gate_up.shape != (E, 2 * ff, W) or down.shape != (E, W, ff) or (T2, W2) != (T, W) or (h is not None and h.dtype != torch.float32)
+    if (gate_up.shape != (E, ff if plain else 2 * ff, W) or down.shape != (E, W, ff) or (T2, W2) != (T, W) or (h is not None and h.dtype != torch.float32)
             or ids.shape != (T, top) or weights.shape != (T, top)):
         raise KernelError(f"experts: x {tuple(x.shape)}, gate/up {tuple(gate_up.shape)}, down {tuple(down.shape)}, "
                           f"ids {tuple(ids.shape)}")
@@ -1865,18 +1921,19 @@ def moe_experts(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, ids:
                                                  _ptr(h), _c_int(ldh), _c_int(T), _c_int(W), _c_int(ff), _c_int(top),
                                                  _c_int(E), _c_int(rows), _ptr(pos), _ptr(row_token), _ptr(tile_expert),
                                                  _ptr(xs), _ptr(act), _ptr(y), _c_int(1 if accumulate else 0),
-                                                 _c_int(act_kind), _c_float(limit), _ptr(identity_w), _ptr(row_scale), _stream()),
+                                                 _c_int(act_kind), _c_float(limit), _ptr(identity_w), _ptr(row_scale),
+                                                 _c_int(1 if plain else 0), _stream()),
                "experts (sorted)", 5 if h is not None else 4)
         return None if h is not None else PairRows(y, pos, None if input_weights else weights, top)
     act = get("moe_act", (T * top, ff), x.dtype)
-    up = gate_up[:, ff:, :]
+    gate, up = (None, gate_up) if plain else (gate_up, gate_up[:, ff:, :])
     # few pairs: the weights are read once per expert, the results of a pair stand in y until they are added
     few = 1 < T * top <= MOE_FEW_MAX_PAIRS and W % 4 == 0 and ldh % 4 == 0 and (h is None or h.data_ptr() % 16 == 0)
     if h is None and (identity_w is not None or not moe_leaves_apart(T, top, W, ff, x)):
         raise KernelError("experts: a step of this form adds its results itself")
     y = get("moe_pair_out", (T * top, W), torch.float32) if few else None
-    _check(_lib().ferris_moe_experts_token_major(_ptr(x), _c_int(ldx), _c_int(_dt(x, "experts")), _ptr(gate_up), _ptr(up),
-                                                 ctypes.c_longlong(2 * ff * W), _ptr(down), _ptr(ids), _ptr(weights),
+    _check(_lib().ferris_moe_experts_token_major(_ptr(x), _c_int(ldx), _c_int(_dt(x, "experts")), _ptr(gate), _ptr(up),
+                                                 ctypes.c_longlong((1 if plain else 2) * ff * W), _ptr(down), _ptr(ids), _ptr(weights),
                                                  _ptr(act), _ptr(h), _c_int(ldh), _c_int(T), _c_int(W), _c_int(ff),
                                                  _c_int(top), _c_int(1 if accumulate else 0),
                                                  _ptr(y) if few else ctypes.c_void_p(0), _c_int(E), _c_int(act_kind),
@@ -2037,9 +2094,9 @@ def attention_step(qkv, out, k_cache, v_cache, meta, ctx, num_heads, num_kv_head
 
 def paged_attention(qkv, out, k_cache, v_cache, block_tables, ctx, num_heads, num_kv_heads, head_dim, window, scale,
                     score_slopes=None, v_head_dim: Optional[int] = None, values_in_keys: bool = False,
-                    chunk: int = 0, fp32_weights: bool = False, pooled: Optional[PooledKeys] = None):
+                    chunk: int = 0, fp32_weights: bool = False, pooled: Optional[PooledKeys] = None, keep_first: int = 0):
     """Attention of the step's tokens over the paged cache (their own keys are in it already).
-    ``chunk``, ``pooled``: see ``paged_attention_simt``.  ``fp32_weights``: the softmax's weights and the weighted sum stay in 32-bit
+    ``chunk``, ``pooled``, ``keep_first``: see ``paged_attention_simt``.  ``fp32_weights``: the softmax's weights and the weighted sum stay in 32-bit
     (the tensor-core kernels round the weights to bf16 for their second product), so the general kernel runs.
     ``ctx`` is the step context.  bf16 with head size 64 / 128 runs on the tensor cores: the split-KV
     kernel when every request brings one token, the prefill kernel otherwise; every other geometry, the
@@ -2048,11 +2105,11 @@ def paged_attention(qkv, out, k_cache, v_cache, block_tables, ctx, num_heads, nu
     _need(k_cache, "key cache", qkv.dtype)
     if isinstance(score_slopes, ScoreTerms) and not score_slopes.any():
         score_slopes = None
-    if values_in_keys or chunk or fp32_weights or pooled is not None or (v_head_dim is not None and v_head_dim != head_dim):
+    if values_in_keys or chunk or fp32_weights or pooled is not None or keep_first or (v_head_dim is not None and v_head_dim != head_dim):
         paged_attention_simt(qkv, out, k_cache, v_cache, block_tables, ctx.token_seq, ctx.positions, num_heads,
                              num_kv_heads, head_dim, window, scale, score_slopes=score_slopes, v_head_dim=v_head_dim,
                              max_q_len=ctx.max_q_len, max_kv_len=ctx.max_kv_len, workspace=ctx.workspace,
-                             values_in_keys=values_in_keys, chunk=chunk, pooled=pooled)
+                             values_in_keys=values_in_keys, chunk=chunk, pooled=pooled, keep_first=keep_first)
         return
     _need(v_cache, "value cache", qkv.dtype)
     _need(block_tables, "block tables", torch.int32)

@@ -31,7 +31,8 @@ Options beyond the reference's layer, each a parameter of its own:
   ``output_gate``       {"name", "kind"}: a matrix [heads x v_head_dim, H] named ``name`` under the prefix, held as further
                         rows of the fused input matrix; the heads side by side are multiplied element by element by
                         sigmoid ("sigmoid") or SiLU ("silu") of that projection of the mixer's input before the output
-                        product
+                        product; with "per_head": True a matrix [heads, H], one number per head, whose sigmoid multiplies
+                        the head where the attention kernel stores it
   ``output_scale``      a factor on the mixer's result (applied to the rows that enter the output product)
   ``chunk``             instead of a window: positions are counted off in chunks of that many from 0, and a token
                         sees the keys of its own chunk up to itself
@@ -39,6 +40,8 @@ Options beyond the reference's layer, each a parameter of its own:
                         positions (counted off from 0) that lies wholly before the window: the means of the run's keys
                         and values as the cache holds them, kept in pages of their own (one row a run), in one softmax
                         with the tokens
+  ``keep_first``        (with a window) the request's first so many tokens stay visible whatever the window has passed
+  ``softcap``           a scaled product x of query and key becomes softcap * tanh(x / softcap)
   ``value_mix``         {"lambda": tensor name, "role": "source" or "mix"}: a layer with "mix" stores (1 - lambda) v +
                         lambda v1 as its values, v1 being the values that the layer with "source" projected for the same
                         token in this pass; the source's own number is read if the folder has it, and not used
@@ -61,6 +64,7 @@ import torch
 from ..kernels import ops
 from .base import CombinedNeed, LayerCache, Mixer, PagedKV, PositionEncoding, TensorSpec
 from .plan import PartSpec, build_part, register_part
+from .recurrent import _fused_rows
 
 
 class GroupedQueryAttention(Mixer):
@@ -79,7 +83,8 @@ class GroupedQueryAttention(Mixer):
                  bias_names: Optional[dict] = None, sink_name: Optional[str] = None,
                  values_from_keys: bool = False, qk_norm: Optional[dict] = None, chunk: Optional[int] = None,
                  fp32_weights: bool = False, output_gate: Optional[dict] = None, output_scale: float = 1.0,
-                 pool: Optional[int] = None, value_mix: Optional[dict] = None):
+                 pool: Optional[int] = None, value_mix: Optional[dict] = None, keep_first: int = 0,
+                 softcap: Optional[float] = None):
         if num_heads % num_kv_heads:
             raise ValueError(f"{num_heads} heads cannot share {num_kv_heads} kv heads")
         self.hidden_size, self.num_heads = int(hidden_size), int(num_heads)
@@ -110,6 +115,12 @@ class GroupedQueryAttention(Mixer):
         self.pool = None if pool is None else int(pool)
         if self.pool is not None and (self.pool <= 0 or not self.window or self.window < 0):
             raise ValueError(f"pooled runs of {pool} positions stand before a window ({window})")
+        self.keep_first = int(keep_first or 0)
+        if self.keep_first < 0 or (self.keep_first and (not self.window or self.window < 0 or self.pool is not None)):
+            raise ValueError(f"{keep_first} kept tokens stand before a window ({window}) without pooled runs")
+        self.softcap = float(softcap or 0.0)
+        if self.softcap < 0.0:
+            raise ValueError(f"a soft cap of {softcap} on the scores: a positive number is needed")
         self.value_mix = None
         if value_mix is not None:
             self.value_mix = (value_mix["lambda"], value_mix["role"])
@@ -122,19 +133,24 @@ class GroupedQueryAttention(Mixer):
         if self.pool is not None and (type(self.position).score_slopes is not PositionEncoding.score_slopes
                                       or type(self.position).score_log_penalty is not PositionEncoding.score_log_penalty):
             raise ValueError("pooled runs go with no distance penalty: a run has no distance of its own")
-        self.output_gate = None
+        self.output_gate, self.gate_per_head = None, False
         if output_gate is not None:
             self.output_gate = (output_gate["name"], output_gate.get("kind", "sigmoid"))
             if self.output_gate[1] not in ("sigmoid", "silu"):
                 raise ValueError(f"output gate '{self.output_gate[1]}' is not known (sigmoid, silu)")
+            self.gate_per_head = bool(output_gate.get("per_head", False))
+            if self.gate_per_head and self.output_gate[1] != "sigmoid":
+                raise ValueError("a gate per head is a sigmoid")
         self.output_scale = float(output_scale)
-        if self.output_scale != 1.0 and self.output_gate is None:
-            raise ValueError("a factor on the attention's result rides in the kernel of its output gate: it needs one")
+        if self.output_scale != 1.0 and (self.output_gate is None or self.gate_per_head):
+            raise ValueError("a factor on the attention's result rides in the kernel of its output gate: it needs one "
+                             "(element by element)")
         self.q_norm_weight = self.k_norm_weight = None
         self.q_size = self.num_heads * self.head_dim
         self.kv_size = self.num_kv_heads * self.head_dim
         self.v_size = 0 if self.values_from_keys else self.num_kv_heads * self.v_head_dim
         self.o_size = self.num_heads * self.v_head_dim
+        self.gate_size = 0 if self.output_gate is None else (self.num_heads if self.gate_per_head else self.o_size)
         # the plain layer (the reference's) keeps its fused kernels; any option sends the step the general way
         self.sink_name, self.sink = sink_name, None
         # norm over the whole projection, rotation of either layout and the cache write are one kernel of their own
@@ -145,7 +161,7 @@ class GroupedQueryAttention(Mixer):
         self.plain = (self.v_head_dim == self.head_dim and self.qk_unit_norm_eps is None
                       and self.output_gate is None and self.output_scale == 1.0
                       and self.query_temperature is None and sink_name is None and not self.rotary_prepare
-                      and self.chunk is None and not self.fp32_weights
+                      and self.chunk is None and not self.fp32_weights and not self.keep_first and not self.softcap
                       and not getattr(self.position, "learned_scores", False))
         if not self.plain and not hasattr(self.position, "table") and getattr(self.position, "rotary_dim", 0):
             raise ValueError("unit-norm keys, a query temperature or value heads of their own size go with a "
@@ -173,7 +189,7 @@ class GroupedQueryAttention(Mixer):
             specs += [TensorSpec(f"{prefix}.{self.qk_norm[1]}", (nq,), "norm"),
                       TensorSpec(f"{prefix}.{self.qk_norm[2]}", (nk,), "norm")]
         if self.output_gate is not None:
-            specs.append(TensorSpec(f"{prefix}.{self.output_gate[0]}", (self.o_size, H), "matrix"))
+            specs.append(TensorSpec(f"{prefix}.{self.output_gate[0]}", (self.gate_size, H), "matrix"))
         if self.bias_names:
             specs += [TensorSpec(f"{prefix}.{self.bias_names[n]}", (size,), "bias")
                       for n, size in zip(self._inputs, (Q, KV, self.v_size))]
@@ -199,7 +215,8 @@ class GroupedQueryAttention(Mixer):
         w = [tensors.pop(self._matrix_name(prefix, n)) for n in self._inputs]
         if self.output_gate is not None:  # the gate's projection rides in the same product
             w.append(tensors.pop(f"{prefix}.{self.output_gate[0]}"))
-        self.qkv_weight = torch.cat(w, dim=0).contiguous()
+        # (a gate of one number per head may leave the rows of the product's output off 16 bytes: filled up with zero rows)
+        self.qkv_weight = _fused_rows(w) if self.gate_per_head else torch.cat(w, dim=0).contiguous()
         if self.bias_names:
             biases = [tensors.pop(f"{prefix}.{self.bias_names[n]}") for n in self._inputs]
         else:
@@ -215,7 +232,7 @@ class GroupedQueryAttention(Mixer):
         if any(b is not None for b in biases):
             sizes = (self.q_size, self.kv_size, self.v_size)[:len(biases)]
             if self.output_gate is not None:
-                biases, sizes = biases + [None], sizes + (self.o_size,)
+                biases, sizes = biases + [None], sizes + (self.qkv_weight.shape[0] - sum(sizes),)
             parts = [
                 b if b is not None else torch.zeros(n, dtype=torch.float32, device=self.qkv_weight.device)
                 for b, n in zip(biases, sizes)
@@ -228,7 +245,8 @@ class GroupedQueryAttention(Mixer):
     # -------------------------------------------------------------------- cache
     def cache_need(self):
         dv = None if self.v_head_dim == self.head_dim else self.v_head_dim
-        need = PagedKV(self.num_kv_heads, self.head_dim, self.window, dv, chunk=self.chunk, run=self.pool)
+        need = PagedKV(self.num_kv_heads, self.head_dim, self.window, dv, chunk=self.chunk, run=self.pool,
+                       keep_first=self.keep_first)
         if self.pool is None:
             return need
         return CombinedNeed((need, PagedKV(self.num_kv_heads, self.head_dim, None, dv, stride=self.pool)))
@@ -250,7 +268,7 @@ class GroupedQueryAttention(Mixer):
             ops.gemm(x, self.qkv_weight, self.qkv_bias, qkv)
             gate = None
             if self.output_gate is not None:
-                qkv, gate = qkv[:, :n_qkv], qkv[:, n_qkv:]
+                qkv, gate = qkv[:, :n_qkv], qkv[:, n_qkv:n_qkv + self.gate_size]
             if self.rotary_prepare:
                 rotary = self.position.table(qkv.device) if hasattr(self.position, "table") else None
                 extra = {}
@@ -272,11 +290,12 @@ class GroupedQueryAttention(Mixer):
             out = ctx.workspace.get("attn_out", (T, self.o_size), x.dtype)
             log = self.position.score_log_penalty(nh, qkv.device)
             terms = ops.ScoreTerms(slopes=self.position.score_slopes(nh, qkv.device), sink=self.sink,
-                                   log_r1=None if log is None else log[0], log_r2=None if log is None else log[1])
+                                   log_r1=None if log is None else log[0], log_r2=None if log is None else log[1],
+                                   softcap=self.softcap, gate=gate if self.gate_per_head else None)
             ops.paged_attention(qkv, out, cache.k, cache.v, meta.block_tables, ctx, nh, nkv, d, self.window or 0,
                                 self.scale, score_slopes=terms, v_head_dim=dv, chunk=self.chunk or 0,
-                                fp32_weights=self.fp32_weights, pooled=pooled)
-            if gate is not None:
+                                fp32_weights=self.fp32_weights, pooled=pooled, keep_first=self.keep_first)
+            if gate is not None and not self.gate_per_head:
                 ops.gate_mul(out, gate, out, self.output_gate[1], self.output_scale)
             ops.gemm(out, self.o_weight, None, h, accumulate=accumulate)
             return

@@ -32,6 +32,8 @@ class PagedKV:
     kept, for a mixer whose keys carry their values).
     ``run`` (with ``window``): positions are counted off in runs of that many from 0, and the pages of a run that is not
     complete yet stay although the window may have passed its first positions (its rows are pooled when it is complete).
+    ``keep_first`` (with ``window``): the request's first so many tokens stay readable whatever the window has passed, so their
+    pages stay until the request ends.
     ``stride``: one row for every ``stride`` WHOLE tokens instead of one per token: row r stands for the tokens
     r * stride .. r * stride + stride - 1 and exists once the last of them is in the cache."""
 
@@ -42,9 +44,10 @@ class PagedKV:
     chunk: Optional[int] = None
     run: Optional[int] = None
     stride: int = 1
+    keep_first: int = 0
 
     def first_needed(self, num_tokens: int) -> int:
-        """The lowest row that a query at position ``num_tokens`` or later can still read."""
+        """The lowest row beyond the kept first ones that a query at position ``num_tokens`` or later can still read."""
         if self.chunk is not None:
             return num_tokens - num_tokens % self.chunk
         if self.window is not None:
@@ -62,7 +65,7 @@ class PagedKV:
         if self.chunk is not None:
             return self.chunk
         if self.window is not None:
-            return self.window if self.run is None else max(self.window, self.run)
+            return self.keep_first + (self.window if self.run is None else max(self.window, self.run))
         return None
 
     @property

@@ -6,7 +6,8 @@ The pre-norm residual block, one branch after the other:
 
 The parallel block, both branches from the same h:
   h += mixer(norm_1(h)) + feed_forward(norm_2(h))
-Both norms are taken before either branch adds, into buffers of their own.  A layer may have no feed-forward.
+Both norms are taken before either branch adds, into buffers of their own.  A layer may have no feed-forward.  Without a
+second norm both branches read the first one's rows: h += mixer(norm(h)) + feed_forward(norm(h)).
 
 The sums are made in the fp32 residual stream by the last matrix product of each branch.
 
@@ -26,6 +27,8 @@ from .plan import build_part, register_part
 
 
 class PreNormResidualBlock(Block):
+    shares_norm = False  # whether a feed-forward without a norm of its own reads the mixer's
+
     def __init__(self, hidden_size: int, mixer, feed_forward, mixer_norm, feed_forward_norm,
                  mixer_prefix: str = "self_attn", feed_forward_prefix: str = "mlp",
                  mixer_norm_prefix: str = "input_layernorm",
@@ -33,6 +36,8 @@ class PreNormResidualBlock(Block):
         self.hidden_size = int(hidden_size)
         self.mixer, self.feed_forward = mixer, feed_forward
         self.mixer_norm, self.feed_forward_norm = mixer_norm, feed_forward_norm
+        if feed_forward is not None and feed_forward_norm is None and not self.shares_norm:
+            raise ValueError("the layer's feed-forward has no norm of its own")
         self._names = (mixer_prefix, feed_forward_prefix, mixer_norm_prefix, feed_forward_norm_prefix)
 
     def _children(self, prefix):
@@ -83,7 +88,10 @@ class PreNormResidualBlock(Block):
 
 class ParallelResidualBlock(PreNormResidualBlock):
     """h += mixer(norm_1(h)) + feed_forward(norm_2(h)); ``feed_forward`` None: the mixer's branch alone (the
-    second norm's tensor is then read if the folder has it, and not used)."""
+    second norm's tensor is then read if the folder has it, and not used); ``feed_forward_norm`` None: both branches read
+    norm_1(h)."""
+
+    shares_norm = True
 
     def __init__(self, hidden_size: int, mixer, feed_forward, mixer_norm, feed_forward_norm,
                  mixer_prefix: str = "mix", feed_forward_prefix: str = "mlp", mixer_norm_prefix: str = "norm1",
@@ -120,7 +128,8 @@ class ParallelResidualBlock(PreNormResidualBlock):
     def forward(self, h, ctx, cache, owns_cache):
         T = h.shape[0]
         x1 = ctx.workspace.get("block_normed", (T, self.hidden_size), ctx.act_dtype)
-        if self.feed_forward is None:
+        x2 = x1
+        if self.feed_forward is None or self.feed_forward_norm is None:
             self.mixer_norm.forward(h, x1)
         else:
             x2 = ctx.workspace.get("block_normed_2", (T, self.hidden_size), ctx.act_dtype)
@@ -137,6 +146,7 @@ class OutputNormBlock(ParallelResidualBlock):
     """h += norm_1(mixer(h)); h += norm_2(feed_forward(h)); ``feed_forward`` None: the mixer's half alone (the second norm's
     tensor is then read if the folder has it, and not used)."""
 
+    shares_norm = False
     keeps_rows = True
 
     @staticmethod

@@ -1,5 +1,5 @@
 """Feed-forwards as parts: the gated SiLU one (SwiGLU), a plain one with a choice of activation, and a mixture of
-gated SiLU experts of which every token uses a few.
+experts (gated or plain) of which every token uses a few.
 
   u = y W_up^T;  g = y W_gate^T;  m = u * (g * sigmoid(g));  h += m W_down^T
 (crates/ferrisinfer-runtime/src/reference.rs:346-368; the reference's w1 is up_proj and w3 is
@@ -149,7 +149,8 @@ class MixtureOfExperts(FeedForward):
 
     ``sigmoid_scores``: the weights are the sigmoids of the chosen outputs, as they are (not with ``scored``).
     ``input_weights``: a weight multiplies its expert's input instead of its result: out = sum_e expert_e(weight_e y).
-    ``router_bias_name`` None: the router has no bias."""
+    ``router_bias_name`` None: the router has no bias.
+    ``gated`` False: an expert is W_down_e a(W_up_e y) without a gate, ``activation`` one of ``ops.PLAIN_ACTIVATIONS``."""
 
     graph_safe = True
     can_overwrite = True
@@ -158,7 +159,7 @@ class MixtureOfExperts(FeedForward):
                  router_bias_name: Optional[str] = "router.b", expert_prefix: str = "e", gate_name: str = "gate",
                  up_name: str = "up", down_name: str = "down", scored: dict = None, identity: int = 0,
                  activation: str = "silu", limit: float = 0.0, sigmoid_scores: bool = False,
-                 input_weights: bool = False):
+                 input_weights: bool = False, gated: bool = True):
         self.hidden_size, self.intermediate_size = int(hidden_size), int(intermediate_size)
         self.sigmoid_scores, self.input_weights = bool(sigmoid_scores), bool(input_weights)
         if self.sigmoid_scores and scored is not None:
@@ -169,8 +170,10 @@ class MixtureOfExperts(FeedForward):
         self.outputs = self.experts + self.identity  # of the router
         if not (1 <= self.top <= self.outputs) or self.identity < 0:
             raise ValueError(f"{self.top} of {self.experts} + {self.identity} experts cannot be chosen")
-        if activation not in ops.GATED_ACTIVATIONS:
-            raise ValueError(f"gated activation '{activation}' is not known ({', '.join(ops.GATED_ACTIVATIONS)})")
+        self.gated = bool(gated)
+        kinds = ops.GATED_ACTIVATIONS if self.gated else ops.PLAIN_ACTIVATIONS
+        if activation not in kinds:
+            raise ValueError(f"experts' activation '{activation}' is not known ({', '.join(kinds)})")
         self.activation, self.limit = activation, float(limit)
         self.scored = None
         if scored is not None:
@@ -192,8 +195,9 @@ class MixtureOfExperts(FeedForward):
         r, rb, _, g, u, d = self._names
         specs = []
         for e in range(self.experts):
-            specs += [TensorSpec(self._expert(prefix, e, g), (I, H), "matrix"),
-                      TensorSpec(self._expert(prefix, e, u), (I, H), "matrix"),
+            if self.gated:
+                specs.append(TensorSpec(self._expert(prefix, e, g), (I, H), "matrix"))
+            specs += [TensorSpec(self._expert(prefix, e, u), (I, H), "matrix"),
                       TensorSpec(self._expert(prefix, e, d), (H, I), "matrix")]
         if self.scored is not None:
             specs.append(TensorSpec(f"{prefix}.{r}", (self.outputs, H), "matrix"))
@@ -206,7 +210,8 @@ class MixtureOfExperts(FeedForward):
     def bind(self, tensors, prefix):
         r, rb, _, g, u, d = self._names
         if self.experts:
-            self.gate_up = torch.stack([torch.cat([tensors.pop(self._expert(prefix, e, g)), tensors.pop(self._expert(prefix, e, u))])
+            names = (g, u) if self.gated else (u,)
+            self.gate_up = torch.stack([torch.cat([tensors.pop(self._expert(prefix, e, n)) for n in names])
                                         for e in range(self.experts)]).contiguous()
             self.down = torch.stack([tensors.pop(self._expert(prefix, e, d)) for e in range(self.experts)]).contiguous()
         self.router = tensors[f"{prefix}.{r}"]
@@ -217,7 +222,7 @@ class MixtureOfExperts(FeedForward):
             self.router_bias = tensors[f"{prefix}.{rb}"] if rb else None
         if self.experts == 0:  # identity experts only: the kernels still want matrices to point at
             W, I = self.hidden_size, self.intermediate_size
-            self.gate_up = self.router.new_zeros(1, 2 * I, W)
+            self.gate_up = self.router.new_zeros(1, (2 if self.gated else 1) * I, W)
             self.down = self.router.new_zeros(1, W, I)
 
     def forward(self, x, h, ctx, accumulate: bool = True):
@@ -241,7 +246,8 @@ class MixtureOfExperts(FeedForward):
             return None
         ops.moe_router(x, self.router, self.router_bias, ids, weights, self.top, scored=scored, sigmoid=self.sigmoid_scores)
         return ops.moe_experts(x, self.gate_up, self.down, ids, weights, h, ctx.workspace, accumulate=accumulate,
-                               activation=self.activation, limit=self.limit, identity_w=identity_w, input_weights=self.input_weights)
+                               activation=self.activation, limit=self.limit, identity_w=identity_w, input_weights=self.input_weights,
+                               plain=not self.gated)
 
 
 register_part("feed_forward", "swiglu", SwiGLU)

@@ -32,8 +32,8 @@ class DecoderModel:
         self.final_norm = build_part("norm", plan.final_norm)
         self.output = build_part("output", plan.output)
         self.bound = False
-        # a callable (run-order index, residual stream) that sees the residual stream after every run of a layer:
-        # for tests and debugging; a model with one is stepped without graphs
+        # a callable (run-order index, residual stream) that sees the residual stream after every run of a layer (in the
+        # model's own units): for tests and debugging; a model with one is stepped without graphs
         self.after_run = None
 
     def _build_layer(self, lp: LayerPlan):
@@ -43,7 +43,7 @@ class DecoderModel:
             mixer=build_part("mixer", lp.mixer),
             feed_forward=None if lp.feed_forward is None else build_part("feed_forward", lp.feed_forward),
             mixer_norm=build_part("norm", lp.mixer_norm),
-            feed_forward_norm=build_part("norm", lp.feed_forward_norm),
+            feed_forward_norm=None if lp.feed_forward_norm is None else build_part("norm", lp.feed_forward_norm),
         )
 
     @property
@@ -125,7 +125,7 @@ class DecoderModel:
                 flush_pending_write(ctx, h, S)
                 if S > 1:
                     ops.streams_sum(h, row, S)
-                self.after_run(i, row)
+                self.after_run(i, row if self.plan.residual_unit == 1.0 else row * self.plan.residual_unit)
         flush_pending_write(ctx, h, S)  # what the last layer of a block kind over residual streams left undone
         if logits_index is None or logits_index.numel() == 0:
             return None

@@ -49,13 +49,13 @@ class TensorSpec:
 @dataclass(frozen=True)
 class LayerPlan:
     """One layer: a block kind wiring two norms, a mixer and a feed-forward (None: the layer has none, where
-    its block kind allows that)."""
+    its block kind allows that; ``feed_forward_norm`` None: both read the mixer's norm, where the block kind allows that)."""
 
     prefix: str  # tensor-name prefix, e.g. "model.layers.3"
     mixer: PartSpec
     feed_forward: Optional[PartSpec]
     mixer_norm: PartSpec
-    feed_forward_norm: PartSpec
+    feed_forward_norm: Optional[PartSpec]
     block: PartSpec = PartSpec("pre_norm_residual")
 
 
@@ -95,10 +95,16 @@ class ModelPlan:
     residual_streams: int = 1
     # True where positions index a table of max_positions rows: no request may grow beyond it, whatever the engine allows
     positions_bounded: bool = False
+    # The residual stream is held divided by this number.  A model that adds m times its sublayers' results, x <- x + m y, is
+    # run as x / m <- x / m + y: the plan's embedding is divided by m, and a norm over x / m with eps / m^2 is the norm over x
+    # with eps, so the factor costs nothing and no weight is rounded again.
+    residual_unit: float = 1.0
 
     def validate(self) -> None:
         if self.residual_streams < 1:
             raise ValueError(f"{self.residual_streams} residual streams")
+        if not self.residual_unit > 0.0:
+            raise ValueError(f"a residual stream held in units of {self.residual_unit}")
         if self.residual_streams > 1 and any(step.add_embedding for step in self.run_order):
             raise ValueError("adding the embedding output again is not defined over several residual streams")
         for i, step in enumerate(self.run_order):

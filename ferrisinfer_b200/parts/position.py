@@ -13,7 +13,10 @@ are fp32, formed in the kernel that also writes the cache.
 ("half") or (2i, 2i + 1) ("interleaved"), optionally with YaRN scaling: with c(r) = rotary_dim ln(original / (2 pi r)) /
 (2 ln base), lo = max(floor(c(fast)), 0), hi = min(ceil(c(slow)), rotary_dim - 1) and ramp_i = clamp((i - lo) /
 max(hi - lo, 0.001), 0, 1), frequency i becomes f_i / factor * ramp_i + f_i (1 - ramp_i), and every cosine and sine is
-multiplied by 0.1 ln(factor) + 1.  It is applied by the kernel that prepares a mixer's queries and keys.
+multiplied by 0.1 ln(factor) + 1; or with a scaling by wavelength (``kind`` "wavelength", as Llama 3.1 has it): with
+w_i = 2 pi / f_i a frequency stays where w_i < original / high, becomes f_i / factor where w_i > original / low, and between
+the two (1 - s) f_i / factor + s f_i with s = (original / w_i - low) / (high - low); cosines and sines as they are.  It is
+applied by the kernel that prepares a mixer's queries and keys.
 
 ``NoPosition``: nothing is encoded (the keys go to the cache as they are).
 
@@ -80,7 +83,8 @@ class ScaledRotary(PositionEncoding):
     graph_safe = True
 
     def __init__(self, rotary_dim: int, base: float, layout: str = "half", scaling: dict = None):
-        """``scaling``: None, or the four numbers ``factor``, ``original``, ``fast``, ``slow`` of a YaRN scaling."""
+        """``scaling``: None, the four numbers ``factor``, ``original``, ``fast``, ``slow`` of a YaRN scaling, or with ``kind``
+        "wavelength" the four numbers ``factor``, ``original``, ``low``, ``high``."""
         if layout not in ("half", "interleaved"):
             raise ValueError(f"rotary layout '{layout}' is not known (half, interleaved)")
         if rotary_dim < 0 or rotary_dim % 2:
@@ -90,7 +94,22 @@ class ScaledRotary(PositionEncoding):
         R = self.rotary_dim
         freq = [self.base ** (-2.0 * i / R) for i in range(R // 2)]
         self.magnitude = 1.0
-        if self.scaling and R:
+        kind = self.scaling.get("kind", "yarn") if self.scaling else None
+        if kind not in (None, "yarn", "wavelength"):
+            raise ValueError(f"rotary scaling '{kind}' is not known (yarn, wavelength)")
+        if kind == "wavelength":
+            factor, original = float(self.scaling["factor"]), float(self.scaling["original"])
+            low, high = float(self.scaling["low"]), float(self.scaling["high"])
+            if factor <= 0 or original <= 0 or low <= 0 or high <= 0 or self.base <= 0:
+                raise ValueError(f"rotary scaling {self.scaling} with base {self.base}: positive numbers are needed")
+            for i, f in enumerate(freq):
+                wave = 2.0 * math.pi / f
+                if wave > original / low:
+                    freq[i] = f / factor
+                elif wave >= original / high and high != low:
+                    s = (original / wave - low) / (high - low)
+                    freq[i] = (1.0 - s) * f / factor + s * f
+        elif kind == "yarn" and R:
             factor, original = float(self.scaling["factor"]), float(self.scaling["original"])
             fast, slow = float(self.scaling["fast"]), float(self.scaling["slow"])
             if factor <= 0 or original <= 0 or fast <= 0 or slow <= 0 or self.base <= 1.0:

@@ -7,6 +7,11 @@
     S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q          (the read-out sees the token's own write)
   h += (rmsnorm_per_head(o) * n * SiLU(y Wg^T)) Wo^T,   n of size vdim, shared by the heads.
 
+``ChannelDeltaRule``: the same rule with a decay per key channel and low-rank projections for the decay and the output gate:
+    z = (y Wa1^T) Wa2^T + dt_bias, heads x dim;  g = exp(-exp(A_log_h) softplus(z)) acts on the rows of S one by one;
+    S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
+  h += (rmsnorm_per_head(o) * n * sigmoid((y Wg1^T) Wg2^T)) Wo^T,   n of size vdim, shared by the heads.
+
 ``StateSpaceDuality`` (a selective state-space layer in its attention-like reading):
   y W_in^T = [z: inner | x: inner | B: groups x N | C: groups x N | dt: heads], inner = heads x vdim;
   x, B, C = SiLU(conv(.) + bias);  dt = softplus(dt + dt_bias);  per head (group h / (heads / groups)):
@@ -47,6 +52,30 @@ def _fused_rows(parts: list) -> torch.Tensor:
     if pad:
         w = torch.cat([w, torch.zeros(pad, w.shape[1], dtype=w.dtype, device=w.device)], dim=0)
     return w.contiguous()
+
+
+def _fused_parts(parts: list) -> tuple:
+    """(matrix, first rows): the matrices one below the other, each filled up with zero rows to a multiple of eight, so that
+    every part's columns of the product's output start on 16 bytes in either type."""
+    rows, offsets = [], []
+    at = 0
+    for p in parts:
+        offsets.append(at)
+        rows.append(_fused_rows([p]))
+        at += rows[-1].shape[0]
+    return torch.cat(rows, dim=0).contiguous(), offsets
+
+
+def _low_rank(first: torch.Tensor, second: torch.Tensor, where: str) -> tuple:
+    """The two matrices of a low-rank projection, W2 (W1 y), with zero rows of the first and zero columns of the second that
+    make the inner size a multiple of eight."""
+    if first.shape[0] != second.shape[1]:
+        raise ValueError(f"{where}: the two matrices do not meet ({tuple(first.shape)} and {tuple(second.shape)})")
+    pad = (-first.shape[0]) % 8
+    if pad:
+        first = torch.cat([first, first.new_zeros(pad, first.shape[1])], dim=0)
+        second = torch.cat([second, second.new_zeros(second.shape[0], pad)], dim=1)
+    return first, second.contiguous()
 
 
 class GatedDeltaRule(Mixer):
@@ -116,6 +145,69 @@ class GatedDeltaRule(Mixer):
                              delta_rule=True, qscale=qscale, kscale=kscale, write_state=owns_cache)
         y = ws.get("recurrent_gated", (T, V), ctx.act_dtype)
         ops.gated_group_norm(o, proj[:, C:C + V], self.norm_weight, self.norm_eps, y, group=dv, gate_kind="silu")
+        ops.gemm(y, self.o_weight, None, h, accumulate=accumulate)
+
+
+class ChannelDeltaRule(GatedDeltaRule):
+    """The inner sizes of the two low-rank projections stand in no configuration key: the folder's tensors decide (a random
+    folder draws 16)."""
+
+    def tensor_specs(self, prefix):
+        H, nh = self.hidden_size, self.num_heads
+        channels = nh * self.head_dim
+        specs = []
+        for n, size in (("q", self.qk_size), ("k", self.qk_size), ("v", self.v_size)):
+            specs += [TensorSpec(f"{prefix}.{n}", (size, H), "matrix"),
+                      TensorSpec(f"{prefix}.{n}.conv", (size, self.taps), "vector")]
+        return specs + [
+            TensorSpec(f"{prefix}.b", (nh, H), "matrix"),
+            TensorSpec(f"{prefix}.A_log", (nh,), "vector"),
+            TensorSpec(f"{prefix}.norm", (self.v_head_dim,), "norm"),
+            TensorSpec(f"{prefix}.a1", (-16, H), "matrix"),
+            TensorSpec(f"{prefix}.a2", (channels, -16), "matrix"),
+            TensorSpec(f"{prefix}.dt_bias", (channels,), "vector"),
+            TensorSpec(f"{prefix}.g1", (-16, H), "matrix"),
+            TensorSpec(f"{prefix}.g2", (self.v_size, -16), "matrix"),
+            TensorSpec(f"{prefix}.o", (H, self.v_size), "matrix"),
+        ]
+
+    def bind(self, tensors, prefix):
+        pop = lambda n: tensors.pop(f"{prefix}.{n}")
+        a1, self.a2 = _low_rank(pop("a1"), pop("a2"), f"{prefix}: decay")
+        g1, self.g2 = _low_rank(pop("g1"), pop("g2"), f"{prefix}: output gate")
+        # one product: [q | k | v | beta | the two low-rank inputs]
+        qkv = torch.cat([pop("q"), pop("k"), pop("v")], dim=0)
+        self.in_weight, (_, self.b_off, self.a_off, self.g_off) = _fused_parts([qkv, pop("b"), a1, g1])
+        self.conv_weight = torch.cat([pop(f"{n}.conv") for n in "qkv"], dim=0).contiguous()
+        # exp of a head's parameter, formed once in 64-bit and rounded once
+        self.rates = torch.exp(tensors[f"{prefix}.A_log"].to(torch.float64)).to(torch.float32).contiguous()
+        self.dt_bias = tensors[f"{prefix}.dt_bias"]
+        self.norm_weight, self.o_weight = tensors[f"{prefix}.norm"], tensors[f"{prefix}.o"]
+
+    def forward(self, x, h, ctx, cache: LayerCache, owns_cache: bool, accumulate: bool = True):
+        T = x.shape[0]
+        nh, g, d, dv = self.num_heads, self.num_qk_heads, self.head_dim, self.v_head_dim
+        QK, V, C = self.qk_size, self.v_size, self.conv_size
+        history, state = cache.parts
+        ws = ctx.workspace
+        proj = ws.get("recurrent_in", (T, self.in_weight.shape[0]), ctx.act_dtype)
+        ops.gemm(x, self.in_weight, None, proj)
+        conv = ws.get("recurrent_conv", (T, C), ctx.act_dtype)
+        ops.short_conv(proj[:, :C], conv, self.conv_weight, None if history is None else history.state, ctx,
+                       advance=owns_cache, residual=False, silu=True)
+        z = ws.get("recurrent_row_decay", (T, nh * d), torch.float32)
+        ops.gemm(proj[:, self.a_off:self.a_off + self.a2.shape[1]], self.a2, self.dt_bias, z)
+        gate = ws.get("recurrent_gate", (T, V), ctx.act_dtype)
+        ops.gemm(proj[:, self.g_off:self.g_off + self.g2.shape[1]], self.g2, None, gate)
+        beta = ws.get("recurrent_beta", (T, nh), torch.float32)
+        qscale, kscale = ws.get("recurrent_qscale", (T, g), torch.float32), ws.get("recurrent_kscale", (T, g), torch.float32)
+        ops.recurrence_gates(proj, None, self.b_off, None, None, None, beta, nh,
+                             unit_norm=(conv, 0, QK, g, d, self.unit_norm_eps, d ** -0.5, qscale, kscale))
+        o = ws.get("recurrent_out", (T, V), torch.float32)
+        ops.gated_recurrence(conv[:, :QK], conv[:, QK:2 * QK], conv[:, 2 * QK:], None, beta, o, state.state, ctx, nh, g, d, dv,
+                             delta_rule=True, qscale=qscale, kscale=kscale, write_state=owns_cache, row_decay=(z, self.rates))
+        y = ws.get("recurrent_gated", (T, V), ctx.act_dtype)
+        ops.gated_group_norm(o, gate, self.norm_weight, self.norm_eps, y, group=dv, gate_kind="sigmoid")
         ops.gemm(y, self.o_weight, None, h, accumulate=accumulate)
 
 
@@ -341,4 +433,5 @@ class GatedLinearAttention(Mixer):
 register_part("mixer", "gated_linear_unit", GatedLinearUnit)
 register_part("mixer", "gated_linear_attention", GatedLinearAttention)
 register_part("mixer", "gated_delta_rule", GatedDeltaRule)
+register_part("mixer", "channel_delta_rule", ChannelDeltaRule)
 register_part("mixer", "state_space_duality", StateSpaceDuality)

@@ -507,8 +507,8 @@ def test_attention_over_a_shared_latent_against_the_plain_mixer(device, nh, d, r
             ctx = fake_ctx(device, [n], [pos], [0])
             rows = proj[pos:pos + n].to(device).contiguous()
             q_att = torch.empty(n, nh * row, dtype=dtype, device=device)
-            ops.latent_prepare(rows, 0, Q, norm_w.to(device), 1e-5, ctx.positions, freq, dims, slots[pos:pos + n].contiguous(), k,
-                               q_att, nh, d, r, rank)
+            ops.latent_prepare(ctx.positions, ops.RotaryTable(freq, dims), 1e-5, nh, d, r, rank, queries=(rows[:, :Q], q_att),
+                               keys=(rows[:, Q:Q + row], norm_w.to(device), slots[pos:pos + n].contiguous(), k))
             ops.head_gemm(rows, d + r, uk_d, q_att, row)
             mixed = torch.empty(n, nh * rank, dtype=dtype, device=device)
             extra = dict(max_kv_len=pos + n, workspace=ws) if ws is not None and n == 1 else {}
