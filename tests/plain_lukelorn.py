@@ -92,7 +92,8 @@ def attention(h, w, p, m, positions, past=None):
     """``past``: (keys [P, G, d], values [P, G, dv]) of every token before h[0]."""
     T = h.shape[0]
     H, G, d, dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
-    freq = frequencies(m["rot"]["dims"], m["rot"]["base"], m["rot"].get("scaling"))
+    rot = m.get("rot") or {"dims": 0, "base": 1.0}
+    freq = frequencies(rot["dims"], rot["base"], rot.get("scaling"))
     q = rotate_pairs((h @ w[p + ".q"].T).reshape(T, H, d), positions, freq)
     k = rotate_pairs((h @ w[p + ".k"].T).reshape(T, G, d), positions, freq)
     v = (h @ w[p + ".v"].T).reshape(T, G, dv)
@@ -115,7 +116,8 @@ def latent_attention(h, w, p, m, eps, positions, past=None):
     q = (cq @ w[p + ".uq"].T).reshape(T, H, d + r)
     dkv = h @ w[p + ".dkv"].T
     c = rms_div(dkv[:, :rank], eps) * w[p + ".dkv.norm"]
-    freq = frequencies(m["rot"]["dims"], m["rot"]["base"])
+    rot = m.get("rot") or {"dims": 0, "base": 1.0}
+    freq = frequencies(rot["dims"], rot["base"])
     q_rot = rotate_pairs(q[..., d:], positions, freq)
     k_rot = rotate_pairs(dkv[:, None, rank:], positions, freq)[:, 0]
     if past is not None:
