@@ -1,9 +1,11 @@
 """Designs side by side at equal layer sizes: the Kugilix decoder beside the Qwen2 dense decoder, or (``design`` =
 "nusudra" / "netinex") the Nusudra or the Netinex decoder beside both, or (``design`` = "sumevik") the Sumevik decoder
 beside the Netinex decoder (the closest existing design: attention within chunks, a linear recurrence, experts) and
-Qwen2, or (``design`` = "retezen") the Retezen decoder beside the same two, random weights.
+Qwen2, or (``design`` = "retezen") the Retezen decoder beside the same two, or (``design`` = "lukelorn") the Lukelorn decoder
+beside the Nusudra decoder (the closest existing design: a delta rule, attention over a latent), Retezen (attention on tensor
+cores, experts with weights on their inputs) and Qwen2, random weights.
 
-Called by ``bench.py --designs [--design nusudra|netinex|sumevik|retezen]``.  For each of a few sizes that resemble a real model's layers it measures, through
+Called by ``bench.py --designs [--design nusudra|netinex|sumevik|retezen|lukelorn]``.  For each of a few sizes that resemble a real model's layers it measures, through
 the step function, the prefill of one prompt and decode steps at two batch sizes for both designs, and times the
 kernels that only the Kugilix design has (decayed linear attention, the windowed attention with slopes, the short
 convolution, the norms in groups, the gated norm, the activation) alone, with what they reach of the measured copy
@@ -154,6 +156,41 @@ def retezen_config(s: dict) -> dict:
     return {"architecture": "Retezen", "vocab": VOCAB, "width": s["width"], "max_positions": 8192, "norm": {"eps": 1e-6},
             "logit_scale": 0.7, "layers": [{"type": "attention", "mixer": mixer, "mlp": moe if i else dense}
                                            for i in range(kugilix_runs(s))]}
+
+
+LUKELORN_KEEP = 64  # first tokens that stay visible beside the window
+LUKELORN_ORDER = ("latent_attention", "attention", "channel_delta")
+
+
+def lukelorn_expert_ff(s: dict) -> int:
+    """An expert's inner size such that the ``TOP`` experts a token uses hold as many weights as the plain feed-forward."""
+    return s["ff"] // TOP
+
+
+def lukelorn_q_rank(s: dict) -> int:
+    return 3 * s["width"] // 8
+
+
+def lukelorn_config(s: dict) -> dict:
+    """As many layers as the Kugilix model has layer runs, its three mixers in turn; the same width, heads, head size; windows
+    as long as the other designs'; the latent row of the Nusudra model (192 + 64), queries through a latent of three eighths of
+    the width; a gated feed-forward of as many weights as the plain one in the first layer, ``TOP`` of ``EXPERTS`` experts in
+    the others; no layer's tensors run twice."""
+    H, G, d = s["heads"], s["kv_heads"], s["dim"]
+    mixers = {
+        "latent_attention": {"heads": H, "dim": d, "rot_dim": 64, "vdim": d, "q_rank": lukelorn_q_rank(s), "kv_rank": 192,
+                             "scale": 1.0 / math.sqrt(d + 64), "rot": {"base": 1e6, "dims": 64}, "mask": {"size": WINDOW}},
+        "attention": {"heads": H, "kv_heads": G, "dim": d, "vdim": d, "scale": 1.0 / math.sqrt(d), "softcap": 50.0,
+                      "rot": {"base": 5e5, "dims": d, "scaling": {"factor": 4.0, "low": 1.0, "high": 4.0, "original": 2048}},
+                      "mask": {"size": WINDOW, "keep_first": LUKELORN_KEEP}},
+        "channel_delta": {"heads": H, "kv_heads": G, "dim": d, "vdim": d, "conv": 4},
+    }
+    moe = {"kind": "moe", "expert": {"ff": lukelorn_expert_ff(s)}, "router": {"experts": EXPERTS, "top": TOP}}
+    dense = {"kind": "dense", "ff": sumevik_dense_ff(s)}
+    layers = [{"type": LUKELORN_ORDER[i % 3], "mixer": mixers[LUKELORN_ORDER[i % 3]], "mlp": moe if i else dense}
+              for i in range(kugilix_runs(s))]
+    return {"architecture": "Lukelorn", "vocab": VOCAB, "width": s["width"], "norm": {"eps": 1e-6}, "residual_mult": 0.5,
+            "layers": layers}
 
 
 def _timed(fn, flush, warmup=3, iters=5, reps=1):
@@ -808,11 +845,160 @@ def retezen_kernel_numbers(s: dict, peaks: dict) -> dict:
     return out
 
 
+def lukelorn_kernel_numbers(s: dict, peaks: dict) -> dict:
+    """The Lukelorn design's own kernels alone at the layer sizes ``s``, measured as ``kernel_numbers`` measures, each beside the
+    like kernel of the designs that were there before (the delta rule with a decay per head, attention over a window alone, over
+    a latent without one, experts with a gate of as many weights)."""
+    import torch
+    from types import SimpleNamespace
+
+    from ferrisinfer_b200.engine.workspace import Workspace
+    from ferrisinfer_b200.kernels import ops
+    from ferrisinfer_b200.parts.position import ScaledRotary
+
+    dev = torch.device("cuda")
+    bf = torch.bfloat16
+    flush = torch.zeros(96 << 20, dtype=torch.float32, device=dev)  # 384 MB
+    W, H, G, d = s["width"], s["heads"], s["kv_heads"], s["dim"]
+    hbm, tensor = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
+    ws = Workspace(dev)
+    out = {}
+
+    def ctx_of(q_lens, start):
+        S = len(q_lens)
+        q_start = [0]
+        for n in q_lens:
+            q_start.append(q_start[-1] + n)
+        i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+        return SimpleNamespace(num_tokens=q_start[-1], num_seqs=S, max_q_len=max(q_lens), workspace=ws,
+                               max_kv_len=start + max(q_lens),
+                               token_seq=i32([i for i in range(S) for _ in range(q_lens[i])]),
+                               positions=i32([start + j for i in range(S) for j in range(q_lens[i])]),
+                               seq_q_start=i32(q_start), seq_start_pos=i32([start] * S), seq_state_slot=i32(list(range(S))))
+
+    def record(name, seconds, bytes_=None, flops=None, tensor_flops=None):
+        e = {"us": round(seconds * 1e6, 1)}
+        if bytes_ is not None:
+            e["GBps"] = round(bytes_ / seconds / 1e9, 1)
+            e["frac_hbm"] = round(bytes_ / seconds / hbm, 3)
+        if flops is not None:
+            e["TFLOPs_fp32"] = round(flops / seconds / 1e12, 2)
+            e["frac_fp32_nominal"] = round(flops / seconds / (FP32_NOMINAL_TFLOPS * 1e12), 3)
+        if tensor_flops is not None:
+            e["TFLOPs_bf16"] = round(tensor_flops / seconds / 1e12, 1)
+            e["frac_bf16_measured"] = round(tensor_flops / seconds / tensor, 3)
+        out[name] = e
+
+    rank, rot, qr = 192, 64, lukelorn_q_rank(s)
+    randn = lambda *shape: torch.randn(*shape, device=dev)
+    for name, batch, q_len, ctx_len in (("decode_b64", 64, 1, 2047), ("decode_b8", 8, 1, 2047), ("prefill_2048", 1, 2048, 0)):
+        T = batch * q_len
+        reps = 10 if T <= 64 else 1
+        pages_each = (ctx_len + q_len + 15) // 16
+        tables = torch.arange(batch * pages_each, dtype=torch.int32, device=dev).view(batch, pages_each)
+        ctx = ctx_of([q_len] * batch, ctx_len)
+        slots = (tables[ctx.token_seq.long(), (ctx.positions // 16).long()] * 16 + ctx.positions % 16).int()
+        # ---- attention: a window with kept tokens, a soft cap, a sink and gates, beside the window alone
+        k = randn(batch * pages_each + 1, G, 16, d).to(bf)
+        v = torch.randn_like(k)
+        width = (H + 2 * G) * d + H
+        qkv = randn(T, (width + 7) // 8 * 8).to(bf)
+        o = torch.empty(T, H * d, dtype=bf, device=dev)
+        terms = ops.ScoreTerms(sink=torch.zeros(H, device=dev), softcap=50.0, gate=qkv[:, (H + 2 * G) * d:width])
+        seen = [min(WINDOW, ctx_len + j + 1) for j in range(q_len)]
+        kept = [min(LUKELORN_KEEP, max(0, ctx_len + j + 1 - WINDOW)) for j in range(q_len)]
+        for what, keep, t_, keys in (("kept_capped_attention", LUKELORN_KEEP, terms, sum(seen) + sum(kept)),
+                                     ("window_attention", 0, None, sum(seen))):
+            t = _timed(lambda: ops.paged_attention_simt(qkv, o, k, v, tables, ctx.token_seq, ctx.positions, H, G, d, WINDOW,
+                                                        1.0 / math.sqrt(d), score_slopes=t_, v_head_dim=d, max_q_len=q_len,
+                                                        max_kv_len=ctx_len + q_len, workspace=ws, keep_first=keep), flush, reps=reps)
+            record(f"{what}_{name}", t, flops=4.0 * keys * batch * H * d,
+                   bytes_=batch * G * keys * 2 * d * 2 + T * H * d * 4 if q_len == 1 else None)
+        table = ScaledRotary(d, 5e5, "interleaved", {"kind": "wavelength", "factor": 4.0, "low": 1.0, "high": 4.0, "original": 2048}).table(dev)
+        rows = qkv[:, :(H + 2 * G) * d]
+        t = _timed(lambda: ops.qk_norm_rotary_cache_write(rows, ctx, slots, k, v, H, G, d, d, None, None, 0.0, table), flush, reps=10)
+        record(f"rotary_cache_write_{name}", t, bytes_=T * (2 * H * d + 4 * G * d) * 2)
+        # ---- attention over the latent, in a window and over every key
+        kl = randn(batch * pages_each + 1, 1, 16, rank + rot).to(bf)
+        ql = randn(T, H * (rank + rot)).to(bf)
+        ol = torch.empty(T, H * rank, dtype=bf, device=dev)
+        for what, window in (("latent_window_attention", WINDOW), ("latent_attention", 0)):
+            keys = (sum(seen) if window else sum(ctx_len + j + 1 for j in range(q_len))) * batch
+            t = _timed(lambda: ops.paged_attention_simt(ql, ol, kl, None, tables, ctx.token_seq, ctx.positions, H, 1, rank + rot,
+                                                        window, 0.07, v_head_dim=rank, max_q_len=q_len, max_kv_len=ctx_len + q_len,
+                                                        workspace=ws, values_in_keys=True), flush, reps=reps)
+            record(f"{what}_{name}", t, flops=2.0 * keys * H * (2 * rank + rot),
+                   bytes_=keys * (rank + rot) * 2 + T * H * (2 * rank + rot) * 2 if q_len == 1 else None)
+        lrot = ScaledRotary(rot, 1e6, "interleaved").table(dev)
+        proj = randn(T, qr + rank + rot + H).to(bf)
+        q = randn(T, H * (d + rot)).to(bf)
+        nq, nc = torch.ones(qr, device=dev), torch.ones(rank, device=dev)
+        cq = torch.empty(T, qr, dtype=bf, device=dev)
+        t = _timed(lambda: ops.latent_prepare(ctx.positions, lrot, 1e-6, H, d, rot, rank, keys=(proj[:, qr:qr + rank + rot], nc, slots, kl),
+                                              q_latent=(proj[:, :qr], nq, cq)), flush, reps=10)
+        record(f"latent_norms_cache_write_{name}", t, bytes_=T * (2 * qr + 2 * (rank + rot)) * 2)
+        t = _timed(lambda: ops.latent_prepare(ctx.positions, lrot, 1e-6, H, d, rot, rank, queries=(q, ql)), flush, reps=10)
+        record(f"latent_query_rotation_{name}", t, bytes_=T * 2 * H * rot * 2)
+        uk = (randn(H, d, rank) / math.sqrt(d)).to(bf)
+        t = _timed(lambda: ops.head_gemm(q, d + rot, uk, ql, rank + rot), flush, reps=reps)
+        record(f"head_product_{name}", t, tensor_flops=2.0 * T * H * d * rank, bytes_=H * d * rank * 2 + T * H * (d + rank) * 2)
+        # ---- the recurrence: decays per channel beside a decay per head, and what stands around it
+        S = batch
+        kq, kk = (randn(T, G * d) / math.sqrt(d)).to(bf), (randn(T, G * d) / math.sqrt(d)).to(bf)
+        vv, beta = randn(T, H * d).to(bf), torch.full((T, H), 0.5, device=dev)
+        z, rates, decay = randn(T, H * d) - 3.0, torch.ones(H, device=dev), torch.full((T, H), 0.97, device=dev)
+        state, og = torch.zeros(S + 1, H, d, d, device=dev), torch.empty(T, H * d, device=dev)
+        moved = 2 * S * H * d * d * 4 + T * (2 * G * d + H * d) * 2 + T * H * d * 4
+        t = _timed(lambda: ops.gated_recurrence(kq, kk, vv, None, beta, og, state, ctx, H, G, d, d, delta_rule=True,
+                                                row_decay=(z, rates)), flush, reps=reps)
+        record(f"channel_delta_{name}", t, bytes_=moved + T * H * d * 4, flops=7.0 * T * H * d * d)
+        if q_len > 1:
+            t = _timed(lambda: ops.gated_recurrence(kq, kk, vv, None, beta, og, state, ctx, H, G, d, d, delta_rule=True,
+                                                    row_decay=(z, rates), chunks=False), flush, reps=reps)
+            record(f"channel_delta_token_by_token_{name}", t, bytes_=moved + T * H * d * 4, flops=7.0 * T * H * d * d)
+        t = _timed(lambda: ops.gated_recurrence(kq, kk, vv, decay, beta, og, state, ctx, H, G, d, d, delta_rule=True), flush, reps=reps)
+        record(f"delta_rule_{name}", t, bytes_=moved, flops=6.0 * T * H * d * d)
+        C = (2 * G + H) * d
+        wide, conv = randn(T, C + 64).to(bf), torch.empty(T, C, dtype=bf, device=dev)
+        cw, cs = randn(C, 4) * 0.1, torch.zeros(S + 1, 3, C, device=dev)
+        t = _timed(lambda: ops.short_conv(wide[:, :C], conv, cw, cs, ctx, residual=False, silu=True), flush, reps=reps)
+        record(f"conv_silu_{name}", t, bytes_=T * C * 4 + (S * 3 * C * 8 if q_len == 1 else 0))
+        a1, a2, dt = randn(T, d).to(bf), (randn(H * d, d) / math.sqrt(d)).to(bf), torch.zeros(H * d, device=dev)
+        t = _timed(lambda: ops.gemm(a1, a2, dt, z), flush, reps=reps)
+        record(f"decay_product_{name}", t, bytes_=T * (d * 2 + H * d * 4) + H * d * d * 2, tensor_flops=2.0 * T * H * d * d)
+        y, gate = torch.empty(T, H * d, dtype=bf, device=dev), randn(T, H * d).to(bf)
+        nw = torch.ones(d, device=dev)
+        t = _timed(lambda: ops.gated_group_norm(og, gate, nw, 1e-6, y, group=d, gate_kind="sigmoid"), flush, reps=reps)
+        record(f"gated_head_norm_{name}", t, bytes_=T * H * d * (4 + 2 + 2))
+        qs, ks = torch.empty(T, G, device=dev), torch.empty(T, G, device=dev)
+        t = _timed(lambda: ops.recurrence_gates(gate, None, 0, None, None, None, beta, H,
+                                                unit_norm=(conv, 0, G * d, G, d, 1e-6, d ** -0.5, qs, ks)), flush, reps=reps)
+        record(f"beta_unit_norms_{name}", t, bytes_=T * (2 * G * d * 2 + H * 2 + H * 4 + 2 * G * 4))
+    # ---- experts without a gate beside gated ones of as many weights, weights on their inputs
+    router = randn(EXPERTS, W).to(bf)
+    for tag, T in (("b64", 64), ("b8", 8), ("2048", 2048)):
+        x = randn(T, W).to(bf)
+        hrow = torch.zeros(T, W, device=dev)
+        ids, wts = torch.empty(T, TOP, dtype=torch.int32, device=dev), torch.empty(T, TOP, device=dev)
+        t = _timed(lambda: ops.moe_router(x, router, None, ids, wts, TOP, sigmoid=True), flush, reps=10)
+        record(f"sigmoid_router_{tag}", t, bytes_=T * W * 2 + EXPERTS * W * 2)
+        distinct = int(torch.unique(ids).numel())
+        for what, plain, eff in (("experts_plain", True, lukelorn_expert_ff(s)), ("experts_gated", False, netinex_expert_ff(s))):
+            n = 2 if plain else 3
+            up = (randn(EXPERTS, (n - 1) * eff, W) / math.sqrt(W)).to(bf)
+            down = (randn(EXPERTS, W, eff) / math.sqrt(eff)).to(bf)
+            t = _timed(lambda: ops.moe_experts(x, up, down, ids, wts, hrow, ws, accumulate=True, input_weights=True, plain=plain,
+                                               activation="relu2" if plain else "silu"), flush)
+            record(f"{what}_{tag}", t, bytes_=distinct * n * W * eff * 2 + T * W * (2 + 8), tensor_flops=2.0 * T * TOP * n * W * eff)
+            out[f"{what}_{tag}"]["distinct_experts"] = distinct
+    return out
+
+
 def run(build_engine, time_decode, time_prefill, peaks, steps=32, warmup=4, sizes=("small", "1B-like"), context=2048,
         prompt=2048, batches=(8, 64), kernels_at="1B-like", design="kugilix") -> dict:
     """``build_engine(cfg, batch, context, extra_tokens)``, ``time_decode`` and ``time_prefill`` are bench.py's.
     ``design`` "kugilix": that design beside Qwen2; "nusudra" or "netinex": that design beside both; "sumevik" or "retezen":
-    that design beside Netinex and Qwen2."""
+    that design beside Netinex and Qwen2; "lukelorn": that design beside Nusudra, Retezen and Qwen2."""
     import torch
 
     result = {"context": context, "prompt_tokens": prompt, "window": WINDOW, "sizes": {}}
@@ -827,6 +1013,9 @@ def run(build_engine, time_decode, time_prefill, peaks, steps=32, warmup=4, size
         if design in ("sumevik", "retezen"):
             own = sumevik_config(s) if design == "sumevik" else retezen_config(s)
             designs = ((design, own), ("netinex", netinex_config(s)), ("qwen2", qwen2_config(s)))
+        if design == "lukelorn":
+            designs = ((design, lukelorn_config(s)), ("nusudra", nusudra_config(s)), ("retezen", retezen_config(s)),
+                       ("qwen2", qwen2_config(s)))
         for design_name, cfg in designs:
             numbers = {}
             engine = build_engine(cfg, 1, context, extra_tokens=prompt)
@@ -846,7 +1035,10 @@ def run(build_engine, time_decode, time_prefill, peaks, steps=32, warmup=4, size
                 torch.cuda.empty_cache()
             entry[design_name] = numbers
         result["sizes"][name] = entry
-    if kernels_at and design == "retezen":
+    if kernels_at and design == "lukelorn":
+        result["kernels_lukelorn"] = {"at": kernels_at, "expert_ff": lukelorn_expert_ff(SIZES[kernels_at]), "experts": EXPERTS,
+                                      "top": TOP, "keep_first": LUKELORN_KEEP, **lukelorn_kernel_numbers(SIZES[kernels_at], peaks)}
+    elif kernels_at and design == "retezen":
         result["kernels_retezen"] = {"at": kernels_at, "expert_ff": netinex_expert_ff(SIZES[kernels_at]), "experts": EXPERTS,
                                      "top": TOP, "pool": RETEZEN_POOL, **retezen_kernel_numbers(SIZES[kernels_at], peaks)}
         result["kernels_netinex"] = {"at": kernels_at, "expert_ff": netinex_expert_ff(SIZES[kernels_at]),

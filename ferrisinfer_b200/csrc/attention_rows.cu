@@ -1,6 +1,6 @@
 // The general attention over a bf16 cache on tensor cores, with the softmax's weights in 32-bit: head sizes of any multiple
-// of eight up to 256 (the values' may differ), any page size, any grouping of heads, a window, a chunk or every key, pooled
-// keys before the window, a sink.  The formulas and arguments are those of attention_simt.cu.
+// of eight up to 256 (the values' may differ, or lie in the keys), any page size, any grouping of heads, a window, a chunk or
+// every key, pooled keys before the window or first tokens that it keeps, a soft cap, a sink, gates.  The formulas and arguments are those of attention_simt.cu.
 //
 // q . k is a product of bf16 numbers with fp32 sums, as exact as FMAs on the widened numbers.  The second product, weights
 // times values, must not round the weights to bf16: a weight p is cut into three bf16 parts, p1 = bf16(p), p2 = bf16(p - p1),
@@ -72,6 +72,7 @@ struct AttentionArgs {
     float scale_cap;  // 0: no cap
     const bf16* gate;  // the heads' gates, rows ldgate apart (null: none)
     int ldgate;
+    int values_in_keys;  // a value is the first dv elements of its key: the keys' tile serves both products, v is not read
 };
 // sigmoid of the gate of head h at token t
 __device__ __forceinline__ float gate_of(const AttentionArgs& p, int t, int h) {
@@ -241,7 +242,8 @@ __global__ void __launch_bounds__(AR_THREADS, D <= 128 ? 3 : 2) attention_rows_k
                 const bf16* vs = (run ? reinterpret_cast<const bf16*>(p.pk.v) : p.v) + row * dv;
                 const uint32_t dst = base + (i & 1) * STAGE + key * PITCH;
                 for (int c = part; c < (d >> 3); c += TPK) copy16_or_zero(dst + c * 16, ks + 8 * c, there);
-                for (int c = part; c < (dv >> 3); c += TPK) copy16_or_zero(dst + V_OFF + c * 16, vs + 8 * c, there);
+                if (!p.values_in_keys)
+                    for (int c = part; c < (dv >> 3); c += TPK) copy16_or_zero(dst + V_OFF + c * 16, vs + 8 * c, there);
             }
             ar_commit();
         };
@@ -319,7 +321,7 @@ __global__ void __launch_bounds__(AR_THREADS, D <= 128 ? 3 : 2) attention_rows_k
             }
             softmax_step<NT, DT>(s, m, l, o);
 #pragma unroll
-            for (int kk = 0; kk < KT / 16; ++kk) weights_times_values<NT, DT>(o, s, kk, kb + V_OFF, PITCH, dv);
+            for (int kk = 0; kk < KT / 16; ++kk) weights_times_values<NT, DT>(o, s, kk, p.values_in_keys ? kb : kb + V_OFF, PITCH, dv);
             __syncthreads();  // the stage is read: the copies after next may overwrite it
         }
         ta = tb + 1;
@@ -437,7 +439,8 @@ __global__ void __launch_bounds__(AR_THREADS) attention_single_rows_kernel(const
                 }
             } else {
                 for (int x = part; x < (d >> 3); x += 2) copy16_or_zero(dst + key * PITCH + x * 16, ks + 8 * x, there);
-                for (int x = part; x < (dv >> 3); x += 2) copy16_or_zero(dst + V_OFF + key * PITCH + x * 16, vs + 8 * x, there);
+                if (!p.values_in_keys)
+                    for (int x = part; x < (dv >> 3); x += 2) copy16_or_zero(dst + V_OFF + key * PITCH + x * 16, vs + 8 * x, there);
             }
         }
         ar_commit();
@@ -504,7 +507,7 @@ __global__ void __launch_bounds__(AR_THREADS) attention_single_rows_kernel(const
         split3(w[2], w[3], pw[0][1], pw[1][1], pw[2][1]);
 #pragma unroll
         for (int x = 0; x < 3; ++x) pw[x][0] = movmatrix_trans(pw[x][0]), pw[x][1] = movmatrix_trans(pw[x][1]);
-        const uint32_t v_at = kb + V_OFF + (uint32_t)((lane & 7) + (lane >> 4) * 8) * PITCH + ((lane >> 3) & 1) * 16;
+        const uint32_t v_at = kb + (!FAST && p.values_in_keys ? 0 : V_OFF) + (uint32_t)((lane & 7) + (lane >> 4) * 8) * PITCH + ((lane >> 3) & 1) * 16;
 #pragma unroll
         for (int n = 0; n < MT; n += 4) {  // four accumulators in turn
             if (16 * n < dv) {
@@ -641,7 +644,7 @@ int launch_single_form(const AttentionArgs& p, int splits, cudaStream_t s) {
 
 template <int D, bool POOL>
 int launch_single(const AttentionArgs& p, int splits, cudaStream_t s) {
-    const bool fast = p.d == D && p.dv == D && p.page_size % AS_KEYS == 0;
+    const bool fast = !p.values_in_keys && p.d == D && p.dv == D && p.page_size % AS_KEYS == 0;
     return fast ? launch_single_form<D, POOL, true>(p, splits, s) : launch_single_form<D, POOL, false>(p, splits, s);
 }
 
@@ -654,20 +657,23 @@ FERRIS_API int ferris_attention_rows_takes(int nh, int nkv, int d, int dv, int p
     return portions ? nh / nkv <= AR_ROWS : 1;
 }
 
-// Arguments as ferris_paged_attention_simt, bf16 throughout, no distance penalty, values in rows of their own.  portions:
+// Arguments as ferris_paged_attention_simt, bf16 throughout, no distance penalty; v_stride is 0 (values in rows of their own)
+// or d, with v_cache the key cache (a value is the first dv elements of its key).  portions:
 // requests bring several tokens each (the kernel of 64-row blocks); else kv_span is the most keys a token sees (0: unknown),
 // by which they are cut into shares.
 FERRIS_API int ferris_attention_rows(const void* q, int ldq, void* out, int ldo, const void* k_cache, const void* v_cache,
                                      const int* block_tables, int max_blocks, const int* token_seq, const int* positions,
                                      int tokens, int nh, int nkv, int d, int dv, int page_size, int window, float scale,
-                                     const float* sink, const void* pool_k, const void* pool_v, const int* pool_tables,
+                                     const float* sink, int v_stride, const void* pool_k, const void* pool_v, const int* pool_tables,
                                      int pool_max_blocks, int pool_every, int keep, float softcap, const void* gate, int ldgate,
                                      int portions, int kv_span, void* stream) {
     if (tokens <= 0) return FERRIS_OK;
     if (!ferris_attention_rows_takes(nh, nkv, d, dv, portions))
         FERRIS_REFUSE("attention rows: %d heads over %d kv heads of %d / %d are not taken", nh, nkv, d, dv);
     if (page_size <= 0 || max_blocks <= 0) FERRIS_REFUSE("attention: page_size=%d max_blocks=%d", page_size, max_blocks);
-    const ScoreTerms st = {nullptr, nullptr, nullptr, sink, 0, softcap, gate, ldgate};
+    if (v_stride != 0 && (v_stride != d || dv > d || v_cache != k_cache))
+        FERRIS_REFUSE("attention rows: values %d elements apart in keys of %d", v_stride, d);
+    const ScoreTerms st = {nullptr, nullptr, nullptr, sink, v_stride, softcap, gate, ldgate};
     const PooledKeys pk = keys_beside(pool_k, pool_v, pool_tables, pool_max_blocks, pool_every, keep, k_cache, v_cache, block_tables, max_blocks);
     if (int rc = check_pooled(pk, window, st)) return rc;
     if ((((uintptr_t)q | (uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)pool_k | (uintptr_t)pool_v) & 15) != 0 || ldq % 8 ||
@@ -676,7 +682,7 @@ FERRIS_API int ferris_attention_rows(const void* q, int ldq, void* out, int ldo,
     const AttentionArgs p = {(const bf16*)q, (bf16*)out, (const bf16*)k_cache, (const bf16*)v_cache, block_tables, token_seq,
                              positions, sink, pk, ldq, ldo, max_blocks, tokens, nh, nkv, d, dv, page_size, window,
                              (softcap > 0.0f ? softcap : scale) * LOG2E, softcap > 0.0f ? scale / softcap : 0.0f,
-                             (const bf16*)gate, ldgate};
+                             (const bf16*)gate, ldgate, v_stride > 0 ? 1 : 0};
     cudaStream_t s = (cudaStream_t)stream;
     const bool pool = pk.every > 0 || pk.keep > 0;
     const int bucket = rows_bucket(d, dv);

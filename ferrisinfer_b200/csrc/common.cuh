@@ -221,6 +221,8 @@ __device__ __forceinline__ float ferris_gated_act(float g, float u, int kind, fl
     return (g / (1.0f + expf(-g))) * u;
 }
 
+__device__ __forceinline__ float ferris_softplus(float v) { return fmaxf(v, 0.0f) + log1pf(expf(-fabsf(v))); }
+
 __device__ __forceinline__ float to_float(float v) { return v; }
 __device__ __forceinline__ float to_float(bf16 v) { return __bfloat162float(v); }
 

@@ -1,0 +1,379 @@
+// The delta rule with a decay per key channel over portions of prompts, sixteen tokens at a time.
+//
+// Per (request, head), with rows r of S as key channels, d_t[r] <= 0 the logarithm of row r's decay at token t:
+//     S <- diag(exp(d_t)) S;  u_t = b_t (v_t - S^T k_t);  S <- S + k_t u_t^T;  o_t = S^T q_t
+// Walking the tokens one by one is a chain of dependent steps.  A chunk of C = 16 tokens has a closed form instead (the
+// compact form of a product of rank-one corrections; Bischof and Van Loan's WY representation is its ancestor).  With
+// L_t = d_1 + .. + d_t inside the chunk and S_0 the state at its start,
+//     D_t = (k_t exp(L_t))^T S_0,   E_t = (q_t exp(L_t))^T S_0
+//     A_ti = sum_r k_t k_i exp(L_t - L_i)  (i < t),   B_ti = sum_r q_t k_i exp(L_t - L_i)  (i <= t)
+//     u_t = b_t (v_t - D_t - sum_(i<t) A_ti u_i)   i.e.  u = M (v - D),  M = (I + diag(b) A)^-1 diag(b)
+//     o_t = E_t + sum_(i<=t) B_ti u_i
+//     S_C = diag(exp(L_C)) S_0 + sum_i (k_i exp(L_C - L_i)) u_i^T
+// Every exponent is of a difference that is not positive, so nothing overflows however fast a channel forgets, and the state
+// moves on as S + (expm1(L_C) S + ..): a decay close to one is never rounded to 24 bits.  All of it is fp32.
+//
+// Two kernels.  What does not depend on the state (k_t exp(L_t), q_t exp(L_t), k_i exp(L_C - L_i), M, B, expm1(L_C)) is formed
+// for all chunks side by side, a block per (chunk, head).  Then a block per (request, head, run of columns of S) walks the
+// chunks: as in gated_recurrence.cu a few lanes share a column and hold eight rows each; here the sixteen tokens' products
+// with S_0 are independent of one another, their sums over the lanes are reduced together (a lane ends with a token's sum, in
+// 16 + 8 + .. exchanges instead of 16 x log2), and only the 16 x 16 products with M and B tie the tokens together.  The next
+// chunk's rows come in by asynchronous copies meanwhile.
+#include <math.h>
+
+#include "common.cuh"
+
+namespace {
+
+constexpr int DC_TOKENS = 16;
+constexpr int DC_THREADS = 128;
+constexpr int DC_PREP_THREADS = 256;
+constexpr int DC_KPL = 8;     // rows of the state that a lane holds
+constexpr int DC_PITCH = 20;  // floats between the rows of 16 x 16 matrices in shared memory: rows start in different banks
+
+// kt, qt, kh: [tokens, heads, dim]; mm, bm: [tokens, heads, 16]; dm: [places, heads, dim], the place of a chunk being
+// (its first row) / 16 + its request's index in the step, which no two chunks share.
+struct DeltaChunks {
+    float* kt;
+    float* qt;
+    float* kh;
+    float* mm;
+    float* bm;
+    float* dm;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(DC_PREP_THREADS) delta_chunk_prepare_kernel(
+    const T* q, int ldq, const T* k, int ldk, const float* z, int ldz, const float* __restrict__ rates, const float* beta,
+    const float* qscale, const float* kscale, const int* __restrict__ seq_q_start, int chunks_max, int heads, int qk_heads, int dim,
+    const DeltaChunks w) {
+    extern __shared__ __align__(16) float dc_smem[];
+    const int pitch = dim + 1;
+    float* Ls = dc_smem;                     // [16][dim + 1]: logarithms, then their sums from the chunk's start
+    float* Ks = Ls + DC_TOKENS * pitch;      // keys and queries with their factors
+    float* Qs = Ks + DC_TOKENS * pitch;
+    __shared__ float As[DC_TOKENS][DC_TOKENS + 1], bs[DC_TOKENS];
+    pdl_wait();
+    pdl_launch_dependents();
+    const int seq = blockIdx.x / chunks_max, head = blockIdx.y;
+    const int row0 = seq_q_start[seq], row1 = seq_q_start[seq + 1];
+    const int first = row0 + (blockIdx.x % chunks_max) * DC_TOKENS;
+    if (first >= row1) return;
+    const int n = min(DC_TOKENS, row1 - first);
+    const int qh = head / (heads / qk_heads);
+    const float rate = rates[head];
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    for (int x = tid; x < n * dim; x += DC_PREP_THREADS) {
+        const int t = x / dim, c = x - t * dim;
+        const size_t row = (size_t)(first + t);
+        Ls[t * pitch + c] = -ferris_softplus(z[row * ldz + (size_t)head * dim + c]) * rate;
+        Ks[t * pitch + c] = to_float(k[row * ldk + (size_t)qh * dim + c]) * (kscale ? kscale[row * qk_heads + qh] : 1.0f);
+        Qs[t * pitch + c] = to_float(q[row * ldq + (size_t)qh * dim + c]) * (qscale ? qscale[row * qk_heads + qh] : 1.0f);
+    }
+    if (tid < DC_TOKENS) bs[tid] = tid < n ? beta[(size_t)(first + tid) * heads + head] : 0.0f;
+    __syncthreads();
+    for (int c = tid; c < dim; c += DC_PREP_THREADS) {
+        float sum = 0.0f;
+        for (int t = 0; t < n; ++t) sum += Ls[t * pitch + c], Ls[t * pitch + c] = sum;
+        w.dm[((size_t)(first / DC_TOKENS + seq) * heads + head) * dim + c] = expm1f(sum);
+    }
+    __syncthreads();
+    for (int x = tid; x < n * dim; x += DC_PREP_THREADS) {
+        const int t = x / dim, c = x - t * dim;
+        const size_t at = ((size_t)(first + t) * heads + head) * dim + c;
+        const float L = Ls[t * pitch + c], e = expf(L), kv = Ks[t * pitch + c];
+        w.kt[at] = kv * e;
+        w.qt[at] = Qs[t * pitch + c] * e;
+        w.kh[at] = kv * expf(Ls[(n - 1) * pitch + c] - L);
+    }
+    // a warp takes tokens w and 15 - w: seventeen pairs each
+    for (int half = 0; half < 2; ++half) {
+        const int t = half ? DC_TOKENS - 1 - warp : warp;
+        if (t >= n) continue;
+        for (int i = 0; i <= t; ++i) {
+            float a = 0.0f, b = 0.0f;
+            for (int c = lane; c < dim; c += 32) {
+                const float e = expf(Ls[t * pitch + c] - Ls[i * pitch + c]) * Ks[i * pitch + c];
+                a = fmaf(Ks[t * pitch + c], e, a), b = fmaf(Qs[t * pitch + c], e, b);
+            }
+            a = warp_sum(a), b = warp_sum(b);
+            if (lane == 0) {
+                As[t][i] = a;
+                w.bm[((size_t)(first + t) * heads + head) * DC_TOKENS + i] = b;
+            }
+        }
+        if (lane > t && lane < DC_TOKENS) w.bm[((size_t)(first + t) * heads + head) * DC_TOKENS + lane] = 0.0f;
+    }
+    __syncthreads();
+    if (tid < DC_TOKENS) {  // a column of M each: M_tj = b_t (delta_tj - sum_(i<t) A_ti M_ij)
+        float m[DC_TOKENS];
+#pragma unroll
+        for (int t = 0; t < DC_TOKENS; ++t) {
+            float acc = t == tid ? 1.0f : 0.0f;
+            if (t < n) {
+#pragma unroll
+                for (int i = 0; i < t; ++i) acc = fmaf(-As[t][i], m[i], acc);
+                m[t] = bs[t] * acc;
+                w.mm[((size_t)(first + t) * heads + head) * DC_TOKENS + tid] = m[t];
+            } else {
+                m[t] = 0.0f;
+            }
+        }
+    }
+}
+
+__device__ __forceinline__ void dc_copy16(float* dst, const float* src) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+}
+
+// The sums over the LANES lanes of a column of sixteen numbers a lane: afterwards lane `sub` holds those of tokens
+// sub * PER .. (LANES <= 16), or that of token sub / 2 (LANES = 32), in the first elements of x.
+template <int LANES>
+__device__ __forceinline__ void reduce_tokens(float (&x)[DC_TOKENS], int sub) {
+    int width = DC_TOKENS;
+#pragma unroll
+    for (int o = LANES / 2; o > 0; o >>= 1) {
+        if (width > 1) {
+            width >>= 1;
+            const bool upper = sub & o;
+#pragma unroll
+            for (int j = 0; j < DC_TOKENS / 2; ++j) {
+                if (j < width) {
+                    const float keep = upper ? x[j + width] : x[j], give = upper ? x[j] : x[j + width];
+                    x[j] = keep + __shfl_xor_sync(0xffffffffu, give, o);
+                }
+            }
+        } else {
+            x[0] += __shfl_xor_sync(0xffffffffu, x[0], o);
+        }
+    }
+}
+
+template <int LANES>
+struct DeltaStage {
+    static constexpr int ROWS = DC_KPL * LANES;
+    float kt[DC_TOKENS][ROWS], qt[DC_TOKENS][ROWS], kh[DC_TOKENS][ROWS];
+    float dm[ROWS];
+    float mm[DC_TOKENS][DC_PITCH], bm[DC_TOKENS][DC_PITCH];
+};
+
+template <typename T, int LANES>
+__global__ void __launch_bounds__(DC_THREADS) delta_chunk_walk_kernel(
+    const DeltaChunks w, const T* v, int ldv, float* __restrict__ out, int ldo, float* state, const int* __restrict__ seq_q_start,
+    const int* __restrict__ seq_state_slot, int heads, int dim, int vdim, int write_state) {
+    constexpr int COLS = DC_THREADS / LANES;  // columns of a block
+    constexpr int PER = LANES >= DC_TOKENS ? 1 : DC_TOKENS / LANES;  // tokens whose sums a lane ends with
+    extern __shared__ __align__(16) float dc_smem[];
+    DeltaStage<LANES>* stages = reinterpret_cast<DeltaStage<LANES>*>(dc_smem);
+    __shared__ __align__(16) float ws[COLS][DC_PITCH], us[COLS][DC_PITCH];
+    pdl_wait();
+    pdl_launch_dependents();
+    const int seq = blockIdx.x, head = blockIdx.y, tid = threadIdx.x;
+    const int sub = tid % LANES, cl = tid / LANES;
+    const int col = blockIdx.z * COLS + cl;
+    const bool active = col < vdim;
+    const int row0 = seq_q_start[seq], row1 = seq_q_start[seq + 1];
+    if (row1 <= row0) return;
+    // both stages start as zeros: rows of the state beyond the head's size, and tokens beyond a chunk's last
+    for (int i = tid; i < (int)(2 * sizeof(DeltaStage<LANES>) / sizeof(float)); i += DC_THREADS) dc_smem[i] = 0.0f;
+    float* S = state + (((size_t)seq_state_slot[seq] * heads + head) * vdim + (active ? col : 0)) * (size_t)dim;
+    float s[DC_KPL];
+#pragma unroll
+    for (int g = 0; g < 2; ++g) {
+        const int r = (g * LANES + sub) * 4;
+        float4 x = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (active && r < dim) x = *reinterpret_cast<const float4*>(S + r);
+        s[4 * g] = x.x, s[4 * g + 1] = x.y, s[4 * g + 2] = x.z, s[4 * g + 3] = x.w;
+    }
+    const int mine = LANES == 32 ? sub >> 1 : sub * PER;  // the first token whose sums this lane ends with
+    const bool writes = LANES != 32 || !(sub & 1);
+    __syncthreads();
+    const int d4 = dim >> 2;
+    auto fetch = [&](int first, DeltaStage<LANES>& st) {
+        if (first < row1) {
+            const int n = min(DC_TOKENS, row1 - first);
+            for (int x = tid; x < n * d4; x += DC_THREADS) {
+                const int t = x / d4, c = (x - t * d4) * 4;
+                const size_t at = ((size_t)(first + t) * heads + head) * dim + c;
+                dc_copy16(&st.kt[t][c], w.kt + at);
+                dc_copy16(&st.qt[t][c], w.qt + at);
+                dc_copy16(&st.kh[t][c], w.kh + at);
+            }
+            for (int x = tid; x < d4; x += DC_THREADS)
+                dc_copy16(&st.dm[4 * x], w.dm + ((size_t)(first / DC_TOKENS + seq) * heads + head) * dim + 4 * x);
+            if (tid < n * 4) {
+                const int t = tid >> 2, c = (tid & 3) * 4;
+                const size_t at = ((size_t)(first + t) * heads + head) * DC_TOKENS + c;
+                dc_copy16(&st.mm[t][c], w.mm + at);
+                dc_copy16(&st.bm[t][c], w.bm + at);
+            }
+            if (n < DC_TOKENS) {  // the last chunk: what an earlier one left behind the last token
+                for (int x = tid; x < (DC_TOKENS - n) * d4; x += DC_THREADS) {
+                    const int t = n + x / d4, c = (x % d4) * 4;
+                    const float4 zero = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+                    *reinterpret_cast<float4*>(&st.kt[t][c]) = zero;
+                    *reinterpret_cast<float4*>(&st.qt[t][c]) = zero;
+                    *reinterpret_cast<float4*>(&st.kh[t][c]) = zero;
+                }
+                for (int x = tid; x < (DC_TOKENS - n) * DC_TOKENS; x += DC_THREADS)
+                    st.mm[n + x / DC_TOKENS][x % DC_TOKENS] = 0.0f, st.bm[n + x / DC_TOKENS][x % DC_TOKENS] = 0.0f;
+            }
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    T pv[PER];
+    auto request_v = [&](int first) {
+#pragma unroll
+        for (int j = 0; j < PER; ++j) {
+            const int t = first + mine + j;
+            pv[j] = from_float<T>(0.0f);
+            if (t < row1 && active) pv[j] = v[(size_t)t * ldv + (size_t)head * vdim + col];
+        }
+    };
+    fetch(row0, stages[0]);
+    request_v(row0);
+    int buf = 0;
+    for (int first = row0; first < row1; first += DC_TOKENS, buf ^= 1) {
+        fetch(first + DC_TOKENS, stages[buf ^ 1]);
+        float vv[PER];
+#pragma unroll
+        for (int j = 0; j < PER; ++j) vv[j] = to_float(pv[j]);
+        request_v(first + DC_TOKENS);
+        asm volatile("cp.async.wait_group 1;" ::: "memory");
+        __syncthreads();
+        const DeltaStage<LANES>& st = stages[buf];
+        float D[DC_TOKENS], E[DC_TOKENS];
+#pragma unroll
+        for (int t = 0; t < DC_TOKENS; ++t) {
+            const float4 a = *reinterpret_cast<const float4*>(&st.kt[t][4 * sub]);
+            const float4 b = *reinterpret_cast<const float4*>(&st.kt[t][4 * (LANES + sub)]);
+            D[t] = fmaf(a.x, s[0], fmaf(a.y, s[1], fmaf(a.z, s[2], a.w * s[3])));
+            D[t] = fmaf(b.x, s[4], fmaf(b.y, s[5], fmaf(b.z, s[6], fmaf(b.w, s[7], D[t]))));
+            const float4 c = *reinterpret_cast<const float4*>(&st.qt[t][4 * sub]);
+            const float4 e = *reinterpret_cast<const float4*>(&st.qt[t][4 * (LANES + sub)]);
+            E[t] = fmaf(c.x, s[0], fmaf(c.y, s[1], fmaf(c.z, s[2], c.w * s[3])));
+            E[t] = fmaf(e.x, s[4], fmaf(e.y, s[5], fmaf(e.z, s[6], fmaf(e.w, s[7], E[t]))));
+        }
+        reduce_tokens<LANES>(D, sub);
+        reduce_tokens<LANES>(E, sub);
+#pragma unroll
+        for (int j = 0; j < PER; ++j)
+            if (writes) ws[cl][mine + j] = vv[j] - D[j];
+        __syncwarp();
+        float x[DC_TOKENS];
+#pragma unroll
+        for (int i = 0; i < DC_TOKENS; i += 4) {
+            const float4 f = *reinterpret_cast<const float4*>(&ws[cl][i]);
+            x[i] = f.x, x[i + 1] = f.y, x[i + 2] = f.z, x[i + 3] = f.w;
+        }
+#pragma unroll
+        for (int j = 0; j < PER; ++j) {
+            float u0 = 0.0f, u1 = 0.0f;
+#pragma unroll
+            for (int i = 0; i < DC_TOKENS; i += 4) {
+                const float4 m = *reinterpret_cast<const float4*>(&st.mm[mine + j][i]);
+                u0 = fmaf(m.x, x[i], u0), u1 = fmaf(m.y, x[i + 1], u1), u0 = fmaf(m.z, x[i + 2], u0), u1 = fmaf(m.w, x[i + 3], u1);
+            }
+            if (writes) us[cl][mine + j] = u0 + u1;
+        }
+        __syncwarp();
+#pragma unroll
+        for (int i = 0; i < DC_TOKENS; i += 4) {
+            const float4 f = *reinterpret_cast<const float4*>(&us[cl][i]);
+            x[i] = f.x, x[i + 1] = f.y, x[i + 2] = f.z, x[i + 3] = f.w;
+        }
+#pragma unroll
+        for (int j = 0; j < PER; ++j) {
+            float o0 = E[j], o1 = 0.0f;
+#pragma unroll
+            for (int i = 0; i < DC_TOKENS; i += 4) {
+                const float4 m = *reinterpret_cast<const float4*>(&st.bm[mine + j][i]);
+                o0 = fmaf(m.x, x[i], o0), o1 = fmaf(m.y, x[i + 1], o1), o0 = fmaf(m.z, x[i + 2], o0), o1 = fmaf(m.w, x[i + 3], o1);
+            }
+            const int t = first + mine + j;
+            if (writes && active && t < row1) out[(size_t)t * ldo + (size_t)head * vdim + col] = o0 + o1;
+        }
+        float acc[DC_KPL];
+#pragma unroll
+        for (int i = 0; i < DC_KPL; ++i) acc[i] = 0.0f;
+#pragma unroll
+        for (int t = 0; t < DC_TOKENS; ++t) {
+            const float4 a = *reinterpret_cast<const float4*>(&st.kh[t][4 * sub]);
+            const float4 b = *reinterpret_cast<const float4*>(&st.kh[t][4 * (LANES + sub)]);
+            acc[0] = fmaf(a.x, x[t], acc[0]), acc[1] = fmaf(a.y, x[t], acc[1]), acc[2] = fmaf(a.z, x[t], acc[2]), acc[3] = fmaf(a.w, x[t], acc[3]);
+            acc[4] = fmaf(b.x, x[t], acc[4]), acc[5] = fmaf(b.y, x[t], acc[5]), acc[6] = fmaf(b.z, x[t], acc[6]), acc[7] = fmaf(b.w, x[t], acc[7]);
+        }
+        const float4 m0 = *reinterpret_cast<const float4*>(&st.dm[4 * sub]), m1 = *reinterpret_cast<const float4*>(&st.dm[4 * (LANES + sub)]);
+        s[0] += fmaf(m0.x, s[0], acc[0]), s[1] += fmaf(m0.y, s[1], acc[1]), s[2] += fmaf(m0.z, s[2], acc[2]), s[3] += fmaf(m0.w, s[3], acc[3]);
+        s[4] += fmaf(m1.x, s[4], acc[4]), s[5] += fmaf(m1.y, s[5], acc[5]), s[6] += fmaf(m1.z, s[6], acc[6]), s[7] += fmaf(m1.w, s[7], acc[7]);
+        __syncthreads();  // the stage is read: the copies after next may overwrite it
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    if (write_state && active) {
+#pragma unroll
+        for (int g = 0; g < 2; ++g) {
+            const int r = (g * LANES + sub) * 4;
+            if (r < dim) *reinterpret_cast<float4*>(S + r) = make_float4(s[4 * g], s[4 * g + 1], s[4 * g + 2], s[4 * g + 3]);
+        }
+    }
+}
+
+template <typename T, int LANES>
+int launch_walk(const DeltaChunks& w, const void* v, int ldv, float* out, int ldo, float* state, const int* seq_q_start,
+                const int* seq_state_slot, int seqs, int heads, int dim, int vdim, int write_state, cudaStream_t s) {
+    constexpr int COLS = DC_THREADS / LANES;
+    const size_t smem = 2 * sizeof(DeltaStage<LANES>);
+    const int rc = ferris_allow_dynamic_smem((const void*)delta_chunk_walk_kernel<T, LANES>, smem);
+    if (rc != FERRIS_OK) return rc;
+    ferris_launch(delta_chunk_walk_kernel<T, LANES>, dim3(seqs, heads, (vdim + COLS - 1) / COLS), dim3(DC_THREADS), smem, s, w,
+                  (const T*)v, ldv, out, ldo, state, seq_q_start, seq_state_slot, heads, dim, vdim, write_state);
+    FERRIS_LAUNCH_CHECK();
+}
+
+}  // namespace
+
+// Floats of scratch that ferris_delta_chunks wants.
+FERRIS_API long long ferris_delta_chunks_scratch(int tokens, int seqs, int heads, int dim) {
+    const long long rows = (long long)tokens * heads, places = tokens / DC_TOKENS + seqs + 1;
+    return rows * (3LL * dim + 2 * DC_TOKENS) + places * heads * dim;
+}
+
+// Arguments as ferris_gated_recurrence with row decays (z, rates); dim a multiple of four, every pointer but v's on 16 bytes;
+// longest: the most tokens a request brings.
+FERRIS_API int ferris_delta_chunks(const void* q, int ldq, const void* k, int ldk, const void* v, int ldv, int dtype, const float* z,
+                                   int ldz, const float* rates, const float* beta, const float* qscale, const float* kscale,
+                                   float* out, int ldo, float* state, const int* seq_q_start, const int* seq_state_slot, int tokens,
+                                   int seqs, int heads, int qk_heads, int dim, int vdim, int write_state, int longest, float* scratch,
+                                   long long scratch_floats, void* stream) {
+    if (seqs <= 0 || tokens <= 0) return FERRIS_OK;
+    if (heads <= 0 || qk_heads <= 0 || heads % qk_heads) FERRIS_REFUSE("delta chunks: %d heads over %d q/k heads", heads, qk_heads);
+    if (dim <= 0 || dim > 256 || dim % 4 || vdim <= 0) FERRIS_REFUSE("delta chunks: heads of %d x %d (multiples of 4, at most 256 rows)", dim, vdim);
+    if (heads > 65535 || (vdim + 3) / 4 > 65535 || longest <= 0) FERRIS_REFUSE("delta chunks: too many heads or columns for one launch, or no length");
+    if (!z || !rates || !beta || !scratch || scratch_floats < ferris_delta_chunks_scratch(tokens, seqs, heads, dim))
+        FERRIS_REFUSE("delta chunks: decays, step sizes or scratch are missing");
+    if (((uintptr_t)state | (uintptr_t)scratch) & 15) FERRIS_REFUSE("delta chunks: state and scratch must start on 16 bytes");
+    const long long chunks_max = (longest + DC_TOKENS - 1) / DC_TOKENS;
+    if (chunks_max * seqs > 2147483647LL) FERRIS_REFUSE("delta chunks: %d requests of up to %d tokens are more than one launch takes", seqs, longest);
+    const size_t rows = (size_t)tokens * heads;
+    DeltaChunks w;
+    w.kt = scratch, w.qt = w.kt + rows * dim, w.kh = w.qt + rows * dim;
+    w.mm = w.kh + rows * dim, w.bm = w.mm + rows * DC_TOKENS, w.dm = w.bm + rows * DC_TOKENS;
+    cudaStream_t s = (cudaStream_t)stream;
+    const size_t smem = 3 * (size_t)DC_TOKENS * (dim + 1) * sizeof(float);
+    const dim3 grid((unsigned)(chunks_max * seqs), heads);
+#define FERRIS_DC_GO(T)                                                                                                      \
+    do {                                                                                                                     \
+        int rc = ferris_allow_dynamic_smem((const void*)delta_chunk_prepare_kernel<T>, smem);                                 \
+        if (rc != FERRIS_OK) return rc;                                                                                      \
+        ferris_launch(delta_chunk_prepare_kernel<T>, grid, dim3(DC_PREP_THREADS), smem, s, (const T*)q, ldq, (const T*)k, ldk, z, \
+                      ldz, rates, beta, qscale, kscale, seq_q_start, (int)chunks_max, heads, qk_heads, dim, w);               \
+        if (dim <= 32) return launch_walk<T, 4>(w, v, ldv, out, ldo, state, seq_q_start, seq_state_slot, seqs, heads, dim, vdim, write_state, s); \
+        if (dim <= 64) return launch_walk<T, 8>(w, v, ldv, out, ldo, state, seq_q_start, seq_state_slot, seqs, heads, dim, vdim, write_state, s); \
+        if (dim <= 128) return launch_walk<T, 16>(w, v, ldv, out, ldo, state, seq_q_start, seq_state_slot, seqs, heads, dim, vdim, write_state, s); \
+        return launch_walk<T, 32>(w, v, ldv, out, ldo, state, seq_q_start, seq_state_slot, seqs, heads, dim, vdim, write_state, s); \
+    } while (0)
+    if (dtype == FERRIS_F32) FERRIS_DC_GO(float);
+    if (dtype == FERRIS_BF16) FERRIS_DC_GO(bf16);
+#undef FERRIS_DC_GO
+    FERRIS_REFUSE("delta chunks: unknown dtype %d", dtype);
+}

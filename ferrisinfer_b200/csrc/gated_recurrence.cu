@@ -12,7 +12,8 @@
 // Either form also takes a decay per ROW of the state (per key channel) that changes with every token, given as
 // fp32 numbers z per (token, head, row): the row's decay is sigmoid(z)^power = exp(-softplus(-z) * power), or, with a rate
 // per head, exp(-softplus(z) * rate[head]), formed in fp32 where the rows are staged; the decay per head is then left out
-// (gated linear attention; a delta rule whose channels forget at their own pace).  What is staged is
+// (gated linear attention; a delta rule whose channels forget at their own pace, whose portions of prompts have a form of
+// their own in delta_chunks.cu).  What is staged is
 // the decay MINUS ONE, expm1(-softplus(-z) power), and a row moves on as s + ((decay - 1) s + k u): a decay close to one
 // rounded to 24 bits is off by a fixed share of what it takes away, with the same sign at every step where the row's
 // decay hardly changes, which over a thousand tokens shows in 32-bit logits; this way only the sum rounds, at the state's
@@ -44,9 +45,8 @@ constexpr int GR_KPL = 8;    // rows of the state that a lane holds
 constexpr int GR_STAGE = 16;  // tokens in shared memory at a time
 constexpr int GR_MAX_DIM = 256;
 
-__device__ __forceinline__ float softplus_g(float v) { return fmaxf(v, 0.0f) + log1pf(expf(-fabsf(v))); }
 // the logarithm of a row's decay: sign = -1 and rate = power, or sign = 1 and rate = the head's
-__device__ __forceinline__ float row_log_decay(float z, float sign, float rate) { return -softplus_g(sign * z) * rate; }
+__device__ __forceinline__ float row_log_decay(float z, float sign, float rate) { return -ferris_softplus(sign * z) * rate; }
 
 // decay[t, h] = exp(-exp(A_log[h]) * dt), dt = softplus(a[t, h] + dt_bias[h]);  beta[t, h] = sigmoid(b[t, h]) (kind 0)
 // or dt itself (kind 1).  With unit norms: qscale[t, g] = q_mul / sqrt(sum q^2 + eps), kscale[t, g] = 1 / sqrt(sum k^2 + eps).
@@ -65,7 +65,7 @@ __global__ void __launch_bounds__(128) recurrence_gates_kernel(const T* proj, in
     for (int h = threadIdx.x; h < heads; h += blockDim.x) {
         float dt = 0.0f;
         if (A_log) {  // without: the step size alone (the decays are formed elsewhere)
-            dt = softplus_g(to_float(row[a_off + h]) + dt_bias[h]);
+            dt = ferris_softplus(to_float(row[a_off + h]) + dt_bias[h]);
             decay[(size_t)t * heads + h] = expf(-expf(A_log[h]) * dt);
         }
         beta[(size_t)t * heads + h] = beta_kind == 0 ? 1.0f / (1.0f + expf(-to_float(row[b_off + h]))) : dt;

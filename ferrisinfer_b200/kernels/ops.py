@@ -832,8 +832,7 @@ def paged_attention_simt(qkv: torch.Tensor, out: torch.Tensor, k_cache: torch.Te
     window's tokens the query sees one row of ``pooled`` for every run of positions that lies wholly before the window.
     ``keep_first`` (with a window, without ``pooled``): beside the window's tokens the query sees the request's first
     ``keep_first`` tokens.
-    bf16 without a distance penalty and with values in rows of their own runs on tensor cores where the geometry allows it
-    (``set_attention_rows``); everything else on CUDA cores."""
+    bf16 without a distance penalty runs on tensor cores where the geometry allows it (``set_attention_rows``); everything else on CUDA cores."""
     dv = int(v_head_dim or head_dim)
     if chunk:
         if window or chunk < 0:
@@ -893,14 +892,14 @@ def paged_attention_simt(qkv: torch.Tensor, out: torch.Tensor, k_cache: torch.Te
     single = max_q_len <= 1 and max_kv_len > 0 and workspace is not None
     # bf16 without a distance penalty: on tensor cores, with the weights' 24 bits kept (the tiled kernel switched off, the
     # CUDA-core form of single tokens is asked for)
-    if (_attention_rows and qkv.dtype == torch.bfloat16 and not v_stride and terms.slopes is None and terms.log_r1 is None
+    if (_attention_rows and qkv.dtype == torch.bfloat16 and terms.slopes is None and terms.log_r1 is None
             and (max_q_len <= 1 or _attention_tiled) and ldq % 8 == 0 and ldo % 2 == 0 and qkv.data_ptr() % 16 == 0
             and _lib().ferris_attention_rows_takes(num_heads, num_kv_heads, head_dim, dv, 1 if max_q_len > 1 else 0)):
         _check(_lib().ferris_attention_rows(
             _ptr(qkv), _c_int(ldq), _ptr(out), _c_int(ldo), _ptr(k_cache), _ptr(v_cache), _ptr(block_tables),
             _c_int(block_tables.shape[1]), _ptr(token_seq), _ptr(positions), _c_int(T), _c_int(num_heads),
             _c_int(num_kv_heads), _c_int(head_dim), _c_int(dv), _c_int(k_cache.shape[2]),
-            _c_int(-chunk if chunk else (window or 0)), _c_float(scale), _ptr(terms.sink), *pool_args,
+            _c_int(-chunk if chunk else (window or 0)), _c_float(scale), _ptr(terms.sink), _c_int(v_stride), *pool_args,
             _c_int(1 if max_q_len > 1 else 0), _c_int(span if single else 0), _stream()), "attention rows")
         return
     fn = _lib().ferris_paged_attention_simt
@@ -1230,18 +1229,23 @@ def recurrence_gates(proj: torch.Tensor, a_off: Optional[int], b_off: Optional[i
     )
 
 
+DELTA_CHUNKS_FROM = 17  # the longest request of a step from which on the channel-decay delta rule runs sixteen tokens at a time
+
+
 def gated_recurrence(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: Optional[torch.Tensor], beta: torch.Tensor,
                      out: torch.Tensor, state: torch.Tensor, ctx, heads: int, qk_heads: int, dim: int, vdim: int,
                      delta_rule: bool, qscale: Optional[torch.Tensor] = None, kscale: Optional[torch.Tensor] = None,
                      skip: Optional[torch.Tensor] = None, write_state: bool = True,
-                     row_decay: Optional[tuple] = None):
+                     row_decay: Optional[tuple] = None, chunks: Optional[bool] = None):
     """The recurrence of the step's tokens, request by request from each request's state (fp32 [slots, heads, vdim, dim]: S transposed):
     plain: S <- decay S + k (beta v)^T, o = S^T q + skip v;  delta rule: S <- decay S, u = beta (v - S^T k), S <- S + k u^T,
     o = S^T q.  ``q``, ``k``: [T, qk_heads x dim] (views with contiguous rows; value head h uses q/k head
     h / (heads / qk_heads)), optionally times one fp32 factor per (token, q/k head) each; ``v``: [T, heads x vdim];
     ``decay``, ``beta``: fp32 [T, heads]; ``out``: fp32 [T, heads x vdim].  ``row_decay`` = (z fp32 [T, heads x dim], rates fp32
     [heads]), with the delta rule and ``decay`` None: every row (key channel) of the state decays by a number of its own,
-    exp(-softplus(z) rate), formed in the kernel."""
+    exp(-softplus(z) rate), formed in the kernel; a step whose longest request brings DELTA_CHUNKS_FROM tokens or more
+    (``chunks`` None; True / False: whatever its length) then runs chunks of sixteen tokens at a time where the heads are a
+    multiple of four (csrc/delta_chunks.cu; scratch from the step's workspace)."""
     T, wq, ldq = _rows(q, "recurrence queries")
     T1, wk, ldk = _rows(k, "recurrence keys")
     T2, wv, ldv = _rows(v, "recurrence values")
@@ -1274,14 +1278,31 @@ def gated_recurrence(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: O
         _need(skip, "skip weights", torch.float32)
         if skip.numel() != heads:
             raise KernelError("recurrence: one skip weight per head is needed")
+    longest = int(getattr(ctx, "max_q_len", 0) or T)
+    if row_decay is not None and skip is None and dim % 4 == 0 and (longest >= DELTA_CHUNKS_FROM if chunks is None else chunks):
+        fn = _lib().ferris_delta_chunks_scratch
+        fn.restype = ctypes.c_longlong
+        floats = int(fn(_c_int(T), _c_int(ctx.num_seqs), _c_int(heads), _c_int(dim)))
+        ws = getattr(ctx, "workspace", None)
+        scratch = ws.get("delta_chunks", (floats,), torch.float32) if ws is not None else \
+            torch.empty(floats, dtype=torch.float32, device=q.device)
+        _check(
+            _lib().ferris_delta_chunks(_ptr(q), _c_int(ldq), _ptr(k), _c_int(ldk), _ptr(v), _c_int(ldv), _c_int(_dt(q, "recurrence")),
+                                       _ptr(z), _c_int(ldz), _ptr(rates), _ptr(beta), _ptr(qscale), _ptr(kscale), _ptr(out),
+                                       _c_int(ldo), _ptr(state), _ptr(ctx.seq_q_start), _ptr(ctx.seq_state_slot), _c_int(T),
+                                       _c_int(ctx.num_seqs), _c_int(heads), _c_int(qk_heads), _c_int(dim), _c_int(vdim),
+                                       _c_int(1 if write_state else 0), _c_int(longest), _ptr(scratch), ctypes.c_longlong(floats),
+                                       _stream()),
+            "delta rule in chunks", 2,
+        )
+        return
     _check(
         _lib().ferris_gated_recurrence(_ptr(q), _c_int(ldq), _ptr(k), _c_int(ldk), _ptr(v), _c_int(ldv),
                                        _c_int(_dt(q, "recurrence")), _ptr(decay), _ptr(beta), _ptr(qscale), _ptr(kscale),
                                        _ptr(skip), _ptr(out), _c_int(ldo), _ptr(state), _ptr(ctx.seq_q_start),
                                        _ptr(ctx.seq_state_slot), _c_int(ctx.num_seqs), _c_int(heads), _c_int(qk_heads),
                                        _c_int(dim), _c_int(vdim), _c_int(1 if delta_rule else 0),
-                                       _c_int(1 if write_state else 0), _c_int(int(getattr(ctx, "max_q_len", 0) or T)),
-                                       _ptr(z), _c_int(ldz), _ptr(rates), _stream()),
+                                       _c_int(1 if write_state else 0), _c_int(longest), _ptr(z), _c_int(ldz), _ptr(rates), _stream()),
         "gated recurrence",
     )
 

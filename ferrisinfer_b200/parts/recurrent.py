@@ -150,7 +150,7 @@ class GatedDeltaRule(Mixer):
 
 class ChannelDeltaRule(GatedDeltaRule):
     """The inner sizes of the two low-rank projections stand in no configuration key: the folder's tensors decide (a random
-    folder draws 16)."""
+    folder draws a head's size)."""
 
     def tensor_specs(self, prefix):
         H, nh = self.hidden_size, self.num_heads
@@ -163,11 +163,11 @@ class ChannelDeltaRule(GatedDeltaRule):
             TensorSpec(f"{prefix}.b", (nh, H), "matrix"),
             TensorSpec(f"{prefix}.A_log", (nh,), "vector"),
             TensorSpec(f"{prefix}.norm", (self.v_head_dim,), "norm"),
-            TensorSpec(f"{prefix}.a1", (-16, H), "matrix"),
-            TensorSpec(f"{prefix}.a2", (channels, -16), "matrix"),
+            TensorSpec(f"{prefix}.a1", (-self.head_dim, H), "matrix"),
+            TensorSpec(f"{prefix}.a2", (channels, -self.head_dim), "matrix"),
             TensorSpec(f"{prefix}.dt_bias", (channels,), "vector"),
-            TensorSpec(f"{prefix}.g1", (-16, H), "matrix"),
-            TensorSpec(f"{prefix}.g2", (self.v_size, -16), "matrix"),
+            TensorSpec(f"{prefix}.g1", (-self.v_head_dim, H), "matrix"),
+            TensorSpec(f"{prefix}.g2", (self.v_size, -self.v_head_dim), "matrix"),
             TensorSpec(f"{prefix}.o", (H, self.v_size), "matrix"),
         ]
 

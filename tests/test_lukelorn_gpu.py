@@ -292,7 +292,8 @@ def plain_delta(q, k, v, z, beta, rates, heads, qk_heads, dim, vdim):
 @pytest.mark.parametrize("heads,qk_heads,dim,vdim", [(4, 2, 32, 24), (3, 3, 15, 9), (2, 1, 64, 64), (6, 2, 100, 33), (2, 2, 128, 128),
                                                       (1, 1, 256, 40), (3, 1, 8, 5)])
 def test_delta_rule_with_a_decay_per_channel(device, heads, qk_heads, dim, vdim, dtype):
-    """Whole, in portions and token by token, from a slot between others."""
+    """Whole, in portions and token by token, from a slot between others; the form that walks the tokens, the one that takes
+    sixteen at a time (portions of no multiple of sixteen too), and whichever a step would take."""
     ops = _ops()
     T = 150
     q, k, v, z, beta = delta_inputs(T, heads, qk_heads, dim, vdim, heads * dim)
@@ -301,7 +302,8 @@ def test_delta_rule_with_a_decay_per_channel(device, heads, qk_heads, dim, vdim,
     want, last = plain_delta(q, k, v, z, beta, rates, heads, qk_heads, dim, vdim)
     want = want.reshape(T, heads * vdim)
     dev = lambda t: t.to(device)
-    for cuts in ([T], [70, 1, 50, 2, 27], [100] + [1] * 50, [2] * 20 + [64, 46]):
+    for cuts, chunks in (([T], None), ([70, 1, 50, 2, 27], None), ([100] + [1] * 50, None), ([2] * 20 + [64, 46], None),
+                         ([T], False), ([T], True), ([16, 48, 17, 1, 2, 15, 33, 18], True), ([1] * 20 + [130], True)):
         state = torch.randn(3, heads, vdim, dim, device=device)
         others = state[:2].clone()
         state[2] = 0.0
@@ -311,8 +313,8 @@ def test_delta_rule_with_a_decay_per_channel(device, heads, qk_heads, dim, vdim,
             sl = slice(pos, pos + n)
             out = torch.empty(n, heads * vdim, device=device)
             ops.gated_recurrence(dev(q[sl]), dev(k[sl]), dev(v[sl]), None, dev(beta[sl]), out, state, ctx, heads, qk_heads, dim, vdim,
-                                 delta_rule=True, row_decay=(dev(z[sl]), dev(rates)))
-            assert torch.allclose(out.cpu().double(), want[sl], atol=1e-4, rtol=2e-4), (cuts[:3], pos)
+                                 delta_rule=True, row_decay=(dev(z[sl]), dev(rates)), chunks=chunks)
+            assert torch.allclose(out.cpu().double(), want[sl], atol=1e-4, rtol=2e-4), (cuts[:3], chunks, pos)
             pos += n
         assert torch.allclose(state[2].cpu().double().transpose(1, 2), last, atol=1e-4, rtol=2e-4)  # S lies transposed
         assert torch.equal(state[:2], others)
@@ -345,6 +347,22 @@ def test_delta_rule_of_several_requests_keeps_their_states_apart(device):
             at += step[i]
             done[i] += step[i]
     assert done == lens
+
+
+def test_delta_rule_whose_channels_forget_at_once(device):
+    """Decays of e^-40 a token beside decays of almost one in the same head: nothing overflows, nothing is lost."""
+    ops = _ops()
+    heads, dim, vdim, T = 2, 32, 16, 100
+    q, k, v, z, beta = delta_inputs(T, heads, heads, dim, vdim, 3)
+    z = torch.where(torch.arange(heads * dim) % 3 == 0, torch.full_like(z, 40.0), torch.where(torch.rand_like(z) < 0.2, z + 30.0, z))
+    rates = torch.ones(heads)
+    want = plain_delta(q, k, v, z, beta, rates, heads, heads, dim, vdim)[0].reshape(T, -1)
+    dev = lambda t: t.to(device)
+    for chunks in (False, True):
+        state, out = torch.zeros(1, heads, vdim, dim, device=device), torch.empty(T, heads * vdim, device=device)
+        ops.gated_recurrence(dev(q), dev(k), dev(v), None, dev(beta), out, state, fake_ctx(device, [T], [0], [0]), heads, heads, dim, vdim,
+                             delta_rule=True, row_decay=(dev(z), dev(rates)), chunks=chunks)
+        assert torch.allclose(out.cpu().double(), want, atol=1e-4, rtol=2e-4), chunks
 
 
 @pytest.mark.parametrize("dtype", [F32, BF16])
