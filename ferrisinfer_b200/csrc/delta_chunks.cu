@@ -19,6 +19,11 @@
 // with S_0 are independent of one another, their sums over the lanes are reduced together (a lane ends with a token's sum, in
 // 16 + 8 + .. exchanges instead of 16 x log2), and only the 16 x 16 products with M and B tie the tokens together.  The next
 // chunk's rows come in by asynchronous copies meanwhile.
+//
+// For bf16 activations the walk runs on tensor cores: a block takes sixteen columns, its four warps share the rows of S, and
+// D^T = S_0^T K^T, E^T = S_0^T Q^T and the sum over the writes are products of tf32 fragments with fp32 sums.  Each operand x is
+// cut into its leading eleven bits and the rest, and the products big x big, big x rest and rest x big are added, which keeps 21
+// bits and more of every product; the state itself is only ever added to in fp32 outside the fragments' accumulators.
 #include <math.h>
 
 #include "common.cuh"
@@ -86,21 +91,35 @@ __global__ void __launch_bounds__(DC_PREP_THREADS) delta_chunk_prepare_kernel(
         w.qt[at] = Qs[t * pitch + c] * e;
         w.kh[at] = kv * expf(Ls[(n - 1) * pitch + c] - L);
     }
+    constexpr float LOG2E = 1.4426950408889634f;
     // a warp takes tokens w and 15 - w: seventeen pairs each
     for (int half = 0; half < 2; ++half) {
         const int t = half ? DC_TOKENS - 1 - warp : warp;
         if (t >= n) continue;
+        float l[8], kv[8], qv[8];  // the token's row, a lane's channels lane, lane + 32, ..
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            const int c = lane + 32 * j;
+            l[j] = kv[j] = qv[j] = 0.0f;
+            if (c < dim) l[j] = Ls[t * pitch + c], kv[j] = Ks[t * pitch + c], qv[j] = Qs[t * pitch + c];
+        }
         for (int i = 0; i <= t; ++i) {
             float a = 0.0f, b = 0.0f;
-            for (int c = lane; c < dim; c += 32) {
-                const float e = expf(Ls[t * pitch + c] - Ls[i * pitch + c]) * Ks[i * pitch + c];
-                a = fmaf(Ks[t * pitch + c], e, a), b = fmaf(Qs[t * pitch + c], e, b);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) {
+                const int c = lane + 32 * j;
+                if (32 * j < dim && c < dim) {
+                    const float e = exp2f((l[j] - Ls[i * pitch + c]) * LOG2E) * Ks[i * pitch + c];
+                    a = fmaf(kv[j], e, a), b = fmaf(qv[j], e, b);
+                }
             }
-            a = warp_sum(a), b = warp_sum(b);
-            if (lane == 0) {
-                As[t][i] = a;
-                w.bm[((size_t)(first + t) * heads + head) * DC_TOKENS + i] = b;
-            }
+            // both sums at once: the lower lanes end with a's, the upper ones with b's
+            const bool upper = lane & 16;
+            float sum = (upper ? b : a) + __shfl_xor_sync(0xffffffffu, upper ? a : b, 16);
+#pragma unroll
+            for (int o = 8; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+            if (lane == 0) As[t][i] = sum;
+            if (lane == 16) w.bm[((size_t)(first + t) * heads + head) * DC_TOKENS + i] = sum;
         }
         if (lane > t && lane < DC_TOKENS) w.bm[((size_t)(first + t) * heads + head) * DC_TOKENS + lane] = 0.0f;
     }
@@ -318,6 +337,238 @@ __global__ void __launch_bounds__(DC_THREADS) delta_chunk_walk_kernel(
     }
 }
 
+// ------------------------------------------------------------------------------------------ the walk on tensor cores
+constexpr int DM_COLS = 16, DM_STAGES = 3, DM_WARPS = DC_THREADS / 32;
+
+__device__ __forceinline__ void dc_copy16_or_zero(float* dst, const float* src, bool there) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src),
+                 "r"(there ? 16 : 0)
+                 : "memory");
+}
+__device__ __forceinline__ void split_tf32(float x, uint32_t& big, uint32_t& rest) {
+    big = __float_as_uint(x) & 0xffffe000u;
+    rest = __float_as_uint(x - __uint_as_float(big));
+}
+__device__ __forceinline__ void mma_tf32_1688(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+
+// Sizes in floats of a stage for heads of `dim`: rows of kt, qt and kh are dim + 8 floats apart, so that the fragments' reads
+// (four or eight tokens by neighbouring rows of S) fall into different banks.
+__host__ __device__ constexpr int dm_pitch(int dim) { return dim + 8; }
+__host__ __device__ constexpr int dm_stage_floats(int dim) { return 3 * DC_TOKENS * dm_pitch(dim) + dim + 2 * DC_TOKENS * DC_PITCH; }
+
+// TILES: eight-row pieces of S that a warp holds at most (warp w's are w, w + 4, ..); dim a multiple of eight.
+template <typename T, int TILES>
+__global__ void __launch_bounds__(DC_THREADS) delta_chunk_walk_mma_kernel(
+    const DeltaChunks w, const T* v, int ldv, float* __restrict__ out, int ldo, float* state, const int* __restrict__ seq_q_start,
+    const int* __restrict__ seq_state_slot, int heads, int dim, int vdim, int write_state) {
+    extern __shared__ __align__(16) float dc_smem[];
+    __shared__ __align__(16) float pd[DM_WARPS][DM_COLS][DC_PITCH], pe[DM_WARPS][DM_COLS][DC_PITCH];
+    __shared__ __align__(16) float ws[DM_COLS][DC_PITCH], us[DM_COLS][DC_PITCH];
+    pdl_wait();
+    pdl_launch_dependents();
+    const int seq = blockIdx.x, head = blockIdx.y, col0 = blockIdx.z * DM_COLS, tid = threadIdx.x;
+    const int warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
+    const int row0 = seq_q_start[seq], row1 = seq_q_start[seq + 1];
+    if (row1 <= row0) return;
+    const int pitch = dm_pitch(dim), stage_floats = dm_stage_floats(dim), tiles = dim >> 3, d4 = dim >> 2;
+    float* S = state + (((size_t)seq_state_slot[seq] * heads + head) * vdim + col0) * (size_t)dim;
+    // S^T as an accumulator fragment: [0], [1]: column g, rows 8 j + 2 t4, + 1; [2], [3]: column g + 8.  The same registers are an A
+    // fragment whose inner index is permuted (slot t4 is row 2 t4, slot t4 + 4 row 2 t4 + 1); B reads its rows the same way.
+    float s[TILES][4];
+#pragma unroll
+    for (int j = 0; j < TILES; ++j) {
+        const int tile = warp + DM_WARPS * j, r = 8 * tile + 2 * t4;
+#pragma unroll
+        for (int a = 0; a < 2; ++a) {
+            float2 x = make_float2(0.0f, 0.0f);
+            if (tile < tiles && col0 + g + 8 * a < vdim) x = *reinterpret_cast<const float2*>(S + (size_t)(g + 8 * a) * dim + r);
+            s[j][2 * a] = x.x, s[j][2 * a + 1] = x.y;
+        }
+    }
+    auto fetch = [&](int first, int stage) {
+        if (first < row1) {
+            float* kt = dc_smem + stage * stage_floats;
+            float* dm = kt + 3 * DC_TOKENS * pitch;
+            float* mm = dm + dim;
+            float* bm = mm + DC_TOKENS * DC_PITCH;
+            for (int x = tid; x < DC_TOKENS * d4; x += DC_THREADS) {
+                const int t = x / d4, c = (x - t * d4) * 4;
+                const bool there = first + t < row1;  // tokens beyond the last one are zeros
+                const size_t at = ((size_t)(first + (there ? t : 0)) * heads + head) * dim + c;
+                dc_copy16_or_zero(kt + t * pitch + c, w.kt + at, there);
+                dc_copy16_or_zero(kt + (DC_TOKENS + t) * pitch + c, w.qt + at, there);
+                dc_copy16_or_zero(kt + (2 * DC_TOKENS + t) * pitch + c, w.kh + at, there);
+            }
+            for (int x = tid; x < d4; x += DC_THREADS)
+                dc_copy16_or_zero(dm + 4 * x, w.dm + ((size_t)(first / DC_TOKENS + seq) * heads + head) * dim + 4 * x, true);
+            if (tid < DC_TOKENS * 4) {
+                const int t = tid >> 2, c = (tid & 3) * 4;
+                const bool there = first + t < row1;
+                const size_t at = ((size_t)(first + (there ? t : 0)) * heads + head) * DC_TOKENS + c;
+                dc_copy16_or_zero(mm + t * DC_PITCH + c, w.mm + at, there);
+                dc_copy16_or_zero(bm + t * DC_PITCH + c, w.bm + at, there);
+            }
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    const int cl = tid >> 3, tk = (tid & 7) * 2;  // this thread's column and its two tokens between the products
+    const bool active = col0 + cl < vdim;
+    T pv[2];
+    auto request_v = [&](int first) {
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+            const int t = first + tk + j;
+            pv[j] = from_float<T>(0.0f);
+            if (t < row1 && active) pv[j] = v[(size_t)t * ldv + (size_t)head * vdim + col0 + cl];
+        }
+    };
+    fetch(row0, 0);
+    fetch(row0 + DC_TOKENS, 1);
+    request_v(row0);
+    int stage = 0;
+    for (int first = row0; first < row1; first += DC_TOKENS) {
+        asm volatile("cp.async.wait_group 1;" ::: "memory");
+        __syncthreads();  // the stage is there; everyone is done with the one before, which the next copies overwrite
+        fetch(first + 2 * DC_TOKENS, stage == 0 ? 2 : stage - 1);
+        const float v0 = to_float(pv[0]), v1 = to_float(pv[1]);
+        request_v(first + DC_TOKENS);
+        const float* kt = dc_smem + stage * stage_floats;
+        const float* qt = kt + DC_TOKENS * pitch;
+        const float* kh = qt + DC_TOKENS * pitch;
+        const float* dm = kh + DC_TOKENS * pitch;
+        const float* mm = dm + dim;
+        const float* bm = mm + DC_TOKENS * DC_PITCH;
+        // D^T and E^T over the warp's rows: two token tiles each, the small products in accumulators of their own
+        float D[2][4], Dr[2][4], E[2][4], Er[2][4];
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) D[n][e] = Dr[n][e] = E[n][e] = Er[n][e] = 0.0f;
+#pragma unroll
+        for (int j = 0; j < TILES; ++j) {
+            const int tile = warp + DM_WARPS * j;
+            if (tile < tiles) {
+                uint32_t ab[4], ar[4];
+                split_tf32(s[j][0], ab[0], ar[0]), split_tf32(s[j][2], ab[1], ar[1]);
+                split_tf32(s[j][1], ab[2], ar[2]), split_tf32(s[j][3], ab[3], ar[3]);
+#pragma unroll
+                for (int n = 0; n < 2; ++n) {
+                    const int at = (8 * n + g) * pitch + 8 * tile + 2 * t4;
+                    const float2 x = *reinterpret_cast<const float2*>(kt + at);
+                    const float2 y = *reinterpret_cast<const float2*>(qt + at);
+                    uint32_t xb0, xr0, xb1, xr1, yb0, yr0, yb1, yr1;
+                    split_tf32(x.x, xb0, xr0), split_tf32(x.y, xb1, xr1);
+                    split_tf32(y.x, yb0, yr0), split_tf32(y.y, yb1, yr1);
+                    mma_tf32_1688(D[n], ab, xb0, xb1);
+                    mma_tf32_1688(E[n], ab, yb0, yb1);
+                    mma_tf32_1688(Dr[n], ab, xr0, xr1);
+                    mma_tf32_1688(Er[n], ab, yr0, yr1);
+                    mma_tf32_1688(Dr[n], ar, xb0, xb1);
+                    mma_tf32_1688(Er[n], ar, yb0, yb1);
+                }
+            }
+        }
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int a = 0; a < 2; ++a) {
+                const int c = g + 8 * a, t = 8 * n + 2 * t4;
+                *reinterpret_cast<float2*>(&pd[warp][c][t]) = make_float2(D[n][2 * a] + Dr[n][2 * a], D[n][2 * a + 1] + Dr[n][2 * a + 1]);
+                *reinterpret_cast<float2*>(&pe[warp][c][t]) = make_float2(E[n][2 * a] + Er[n][2 * a], E[n][2 * a + 1] + Er[n][2 * a + 1]);
+            }
+        __syncthreads();
+        float2 e = make_float2(0.0f, 0.0f), x = make_float2(0.0f, 0.0f);
+#pragma unroll
+        for (int q = 0; q < DM_WARPS; ++q) {
+            const float2 a = *reinterpret_cast<const float2*>(&pd[q][cl][tk]), b = *reinterpret_cast<const float2*>(&pe[q][cl][tk]);
+            x.x += a.x, x.y += a.y, e.x += b.x, e.y += b.y;
+        }
+        *reinterpret_cast<float2*>(&ws[cl][tk]) = make_float2(v0 - x.x, v1 - x.y);
+        __syncwarp();  // a column's eight threads are of one warp
+        // u = M w for the thread's two tokens
+        float u0 = 0.0f, u1 = 0.0f, y0 = 0.0f, y1 = 0.0f;
+#pragma unroll
+        for (int i = 0; i < DC_TOKENS; i += 4) {
+            const float4 f = *reinterpret_cast<const float4*>(&ws[cl][i]);
+            const float4 m = *reinterpret_cast<const float4*>(mm + tk * DC_PITCH + i);
+            const float4 n = *reinterpret_cast<const float4*>(mm + (tk + 1) * DC_PITCH + i);
+            u0 = fmaf(m.x, f.x, u0), y0 = fmaf(m.y, f.y, y0), u0 = fmaf(m.z, f.z, u0), y0 = fmaf(m.w, f.w, y0);
+            u1 = fmaf(n.x, f.x, u1), y1 = fmaf(n.y, f.y, y1), u1 = fmaf(n.z, f.z, u1), y1 = fmaf(n.w, f.w, y1);
+        }
+        *reinterpret_cast<float2*>(&us[cl][tk]) = make_float2(u0 + y0, u1 + y1);
+        __syncthreads();
+        // the writes: S^T += U^T K over the chunk's tokens, formed apart from the state and added to it in fp32
+        {
+            uint32_t ub[2][4], ur[2][4];
+#pragma unroll
+            for (int k = 0; k < 2; ++k) {
+                split_tf32(us[g][8 * k + t4], ub[k][0], ur[k][0]), split_tf32(us[g + 8][8 * k + t4], ub[k][1], ur[k][1]);
+                split_tf32(us[g][8 * k + t4 + 4], ub[k][2], ur[k][2]), split_tf32(us[g + 8][8 * k + t4 + 4], ub[k][3], ur[k][3]);
+            }
+#pragma unroll
+            for (int j = 0; j < TILES; ++j) {
+                const int tile = warp + DM_WARPS * j;
+                if (tile < tiles) {
+                    float acc[4] = {0.0f, 0.0f, 0.0f, 0.0f}, rest[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+#pragma unroll
+                    for (int k = 0; k < 2; ++k) {
+                        uint32_t b0, r0, b1, r1;
+                        split_tf32(kh[(8 * k + t4) * pitch + 8 * tile + g], b0, r0);
+                        split_tf32(kh[(8 * k + t4 + 4) * pitch + 8 * tile + g], b1, r1);
+                        mma_tf32_1688(acc, ub[k], b0, b1);
+                        mma_tf32_1688(rest, ub[k], r0, r1);
+                        mma_tf32_1688(rest, ur[k], b0, b1);
+                    }
+                    const float2 m = *reinterpret_cast<const float2*>(dm + 8 * tile + 2 * t4);
+                    s[j][0] += fmaf(m.x, s[j][0], acc[0] + rest[0]), s[j][1] += fmaf(m.y, s[j][1], acc[1] + rest[1]);
+                    s[j][2] += fmaf(m.x, s[j][2], acc[2] + rest[2]), s[j][3] += fmaf(m.y, s[j][3], acc[3] + rest[3]);
+                }
+            }
+        }
+        // o = E + B u
+        {
+            float o0 = e.x, o1 = e.y, z0 = 0.0f, z1 = 0.0f;
+#pragma unroll
+            for (int i = 0; i < DC_TOKENS; i += 4) {
+                const float4 f = *reinterpret_cast<const float4*>(&us[cl][i]);
+                const float4 m = *reinterpret_cast<const float4*>(bm + tk * DC_PITCH + i);
+                const float4 n = *reinterpret_cast<const float4*>(bm + (tk + 1) * DC_PITCH + i);
+                o0 = fmaf(m.x, f.x, o0), z0 = fmaf(m.y, f.y, z0), o0 = fmaf(m.z, f.z, o0), z0 = fmaf(m.w, f.w, z0);
+                o1 = fmaf(n.x, f.x, o1), z1 = fmaf(n.y, f.y, z1), o1 = fmaf(n.z, f.z, o1), z1 = fmaf(n.w, f.w, z1);
+            }
+            float* dst = out + (size_t)(first + tk) * ldo + (size_t)head * vdim + col0 + cl;
+            if (active && first + tk < row1) dst[0] = o0 + z0;
+            if (active && first + tk + 1 < row1) dst[ldo] = o1 + z1;
+        }
+        stage = stage + 1 == DM_STAGES ? 0 : stage + 1;
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    if (!write_state) return;
+#pragma unroll
+    for (int j = 0; j < TILES; ++j) {
+        const int tile = warp + DM_WARPS * j, r = 8 * tile + 2 * t4;
+#pragma unroll
+        for (int a = 0; a < 2; ++a)
+            if (tile < tiles && col0 + g + 8 * a < vdim)
+                *reinterpret_cast<float2*>(S + (size_t)(g + 8 * a) * dim + r) = make_float2(s[j][2 * a], s[j][2 * a + 1]);
+    }
+}
+
+template <typename T, int TILES>
+int launch_walk_mma(const DeltaChunks& w, const void* v, int ldv, float* out, int ldo, float* state, const int* seq_q_start,
+                    const int* seq_state_slot, int seqs, int heads, int dim, int vdim, int write_state, cudaStream_t s) {
+    const size_t smem = (size_t)DM_STAGES * dm_stage_floats(dim) * sizeof(float);
+    const int rc = ferris_allow_dynamic_smem((const void*)delta_chunk_walk_mma_kernel<T, TILES>, smem);
+    if (rc != FERRIS_OK) return rc;
+    ferris_launch(delta_chunk_walk_mma_kernel<T, TILES>, dim3(seqs, heads, (vdim + DM_COLS - 1) / DM_COLS), dim3(DC_THREADS), smem, s, w,
+                  (const T*)v, ldv, out, ldo, state, seq_q_start, seq_state_slot, heads, dim, vdim, write_state);
+    FERRIS_LAUNCH_CHECK();
+}
+
 template <typename T, int LANES>
 int launch_walk(const DeltaChunks& w, const void* v, int ldv, float* out, int ldo, float* state, const int* seq_q_start,
                 const int* seq_state_slot, int seqs, int heads, int dim, int vdim, int write_state, cudaStream_t s) {
@@ -372,6 +623,19 @@ FERRIS_API int ferris_delta_chunks(const void* q, int ldq, const void* k, int ld
         if (dim <= 128) return launch_walk<T, 16>(w, v, ldv, out, ldo, state, seq_q_start, seq_state_slot, seqs, heads, dim, vdim, write_state, s); \
         return launch_walk<T, 32>(w, v, ldv, out, ldo, state, seq_q_start, seq_state_slot, seqs, heads, dim, vdim, write_state, s); \
     } while (0)
+    if (dtype == FERRIS_BF16 && dim % 8 == 0) {
+        int rc = ferris_allow_dynamic_smem((const void*)delta_chunk_prepare_kernel<bf16>, smem);
+        if (rc != FERRIS_OK) return rc;
+        ferris_launch(delta_chunk_prepare_kernel<bf16>, grid, dim3(DC_PREP_THREADS), smem, s, (const bf16*)q, ldq, (const bf16*)k, ldk, z,
+                      ldz, rates, beta, qscale, kscale, seq_q_start, (int)chunks_max, heads, qk_heads, dim, w);
+#define FERRIS_DM_GO(TILES) \
+    return launch_walk_mma<bf16, TILES>(w, v, ldv, out, ldo, state, seq_q_start, seq_state_slot, seqs, heads, dim, vdim, write_state, s)
+        if (dim <= 32) FERRIS_DM_GO(1);
+        if (dim <= 64) FERRIS_DM_GO(2);
+        if (dim <= 128) FERRIS_DM_GO(4);
+        FERRIS_DM_GO(8);
+#undef FERRIS_DM_GO
+    }
     if (dtype == FERRIS_F32) FERRIS_DC_GO(float);
     if (dtype == FERRIS_BF16) FERRIS_DC_GO(bf16);
 #undef FERRIS_DC_GO

@@ -419,6 +419,58 @@ __global__ void __launch_bounds__(256) gated_group_norm_kernel(const float* o, i
     }
 }
 
+// The same for groups of whole 16-byte pieces of o, at most four a lane, which stay in registers between the sum of squares and
+// the scaling; the gate behind the norm.  A warp per group, the groups of all rows in one line.
+__device__ __forceinline__ float4 gate_load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 gate_load4(const bf16* p) {
+    const uint2 u = *reinterpret_cast<const uint2*>(p);
+    return make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xffff0000u), __uint_as_float(u.y << 16), __uint_as_float(u.y & 0xffff0000u));
+}
+__device__ __forceinline__ void gate_store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void gate_store4(bf16* p, float4 v) {
+    __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<uint32_t*>(&a), *reinterpret_cast<uint32_t*>(&b));
+}
+
+template <typename T, int PIECES>  // 16-byte pieces of o a lane holds: group <= 128 * PIECES
+__global__ void __launch_bounds__(256) gated_group_norm_vec_kernel(const float* o, int ldi, const T* gate, int ldg,
+                                                                   const float* __restrict__ w, int wlen, T* __restrict__ out, int ldo,
+                                                                   int rows, int groups, int group, float eps, int gate_kind) {
+    pdl_wait();
+    pdl_launch_dependents();
+    const int lane = threadIdx.x & 31;
+    const long long item = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (item >= (long long)rows * groups) return;
+    const int t = (int)(item / groups), base = (int)(item % groups) * group;
+    float4 x[PIECES], g[PIECES];
+    float ss = 0.0f;
+#pragma unroll
+    for (int i = 0; i < PIECES; ++i) {
+        const int c = (i * 32 + lane) * 4;
+        x[i] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (c < group) {
+            x[i] = *reinterpret_cast<const float4*>(o + (size_t)t * ldi + base + c);
+            if (gate) g[i] = gate_load4(gate + (size_t)t * ldg + base + c);
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < PIECES; ++i) ss = fmaf(x[i].x, x[i].x, fmaf(x[i].y, x[i].y, fmaf(x[i].z, x[i].z, fmaf(x[i].w, x[i].w, ss))));
+    const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)group + eps);
+    auto gated = [&](float z) {
+        const float sg = 1.0f / (1.0f + expf(-z));
+        return gate_kind == 1 ? z * sg : sg;
+    };
+#pragma unroll
+    for (int i = 0; i < PIECES; ++i) {
+        const int c = (i * 32 + lane) * 4;
+        if (c >= group) continue;
+        const float4 wv = *reinterpret_cast<const float4*>(w + (base + c) % wlen);
+        float4 y = make_float4(x[i].x * inv * wv.x, x[i].y * inv * wv.y, x[i].z * inv * wv.z, x[i].w * inv * wv.w);
+        if (gate) y.x *= gated(g[i].x), y.y *= gated(g[i].y), y.z *= gated(g[i].z), y.w *= gated(g[i].w);
+        gate_store4(out + (size_t)t * ldo + base + c, y);
+    }
+}
+
 template <typename T, bool DELTA, bool AHEAD, bool ROWDECAY = false, int MODE = 0>
 int launch_recurrence(const void* q, int ldq, const void* k, int ldk, const void* v, int ldv, const float* decay,
                       const float* beta, const float* qscale, const float* kscale, const float* skip, float* out, int ldo,
@@ -561,6 +613,22 @@ FERRIS_API int ferris_gated_group_norm(const float* o, int ldi, const void* gate
     const int groups = n / group;
     const int threads = group >= 512 ? 256 : (groups >= 8 ? 256 : (groups >= 4 ? 128 : (groups >= 2 ? 64 : 32)));
     cudaStream_t s = (cudaStream_t)stream;
+    const size_t four = dtype == FERRIS_F32 ? 16 : 8;  // bytes of four elements of gate and out
+    if ((dtype == FERRIS_F32 || dtype == FERRIS_BF16) && !(gate && gate_first) && group % 4 == 0 && group <= 512 && wlen % 4 == 0 && ldi % 4 == 0 &&
+        ldo % 4 == 0 && ldg % 4 == 0 && (((uintptr_t)o | (uintptr_t)w) & 15) == 0 && (uintptr_t)out % four == 0 && (uintptr_t)gate % four == 0) {
+        const long long blocks = ((long long)rows * groups + 7) / 8;
+        if (blocks > 2147483647LL) FERRIS_REFUSE("gated group norm: %d rows are more than one launch takes", rows);
+#define FERRIS_GGN(T, P)                                                                                                   \
+    ferris_launch(gated_group_norm_vec_kernel<T, P>, dim3((unsigned)blocks), dim3(256), 0, s, o, ldi, (const T*)gate, ldg, w, wlen, \
+                  (T*)out, ldo, rows, groups, group, eps, gate_kind)
+        if (dtype == FERRIS_F32) {
+            if (group <= 128) FERRIS_GGN(float, 1); else FERRIS_GGN(float, 4);
+        } else {
+            if (group <= 128) FERRIS_GGN(bf16, 1); else FERRIS_GGN(bf16, 4);
+        }
+#undef FERRIS_GGN
+        FERRIS_LAUNCH_CHECK();
+    }
     if (dtype == FERRIS_F32)
         ferris_launch(gated_group_norm_kernel<float>, dim3(rows), dim3(threads), 0, s, o, ldi, (const float*)gate, ldg, w, wlen, (float*)out, ldo, n, group, eps, gate_kind, gate_first);
     else if (dtype == FERRIS_BF16)

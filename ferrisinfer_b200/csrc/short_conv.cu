@@ -50,6 +50,65 @@ __global__ void __launch_bounds__(256) short_conv_apply_kernel(
     out[(size_t)t * ldo + c] = from_float<T>(acc);
 }
 
+// `apply` for steps of many tokens: a thread takes two neighbouring channels and SC_RUN tokens in a row, holds the TAPS - 1
+// inputs before the next token in registers and reads every row once.  The sums are formed in the same order.
+constexpr int SC_RUN = 16;
+__device__ __forceinline__ float2 sc_load2(const float* p) { return *reinterpret_cast<const float2*>(p); }
+__device__ __forceinline__ float2 sc_load2(const bf16* p) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p)); }
+__device__ __forceinline__ void sc_store2(float* p, float a, float b) { *reinterpret_cast<float2*>(p) = make_float2(a, b); }
+__device__ __forceinline__ void sc_store2(bf16* p, float a, float b) { *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(a, b); }
+
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(128) short_conv_runs_kernel(
+    const T* y, int ldy, T* __restrict__ out, int ldo, const float* __restrict__ w, const float* state,
+    const int* __restrict__ token_seq, const int* __restrict__ positions, const int* __restrict__ seq_start_pos,
+    const int* __restrict__ seq_state_slot, int tokens, int channels, const float* __restrict__ bias, int residual, int act) {
+    constexpr int N = TAPS - 1;
+    pdl_wait();
+    pdl_launch_dependents();
+    const int c = 2 * (blockIdx.y * blockDim.x + threadIdx.x);
+    if (c >= channels) return;
+    const int t0 = blockIdx.x * SC_RUN, t1 = min(tokens, t0 + SC_RUN);
+    float w0[TAPS], w1[TAPS];
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) w0[j] = w[(size_t)c * TAPS + j], w1[j] = w[(size_t)(c + 1) * TAPS + j];
+    const float2 b = bias ? sc_load2(bias + c) : make_float2(0.0f, 0.0f);
+    float2 own[SC_RUN];  // all rows of the run are requested before the first is used
+#pragma unroll
+    for (int i = 0; i < SC_RUN; ++i)
+        if (t0 + i < t1) own[i] = sc_load2(y + (size_t)(t0 + i) * ldy + c);
+    float2 past[N > 0 ? N : 1];  // the inputs N, N - 1, .. 1 positions before the token
+    int seq = -1;
+#pragma unroll
+    for (int i = 0; i < SC_RUN; ++i) {
+        const int t = t0 + i;
+        if (t >= t1) break;
+        if (token_seq[t] != seq) {  // the run's or a request's first token: rows of the step before it, else the state
+            seq = token_seq[t];
+            const int pos = positions[t], start = seq_start_pos[seq];
+            const float* st = state + (size_t)seq_state_slot[seq] * N * channels + c;
+#pragma unroll
+            for (int j = 0; j < N; ++j) {
+                const int back = N - j, p = pos - back;
+                past[j] = make_float2(0.0f, 0.0f);
+                if (p >= start)
+                    past[j] = sc_load2(y + (size_t)(t - back) * ldy + c);
+                else if (p >= 0)
+                    past[j] = sc_load2(st + (size_t)(p - start + N) * channels);
+            }
+        }
+        float a0 = (residual ? own[i].x : 0.0f) + b.x, a1 = (residual ? own[i].y : 0.0f) + b.y;
+#pragma unroll
+        for (int j = 0; j < N; ++j) a0 = fmaf(w0[j], past[j].x, a0), a1 = fmaf(w1[j], past[j].y, a1);
+        a0 = fmaf(w0[N], own[i].x, a0), a1 = fmaf(w1[N], own[i].y, a1);
+        if (act) a0 = a0 / (1.0f + expf(-a0)), a1 = a1 / (1.0f + expf(-a1));
+        sc_store2(out + (size_t)t * ldo + c, a0, a1);
+#pragma unroll
+        for (int j = 0; j + 1 < N; ++j) past[j] = past[j + 1];
+        if (N > 0) past[N - 1] = own[i];
+    }
+}
+
 template <typename T>
 __global__ void __launch_bounds__(256) short_conv_advance_kernel(const T* y, int ldy, float* state,
                                                                  const int* __restrict__ seq_q_start,
@@ -126,6 +185,25 @@ FERRIS_API int ferris_short_conv(const void* y, int ldy, void* out, int ldo, int
     if (single_tokens && advance && tokens == seqs && dtype == FERRIS_BF16) {
         ferris_launch(short_conv_single_kernel<bf16>, grid_a, block, 0, s, (const bf16*)y, ldy, (bf16*)out, ldo, w, state,
                       positions, seq_state_slot, channels, taps, bias, residual, act);
+        FERRIS_LAUNCH_CHECK();
+    }
+    const size_t pair = dtype == FERRIS_F32 ? 8 : 4;  // bytes of two channels
+    if ((dtype == FERRIS_F32 || dtype == FERRIS_BF16) && tokens >= 2 * SC_RUN && taps >= 2 && taps <= 4 && !((channels | ldy | ldo) & 1) &&
+        (uintptr_t)y % pair == 0 && (uintptr_t)out % pair == 0 && (((uintptr_t)state | (uintptr_t)bias) & 7) == 0) {
+        const dim3 grid((tokens + SC_RUN - 1) / SC_RUN, (channels / 2 + 127) / 128);
+#define FERRIS_SC_RUNS(T, TAPS)                                                                                            \
+    ferris_launch(short_conv_runs_kernel<T, TAPS>, grid, dim3(128), 0, s, (const T*)y, ldy, (T*)out, ldo, w, (const float*)state, \
+                  token_seq, positions, seq_start_pos, seq_state_slot, tokens, channels, bias, residual, act)
+#define FERRIS_SC_TAPS(T)                                                                                                  \
+    do {                                                                                                                   \
+        if (taps == 2) FERRIS_SC_RUNS(T, 2); else if (taps == 3) FERRIS_SC_RUNS(T, 3); else FERRIS_SC_RUNS(T, 4);            \
+        if (advance)                                                                                                       \
+            ferris_launch(short_conv_advance_kernel<T>, grid_b, block, 0, s, (const T*)y, ldy, state, seq_q_start,          \
+                          seq_state_slot, channels, taps);                                                                 \
+    } while (0)
+        if (dtype == FERRIS_F32) FERRIS_SC_TAPS(float); else FERRIS_SC_TAPS(bf16);
+#undef FERRIS_SC_TAPS
+#undef FERRIS_SC_RUNS
         FERRIS_LAUNCH_CHECK();
     }
     if (dtype == FERRIS_F32) {

@@ -9,6 +9,7 @@
 #include <math.h>
 
 #include "common.cuh"
+#include "sm100.cuh"
 
 namespace {
 
@@ -354,6 +355,83 @@ __global__ void __launch_bounds__(HG_THREADS) head_gemm_kernel(const T* x, int l
     }
 }
 
+// The same product for long bf16 steps on the tensor cores: a block takes 64 tokens and 64 output columns of a head and walks
+// the inputs 64 at a time through two stages of asynchronous copies; each of its four warps owns 16 tokens.  bf16 operands as
+// stored, fp32 sums.
+constexpr int HM_TOKENS = 64, HM_COLS = 64, HM_K = 64, HM_THREADS = 128;
+constexpr int HM_PITCH = (HM_K + 8) * 2;  // bytes of a row of either tile: eight rows lie in different banks
+
+__device__ __forceinline__ void hm_copy16(uint32_t dst, const void* src, bool there) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(there ? 16 : 0) : "memory");
+}
+
+__global__ void __launch_bounds__(HM_THREADS) head_gemm_mma_kernel(const bf16* x, int ldx, int hsx, const bf16* __restrict__ w,
+                                                                   bf16* __restrict__ out, int ldo, int hso, const bf16* gate,
+                                                                   int ldg, int tokens, int K, int N) {
+    __shared__ __align__(16) uint8_t xs[2][HM_TOKENS * HM_PITCH];
+    __shared__ __align__(16) uint8_t wt[2][HM_K * HM_PITCH];
+    pdl_wait();
+    pdl_launch_dependents();
+    const int t0 = blockIdx.x * HM_TOKENS, h = blockIdx.y, n0 = blockIdx.z * HM_COLS;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const bf16* wh = w + (size_t)h * K * N;
+    auto fetch = [&](int k0, int st) {
+        if (k0 < K) {
+            const uint32_t xb = smem_u32(xs[st]), wb = smem_u32(wt[st]);
+#pragma unroll
+            for (int it = 0; it < HM_TOKENS * (HM_K / 8) / HM_THREADS; ++it) {
+                const int e = it * HM_THREADS + tid, r = e >> 3, c = (e & 7) * 8;
+                const bool in = t0 + r < tokens && k0 + c < K;
+                hm_copy16(xb + r * HM_PITCH + c * 2, in ? x + (size_t)(t0 + r) * ldx + (size_t)h * hsx + k0 + c : x, in);
+                const bool win = k0 + r < K && n0 + c < N;  // the weights' tile has as many rows (inputs) and pieces
+                hm_copy16(wb + r * HM_PITCH + c * 2, win ? wh + (size_t)(k0 + r) * N + n0 + c : wh, win);
+            }
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    float acc[HM_COLS / 8][4];
+#pragma unroll
+    for (int n = 0; n < HM_COLS / 8; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc[n][e] = 0.0f;
+    fetch(0, 0);
+    int st = 0;
+    for (int k0 = 0; k0 < K; k0 += HM_K, st ^= 1) {
+        fetch(k0 + HM_K, st ^ 1);
+        asm volatile("cp.async.wait_group 1;" ::: "memory");
+        __syncthreads();
+        const uint32_t a_at = smem_u32(xs[st]) + (uint32_t)(16 * warp + (lane & 7) + ((lane >> 3) & 1) * 8) * HM_PITCH + (lane >> 4) * 16;
+        const uint32_t b_at = smem_u32(wt[st]) + (uint32_t)(((lane >> 3) & 1) * 8 + (lane & 7)) * HM_PITCH + (lane >> 4) * 16;
+#pragma unroll
+        for (int kk = 0; kk < HM_K / 16; ++kk) {
+            uint32_t a[4];
+            ldmatrix_x4(a, a_at + kk * 32);
+#pragma unroll
+            for (int n = 0; n < HM_COLS / 8; n += 2) {
+                uint32_t b[4];
+                ldmatrix_x4_trans(b, b_at + kk * 16 * HM_PITCH + n * 16);
+                mma_bf16_16816(acc[n], a, b[0], b[1]);
+                mma_bf16_16816(acc[n + 1], a, b[2], b[3]);
+            }
+        }
+        __syncthreads();  // the stage is read: the copies after next may overwrite it
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+#pragma unroll
+    for (int a = 0; a < 2; ++a) {
+        const int t = t0 + 16 * warp + (lane >> 2) + 8 * a;
+        if (t >= tokens) continue;
+        const float g = gate ? 1.0f / (1.0f + expf(-to_float(gate[(size_t)t * ldg + h]))) : 1.0f;
+        bf16* row = out + (size_t)t * ldo + (size_t)h * hso;
+#pragma unroll
+        for (int n = 0; n < HM_COLS / 8; ++n) {
+            const int c = n0 + 8 * n + 2 * (lane & 3);
+            if (c < N) *reinterpret_cast<uint32_t*>(row + c) = pack_bf16(acc[n][2 * a] * g, acc[n][2 * a + 1] * g);
+        }
+    }
+}
+constexpr int HM_MIN_TOKENS = 48;  // shorter steps keep the kernel above: its blocks of eight tokens fill more SMs
+
 }  // namespace
 
 FERRIS_API int ferris_streams_expand(const float* h, float* xs, int tokens, int streams, int width, void* stream) {
@@ -484,6 +562,12 @@ FERRIS_API int ferris_head_gemm(const void* x, int ldx, int hsx, const void* w, 
     const size_t smem = ((size_t)HG_TOKENS * K + (size_t)(HG_PARTS - 1) * HG_TOKENS * HG_COLS) * sizeof(float);
     if (smem > 200 * 1024) FERRIS_REFUSE("head gemm: %d inputs a head are more than shared memory holds", K);
     cudaStream_t s = (cudaStream_t)stream;
+    if (dtype == FERRIS_BF16 && tokens >= HM_MIN_TOKENS && K % 8 == 0 && N % 8 == 0 && ldx % 8 == 0 && hsx % 8 == 0 && ldo % 2 == 0 &&
+        hso % 2 == 0 && (((uintptr_t)x | (uintptr_t)w) & 15) == 0 && ((uintptr_t)out & 3) == 0) {
+        ferris_launch(head_gemm_mma_kernel, dim3((tokens + HM_TOKENS - 1) / HM_TOKENS, heads, (N + HM_COLS - 1) / HM_COLS), dim3(HM_THREADS), 0,
+                      s, (const bf16*)x, ldx, hsx, (const bf16*)w, (bf16*)out, ldo, hso, (const bf16*)gate, ldg, tokens, K, N);
+        FERRIS_LAUNCH_CHECK();
+    }
     const dim3 grid((tokens + HG_TOKENS - 1) / HG_TOKENS, heads, (N + HG_COLS - 1) / HG_COLS), block(HG_THREADS);
     if (dtype == FERRIS_F32) {
         int e_ = ferris_allow_dynamic_smem((const void*)head_gemm_kernel<float>, smem);
