@@ -20,7 +20,7 @@
 // 16 + 8 + .. exchanges instead of 16 x log2), and only the 16 x 16 products with M and B tie the tokens together.  The next
 // chunk's rows come in by asynchronous copies meanwhile.
 //
-// For bf16 activations the walk runs on tensor cores: a block takes sixteen columns, its four warps share the rows of S, and
+// For bf16 activations the walk runs on tensor cores: a block takes sixteen columns, its eight warps share the rows of S, and
 // D^T = S_0^T K^T, E^T = S_0^T Q^T and the sum over the writes are products of tf32 fragments with fp32 sums.  Each operand x is
 // cut into its leading eleven bits and the rest, and the products big x big, big x rest and rest x big are added, which keeps 21
 // bits and more of every product; the state itself is only ever added to in fp32 outside the fragments' accumulators.
@@ -36,22 +36,39 @@ constexpr int DC_PREP_THREADS = 256;
 constexpr int DC_KPL = 8;     // rows of the state that a lane holds
 constexpr int DC_PITCH = 20;  // floats between the rows of 16 x 16 matrices in shared memory: rows start in different banks
 
-// kt, qt, kh: [tokens, heads, dim]; mm, bm: [tokens, heads, 16]; dm: [places, heads, dim], the place of a chunk being
-// (its first row) / 16 + its request's index in the step, which no two chunks share.
-struct DeltaChunks {
-    float* kt;
-    float* qt;
-    float* kh;
-    float* mm;
-    float* bm;
-    float* dm;
+// What a chunk of a head hands to the walk, in one piece of memory that a stage of shared memory takes as it is: kt, qt, kh
+// [16][dim + 8], the products' rows (the pitch keeps the fragments' reads in different banks); dm [dim]; mm, bm [16][20].  Tokens
+// beyond a chunk's last are zeros.  The place of a chunk is (its first row) / 16 + its request's index in the step, which no two
+// chunks share.
+__host__ __device__ constexpr int dc_pitch(int dim) { return dim + 8; }
+__host__ __device__ constexpr int dc_stage_floats(int dim) { return 3 * DC_TOKENS * dc_pitch(dim) + dim + 2 * DC_TOKENS * DC_PITCH; }
+struct DeltaStage {
+    float *kt, *qt, *kh, *dm, *mm, *bm;
 };
+__device__ __forceinline__ DeltaStage dc_stage(float* base, int dim) {
+    DeltaStage st;
+    st.kt = base, st.qt = st.kt + DC_TOKENS * dc_pitch(dim), st.kh = st.qt + DC_TOKENS * dc_pitch(dim);
+    st.dm = st.kh + DC_TOKENS * dc_pitch(dim), st.mm = st.dm + dim, st.bm = st.mm + DC_TOKENS * DC_PITCH;
+    return st;
+}
+__device__ __forceinline__ float* dc_place(float* scratch, int first, int seq, int head, int heads, int dim) {
+    return scratch + ((size_t)(first / DC_TOKENS + seq) * heads + head) * dc_stage_floats(dim);
+}
+// a stage's piece of memory into shared memory, 16 bytes at a time
+__device__ __forceinline__ void dc_fetch(float* dst, const float* src, int floats, int threads) {
+    const uint32_t to = (uint32_t)__cvta_generic_to_shared(dst);
+    for (int x = threadIdx.x * 4; x < floats; x += threads * 4)
+        asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(to + x * 4), "l"(src + x) : "memory");
+}
+__device__ __forceinline__ void dc_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void dc_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
 template <typename T>
 __global__ void __launch_bounds__(DC_PREP_THREADS) delta_chunk_prepare_kernel(
     const T* q, int ldq, const T* k, int ldk, const float* z, int ldz, const float* __restrict__ rates, const float* beta,
     const float* qscale, const float* kscale, const int* __restrict__ seq_q_start, int chunks_max, int heads, int qk_heads, int dim,
-    const DeltaChunks w) {
+    float* scratch) {
     extern __shared__ __align__(16) float dc_smem[];
     const int pitch = dim + 1;
     float* Ls = dc_smem;                     // [16][dim + 1]: logarithms, then their sums from the chunk's start
@@ -68,34 +85,49 @@ __global__ void __launch_bounds__(DC_PREP_THREADS) delta_chunk_prepare_kernel(
     const int qh = head / (heads / qk_heads);
     const float rate = rates[head];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    for (int x = tid; x < n * dim; x += DC_PREP_THREADS) {
-        const int t = x / dim, c = x - t * dim;
-        const size_t row = (size_t)(first + t);
-        Ls[t * pitch + c] = -ferris_softplus(z[row * ldz + (size_t)head * dim + c]) * rate;
-        Ks[t * pitch + c] = to_float(k[row * ldk + (size_t)qh * dim + c]) * (kscale ? kscale[row * qk_heads + qh] : 1.0f);
-        Qs[t * pitch + c] = to_float(q[row * ldq + (size_t)qh * dim + c]) * (qscale ? qscale[row * qk_heads + qh] : 1.0f);
+    const DeltaStage st = dc_stage(dc_place(scratch, first, seq, head, heads, dim), dim);
+    // an element (token, channel) a thread at a time: the next one is DC_PREP_THREADS further on
+    const int step_t = DC_PREP_THREADS / dim, step_c = DC_PREP_THREADS - step_t * dim;
+    const int t_mine = tid / dim, c_mine = tid - t_mine * dim;
+    for (int t = t_mine, c = c_mine; t < DC_TOKENS;) {
+        if (t < n) {
+            const size_t row = (size_t)(first + t);
+            Ls[t * pitch + c] = -ferris_softplus(z[row * ldz + (size_t)head * dim + c]) * rate;
+            Ks[t * pitch + c] = to_float(k[row * ldk + (size_t)qh * dim + c]) * (kscale ? kscale[row * qk_heads + qh] : 1.0f);
+            Qs[t * pitch + c] = to_float(q[row * ldq + (size_t)qh * dim + c]) * (qscale ? qscale[row * qk_heads + qh] : 1.0f);
+        }
+        t += step_t, c += step_c;
+        if (c >= dim) c -= dim, ++t;
     }
     if (tid < DC_TOKENS) bs[tid] = tid < n ? beta[(size_t)(first + tid) * heads + head] : 0.0f;
     __syncthreads();
     for (int c = tid; c < dim; c += DC_PREP_THREADS) {
         float sum = 0.0f;
         for (int t = 0; t < n; ++t) sum += Ls[t * pitch + c], Ls[t * pitch + c] = sum;
-        w.dm[((size_t)(first / DC_TOKENS + seq) * heads + head) * dim + c] = expm1f(sum);
+        st.dm[c] = expm1f(sum);
     }
     __syncthreads();
-    for (int x = tid; x < n * dim; x += DC_PREP_THREADS) {
-        const int t = x / dim, c = x - t * dim;
-        const size_t at = ((size_t)(first + t) * heads + head) * dim + c;
-        const float L = Ls[t * pitch + c], e = expf(L), kv = Ks[t * pitch + c];
-        w.kt[at] = kv * e;
-        w.qt[at] = Qs[t * pitch + c] * e;
-        w.kh[at] = kv * expf(Ls[(n - 1) * pitch + c] - L);
+    for (int t = t_mine, c = c_mine; t < DC_TOKENS;) {
+        const int at = t * dc_pitch(dim) + c;
+        if (t < n) {
+            const float L = Ls[t * pitch + c], e = expf(L), kv = Ks[t * pitch + c];
+            st.kt[at] = kv * e;
+            st.qt[at] = Qs[t * pitch + c] * e;
+            st.kh[at] = kv * expf(Ls[(n - 1) * pitch + c] - L);
+        } else {
+            st.kt[at] = st.qt[at] = st.kh[at] = 0.0f;
+        }
+        t += step_t, c += step_c;
+        if (c >= dim) c -= dim, ++t;
     }
     constexpr float LOG2E = 1.4426950408889634f;
     // a warp takes tokens w and 15 - w: seventeen pairs each
     for (int half = 0; half < 2; ++half) {
         const int t = half ? DC_TOKENS - 1 - warp : warp;
-        if (t >= n) continue;
+        if (t >= n) {
+            if (lane < DC_TOKENS) st.bm[t * DC_PITCH + lane] = 0.0f;
+            continue;
+        }
         float l[8], kv[8], qv[8];  // the token's row, a lane's channels lane, lane + 32, ..
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
@@ -119,9 +151,9 @@ __global__ void __launch_bounds__(DC_PREP_THREADS) delta_chunk_prepare_kernel(
 #pragma unroll
             for (int o = 8; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
             if (lane == 0) As[t][i] = sum;
-            if (lane == 16) w.bm[((size_t)(first + t) * heads + head) * DC_TOKENS + i] = sum;
+            if (lane == 16) st.bm[t * DC_PITCH + i] = sum;
         }
-        if (lane > t && lane < DC_TOKENS) w.bm[((size_t)(first + t) * heads + head) * DC_TOKENS + lane] = 0.0f;
+        if (lane > t && lane < DC_TOKENS) st.bm[t * DC_PITCH + lane] = 0.0f;
     }
     __syncthreads();
     if (tid < DC_TOKENS) {  // a column of M each: M_tj = b_t (delta_tj - sum_(i<t) A_ti M_ij)
@@ -133,16 +165,12 @@ __global__ void __launch_bounds__(DC_PREP_THREADS) delta_chunk_prepare_kernel(
 #pragma unroll
                 for (int i = 0; i < t; ++i) acc = fmaf(-As[t][i], m[i], acc);
                 m[t] = bs[t] * acc;
-                w.mm[((size_t)(first + t) * heads + head) * DC_TOKENS + tid] = m[t];
             } else {
                 m[t] = 0.0f;
             }
+            st.mm[t * DC_PITCH + tid] = m[t];
         }
     }
-}
-
-__device__ __forceinline__ void dc_copy16(float* dst, const float* src) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
 }
 
 // The sums over the LANES lanes of a column of sixteen numbers a lane: afterwards lane `sub` holds those of tokens
@@ -168,22 +196,13 @@ __device__ __forceinline__ void reduce_tokens(float (&x)[DC_TOKENS], int sub) {
     }
 }
 
-template <int LANES>
-struct DeltaStage {
-    static constexpr int ROWS = DC_KPL * LANES;
-    float kt[DC_TOKENS][ROWS], qt[DC_TOKENS][ROWS], kh[DC_TOKENS][ROWS];
-    float dm[ROWS];
-    float mm[DC_TOKENS][DC_PITCH], bm[DC_TOKENS][DC_PITCH];
-};
-
 template <typename T, int LANES>
 __global__ void __launch_bounds__(DC_THREADS) delta_chunk_walk_kernel(
-    const DeltaChunks w, const T* v, int ldv, float* __restrict__ out, int ldo, float* state, const int* __restrict__ seq_q_start,
+    float* scratch, const T* v, int ldv, float* __restrict__ out, int ldo, float* state, const int* __restrict__ seq_q_start,
     const int* __restrict__ seq_state_slot, int heads, int dim, int vdim, int write_state) {
     constexpr int COLS = DC_THREADS / LANES;  // columns of a block
     constexpr int PER = LANES >= DC_TOKENS ? 1 : DC_TOKENS / LANES;  // tokens whose sums a lane ends with
     extern __shared__ __align__(16) float dc_smem[];
-    DeltaStage<LANES>* stages = reinterpret_cast<DeltaStage<LANES>*>(dc_smem);
     __shared__ __align__(16) float ws[COLS][DC_PITCH], us[COLS][DC_PITCH];
     pdl_wait();
     pdl_launch_dependents();
@@ -193,8 +212,6 @@ __global__ void __launch_bounds__(DC_THREADS) delta_chunk_walk_kernel(
     const bool active = col < vdim;
     const int row0 = seq_q_start[seq], row1 = seq_q_start[seq + 1];
     if (row1 <= row0) return;
-    // both stages start as zeros: rows of the state beyond the head's size, and tokens beyond a chunk's last
-    for (int i = tid; i < (int)(2 * sizeof(DeltaStage<LANES>) / sizeof(float)); i += DC_THREADS) dc_smem[i] = 0.0f;
     float* S = state + (((size_t)seq_state_slot[seq] * heads + head) * vdim + (active ? col : 0)) * (size_t)dim;
     float s[DC_KPL];
 #pragma unroll
@@ -206,39 +223,14 @@ __global__ void __launch_bounds__(DC_THREADS) delta_chunk_walk_kernel(
     }
     const int mine = LANES == 32 ? sub >> 1 : sub * PER;  // the first token whose sums this lane ends with
     const bool writes = LANES != 32 || !(sub & 1);
-    __syncthreads();
-    const int d4 = dim >> 2;
-    auto fetch = [&](int first, DeltaStage<LANES>& st) {
-        if (first < row1) {
-            const int n = min(DC_TOKENS, row1 - first);
-            for (int x = tid; x < n * d4; x += DC_THREADS) {
-                const int t = x / d4, c = (x - t * d4) * 4;
-                const size_t at = ((size_t)(first + t) * heads + head) * dim + c;
-                dc_copy16(&st.kt[t][c], w.kt + at);
-                dc_copy16(&st.qt[t][c], w.qt + at);
-                dc_copy16(&st.kh[t][c], w.kh + at);
-            }
-            for (int x = tid; x < d4; x += DC_THREADS)
-                dc_copy16(&st.dm[4 * x], w.dm + ((size_t)(first / DC_TOKENS + seq) * heads + head) * dim + 4 * x);
-            if (tid < n * 4) {
-                const int t = tid >> 2, c = (tid & 3) * 4;
-                const size_t at = ((size_t)(first + t) * heads + head) * DC_TOKENS + c;
-                dc_copy16(&st.mm[t][c], w.mm + at);
-                dc_copy16(&st.bm[t][c], w.bm + at);
-            }
-            if (n < DC_TOKENS) {  // the last chunk: what an earlier one left behind the last token
-                for (int x = tid; x < (DC_TOKENS - n) * d4; x += DC_THREADS) {
-                    const int t = n + x / d4, c = (x % d4) * 4;
-                    const float4 zero = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-                    *reinterpret_cast<float4*>(&st.kt[t][c]) = zero;
-                    *reinterpret_cast<float4*>(&st.qt[t][c]) = zero;
-                    *reinterpret_cast<float4*>(&st.kh[t][c]) = zero;
-                }
-                for (int x = tid; x < (DC_TOKENS - n) * DC_TOKENS; x += DC_THREADS)
-                    st.mm[n + x / DC_TOKENS][x % DC_TOKENS] = 0.0f, st.bm[n + x / DC_TOKENS][x % DC_TOKENS] = 0.0f;
-            }
-        }
-        asm volatile("cp.async.commit_group;" ::: "memory");
+    // the lane's two runs of four rows; a run beyond the head's size reads rows that its zero state does not feel, and its sums
+    // over the writes are never used
+    const int floats = dc_stage_floats(dim), pitch = dc_pitch(dim);
+    const bool has[2] = {4 * sub < dim, 4 * (LANES + sub) < dim};
+    const int r0 = has[0] ? 4 * sub : 0, r1 = has[1] ? 4 * (LANES + sub) : 0;
+    auto fetch = [&](int first, int buf) {
+        if (first < row1) dc_fetch(dc_smem + buf * floats, dc_place(scratch, first, seq, head, heads, dim), floats, DC_THREADS);
+        dc_commit();
     };
     T pv[PER];
     auto request_v = [&](int first) {
@@ -249,27 +241,27 @@ __global__ void __launch_bounds__(DC_THREADS) delta_chunk_walk_kernel(
             if (t < row1 && active) pv[j] = v[(size_t)t * ldv + (size_t)head * vdim + col];
         }
     };
-    fetch(row0, stages[0]);
+    fetch(row0, 0);
     request_v(row0);
     int buf = 0;
     for (int first = row0; first < row1; first += DC_TOKENS, buf ^= 1) {
-        fetch(first + DC_TOKENS, stages[buf ^ 1]);
+        fetch(first + DC_TOKENS, buf ^ 1);
         float vv[PER];
 #pragma unroll
         for (int j = 0; j < PER; ++j) vv[j] = to_float(pv[j]);
         request_v(first + DC_TOKENS);
-        asm volatile("cp.async.wait_group 1;" ::: "memory");
+        dc_wait<1>();
         __syncthreads();
-        const DeltaStage<LANES>& st = stages[buf];
+        const DeltaStage st = dc_stage(dc_smem + buf * floats, dim);
         float D[DC_TOKENS], E[DC_TOKENS];
 #pragma unroll
         for (int t = 0; t < DC_TOKENS; ++t) {
-            const float4 a = *reinterpret_cast<const float4*>(&st.kt[t][4 * sub]);
-            const float4 b = *reinterpret_cast<const float4*>(&st.kt[t][4 * (LANES + sub)]);
+            const float4 a = *reinterpret_cast<const float4*>(st.kt + t * pitch + r0);
+            const float4 b = *reinterpret_cast<const float4*>(st.kt + t * pitch + r1);
             D[t] = fmaf(a.x, s[0], fmaf(a.y, s[1], fmaf(a.z, s[2], a.w * s[3])));
             D[t] = fmaf(b.x, s[4], fmaf(b.y, s[5], fmaf(b.z, s[6], fmaf(b.w, s[7], D[t]))));
-            const float4 c = *reinterpret_cast<const float4*>(&st.qt[t][4 * sub]);
-            const float4 e = *reinterpret_cast<const float4*>(&st.qt[t][4 * (LANES + sub)]);
+            const float4 c = *reinterpret_cast<const float4*>(st.qt + t * pitch + r0);
+            const float4 e = *reinterpret_cast<const float4*>(st.qt + t * pitch + r1);
             E[t] = fmaf(c.x, s[0], fmaf(c.y, s[1], fmaf(c.z, s[2], c.w * s[3])));
             E[t] = fmaf(e.x, s[4], fmaf(e.y, s[5], fmaf(e.z, s[6], fmaf(e.w, s[7], E[t]))));
         }
@@ -290,7 +282,7 @@ __global__ void __launch_bounds__(DC_THREADS) delta_chunk_walk_kernel(
             float u0 = 0.0f, u1 = 0.0f;
 #pragma unroll
             for (int i = 0; i < DC_TOKENS; i += 4) {
-                const float4 m = *reinterpret_cast<const float4*>(&st.mm[mine + j][i]);
+                const float4 m = *reinterpret_cast<const float4*>(st.mm + (mine + j) * DC_PITCH + i);
                 u0 = fmaf(m.x, x[i], u0), u1 = fmaf(m.y, x[i + 1], u1), u0 = fmaf(m.z, x[i + 2], u0), u1 = fmaf(m.w, x[i + 3], u1);
             }
             if (writes) us[cl][mine + j] = u0 + u1;
@@ -306,7 +298,7 @@ __global__ void __launch_bounds__(DC_THREADS) delta_chunk_walk_kernel(
             float o0 = E[j], o1 = 0.0f;
 #pragma unroll
             for (int i = 0; i < DC_TOKENS; i += 4) {
-                const float4 m = *reinterpret_cast<const float4*>(&st.bm[mine + j][i]);
+                const float4 m = *reinterpret_cast<const float4*>(st.bm + (mine + j) * DC_PITCH + i);
                 o0 = fmaf(m.x, x[i], o0), o1 = fmaf(m.y, x[i + 1], o1), o0 = fmaf(m.z, x[i + 2], o0), o1 = fmaf(m.w, x[i + 3], o1);
             }
             const int t = first + mine + j;
@@ -317,17 +309,17 @@ __global__ void __launch_bounds__(DC_THREADS) delta_chunk_walk_kernel(
         for (int i = 0; i < DC_KPL; ++i) acc[i] = 0.0f;
 #pragma unroll
         for (int t = 0; t < DC_TOKENS; ++t) {
-            const float4 a = *reinterpret_cast<const float4*>(&st.kh[t][4 * sub]);
-            const float4 b = *reinterpret_cast<const float4*>(&st.kh[t][4 * (LANES + sub)]);
+            const float4 a = *reinterpret_cast<const float4*>(st.kh + t * pitch + r0);
+            const float4 b = *reinterpret_cast<const float4*>(st.kh + t * pitch + r1);
             acc[0] = fmaf(a.x, x[t], acc[0]), acc[1] = fmaf(a.y, x[t], acc[1]), acc[2] = fmaf(a.z, x[t], acc[2]), acc[3] = fmaf(a.w, x[t], acc[3]);
             acc[4] = fmaf(b.x, x[t], acc[4]), acc[5] = fmaf(b.y, x[t], acc[5]), acc[6] = fmaf(b.z, x[t], acc[6]), acc[7] = fmaf(b.w, x[t], acc[7]);
         }
-        const float4 m0 = *reinterpret_cast<const float4*>(&st.dm[4 * sub]), m1 = *reinterpret_cast<const float4*>(&st.dm[4 * (LANES + sub)]);
-        s[0] += fmaf(m0.x, s[0], acc[0]), s[1] += fmaf(m0.y, s[1], acc[1]), s[2] += fmaf(m0.z, s[2], acc[2]), s[3] += fmaf(m0.w, s[3], acc[3]);
-        s[4] += fmaf(m1.x, s[4], acc[4]), s[5] += fmaf(m1.y, s[5], acc[5]), s[6] += fmaf(m1.z, s[6], acc[6]), s[7] += fmaf(m1.w, s[7], acc[7]);
+        const float4 m0 = *reinterpret_cast<const float4*>(st.dm + r0), m1 = *reinterpret_cast<const float4*>(st.dm + r1);
+        if (has[0]) s[0] += fmaf(m0.x, s[0], acc[0]), s[1] += fmaf(m0.y, s[1], acc[1]), s[2] += fmaf(m0.z, s[2], acc[2]), s[3] += fmaf(m0.w, s[3], acc[3]);
+        if (has[1]) s[4] += fmaf(m1.x, s[4], acc[4]), s[5] += fmaf(m1.y, s[5], acc[5]), s[6] += fmaf(m1.z, s[6], acc[6]), s[7] += fmaf(m1.w, s[7], acc[7]);
         __syncthreads();  // the stage is read: the copies after next may overwrite it
     }
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    dc_wait<0>();
     if (write_state && active) {
 #pragma unroll
         for (int g = 0; g < 2; ++g) {
@@ -338,13 +330,8 @@ __global__ void __launch_bounds__(DC_THREADS) delta_chunk_walk_kernel(
 }
 
 // ------------------------------------------------------------------------------------------ the walk on tensor cores
-constexpr int DM_COLS = 16, DM_STAGES = 3, DM_WARPS = DC_THREADS / 32;
+constexpr int DM_COLS = 16, DM_STAGES = 3, DM_WARPS = 8, DM_THREADS = 32 * DM_WARPS;
 
-__device__ __forceinline__ void dc_copy16_or_zero(float* dst, const float* src, bool there) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src),
-                 "r"(there ? 16 : 0)
-                 : "memory");
-}
 __device__ __forceinline__ void split_tf32(float x, uint32_t& big, uint32_t& rest) {
     big = __float_as_uint(x) & 0xffffe000u;
     rest = __float_as_uint(x - __uint_as_float(big));
@@ -355,15 +342,10 @@ __device__ __forceinline__ void mma_tf32_1688(float (&c)[4], const uint32_t (&a)
                  : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
-// Sizes in floats of a stage for heads of `dim`: rows of kt, qt and kh are dim + 8 floats apart, so that the fragments' reads
-// (four or eight tokens by neighbouring rows of S) fall into different banks.
-__host__ __device__ constexpr int dm_pitch(int dim) { return dim + 8; }
-__host__ __device__ constexpr int dm_stage_floats(int dim) { return 3 * DC_TOKENS * dm_pitch(dim) + dim + 2 * DC_TOKENS * DC_PITCH; }
-
-// TILES: eight-row pieces of S that a warp holds at most (warp w's are w, w + 4, ..); dim a multiple of eight.
+// TILES: eight-row pieces of S that a warp holds at most (warp w's are w, w + 8, ..); dim a multiple of eight.
 template <typename T, int TILES>
-__global__ void __launch_bounds__(DC_THREADS) delta_chunk_walk_mma_kernel(
-    const DeltaChunks w, const T* v, int ldv, float* __restrict__ out, int ldo, float* state, const int* __restrict__ seq_q_start,
+__global__ void __launch_bounds__(DM_THREADS) delta_chunk_walk_mma_kernel(
+    float* scratch, const T* v, int ldv, float* __restrict__ out, int ldo, float* state, const int* __restrict__ seq_q_start,
     const int* __restrict__ seq_state_slot, int heads, int dim, int vdim, int write_state) {
     extern __shared__ __align__(16) float dc_smem[];
     __shared__ __align__(16) float pd[DM_WARPS][DM_COLS][DC_PITCH], pe[DM_WARPS][DM_COLS][DC_PITCH];
@@ -374,7 +356,7 @@ __global__ void __launch_bounds__(DC_THREADS) delta_chunk_walk_mma_kernel(
     const int warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
     const int row0 = seq_q_start[seq], row1 = seq_q_start[seq + 1];
     if (row1 <= row0) return;
-    const int pitch = dm_pitch(dim), stage_floats = dm_stage_floats(dim), tiles = dim >> 3, d4 = dim >> 2;
+    const int pitch = dc_pitch(dim), floats = dc_stage_floats(dim), tiles = dim >> 3;
     float* S = state + (((size_t)seq_state_slot[seq] * heads + head) * vdim + col0) * (size_t)dim;
     // S^T as an accumulator fragment: [0], [1]: column g, rows 8 j + 2 t4, + 1; [2], [3]: column g + 8.  The same registers are an A
     // fragment whose inner index is permuted (slot t4 is row 2 t4, slot t4 + 4 row 2 t4 + 1); B reads its rows the same way.
@@ -390,58 +372,27 @@ __global__ void __launch_bounds__(DC_THREADS) delta_chunk_walk_mma_kernel(
         }
     }
     auto fetch = [&](int first, int stage) {
-        if (first < row1) {
-            float* kt = dc_smem + stage * stage_floats;
-            float* dm = kt + 3 * DC_TOKENS * pitch;
-            float* mm = dm + dim;
-            float* bm = mm + DC_TOKENS * DC_PITCH;
-            for (int x = tid; x < DC_TOKENS * d4; x += DC_THREADS) {
-                const int t = x / d4, c = (x - t * d4) * 4;
-                const bool there = first + t < row1;  // tokens beyond the last one are zeros
-                const size_t at = ((size_t)(first + (there ? t : 0)) * heads + head) * dim + c;
-                dc_copy16_or_zero(kt + t * pitch + c, w.kt + at, there);
-                dc_copy16_or_zero(kt + (DC_TOKENS + t) * pitch + c, w.qt + at, there);
-                dc_copy16_or_zero(kt + (2 * DC_TOKENS + t) * pitch + c, w.kh + at, there);
-            }
-            for (int x = tid; x < d4; x += DC_THREADS)
-                dc_copy16_or_zero(dm + 4 * x, w.dm + ((size_t)(first / DC_TOKENS + seq) * heads + head) * dim + 4 * x, true);
-            if (tid < DC_TOKENS * 4) {
-                const int t = tid >> 2, c = (tid & 3) * 4;
-                const bool there = first + t < row1;
-                const size_t at = ((size_t)(first + (there ? t : 0)) * heads + head) * DC_TOKENS + c;
-                dc_copy16_or_zero(mm + t * DC_PITCH + c, w.mm + at, there);
-                dc_copy16_or_zero(bm + t * DC_PITCH + c, w.bm + at, there);
-            }
-        }
-        asm volatile("cp.async.commit_group;" ::: "memory");
+        if (first < row1) dc_fetch(dc_smem + stage * floats, dc_place(scratch, first, seq, head, heads, dim), floats, DM_THREADS);
+        dc_commit();
     };
-    const int cl = tid >> 3, tk = (tid & 7) * 2;  // this thread's column and its two tokens between the products
+    const int cl = tid >> 4, tk = tid & 15;  // this thread's column and token between the products
     const bool active = col0 + cl < vdim;
-    T pv[2];
+    T pv;
     auto request_v = [&](int first) {
-#pragma unroll
-        for (int j = 0; j < 2; ++j) {
-            const int t = first + tk + j;
-            pv[j] = from_float<T>(0.0f);
-            if (t < row1 && active) pv[j] = v[(size_t)t * ldv + (size_t)head * vdim + col0 + cl];
-        }
+        pv = from_float<T>(0.0f);
+        if (first + tk < row1 && active) pv = v[(size_t)(first + tk) * ldv + (size_t)head * vdim + col0 + cl];
     };
     fetch(row0, 0);
     fetch(row0 + DC_TOKENS, 1);
     request_v(row0);
     int stage = 0;
     for (int first = row0; first < row1; first += DC_TOKENS) {
-        asm volatile("cp.async.wait_group 1;" ::: "memory");
+        dc_wait<1>();
         __syncthreads();  // the stage is there; everyone is done with the one before, which the next copies overwrite
         fetch(first + 2 * DC_TOKENS, stage == 0 ? 2 : stage - 1);
-        const float v0 = to_float(pv[0]), v1 = to_float(pv[1]);
+        const float vv = to_float(pv);
         request_v(first + DC_TOKENS);
-        const float* kt = dc_smem + stage * stage_floats;
-        const float* qt = kt + DC_TOKENS * pitch;
-        const float* kh = qt + DC_TOKENS * pitch;
-        const float* dm = kh + DC_TOKENS * pitch;
-        const float* mm = dm + dim;
-        const float* bm = mm + DC_TOKENS * DC_PITCH;
+        const DeltaStage st = dc_stage(dc_smem + stage * floats, dim);
         // D^T and E^T over the warp's rows: two token tiles each, the small products in accumulators of their own
         float D[2][4], Dr[2][4], E[2][4], Er[2][4];
 #pragma unroll
@@ -458,8 +409,8 @@ __global__ void __launch_bounds__(DC_THREADS) delta_chunk_walk_mma_kernel(
 #pragma unroll
                 for (int n = 0; n < 2; ++n) {
                     const int at = (8 * n + g) * pitch + 8 * tile + 2 * t4;
-                    const float2 x = *reinterpret_cast<const float2*>(kt + at);
-                    const float2 y = *reinterpret_cast<const float2*>(qt + at);
+                    const float2 x = *reinterpret_cast<const float2*>(st.kt + at);
+                    const float2 y = *reinterpret_cast<const float2*>(st.qt + at);
                     uint32_t xb0, xr0, xb1, xr1, yb0, yr0, yb1, yr1;
                     split_tf32(x.x, xb0, xr0), split_tf32(x.y, xb1, xr1);
                     split_tf32(y.x, yb0, yr0), split_tf32(y.y, yb1, yr1);
@@ -481,25 +432,19 @@ __global__ void __launch_bounds__(DC_THREADS) delta_chunk_walk_mma_kernel(
                 *reinterpret_cast<float2*>(&pe[warp][c][t]) = make_float2(E[n][2 * a] + Er[n][2 * a], E[n][2 * a + 1] + Er[n][2 * a + 1]);
             }
         __syncthreads();
-        float2 e = make_float2(0.0f, 0.0f), x = make_float2(0.0f, 0.0f);
+        float e = 0.0f, x = 0.0f;
 #pragma unroll
-        for (int q = 0; q < DM_WARPS; ++q) {
-            const float2 a = *reinterpret_cast<const float2*>(&pd[q][cl][tk]), b = *reinterpret_cast<const float2*>(&pe[q][cl][tk]);
-            x.x += a.x, x.y += a.y, e.x += b.x, e.y += b.y;
-        }
-        *reinterpret_cast<float2*>(&ws[cl][tk]) = make_float2(v0 - x.x, v1 - x.y);
-        __syncwarp();  // a column's eight threads are of one warp
-        // u = M w for the thread's two tokens
-        float u0 = 0.0f, u1 = 0.0f, y0 = 0.0f, y1 = 0.0f;
+        for (int q = 0; q < DM_WARPS; ++q) x += pd[q][cl][tk], e += pe[q][cl][tk];
+        ws[cl][tk] = vv - x;
+        __syncwarp();  // a column's sixteen threads are of one warp
+        float u0 = 0.0f, u1 = 0.0f;  // u = M w
 #pragma unroll
         for (int i = 0; i < DC_TOKENS; i += 4) {
             const float4 f = *reinterpret_cast<const float4*>(&ws[cl][i]);
-            const float4 m = *reinterpret_cast<const float4*>(mm + tk * DC_PITCH + i);
-            const float4 n = *reinterpret_cast<const float4*>(mm + (tk + 1) * DC_PITCH + i);
-            u0 = fmaf(m.x, f.x, u0), y0 = fmaf(m.y, f.y, y0), u0 = fmaf(m.z, f.z, u0), y0 = fmaf(m.w, f.w, y0);
-            u1 = fmaf(n.x, f.x, u1), y1 = fmaf(n.y, f.y, y1), u1 = fmaf(n.z, f.z, u1), y1 = fmaf(n.w, f.w, y1);
+            const float4 m = *reinterpret_cast<const float4*>(st.mm + tk * DC_PITCH + i);
+            u0 = fmaf(m.x, f.x, u0), u1 = fmaf(m.y, f.y, u1), u0 = fmaf(m.z, f.z, u0), u1 = fmaf(m.w, f.w, u1);
         }
-        *reinterpret_cast<float2*>(&us[cl][tk]) = make_float2(u0 + y0, u1 + y1);
+        us[cl][tk] = u0 + u1;
         __syncthreads();
         // the writes: S^T += U^T K over the chunk's tokens, formed apart from the state and added to it in fp32
         {
@@ -517,13 +462,13 @@ __global__ void __launch_bounds__(DC_THREADS) delta_chunk_walk_mma_kernel(
 #pragma unroll
                     for (int k = 0; k < 2; ++k) {
                         uint32_t b0, r0, b1, r1;
-                        split_tf32(kh[(8 * k + t4) * pitch + 8 * tile + g], b0, r0);
-                        split_tf32(kh[(8 * k + t4 + 4) * pitch + 8 * tile + g], b1, r1);
+                        split_tf32(st.kh[(8 * k + t4) * pitch + 8 * tile + g], b0, r0);
+                        split_tf32(st.kh[(8 * k + t4 + 4) * pitch + 8 * tile + g], b1, r1);
                         mma_tf32_1688(acc, ub[k], b0, b1);
                         mma_tf32_1688(rest, ub[k], r0, r1);
                         mma_tf32_1688(rest, ur[k], b0, b1);
                     }
-                    const float2 m = *reinterpret_cast<const float2*>(dm + 8 * tile + 2 * t4);
+                    const float2 m = *reinterpret_cast<const float2*>(st.dm + 8 * tile + 2 * t4);
                     s[j][0] += fmaf(m.x, s[j][0], acc[0] + rest[0]), s[j][1] += fmaf(m.y, s[j][1], acc[1] + rest[1]);
                     s[j][2] += fmaf(m.x, s[j][2], acc[2] + rest[2]), s[j][3] += fmaf(m.y, s[j][3], acc[3] + rest[3]);
                 }
@@ -531,22 +476,18 @@ __global__ void __launch_bounds__(DC_THREADS) delta_chunk_walk_mma_kernel(
         }
         // o = E + B u
         {
-            float o0 = e.x, o1 = e.y, z0 = 0.0f, z1 = 0.0f;
+            float o0 = e, o1 = 0.0f;
 #pragma unroll
             for (int i = 0; i < DC_TOKENS; i += 4) {
                 const float4 f = *reinterpret_cast<const float4*>(&us[cl][i]);
-                const float4 m = *reinterpret_cast<const float4*>(bm + tk * DC_PITCH + i);
-                const float4 n = *reinterpret_cast<const float4*>(bm + (tk + 1) * DC_PITCH + i);
-                o0 = fmaf(m.x, f.x, o0), z0 = fmaf(m.y, f.y, z0), o0 = fmaf(m.z, f.z, o0), z0 = fmaf(m.w, f.w, z0);
-                o1 = fmaf(n.x, f.x, o1), z1 = fmaf(n.y, f.y, z1), o1 = fmaf(n.z, f.z, o1), z1 = fmaf(n.w, f.w, z1);
+                const float4 m = *reinterpret_cast<const float4*>(st.bm + tk * DC_PITCH + i);
+                o0 = fmaf(m.x, f.x, o0), o1 = fmaf(m.y, f.y, o1), o0 = fmaf(m.z, f.z, o0), o1 = fmaf(m.w, f.w, o1);
             }
-            float* dst = out + (size_t)(first + tk) * ldo + (size_t)head * vdim + col0 + cl;
-            if (active && first + tk < row1) dst[0] = o0 + z0;
-            if (active && first + tk + 1 < row1) dst[ldo] = o1 + z1;
+            if (active && first + tk < row1) out[(size_t)(first + tk) * ldo + (size_t)head * vdim + col0 + cl] = o0 + o1;
         }
         stage = stage + 1 == DM_STAGES ? 0 : stage + 1;
     }
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    dc_wait<0>();
     if (!write_state) return;
 #pragma unroll
     for (int j = 0; j < TILES; ++j) {
@@ -559,24 +500,24 @@ __global__ void __launch_bounds__(DC_THREADS) delta_chunk_walk_mma_kernel(
 }
 
 template <typename T, int TILES>
-int launch_walk_mma(const DeltaChunks& w, const void* v, int ldv, float* out, int ldo, float* state, const int* seq_q_start,
+int launch_walk_mma(float* scratch, const void* v, int ldv, float* out, int ldo, float* state, const int* seq_q_start,
                     const int* seq_state_slot, int seqs, int heads, int dim, int vdim, int write_state, cudaStream_t s) {
-    const size_t smem = (size_t)DM_STAGES * dm_stage_floats(dim) * sizeof(float);
+    const size_t smem = (size_t)DM_STAGES * dc_stage_floats(dim) * sizeof(float);
     const int rc = ferris_allow_dynamic_smem((const void*)delta_chunk_walk_mma_kernel<T, TILES>, smem);
     if (rc != FERRIS_OK) return rc;
-    ferris_launch(delta_chunk_walk_mma_kernel<T, TILES>, dim3(seqs, heads, (vdim + DM_COLS - 1) / DM_COLS), dim3(DC_THREADS), smem, s, w,
+    ferris_launch(delta_chunk_walk_mma_kernel<T, TILES>, dim3(seqs, heads, (vdim + DM_COLS - 1) / DM_COLS), dim3(DM_THREADS), smem, s, scratch,
                   (const T*)v, ldv, out, ldo, state, seq_q_start, seq_state_slot, heads, dim, vdim, write_state);
     FERRIS_LAUNCH_CHECK();
 }
 
 template <typename T, int LANES>
-int launch_walk(const DeltaChunks& w, const void* v, int ldv, float* out, int ldo, float* state, const int* seq_q_start,
+int launch_walk(float* scratch, const void* v, int ldv, float* out, int ldo, float* state, const int* seq_q_start,
                 const int* seq_state_slot, int seqs, int heads, int dim, int vdim, int write_state, cudaStream_t s) {
     constexpr int COLS = DC_THREADS / LANES;
-    const size_t smem = 2 * sizeof(DeltaStage<LANES>);
+    const size_t smem = 2 * (size_t)dc_stage_floats(dim) * sizeof(float);
     const int rc = ferris_allow_dynamic_smem((const void*)delta_chunk_walk_kernel<T, LANES>, smem);
     if (rc != FERRIS_OK) return rc;
-    ferris_launch(delta_chunk_walk_kernel<T, LANES>, dim3(seqs, heads, (vdim + COLS - 1) / COLS), dim3(DC_THREADS), smem, s, w,
+    ferris_launch(delta_chunk_walk_kernel<T, LANES>, dim3(seqs, heads, (vdim + COLS - 1) / COLS), dim3(DC_THREADS), smem, s, scratch,
                   (const T*)v, ldv, out, ldo, state, seq_q_start, seq_state_slot, heads, dim, vdim, write_state);
     FERRIS_LAUNCH_CHECK();
 }
@@ -585,8 +526,7 @@ int launch_walk(const DeltaChunks& w, const void* v, int ldv, float* out, int ld
 
 // Floats of scratch that ferris_delta_chunks wants.
 FERRIS_API long long ferris_delta_chunks_scratch(int tokens, int seqs, int heads, int dim) {
-    const long long rows = (long long)tokens * heads, places = tokens / DC_TOKENS + seqs + 1;
-    return rows * (3LL * dim + 2 * DC_TOKENS) + places * heads * dim;
+    return (long long)(tokens / DC_TOKENS + seqs + 1) * heads * dc_stage_floats(dim);
 }
 
 // Arguments as ferris_gated_recurrence with row decays (z, rates); dim a multiple of four, every pointer but v's on 16 bytes;
@@ -605,10 +545,6 @@ FERRIS_API int ferris_delta_chunks(const void* q, int ldq, const void* k, int ld
     if (((uintptr_t)state | (uintptr_t)scratch) & 15) FERRIS_REFUSE("delta chunks: state and scratch must start on 16 bytes");
     const long long chunks_max = (longest + DC_TOKENS - 1) / DC_TOKENS;
     if (chunks_max * seqs > 2147483647LL) FERRIS_REFUSE("delta chunks: %d requests of up to %d tokens are more than one launch takes", seqs, longest);
-    const size_t rows = (size_t)tokens * heads;
-    DeltaChunks w;
-    w.kt = scratch, w.qt = w.kt + rows * dim, w.kh = w.qt + rows * dim;
-    w.mm = w.kh + rows * dim, w.bm = w.mm + rows * DC_TOKENS, w.dm = w.bm + rows * DC_TOKENS;
     cudaStream_t s = (cudaStream_t)stream;
     const size_t smem = 3 * (size_t)DC_TOKENS * (dim + 1) * sizeof(float);
     const dim3 grid((unsigned)(chunks_max * seqs), heads);
@@ -617,23 +553,22 @@ FERRIS_API int ferris_delta_chunks(const void* q, int ldq, const void* k, int ld
         int rc = ferris_allow_dynamic_smem((const void*)delta_chunk_prepare_kernel<T>, smem);                                 \
         if (rc != FERRIS_OK) return rc;                                                                                      \
         ferris_launch(delta_chunk_prepare_kernel<T>, grid, dim3(DC_PREP_THREADS), smem, s, (const T*)q, ldq, (const T*)k, ldk, z, \
-                      ldz, rates, beta, qscale, kscale, seq_q_start, (int)chunks_max, heads, qk_heads, dim, w);               \
-        if (dim <= 32) return launch_walk<T, 4>(w, v, ldv, out, ldo, state, seq_q_start, seq_state_slot, seqs, heads, dim, vdim, write_state, s); \
-        if (dim <= 64) return launch_walk<T, 8>(w, v, ldv, out, ldo, state, seq_q_start, seq_state_slot, seqs, heads, dim, vdim, write_state, s); \
-        if (dim <= 128) return launch_walk<T, 16>(w, v, ldv, out, ldo, state, seq_q_start, seq_state_slot, seqs, heads, dim, vdim, write_state, s); \
-        return launch_walk<T, 32>(w, v, ldv, out, ldo, state, seq_q_start, seq_state_slot, seqs, heads, dim, vdim, write_state, s); \
+                      ldz, rates, beta, qscale, kscale, seq_q_start, (int)chunks_max, heads, qk_heads, dim, scratch);               \
+        if (dim <= 32) return launch_walk<T, 4>(scratch, v, ldv, out, ldo, state, seq_q_start, seq_state_slot, seqs, heads, dim, vdim, write_state, s); \
+        if (dim <= 64) return launch_walk<T, 8>(scratch, v, ldv, out, ldo, state, seq_q_start, seq_state_slot, seqs, heads, dim, vdim, write_state, s); \
+        if (dim <= 128) return launch_walk<T, 16>(scratch, v, ldv, out, ldo, state, seq_q_start, seq_state_slot, seqs, heads, dim, vdim, write_state, s); \
+        return launch_walk<T, 32>(scratch, v, ldv, out, ldo, state, seq_q_start, seq_state_slot, seqs, heads, dim, vdim, write_state, s); \
     } while (0)
     if (dtype == FERRIS_BF16 && dim % 8 == 0) {
         int rc = ferris_allow_dynamic_smem((const void*)delta_chunk_prepare_kernel<bf16>, smem);
         if (rc != FERRIS_OK) return rc;
         ferris_launch(delta_chunk_prepare_kernel<bf16>, grid, dim3(DC_PREP_THREADS), smem, s, (const bf16*)q, ldq, (const bf16*)k, ldk, z,
-                      ldz, rates, beta, qscale, kscale, seq_q_start, (int)chunks_max, heads, qk_heads, dim, w);
+                      ldz, rates, beta, qscale, kscale, seq_q_start, (int)chunks_max, heads, qk_heads, dim, scratch);
 #define FERRIS_DM_GO(TILES) \
-    return launch_walk_mma<bf16, TILES>(w, v, ldv, out, ldo, state, seq_q_start, seq_state_slot, seqs, heads, dim, vdim, write_state, s)
-        if (dim <= 32) FERRIS_DM_GO(1);
-        if (dim <= 64) FERRIS_DM_GO(2);
-        if (dim <= 128) FERRIS_DM_GO(4);
-        FERRIS_DM_GO(8);
+    return launch_walk_mma<bf16, TILES>(scratch, v, ldv, out, ldo, state, seq_q_start, seq_state_slot, seqs, heads, dim, vdim, write_state, s)
+        if (dim <= 64) FERRIS_DM_GO(1);
+        if (dim <= 128) FERRIS_DM_GO(2);
+        FERRIS_DM_GO(4);
 #undef FERRIS_DM_GO
     }
     if (dtype == FERRIS_F32) FERRIS_DC_GO(float);
