@@ -397,6 +397,70 @@ def test_a_channel_that_hardly_forgets_over_thousands_of_tokens(device, dtype):
     assert float((got[-1].cpu().double() - want).abs().max()) < 2e-5 * float(want.abs().max())
 
 
+@pytest.mark.parametrize("dtype", [F32, BF16])
+@pytest.mark.parametrize("channels,taps", [(48, 4), (130, 2), (64, 3), (33, 4), (40, 1), (24, 5)])
+def test_convolution_of_unequal_requests_in_one_step(device, channels, taps, dtype):
+    """Portions, single tokens and long prompts side by side over slots out of order, continued in later steps; runs of tokens that
+    begin and end inside requests; a slice of wider rows."""
+    ops = _ops()
+    torch.manual_seed(channels * taps)
+    lens = [70, 1, 40, 3, 19]
+    w = torch.randn(channels, taps)
+    xs = [torch.randn(n + 30, channels).to(dtype) for n in lens]
+    want = [plain.silu(plain.causal_conv(x.double(), w.double())[0]) for x in xs]
+    state = torch.zeros(7, taps - 1, channels, device=device) if taps > 1 else None
+    slots, done = [3, 0, 5, 1, 6], [0] * 5
+    for step in (lens, [1] * 5, [2, 17, 1, 25, 11], [27, 12, 28, 4, 18]):
+        live = [i for i in range(5) if step[i]]
+        ctx = fake_ctx(device, [step[i] for i in live], [done[i] for i in live], [slots[i] for i in live])
+        rows = torch.cat([xs[i][done[i]:done[i] + step[i]] for i in live])
+        wide = torch.randn(rows.shape[0], channels + 10).to(dtype).to(device)
+        wide[:, :channels] = rows.to(device)
+        out = torch.empty(rows.shape[0], channels, dtype=dtype, device=device)
+        ops.short_conv(wide[:, :channels], out, w.to(device), state, ctx, residual=False, silu=True)
+        at = 0
+        for i in live:
+            assert torch.allclose(out[at:at + step[i]].cpu().double(), want[i][done[i]:done[i] + step[i]], **tol_of(dtype)), (step, i)
+            at, done[i] = at + step[i], done[i] + step[i]
+    assert done == [n + 30 for n in lens]
+
+
+@pytest.mark.parametrize("dtype", [F32, BF16])
+@pytest.mark.parametrize("T", [1, 47, 48, 200])
+@pytest.mark.parametrize("heads,K,N,pad", [(3, 64, 128, 16), (4, 48, 40, 8), (2, 200, 72, 0), (5, 13, 21, 3), (16, 128, 192, 64)])
+def test_product_per_head(device, T, heads, K, N, pad, dtype):
+    """Heads apart by more than their sizes, gates, sizes of whole tiles and not; short steps and those on tensor cores."""
+    ops = _ops()
+    torch.manual_seed(T + K)
+    x, w = torch.randn(T, heads * (K + pad)).to(dtype), (torch.randn(heads, K, N) / math.sqrt(K)).to(dtype)
+    gates = torch.randn(T, heads + 2).to(dtype)
+    out = torch.full((T, heads * (N + 8)), 9.0, dtype=dtype, device=device)
+    want = torch.einsum("thk,hkn->thn", x.double().view(T, heads, K + pad)[..., :K], w.double())
+    ops.head_gemm(x.to(device), K + pad, w.to(device), out, N + 8)
+    got = out.view(T, heads, N + 8)
+    assert torch.allclose(got[..., :N].cpu().double(), want, **tol_of(dtype)) and bool((got[..., N:] == 9.0).all())
+    ops.head_gemm(x.to(device), K + pad, w.to(device), out, N + 8, gate=gates.to(device)[:, 1:1 + heads])
+    want = want * torch.sigmoid(gates[:, 1:1 + heads].double())[..., None]
+    assert torch.allclose(out.view(T, heads, N + 8)[..., :N].cpu().double(), want, **tol_of(dtype))
+
+
+@pytest.mark.parametrize("dtype", [F32, BF16])
+@pytest.mark.parametrize("heads,dv", [(3, 64), (2, 128), (4, 33), (1, 512), (2, 700), (5, 8), (2, 200)])
+@pytest.mark.parametrize("kind", ["sigmoid", "silu"])
+def test_norm_per_head_with_its_gate(device, heads, dv, kind, dtype):
+    ops = _ops()
+    torch.manual_seed(heads * dv)
+    T = 37
+    o, w, gate = 2.0 * torch.randn(T, heads * dv), 1.0 + 0.2 * torch.randn(dv), torch.randn(T, heads * dv + 8).to(dtype)
+    g = gate[:, :heads * dv].double()
+    want = (plain.rms_div(o.double().view(T, heads, dv), 1e-4) * w.double()).reshape(T, -1) * (torch.sigmoid(g) if kind == "sigmoid" else plain.silu(g))
+    out = torch.empty(T, heads * dv, dtype=dtype, device=device)
+    ops.gated_group_norm(o.to(device), gate.to(device)[:, :heads * dv], w.to(device), 1e-4, out, group=dv, gate_kind=kind)
+    assert torch.allclose(out.cpu().double(), want, **tol_of(dtype))
+    ops.gated_group_norm(o.to(device), None, w.to(device), 1e-4, out, group=dv)
+    assert torch.allclose(out.cpu().double(), (plain.rms_div(o.double().view(T, heads, dv), 1e-4) * w.double()).reshape(T, -1), **tol_of(dtype))
+
+
 # =========================================================================================== experts
 @pytest.mark.parametrize("dtype,form", [(F32, "few"), (BF16, "few"), (BF16, "sorted"), (F32, "token"), (BF16, "token")])
 @pytest.mark.parametrize("activation", ["relu2", "silu"])
