@@ -846,7 +846,8 @@ def retezen_kernel_numbers(s: dict, peaks: dict) -> dict:
 
 
 def lukelorn_kernel_numbers(s: dict, peaks: dict) -> dict:
-    """The Lukelorn design's own kernels alone at the layer sizes ``s``, measured as ``kernel_numbers`` measures, each beside the
+    """The Lukelorn design's own kernels alone at the layer sizes ``s``, measured as ``kernel_numbers`` measures (prompt portions
+    four launches back to back: a form of two launches would else be timed together with the host's way to both), each beside the
     like kernel of the designs that were there before (the delta rule with a decay per head, attention over a window alone, over
     a latent without one, experts with a gate of as many weights)."""
     import torch
@@ -893,7 +894,7 @@ def lukelorn_kernel_numbers(s: dict, peaks: dict) -> dict:
     randn = lambda *shape: torch.randn(*shape, device=dev)
     for name, batch, q_len, ctx_len in (("decode_b64", 64, 1, 2047), ("decode_b8", 8, 1, 2047), ("prefill_2048", 1, 2048, 0)):
         T = batch * q_len
-        reps = 10 if T <= 64 else 1
+        reps = 10 if T <= 64 else 4
         pages_each = (ctx_len + q_len + 15) // 16
         tables = torch.arange(batch * pages_each, dtype=torch.int32, device=dev).view(batch, pages_each)
         ctx = ctx_of([q_len] * batch, ctx_len)
@@ -988,7 +989,7 @@ def lukelorn_kernel_numbers(s: dict, peaks: dict) -> dict:
             up = (randn(EXPERTS, (n - 1) * eff, W) / math.sqrt(W)).to(bf)
             down = (randn(EXPERTS, W, eff) / math.sqrt(eff)).to(bf)
             t = _timed(lambda: ops.moe_experts(x, up, down, ids, wts, hrow, ws, accumulate=True, input_weights=True, plain=plain,
-                                               activation="relu2" if plain else "silu"), flush)
+                                               activation="relu2" if plain else "silu"), flush, reps=2)
             record(f"{what}_{tag}", t, bytes_=distinct * n * W * eff * 2 + T * W * (2 + 8), tensor_flops=2.0 * T * TOP * n * W * eff)
             out[f"{what}_{tag}"]["distinct_experts"] = distinct
     return out

@@ -1,4 +1,4 @@
-// Attention over the paged cache, general form: any head size up to 512 (the values' may differ
+// Attention over the paged cache, general form: any head size up to 1024 (the values' may differ
 // from the queries' and keys'), any page size, any number of heads and groups, an optional window;
 // fp32 arithmetic throughout whatever the storage type.  One block per (token, query head); the warps of a block split the keys and keep
 // a running maximum, sum and weighted value sum each, merged at the end.
@@ -25,9 +25,9 @@ namespace {
 
 constexpr int ATT_THREADS = 128;
 constexpr int ATT_WARPS = ATT_THREADS / 32;
-constexpr int MAX_PER_LANE = 16;  // head size up to 512 (the forms below this one: up to 256)
+constexpr int MAX_HEAD = 1024;  // (the forms below this one: up to 256)
 
-template <typename T, bool POOL>
+template <typename T, bool POOL, int MAX_PER_LANE>  // elements of a head that a lane holds: 16 (sizes up to 512) or 32
 __global__ void __launch_bounds__(ATT_THREADS)
     paged_attention_simt_kernel(const T* q, int ldq, T* __restrict__ out, int ldo, const T* k_cache, const T* v_cache,
                                 const int* __restrict__ block_tables, int max_blocks,
@@ -783,8 +783,8 @@ FERRIS_API int ferris_paged_attention_simt(const void* q, int ldq, void* out, in
     if (int rc = check_pooled(pk, window, st)) return rc;
     const bool pool = pk.every > 0 || pk.keep > 0;
     if (nh <= 0 || nkv <= 0 || nh % nkv != 0) FERRIS_REFUSE("attention: %d heads over %d kv heads", nh, nkv);
-    if (d <= 0 || d > 32 * MAX_PER_LANE) FERRIS_REFUSE("attention: head size %d not in 1..%d", d, 32 * MAX_PER_LANE);
-    if (dv <= 0 || dv > 32 * MAX_PER_LANE) FERRIS_REFUSE("attention: value head size %d not in 1..%d", dv, 32 * MAX_PER_LANE);
+    if (d <= 0 || d > MAX_HEAD) FERRIS_REFUSE("attention: head size %d not in 1..%d", d, MAX_HEAD);
+    if (dv <= 0 || dv > MAX_HEAD) FERRIS_REFUSE("attention: value head size %d not in 1..%d", dv, MAX_HEAD);
     if (page_size <= 0 || max_blocks <= 0) FERRIS_REFUSE("attention: page_size=%d max_blocks=%d", page_size, max_blocks);
     if (nh > 65535) FERRIS_REFUSE("attention: %d heads are more than one launch takes", nh);
     dim3 grid(tokens, nh);
@@ -854,15 +854,21 @@ FERRIS_API int ferris_paged_attention_simt(const void* q, int ldq, void* out, in
         FERRIS_LAUNCH_CHECK();
     }
 #define FERRIS_ATT(T, POOL)                                                                                               \
-    ferris_launch(paged_attention_simt_kernel<T, POOL>, grid, dim3(ATT_THREADS), smem, s, (const T*)q, ldq, (T*)out, ldo,  \
+    if (d <= 512 && dv <= 512)                                                                                            \
+        FERRIS_ATT_N(T, POOL, 16);                                                                                        \
+    else                                                                                                                  \
+        FERRIS_ATT_N(T, POOL, 32)
+#define FERRIS_ATT_N(T, POOL, N)                                                                                          \
+    ferris_launch(paged_attention_simt_kernel<T, POOL, N>, grid, dim3(ATT_THREADS), smem, s, (const T*)q, ldq, (T*)out, ldo,  \
                   (const T*)k_cache, (const T*)v_cache, block_tables, max_blocks, token_seq, positions, nh, nkv, d, dv,    \
                   page_size, window, scale, st, pk)
     if (dtype == FERRIS_F32) {
-        if (pool) FERRIS_ATT(float, true); else FERRIS_ATT(float, false);
+        if (pool) { FERRIS_ATT(float, true); } else { FERRIS_ATT(float, false); }
     } else {
-        if (pool) FERRIS_ATT(bf16, true); else FERRIS_ATT(bf16, false);
+        if (pool) { FERRIS_ATT(bf16, true); } else { FERRIS_ATT(bf16, false); }
     }
 #undef FERRIS_ATT
+#undef FERRIS_ATT_N
     FERRIS_LAUNCH_CHECK();
 }
 

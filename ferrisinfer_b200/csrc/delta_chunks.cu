@@ -76,7 +76,7 @@ __global__ void __launch_bounds__(DC_PREP_THREADS) delta_chunk_prepare_kernel(
     float* Qs = Ks + DC_TOKENS * pitch;
     __shared__ float As[DC_TOKENS][DC_TOKENS + 1], bs[DC_TOKENS];
     pdl_wait();
-    pdl_launch_dependents();
+    // (the walk is let in when this kernel's blocks end: its blocks would hold half of an SM's registers while they wait)
     const int seq = blockIdx.x / chunks_max, head = blockIdx.y;
     const int row0 = seq_q_start[seq], row1 = seq_q_start[seq + 1];
     const int first = row0 + (blockIdx.x % chunks_max) * DC_TOKENS;

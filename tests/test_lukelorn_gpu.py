@@ -204,7 +204,8 @@ def test_attention_on_tensor_cores_against_cuda_cores(device, nh, nkv, d, dv, wi
 
 @pytest.mark.parametrize("dtype", [F32, BF16])
 @pytest.mark.parametrize("form", ["single", "portion", "shares", "single rows", "portion rows", "shares rows"])
-@pytest.mark.parametrize("nh,rank,rot,window", [(4, 48, 8, 19), (3, 33, 6, 1), (2, 112, 16, 16), (16, 96, 32, 40), (20, 24, 8, 0)])
+@pytest.mark.parametrize("nh,rank,rot,window", [(4, 48, 8, 19), (3, 33, 6, 1), (2, 112, 16, 16), (16, 96, 32, 40), (20, 24, 8, 0),
+                                                (2, 512, 64, 20)])
 def test_latents_in_a_window_one_key_stands_out_at_each_edge(device, nh, rank, rot, window, form, dtype):
     """Keys that carry their values: the loud latent just inside the window takes the weight, the one just outside does not."""
     ops = _ops()
